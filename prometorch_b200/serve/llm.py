@@ -1,16 +1,18 @@
-"""Continuous-batching engine for Hugging Face Llama checkpoints with a paged KV cache.
+"""Continuous-batching engine with a paged KV cache for the models registered in ``models/paged.py`` (Hugging Face Llama
+checkpoints, Kifusun).
 
 Same public surface as the reference's ``LLMEngine`` (torch/serve/llm.h:33-57 for the request types, :299-334 for the
 64-token page pool, :352-437 for ``load / set_weights / generate / submit_request / step / poll_responses``).  The
 reference walks its active requests one after another on the CPU; here one ``step()`` is
 
-* a prompt pass for each newly admitted request (tcgen05 GEMMs, FlashAttention over the prompt, rotary + page write
-  in ``paged_rope_write_kernel``), and
-* ONE batched decode pass for all other active requests: a ``[B, hidden]`` activation runs through the layer GEMMs,
-  ``paged_attn_decode_kernel`` reads each request's pages through the page table, and the sampler picks the next ids
-  on the device.
+* a prompt pass for the newly admitted requests (for Llama: tcgen05 GEMMs, FlashAttention over the prompt, rotary + page
+  write in ``paged_rope_write_kernel``), and
+* ONE batched decode pass for all other active requests: a ``[B, hidden]`` activation runs through the layer GEMMs, an
+  attention kernel reads each request's pages through the page table, and the sampler picks the next ids on the device.
 
-Pages come from one pool shared by all requests and go back to it when a request finishes.  CPU tensors take the
+Pages come from one pool shared by all requests and go back to it when a request finishes, or earlier when every layer of
+the model has a window and the page lies behind all of them.  ``feed`` runs given ids through the same passes and returns
+logits (scoring, replay).  CPU tensors take the
 plain torch path of every op, which is how the scheduling logic is tested without a GPU.
 """
 from __future__ import annotations
@@ -23,8 +25,9 @@ from dataclasses import dataclass, field
 from typing import Callable, Deque, Dict, List, Optional, Sequence, Union
 
 import torch
-import torch.nn.functional as F
 
+from ..models.llama_paged import LlamaConfig, LlamaWeights  # noqa: F401
+from ..models.paged import PagedModel, PromptBatch, entry_of, read_config, resolve_architecture
 from ..ops import paged as P
 
 PAGE = P.PAGE
@@ -57,114 +60,7 @@ class Response:
     throughput_tok_per_s: float = 0.0
 
 
-@dataclass
-class LlamaConfig:
-    vocab_size: int = 32000
-    hidden_size: int = 4096
-    intermediate_size: int = 11008
-    num_hidden_layers: int = 32
-    num_attention_heads: int = 32
-    num_key_value_heads: int = 32
-    max_position_embeddings: int = 4096
-    rms_norm_eps: float = 1e-5
-    rope_theta: float = 10000.0
-    bos_token_id: int = 1
-    eos_token_id: int = 2
-    tie_word_embeddings: bool = False
-
-    @property
-    def head_dim(self) -> int:
-        return self.hidden_size // self.num_attention_heads
-
-    @classmethod
-    def from_json(cls, path: str) -> "LlamaConfig":
-        with open(path) as f:
-            d = json.load(f)
-        c = cls()
-        for k in cls.__dataclass_fields__:
-            if k in d and d[k] is not None:
-                v = d[k]
-                if k == "eos_token_id" and isinstance(v, list):
-                    v = v[0]
-                setattr(c, k, type(getattr(c, k))(v))
-        if "num_key_value_heads" not in d:
-            c.num_key_value_heads = c.num_attention_heads
-        return c
-
-
 from ..io.safetensors import load_checkpoint_dir, load_file as load_safetensors, save_file as save_safetensors  # noqa: E402,F401
-
-
-# ------------------------------------------------------------------------------------------ weights
-class LlamaWeights:
-    """Weights in the layout the engine runs: q/k/v packed into one matrix, gate/up packed into one."""
-
-    def __init__(self, cfg: LlamaConfig):
-        self.cfg = cfg
-        self.tok_emb: Optional[torch.Tensor] = None
-        self.layers: List[Dict[str, torch.Tensor]] = []
-        self.final_norm: Optional[torch.Tensor] = None
-        self.lm_head: Optional[torch.Tensor] = None
-
-    @classmethod
-    def random(cls, cfg: LlamaConfig, seed: int = 0, dtype=torch.float32, device="cpu") -> "LlamaWeights":
-        """Random weights of the right scales (benchmarks and tests); drawn on ``device`` so a large model never sits in
-        host memory."""
-        g = torch.Generator(device=device).manual_seed(seed)
-        D, I, H, Hk, Dh = cfg.hidden_size, cfg.intermediate_size, cfg.num_attention_heads, cfg.num_key_value_heads, cfg.head_dim
-
-        def r(*s, scale):
-            return (torch.randn(*s, generator=g, device=device) * scale).to(dtype)
-
-        def norm_w():
-            return (1 + 0.1 * torch.randn(D, generator=g, device=device)).to(dtype)
-        w = cls(cfg)
-        w.tok_emb = r(cfg.vocab_size, D, scale=1.0)
-        for _ in range(cfg.num_hidden_layers):
-            w.layers.append(dict(attn_norm=norm_w(), wqkv=r((H + 2 * Hk) * Dh, D, scale=D ** -0.5), wo=r(D, H * Dh, scale=(H * Dh) ** -0.5),
-                                 ffn_norm=norm_w(), w_gate_up=r(2 * I, D, scale=D ** -0.5), w_down=r(D, I, scale=I ** -0.5)))
-        w.final_norm = norm_w()
-        w.lm_head = r(cfg.vocab_size, D, scale=D ** -0.5)
-        return w
-
-    @classmethod
-    def from_state_dict(cls, cfg: LlamaConfig, sd: Dict[str, torch.Tensor]) -> "LlamaWeights":
-        """Hugging Face names: ``model.layers.N.self_attn.{q,k,v,o}_proj.weight`` and so on."""
-        w = cls(cfg)
-        if "embed_tokens.weight" in sd and "model.embed_tokens.weight" not in sd:          # a bare LlamaModel checkpoint
-            sd = {("model." + k if not k.startswith("lm_head") else k): v for k, v in sd.items()}
-        w.tok_emb = sd["model.embed_tokens.weight"]
-        for l in range(cfg.num_hidden_layers):
-            p = f"model.layers.{l}."
-            w.layers.append(dict(
-                attn_norm=sd[p + "input_layernorm.weight"],
-                wqkv=torch.cat([sd[p + "self_attn.q_proj.weight"], sd[p + "self_attn.k_proj.weight"], sd[p + "self_attn.v_proj.weight"]]),
-                wo=sd[p + "self_attn.o_proj.weight"], ffn_norm=sd[p + "post_attention_layernorm.weight"],
-                w_gate_up=torch.cat([sd[p + "mlp.gate_proj.weight"], sd[p + "mlp.up_proj.weight"]]), w_down=sd[p + "mlp.down_proj.weight"]))
-        w.final_norm = sd["model.norm.weight"]
-        w.lm_head = sd.get("lm_head.weight", w.tok_emb)
-        return w
-
-    def state_dict(self) -> Dict[str, torch.Tensor]:
-        c = self.cfg
-        H, Hk, Dh, I = c.num_attention_heads, c.num_key_value_heads, c.head_dim, c.intermediate_size
-        sd = {"model.embed_tokens.weight": self.tok_emb, "model.norm.weight": self.final_norm, "lm_head.weight": self.lm_head}
-        for l, L in enumerate(self.layers):
-            p = f"model.layers.{l}."
-            q, k, v = L["wqkv"].split([H * Dh, Hk * Dh, Hk * Dh])
-            g, u = L["w_gate_up"].split([I, I])
-            sd.update({p + "input_layernorm.weight": L["attn_norm"], p + "self_attn.q_proj.weight": q, p + "self_attn.k_proj.weight": k,
-                       p + "self_attn.v_proj.weight": v, p + "self_attn.o_proj.weight": L["wo"],
-                       p + "post_attention_layernorm.weight": L["ffn_norm"], p + "mlp.gate_proj.weight": g,
-                       p + "mlp.up_proj.weight": u, p + "mlp.down_proj.weight": L["w_down"]})
-        return sd
-
-    def to(self, device, dtype) -> "LlamaWeights":
-        w = LlamaWeights(self.cfg)
-        mv = lambda t: t.to(device=device, dtype=dtype).contiguous()
-        w.tok_emb, w.final_norm, w.lm_head = mv(self.tok_emb), mv(self.final_norm), mv(self.lm_head)
-        w.layers = [{k: mv(v) for k, v in L.items()} for L in self.layers]
-        return w
 
 
 class ByteTokenizer:
@@ -206,13 +102,20 @@ def load_hf_tokenizer(model_dir: str):
 class PagedKVCache:
     """One pool of 64-token pages shared by all requests; a page id addresses the same slot in every layer."""
 
-    def __init__(self, num_layers: int, num_kv_heads: int, head_dim: int, max_pages: int, device, dtype, spare: bool = False):
+    def __init__(self, num_layers: int, num_kv_heads: int, head_dim: int, max_pages: int, device, dtype, spare: bool = False,
+                 shapes: Optional[List[tuple]] = None):
+        """``shapes``: (kv heads, key size, value size) per layer, for models whose layers differ."""
         n = max_pages + (1 if spare else 0)                # the spare page (id max_pages) is never handed out
-        self.k = [torch.zeros(n, num_kv_heads, PAGE, head_dim, device=device, dtype=dtype) for _ in range(num_layers)]
-        self.v = [torch.zeros(n, num_kv_heads, PAGE, head_dim, device=device, dtype=dtype) for _ in range(num_layers)]
+        shapes = shapes if shapes is not None else [(num_kv_heads, head_dim, head_dim)] * num_layers
+        self.k = [torch.zeros(n, hk, PAGE, dk, device=device, dtype=dtype) for hk, dk, _ in shapes]
+        self.v = [torch.zeros(n, hk, PAGE, dv, device=device, dtype=dtype) for hk, _, dv in shapes]
         self.max_pages = max_pages
         self.spare_page = max_pages if spare else -1
         self.free_pages: Deque[int] = collections.deque(range(max_pages))
+
+    @classmethod
+    def for_model(cls, model: PagedModel, max_pages: int, device, dtype) -> "PagedKVCache":
+        return cls(0, 0, 0, max_pages, device, dtype, spare=True, shapes=model.kv_shapes())
 
     def alloc_page(self) -> int:
         return self.free_pages.popleft() if self.free_pages else -1
@@ -234,7 +137,8 @@ class RequestState:
     t_start: float
     prompt_ids: List[int] = field(default_factory=list)
     row: int = -1                        # row of the page table while active
-    pages: List[int] = field(default_factory=list)
+    pages: List[int] = field(default_factory=list)       # by place in the sequence; -1: already given back
+    passed: int = 0                      # how many leading pages were given back
     kv_position: int = 0
     output_ids: List[int] = field(default_factory=list)
     prefill_done: bool = False
@@ -255,8 +159,8 @@ class LLMEngine:
         self.device = torch.device(device if device is not None else ("cuda" if torch.cuda.is_available() else "cpu"))
         self.dtype = dtype if dtype is not None else (torch.bfloat16 if self.device.type == "cuda" else torch.float32)
         self.max_pages, self.max_active = max_pages, max_active
-        self.cfg: Optional[LlamaConfig] = None
-        self.weights: Optional[LlamaWeights] = None
+        self.cfg = None
+        self.model: Optional[PagedModel] = None
         self.tokenizer = ByteTokenizer()
         self.kv: Optional[PagedKVCache] = None
         self.pending: Deque[RequestState] = collections.deque()
@@ -278,11 +182,13 @@ class LLMEngine:
 
     # -------------------------------------------------------------------------------------- loading
     def load(self, model_dir: str) -> bool:
-        """A Hugging Face directory: ``config.json``, ``model.safetensors`` (or the shards its index lists), tokenizer."""
-        cj = os.path.join(model_dir, "config.json")
-        if not os.path.exists(cj):
+        """A directory with ``config.json``, ``model.safetensors`` (or the shards its index lists) and, if there is one, a
+        tokenizer.  ``config.json`` picks the model (``models/paged.py``)."""
+        d = read_config(model_dir)
+        if d is None:
             return False
-        cfg = LlamaConfig.from_json(cj)
+        entry = resolve_architecture(d)
+        cfg = entry.config.from_dict(d)
         sd = load_checkpoint_dir(model_dir)
         tok = load_hf_tokenizer(model_dir)
         if tok is not None:
@@ -290,15 +196,14 @@ class LLMEngine:
         if not sd:
             self.cfg = cfg
             return True                           # weights may still arrive through set_weights()
-        self.set_weights(LlamaWeights.from_state_dict(cfg, sd))
+        self.set_weights(entry.weights.from_state_dict(cfg, sd))
         return True
 
-    def set_weights(self, w: LlamaWeights):
+    def set_weights(self, w):
         self.cfg = w.cfg
-        self.weights = w.to(self.device, self.dtype)
+        self.model = entry_of(w.cfg).model(w, self.device, self.dtype)
         c = self.cfg
-        self.cos, self.sin = P.rope_tables(c.max_position_embeddings, c.head_dim, c.rope_theta, self.device)
-        self.kv = PagedKVCache(c.num_hidden_layers, c.num_key_value_heads, c.head_dim, self.max_pages, self.device, self.dtype, spare=True)
+        self.kv = PagedKVCache.for_model(self.model, self.max_pages, self.device, self.dtype)
         self.pt_stride = (c.max_position_embeddings + PAGE - 1) // PAGE
         # one row per active request plus a spare one whose single page absorbs the writes of padding rows
         self.page_table = torch.zeros(self.max_active + 1, self.pt_stride, dtype=torch.int32, device=self.device)
@@ -306,6 +211,10 @@ class LLMEngine:
         self.free_rows = list(range(self.max_active))
         self._graphs = {}
         self.loaded = True
+
+    @property
+    def weights(self):
+        return self.model.weights if self.model is not None else None
 
     # -------------------------------------------------------------------------------------- public API
     def generate(self, prompt, config: Optional[GenerationConfig] = None) -> Response:
@@ -348,6 +257,54 @@ class LLMEngine:
         self.pending.append(RequestState(req.request_id, req.config, list(ids), len(ids), time.perf_counter(), prompt_ids=list(ids),
                                          on_token=req.on_token))
         self._admit_pending()
+
+    # ---- given ids instead of sampled ones
+    def open_sequence(self) -> RequestState:
+        """A sequence whose ids the caller supplies through :meth:`feed`; it holds a page-table row until it is closed."""
+        if not self.free_rows:
+            raise RuntimeError("open_sequence: every page-table row is in use")
+        s = RequestState(-1, GenerationConfig(), [], 0, time.perf_counter())
+        s.row = self.free_rows.pop()
+        return s
+
+    def close_sequence(self, s: RequestState):
+        self._free_pages(s)
+        self.free_rows.append(s.row)
+        s.row = -1
+
+    @torch.no_grad()
+    def feed(self, entries: Sequence[tuple]) -> torch.Tensor:
+        """``entries``: (sequence, its next ids, places among these ids whose logits are wanted).  One batch: a decode pass if
+        every entry goes on by one token, else prompt passes.  Returns fp32 logits ``[wanted, V]`` in the order asked for."""
+        entries = [(s, [int(t) for t in ids], list(want)) for s, ids, want in entries if len(ids)]
+        for s, ids, _ in entries:
+            if s.kv_position + len(ids) > self.cfg.max_position_embeddings:
+                raise ValueError(f"feed: {s.kv_position + len(ids)} tokens exceed the context of {self.cfg.max_position_embeddings}")
+            if not self._ensure_pages(s, s.kv_position + len(ids) - 1):
+                raise RuntimeError("feed: the page pool is empty")
+        out: List[torch.Tensor] = []
+        if entries and all(len(ids) == 1 and s.kv_position > 0 for s, ids, _ in entries):
+            logits = self._forward_rows([[ids[0], s.kv_position, s.row, s.kv_position + 1] for s, ids, _ in entries])
+            out = [logits[i:i + 1] for i, (_, _, want) in enumerate(entries) for _ in want]
+        else:
+            todo = list(entries)
+            while todo:
+                chunk, total = [], 0
+                while todo and (not chunk or total + len(todo[0][1]) <= self.max_prompt_tokens):
+                    total += len(todo[0][1])
+                    chunk.append(todo.pop(0))
+                at, want = 0, []
+                for _, ids, w in chunk:
+                    want += [at + p for p in w]
+                    at += len(ids)
+                batch = self._prompt_batch([(ids, s.kv_position, s.row) for s, ids, _ in chunk], want)
+                out.append(self.model.prompt_pass(self.kv, self.page_table, batch))
+        for s, ids, _ in entries:
+            s.kv_position += len(ids)
+            self._release_passed(s)
+        if self.device.type == "cuda":
+            P.check_status(self.device)
+        return torch.cat(out) if out else torch.empty(0, self.cfg.vocab_size, device=self.device)
 
     def cancel(self, request_id: int) -> bool:
         """Drop a queued request or end a running one at the next step (its pages go back to the pool; it still gets a
@@ -408,6 +365,7 @@ class LLMEngine:
             logits = self._forward_prompts(chunk)
             for i, s in enumerate(chunk):
                 s.kv_position = s.prompt_len
+                self._release_passed(s)
                 s.prefill_done = True
                 self._emit(s, self._sample([s], logits[i:i + 1])[0])
         running = [s for s in running if self._ensure_pages(s, s.kv_position) or self._finish(s)]
@@ -417,6 +375,7 @@ class LLMEngine:
             logits = self._forward_decode(running)
             for s, t in zip(running, self._sample(running, logits)):
                 s.kv_position += 1
+                self._release_passed(s)
                 self._emit(s, t)
         finished = any(s.done for s in self.active)
         self._collect_done()
@@ -480,6 +439,7 @@ class LLMEngine:
                 if s.done or j >= len(draft) or draft[j] != tok:
                     break
                 j += 1
+            self._release_passed(s)
             self.spec_drafted += len(draft)
             self.spec_accepted += j
 
@@ -493,7 +453,7 @@ class LLMEngine:
         except TypeError:                                      # a tokenizer without the add_bos switch
             ids = list(self.tokenizer.encode(prompt))
         bos = self.cfg.bos_token_id
-        if not ids or ids[0] != bos:
+        if bos is not None and (not ids or ids[0] != bos):
             ids = [bos] + ids
         return [min(max(int(i), 0), self.cfg.vocab_size - 1) for i in ids]
 
@@ -523,6 +483,24 @@ class LLMEngine:
             self.page_table[s.row, lo:lo + len(fresh)] = torch.tensor(fresh, dtype=torch.int32, device=self.device)
         return True
 
+    def _release_passed(self, s: RequestState):
+        """Give back the pages no layer can read again: the next token stands at ``kv_position`` and sees the
+        ``cache_window`` latest tokens, itself included."""
+        window = self.model.cache_window()
+        if window is None:
+            return
+        keep = max(0, s.kv_position - window + 1) // PAGE             # first page that is still in a window
+        for i in range(s.passed, min(keep, len(s.pages))):
+            self.kv.free_page(s.pages[i])
+            s.pages[i] = -1
+        s.passed = max(s.passed, min(keep, len(s.pages)))
+
+    def _free_pages(self, s: RequestState):
+        for p in s.pages:
+            if p >= 0:
+                self.kv.free_page(p)
+        s.pages, s.passed = [], 0
+
     def _emit(self, s: RequestState, tok: int):
         self.tokens_generated += 1
         s.output_ids.append(tok)
@@ -544,9 +522,7 @@ class LLMEngine:
             if not s.done:
                 keep.append(s)
                 continue
-            for p in s.pages:
-                self.kv.free_page(p)
-            s.pages = []
+            self._free_pages(s)
             self.free_rows.append(s.row)
             dt = max(time.perf_counter() - s.t_start, 1e-9)
             text = self.tokenizer.decode(s.output_ids)
@@ -554,20 +530,6 @@ class LLMEngine:
         self.active = keep
 
     # -------------------------------------------------------------------------------------- model
-    def _linear(self, x, w):
-        if x.is_cuda:
-            from ..ops.gemm import linear
-            return linear(x, w)
-        return F.linear(x, w)
-
-    def _norm(self, x, w):
-        from ..ops.fused_ops import rms_norm
-        return rms_norm(x, w, self.cfg.rms_norm_eps)
-
-    def _mlp(self, x, L):
-        from ..ops.fused_ops import swiglu
-        return self._linear(swiglu(self._linear(x, L["w_gate_up"])), L["w_down"])
-
     def _forward_prompt(self, s: RequestState) -> torch.Tensor:
         """All prompt tokens of one request; fills its pages; returns the logits of the last position ``[1, V]``."""
         return self._forward_prompts([s])
@@ -588,67 +550,32 @@ class LLMEngine:
             h = self._forward_prompts([s], hidden=True).float().mean(0)
             return h / h.norm().clamp_min(1e-12)
         finally:
-            for p in s.pages:
-                self.kv.free_page(p)
+            self._free_pages(s)
             self.free_rows.append(s.row)
 
-    def _forward_prompts(self, batch: List[RequestState], hidden: bool = False) -> torch.Tensor:
-        """The prompt pass of several new requests at once: their tokens are concatenated, so every projection is one
-        GEMM over all of them; attention runs per request (requests of equal length share a call).  Fills the pages;
-        returns the logits of each request's last position ``[len(batch), V]``."""
-        from ..ops.attention import flash_attention
-        c, w = self.cfg, self.weights
-        H, Hk, Dh = c.num_attention_heads, c.num_key_value_heads, c.head_dim
+    def _prompt_batch(self, parts: List[tuple], want: Optional[List[int]] = None) -> PromptBatch:
+        """``parts``: (ids, first position, page-table row) per sequence; ``want``: places among the concatenated tokens
+        (default: every sequence's last)."""
         dev = self.device
-        lens = [s.prompt_len for s in batch]
+        lens = [len(ids) for ids, _, _ in parts]
         offs = [0]
         for n in lens:
             offs.append(offs[-1] + n)
-        ids = torch.tensor([t for s in batch for t in s.input_ids], dtype=torch.long)
-        pos = torch.cat([torch.arange(n, dtype=torch.int32) for n in lens])
-        req = torch.cat([torch.full((n,), s.row, dtype=torch.int32) for s, n in zip(batch, lens)])
-        ids, pos, req = ids.to(dev), pos.to(dev), req.to(dev)
-        groups: Dict[int, List[int]] = {}
-        for i, n in enumerate(lens):
-            groups.setdefault(n, []).append(i)
-        consecutive = all(g == list(range(g[0], g[0] + len(g))) for g in groups.values())
-        x = w.tok_emb[ids]
-        for l, L in enumerate(w.layers):
-            qkv = self._linear(self._norm(x, L["attn_norm"]), L["wqkv"]).contiguous()
-            k = P.paged_rope_write(qkv, H, Hk, Dh, pos, req, self.page_table, self.cos, self.sin, self.kv.k[l], self.kv.v[l], want_k=True)
-            a = torch.empty(qkv.shape[0], H * Dh, dtype=qkv.dtype, device=dev)
-            for n, members in groups.items():
-                runs = [members] if consecutive else [[i] for i in members]      # equal lengths side by side: one call
-                for run in runs:
-                    lo, hi, nb = offs[run[0]], offs[run[-1] + 1], len(run)
-                    q = qkv[lo:hi, :H * Dh].reshape(nb, n, H, Dh)
-                    v = qkv[lo:hi, (H + Hk) * Dh:].reshape(nb, n, Hk, Dh)
-                    a[lo:hi] = flash_attention(q, k[lo:hi].view(nb, n, Hk, Dh), v, causal=True).reshape(nb * n, H * Dh)
-            x = x + self._linear(a, L["wo"])
-            x = x + self._mlp(self._norm(x, L["ffn_norm"]), L)
-        if hidden:                                             # the embedding path: every position after the final norm
-            return self._norm(x, w.final_norm)
-        last = x[torch.tensor([o - 1 for o in offs[1:]], device=dev)]
-        return self._linear(self._norm(last, w.final_norm), w.lm_head).float()
+        ids = torch.tensor([t for p in parts for t in p[0]], dtype=torch.int32)
+        pos = torch.cat([torch.arange(at, at + n, dtype=torch.int32) for (_, at, _), n in zip(parts, lens)])
+        req = torch.cat([torch.full((n,), row, dtype=torch.int32) for (_, _, row), n in zip(parts, lens)])
+        want = torch.tensor([o - 1 for o in offs[1:]] if want is None else want, dtype=torch.long)
+        return PromptBatch(ids.to(dev), pos.to(dev), req.to(dev), offs, [p[1] for p in parts], want.to(dev))
+
+    def _forward_prompts(self, batch: List[RequestState], hidden: bool = False) -> torch.Tensor:
+        """The prompt pass of several new requests at once: their tokens are concatenated, so every projection is one
+        GEMM over all of them.  Fills the pages; returns the logits of each request's last position ``[len(batch), V]``."""
+        parts = [(s.input_ids, s.kv_position, s.row) for s in batch]
+        return self.model.prompt_pass(self.kv, self.page_table, self._prompt_batch(parts), hidden)
 
     def _decode_layers(self, meta: torch.Tensor, nsplit: int) -> torch.Tensor:
         """The device work of a decode pass.  ``meta [B, 4]`` int32: token id, position, page-table row, cached length."""
-        from ..ops.gemm import linear_add_rms_norm, linear_swiglu
-        c, w = self.cfg, self.weights
-        H, Hk, Dh = c.num_attention_heads, c.num_key_value_heads, c.head_dim
-        B = meta.shape[0]
-        ids, pos, rows, lens = meta[:, 0].long(), meta[:, 1].contiguous(), meta[:, 2].long(), meta[:, 3].contiguous()
-        table = self.page_table[rows]                          # [B, pt_stride] rows in batch order
-        req = torch.arange(B, dtype=torch.int32, device=meta.device)
-        x = w.tok_emb[ids]
-        h = self._norm(x, w.layers[0]["attn_norm"])
-        for l, L in enumerate(w.layers):
-            q = P.qkv_rope_write(h, L["wqkv"], H, Hk, Dh, pos, req, table, self.cos, self.sin, self.kv.k[l], self.kv.v[l])
-            a = P.paged_attention_decode(q, H, Hk, Dh, lens, table, self.kv.k[l], self.kv.v[l], nsplit=nsplit)
-            h, x = linear_add_rms_norm(a, L["wo"], x, L["ffn_norm"], c.rms_norm_eps)
-            nxt = w.layers[l + 1]["attn_norm"] if l + 1 < len(w.layers) else w.final_norm
-            h, x = linear_add_rms_norm(linear_swiglu(h, L["w_gate_up"]), L["w_down"], x, nxt, c.rms_norm_eps)
-        return self._linear(h, w.lm_head).float()
+        return self.model.decode_pass(self.kv, self.page_table, meta, nsplit)
 
     def _forward_decode(self, batch: List[RequestState]) -> torch.Tensor:
         """One new token for every request of the batch; returns logits ``[B, V]``.  On a GPU the pass is a CUDA graph
@@ -663,15 +590,14 @@ class LLMEngine:
         B = len(rows)
         rows = list(rows)
         max_len = max(r[3] for r in rows)
-        Hk = self.cfg.num_key_value_heads
         if dev.type != "cuda" or not self.use_graphs:
             meta = torch.tensor(rows, dtype=torch.int32)
             meta = (meta.pin_memory() if dev.type == "cuda" else meta).to(dev, non_blocking=True)
-            return self._decode_layers(meta, P.pick_splits(B, Hk, max_len))
+            return self._decode_layers(meta, self.model.pick_splits(B, max_len))
         Bb = 1
         while Bb < max(B, min_rows):
             Bb *= 2
-        nsplit = P.pick_splits(Bb, Hk, max_len)
+        nsplit = self.model.pick_splits(Bb, max_len)
         rows += [[0, 0, self.max_active, 1]] * (Bb - B)        # padding: the spare row of the page table
         key = (Bb, nsplit)
         if key not in self._graphs:

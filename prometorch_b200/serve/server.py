@@ -200,7 +200,7 @@ class OracleBackend(ModelBackend):
 
 
 class PagedBackend(ModelBackend):
-    """A Hugging Face Llama directory served by the continuous-batching engine (``serve/llm.py``).  ``concurrent``:
+    """A directory with ``config.json`` and safetensors served by the continuous-batching engine (``serve/llm.py``).  ``concurrent``:
     the handlers do not serialise generations for this backend, so requests that arrive together share decode
     batches (the reference's server takes one generation at a time, promeserve/api_handlers.h:769-790)."""
     concurrent = True
@@ -214,11 +214,12 @@ class PagedBackend(ModelBackend):
         dev = "cpu" if (device == "cuda" and not torch.cuda.is_available()) else device
         self.engine = LLMEngine(device=dev, max_pages=max_pages, max_active=max_active)
         if not self.engine.load(model_dir) or not self.engine.loaded:
-            raise KeyError(f"'{model_dir}' is not a loadable Hugging Face Llama directory")
+            raise KeyError(f"'{model_dir}' is not a loadable model directory")
         self.server = EngineServer(self.engine)
         self.name, self.path, self.model_name = name, model_dir, os.path.basename(os.path.normpath(model_dir))
         self.size = sum(os.path.getsize(os.path.join(model_dir, f)) for f in os.listdir(model_dir) if f.endswith(".safetensors"))
-        n = sum(t.numel() for L in self.engine.weights.layers for t in L.values()) + self.engine.weights.tok_emb.numel()
+        n = self.engine.weights.num_parameters()
+        self.architecture = self.engine.model.architecture
         self.parameter_size = f"{n / 1e9:.1f}B"
 
     def encode(self, text):
