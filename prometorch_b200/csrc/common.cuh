@@ -214,8 +214,9 @@ __device__ __forceinline__ uint64_t global_ns() {
 
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
 __device__ __forceinline__ float gelu_tanh(float x) {
-    const float k = 0.7978845608028654f;
-    return 0.5f * x * (1.0f + tanhf(k * (x + 0.044715f * x * x * x)));
+    // 0.5 x (1 + tanh(u)) = x * sigmoid(2 u): keeps its relative accuracy where 1 + tanh(u) cancels
+    const float k2 = 2.0f * 0.7978845608028654f;
+    return x / (1.0f + __expf(-k2 * (x + 0.044715f * x * x * x)));
 }
 
 }  // namespace ptb

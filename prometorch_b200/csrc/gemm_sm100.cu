@@ -211,6 +211,22 @@ __global__ void __launch_bounds__(256) splitk_reduce_kernel(const float* __restr
     o[1] = __floats2bfloat162_rn(acc.z, acc.w);
 }
 
+// The sum alone, in fp32 (logits).
+__global__ void __launch_bounds__(256) splitk_reduce_f32_kernel(const float* __restrict__ work, int splits, long long mn, int N, float* __restrict__ C,
+                                                                long long ldc) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const long long i4 = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+    if (i4 >= mn) return;
+    float4 acc = *reinterpret_cast<const float4*>(work + i4);
+    for (int s = 1; s < splits; ++s) {
+        const float4 v = *reinterpret_cast<const float4*>(work + (size_t)s * mn + i4);
+        acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
+    }
+    const long long row = i4 / N;
+    *reinterpret_cast<float4*>(C + row * ldc + (i4 - row * N)) = acc;
+}
+
 // Split-K sum fused with what follows a projection in a decoder layer, so the partials are read once and the layer
 // saves a launch: (a) residual add + RMSNorm after the attention-output and MLP-down projections, (b) the gated
 // activation after the packed gate/up projection.
@@ -263,6 +279,53 @@ __global__ void __launch_bounds__(SKN_THREADS) splitk_reduce_norm_kernel(const f
             __nv_bfloat162* y2 = reinterpret_cast<__nv_bfloat162*>(y + row * N + (size_t)c * 4);
             y2[0] = __floats2bfloat162_rn(h[k].x * rs * w0.x, h[k].y * rs * w0.y);
             y2[1] = __floats2bfloat162_rn(h[k].z * rs * w1.x, h[k].w * rs * w1.y);
+        }
+    }
+}
+
+// One CTA per row, for a decoder whose norm sits on the sublayer's output and whose residual stream is fp32:
+// y = sum_s work[s][row];  x += y / rms(y) * g * w;  xb = bf16(x).
+__global__ void __launch_bounds__(SKN_THREADS) splitk_reduce_post_norm_kernel(const float* __restrict__ work, int splits, long long mn, int N,
+                                                                              const float* __restrict__ w, float g, float eps,
+                                                                              float* __restrict__ x, __nv_bfloat16* __restrict__ xb) {
+    __shared__ float red[32];
+    pdl_wait();
+    pdl_launch_dependents();
+    const size_t row = blockIdx.x;
+    const int nc = N / 4;
+    float4 h[SKN_MAXC];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < SKN_MAXC; ++k) {
+        const int c = k * SKN_THREADS + threadIdx.x;
+        if (c < nc) {
+            float4 a = *reinterpret_cast<const float4*>(work + row * N + (size_t)c * 4);
+            for (int s = 1; s < splits; ++s) {
+                const float4 v = *reinterpret_cast<const float4*>(work + (size_t)s * mn + row * N + (size_t)c * 4);
+                a.x += v.x; a.y += v.y; a.z += v.z; a.w += v.w;
+            }
+            h[k] = a;
+            ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+        }
+    }
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    float t = (threadIdx.x & 31) < SKN_THREADS / 32 ? red[threadIdx.x & 31] : 0.f;
+    t = warp_sum(t);
+    const float rs = rsqrtf(t / (float)N + eps) * g;
+#pragma unroll
+    for (int k = 0; k < SKN_MAXC; ++k) {
+        const int c = k * SKN_THREADS + threadIdx.x;
+        if (c < nc) {
+            float4 r = *reinterpret_cast<const float4*>(x + row * N + (size_t)c * 4);
+            float4 m = make_float4(1.f, 1.f, 1.f, 1.f);
+            if (w) m = *reinterpret_cast<const float4*>(w + (size_t)c * 4);
+            r.x += h[k].x * rs * m.x; r.y += h[k].y * rs * m.y; r.z += h[k].z * rs * m.z; r.w += h[k].w * rs * m.w;
+            *reinterpret_cast<float4*>(x + row * N + (size_t)c * 4) = r;
+            __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(xb + row * N + (size_t)c * 4);
+            o[0] = __floats2bfloat162_rn(r.x, r.y);
+            o[1] = __floats2bfloat162_rn(r.z, r.w);
         }
     }
 }
@@ -385,6 +448,34 @@ PTB_API int ptb_gemm_bf16_splitk_add_norm(const void* A, long long lda, const vo
     if (skinny_partials(A, lda, B, ldb, M, N, K, splits, work, status, n_sm, st, &real)) return -1;
     PTB_CUDA_OK(ptb_launch(splitk_reduce_norm_kernel, dim3(M), dim3(SKN_THREADS), 0, st, ptb_pdl_enabled(), work, real, (long long)M * N, N,
                            (const __nv_bfloat16*)resid_in, (__nv_bfloat16*)resid_out, (const __nv_bfloat16*)norm_w, eps, (__nv_bfloat16*)y));
+    PTB_CUDA_OK(cudaGetLastError());
+    return 0;
+}
+
+// The same product with an fp32 result (no bias).
+PTB_API int ptb_gemm_bf16_splitk_f32(const void* A, long long lda, const void* B, long long ldb, float* C, long long ldc, int M, int N, int K,
+                                     int splits, float* work, int* status, int n_sm, cudaStream_t st) {
+    if (M <= 0 || N <= 0 || K <= 0) return 0;
+    int real = 0;
+    if (skinny_partials(A, lda, B, ldb, M, N, K, splits, work, status, n_sm, st, &real)) return -1;
+    const long long mn = (long long)M * N;
+    PTB_CUDA_OK(ptb_launch(splitk_reduce_f32_kernel, dim3((unsigned)((mn / 4 + 255) / 256)), dim3(256), 0, st, ptb_pdl_enabled(), (const float*)work, real, mn,
+                           N, C, ldc));
+    PTB_CUDA_OK(cudaGetLastError());
+    return 0;
+}
+
+// The same product followed, in the reduce launch, by `x += P / rms(P) * g * w; xb = bf16(x)` (x fp32 [M, N] contiguous, w an
+// optional fp32 vector; N <= 8192).
+PTB_API int ptb_gemm_bf16_splitk_post_norm(const void* A, long long lda, const void* B, long long ldb, int M, int N, int K, int splits,
+                                           float* work, const float* w, float g, float eps, float* x, void* xb, int* status, int n_sm,
+                                           cudaStream_t st) {
+    if (M <= 0 || N <= 0 || K <= 0) return 0;
+    if (N > 4 * SKN_THREADS * SKN_MAXC) { ptb_set_error("gemm split-K + norm: N %d above %d", N, 4 * SKN_THREADS * SKN_MAXC); return -1; }
+    int real = 0;
+    if (skinny_partials(A, lda, B, ldb, M, N, K, splits, work, status, n_sm, st, &real)) return -1;
+    PTB_CUDA_OK(ptb_launch(splitk_reduce_post_norm_kernel, dim3(M), dim3(SKN_THREADS), 0, st, ptb_pdl_enabled(), (const float*)work, real,
+                           (long long)M * N, N, w, g, eps, x, (__nv_bfloat16*)xb));
     PTB_CUDA_OK(cudaGetLastError());
     return 0;
 }
