@@ -222,9 +222,12 @@ class PagedKifusun(PagedModel):
 
     def prompt_pass(self, kv, page_table, batch: PromptBatch, hidden: bool = False) -> torch.Tensor:
         top = max(at + n for at, n in zip(batch.starts, batch.lens()))
+        tiles = A.PromptTiles.of(batch.offs, batch.starts, batch.rows, self.device) if batch.offs[-1] >= A.TILES_FROM else None
 
         def attend(l, q):
             a = self.attn[l]
+            if tiles is not None and A.tiles_supported(q, a):
+                return A.gated_attention_tiles(q, a, tiles, page_table, kv.k[l], kv.v[l])
             return A.gated_attention(q, a, batch.pos, batch.req, page_table, kv.k[l], kv.v[l], A.pick_splits(q.shape[0], a.window, top), top)
         stream = self._layers(S.embed_residual(batch.ids, self.weights.embed, self.cfg.embed_scale), kv, page_table, batch.pos, batch.req, attend)
         if hidden:

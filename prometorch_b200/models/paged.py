@@ -23,6 +23,7 @@ class PromptBatch:
     req: torch.Tensor                  # [n] int32, row of the page table
     offs: List[int]
     starts: List[int]
+    rows: List[int]                    # page-table row of every sequence
     want: Optional[torch.Tensor] = None      # [m] int64, places among the n tokens whose logits are asked for
 
     def lens(self) -> List[int]:

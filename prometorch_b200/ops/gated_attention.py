@@ -8,7 +8,7 @@ from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass
-from typing import Optional
+from typing import List, Optional, Tuple
 
 import torch
 
@@ -27,6 +27,10 @@ def _decls(L):
     L.ptb_gated_rows_work_floats.restype = ll
     L.ptb_gated_attn_rows.argtypes = [vp, vp, ci, ci, ci, ci, ci, ci, vp, ci, vp, ci, vp, ci, ci, vp, vp, vp, ci, vp, ci, cf, cf, ci, vp, ci, vp, ci, vp]
     L.ptb_gated_attn_rows.restype = ci
+    L.ptb_gated_tiles_supported.argtypes = [ci, ci, ci, ci]
+    L.ptb_gated_tiles_supported.restype = ci
+    L.ptb_gated_attn_tiles.argtypes = [vp, vp, vp, ci, ci, ci, ci, ci, ci, vp, ci, ci, vp, vp, vp, ci, vp, ci, cf, cf, vp, ci, ci, vp, vp]
+    L.ptb_gated_attn_tiles.restype = ci
 
 
 def stored(size: int) -> int:
@@ -162,6 +166,53 @@ def gated_attention(q: torch.Tensor, a: GatedAttention, pos: torch.Tensor, req: 
                                             k_pages.shape[0], k_pages.data_ptr(), v_pages.data_ptr(), a.bias.data_ptr(), a.bias.shape[1],
                                             N.ptr(a.talk), a.window, float(a.scale), float(a.softcap), int(max_len), N.ptr(work), nsplit,
                                             _status(q.device).data_ptr(), int(q.dtype == torch.bfloat16), st), "gated_attn_rows")
+    return out
+
+
+QUERY_TILE = 32                        # queries per tile of csrc/gated_prefill.cu
+TILES_FROM = 64                        # rows of a prompt pass from which the tile kernels are the better choice
+WEIGHTS_BYTES = 96 << 20               # scratch of the tile kernels per launch: it should stay in L2 between the two of them
+
+
+@dataclass
+class PromptTiles:
+    """The query tiles of a prompt pass: on the device ``[tiles, 4]`` int32 (first row, its position, rows, page-table row)."""
+    host: List[Tuple[int, int, int, int]]
+    device: torch.Tensor
+    n: int
+
+    @classmethod
+    def of(cls, offs: List[int], starts: List[int], rows: List[int], device) -> "PromptTiles":
+        host = [(lo + i, at + i, min(QUERY_TILE, hi - lo - i), r) for lo, hi, at, r in zip(offs, offs[1:], starts, rows)
+                for i in range(0, hi - lo, QUERY_TILE)]
+        return cls(host, torch.tensor(host, dtype=torch.int32).to(device), offs[-1])
+
+    def width(self, window: int) -> int:
+        """Columns of the weights' band: whole 64-key blocks from the first one a tile sees to its last query."""
+        return max((at + n - max(0, at - window + 1) // PAGE * PAGE + PAGE - 1) // PAGE * PAGE for _, at, n, _ in self.host)
+
+
+def tiles_supported(q: torch.Tensor, a: GatedAttention) -> bool:
+    return q.is_cuda and q.dtype == torch.bfloat16 and bool(N.lib().ptb_gated_tiles_supported(a.heads, a.kv_heads, a.dim_stored, a.vdim_stored))
+
+
+def gated_attention_tiles(q: torch.Tensor, a: GatedAttention, tiles: PromptTiles, page_table: torch.Tensor, k_pages: torch.Tensor,
+                          v_pages: torch.Tensor, sms: int = 148) -> torch.Tensor:
+    """A prompt pass's rows against the pages, on the tensor cores (sizes: :func:`tiles_supported`)."""
+    H, n, nt = a.heads, q.shape[0], len(tiles.host)
+    out = torch.empty(n, H * a.vdim, dtype=q.dtype, device=q.device)
+    KW = tiles.width(a.window)
+    step = max(1, min(nt, WEIGHTS_BYTES // (2 * H * QUERY_TILE * KW), 65535))
+    step = -(-nt // -(-nt // step))                                    # equal shares
+    weights = torch.empty(step * H * QUERY_TILE * KW, dtype=torch.bfloat16, device=q.device)
+    st = torch.cuda.current_stream(q.device).cuda_stream
+    for lo in range(0, nt, step):
+        m = min(step, nt - lo)
+        splits = max(1, min(KW // 64, -(-2 * sms // (2 * m))))
+        N.check(N.lib().ptb_gated_attn_tiles(q.data_ptr(), out.data_ptr(), tiles.device[lo:].data_ptr(), m, H, a.kv_heads, a.dim_stored, a.vdim,
+                                             a.vdim_stored, page_table.data_ptr(), page_table.stride(0), k_pages.shape[0], k_pages.data_ptr(),
+                                             v_pages.data_ptr(), a.bias.data_ptr(), a.bias.shape[1], N.ptr(a.talk), a.window, float(a.scale),
+                                             float(a.softcap), weights.data_ptr(), KW, splits, _status(q.device).data_ptr(), st), "gated_attn_tiles")
     return out
 
 

@@ -565,7 +565,7 @@ class LLMEngine:
         pos = torch.cat([torch.arange(at, at + n, dtype=torch.int32) for (_, at, _), n in zip(parts, lens)])
         req = torch.cat([torch.full((n,), row, dtype=torch.int32) for (_, _, row), n in zip(parts, lens)])
         want = torch.tensor([o - 1 for o in offs[1:]] if want is None else want, dtype=torch.long)
-        return PromptBatch(ids.to(dev), pos.to(dev), req.to(dev), offs, [p[1] for p in parts], want.to(dev))
+        return PromptBatch(ids.to(dev), pos.to(dev), req.to(dev), offs, [p[1] for p in parts], [p[2] for p in parts], want.to(dev))
 
     def _forward_prompts(self, batch: List[RequestState], hidden: bool = False) -> torch.Tensor:
         """The prompt pass of several new requests at once: their tokens are concatenated, so every projection is one
