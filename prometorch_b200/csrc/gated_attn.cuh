@@ -31,25 +31,31 @@ struct GatedAttnParams {
     int* status;
 };
 
-// cap * tanh(s / cap) without the cancellation of 1 - 2 / (exp + 1) near zero: there, the Taylor series of tanh through x^15
-// (below 0.5 the next term is smaller than 1e-8 of the value).
-__device__ __forceinline__ float soft_cap(float s, float cap, float inv_cap) {
-    const float x = s * inv_cap, ax = fabsf(x);
-    float t;
-    if (ax < 0.5f) {
-        const float u = x * x;
-        float p = -929569.f / 638512875.f;
-        p = fmaf(p, u, 21844.f / 6081075.f);
-        p = fmaf(p, u, -1382.f / 155925.f);
-        p = fmaf(p, u, 62.f / 2835.f);
-        p = fmaf(p, u, -17.f / 315.f);
-        p = fmaf(p, u, 2.f / 15.f);
-        p = fmaf(p, u, -1.f / 3.f);
-        t = fmaf(x * u, p, x);
-    } else {
-        t = copysignf(1.f - __fdividef(2.f, __expf(2.f * fminf(ax, 40.f)) + 1.f), x);
-    }
-    return cap * t;
+// tanh without the cancellation of 1 - 2 / (exp + 1) near zero: there, its Taylor series through x^15 (below 0.5 the next term is
+// smaller than 1e-8 of the value).
+constexpr float TANH_SERIES_MAX = 0.5f;
+__device__ __forceinline__ float tanh_series(float x) {
+    const float u = x * x;
+    float p = -929569.f / 638512875.f;
+    p = fmaf(p, u, 21844.f / 6081075.f);
+    p = fmaf(p, u, -1382.f / 155925.f);
+    p = fmaf(p, u, 62.f / 2835.f);
+    p = fmaf(p, u, -17.f / 315.f);
+    p = fmaf(p, u, 2.f / 15.f);
+    p = fmaf(p, u, -1.f / 3.f);
+    return fmaf(x * u, p, x);
+}
+__device__ __forceinline__ float tanh_any(float x) {
+    const float ax = fabsf(x), e = copysignf(1.f - __fdividef(2.f, __expf(2.f * fminf(ax, 40.f)) + 1.f), x);
+    return ax < TANH_SERIES_MAX ? tanh_series(x) : e;
+}
+__device__ __forceinline__ float soft_cap(float s, float cap, float inv_cap) { return cap * tanh_any(s * inv_cap); }
+// 1 / (1 + 2^z): with z = -s log2(e) the sigmoid of s; 2^z may overflow to infinity, whose reciprocal is 0.
+__device__ __forceinline__ float sigmoid_ex2(float z) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(z));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+    return r;
 }
 __device__ __forceinline__ float sigmoid_w(float s) { return __fdividef(1.f, 1.f + __expf(fminf(-s, 80.f))); }
 

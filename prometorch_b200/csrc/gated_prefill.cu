@@ -71,7 +71,8 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
         }
         reinterpret_cast<uint32_t*>(talk_f)[e] = v;
     }
-    for (int e = threadIdx.x; e < NBUF * BUF / 16; e += W_THREADS) reinterpret_cast<uint4*>(smem)[e] = make_uint4(0, 0, 0, 0);   // chunks past U
+    if (U < NC)                                                        // chunks past U
+        for (int e = threadIdx.x; e < NBUF * BUF / 16; e += W_THREADS) reinterpret_cast<uint4*>(smem)[e] = make_uint4(0, 0, 0, 0);
     __syncthreads();
     pdl_wait();
     pdl_launch_dependents();
@@ -94,6 +95,8 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
     const __nv_bfloat16* q = (const __nv_bfloat16*)A.q + (size_t)(T.tok0 + half) * H * A.Dp;
     const __nv_bfloat16* kp = (const __nv_bfloat16*)A.k_pages;
     const uint4 zero4 = make_uint4(0, 0, 0, 0);
+    // score = y_scale * tanh(x_scale * dot), or scale * dot without a cap
+    const float x_scale = A.scale * A.inv_cap, y_scale = A.cap > 0.f ? A.cap : A.scale;
     auto load_q = [&](int h, int row, int ch) {
         return (h < H && row < nq && ch < nch) ? *reinterpret_cast<const uint4*>(q + ((size_t)row * H + h) * A.Dp + ch * 8) : zero4;
     };
@@ -108,12 +111,26 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
                     qa[hd][s][1] = load_q((warp % U) * 4 + hd, g + 8, 4 * s + t);
                 }
     }
+    // the next eight keys are on their way while the weights of the current ones are formed
+    uint4 kb[KEEP && SAMEC ? KS : 1];
+    auto fetch = [&](int step, int n) {
+        if constexpr (KEEP && SAMEC) {
+            const int j = band.k0 + step * KT + n * 8 + g, col = j / GA_PAGE;
+            const int page = min(max(col < A.pt_stride ? table[col] : 0, 0), A.n_pages - 1);
+            const uint4* kr = reinterpret_cast<const uint4*>(kp + (((size_t)page * A.G + (warp % U) * 4 / R) * GA_PAGE + j % GA_PAGE) * A.Dp);
+#pragma unroll
+            for (int s = 0; s < KS; ++s) kb[s] = 4 * s + t < nch ? kr[4 * s + t] : zero4;
+        }
+    };
+    if (active && s_lo < s_hi) fetch(s_lo, n_lo);
     for (int step = s_lo; step < s_hi; ++step) {
         const int j0 = band.k0 + step * KT;
         unsigned char* buf = smem + (NBUF == 2 ? (step & 1) * BUF : 0);
         // a step no query of this half sees carries zeros
         const bool dead = j0 > q_pos + nq - 1 || j0 + KT - 1 < q_pos - A.window + 1;
-        if (!dead) {
+        if (dead) {
+            if (active && step + 1 < s_hi) fetch(step + 1, n_lo);
+        } else {
             const int col = j0 / GA_PAGE;
             int page = col < A.pt_stride ? table[col] : -1;
             if (page < 0 || page >= A.n_pages) {
@@ -123,9 +140,11 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
             const bool edge = page < 0 || j0 + KT - 1 > q_pos || j0 < q_pos + 15 - A.window + 1 || nq < 16;
             const bool far = q_pos - (j0 + KT - 1) >= A.nb - 1;        // one bias per head
             for (int u = single ? warp % U : warp; active && u < U; u += single ? U : W_WARPS) {
+                const float* bias_u = A.bias + (size_t)u * 4 * A.nb;
+                const int hd_max = min(3, H - 1 - u * 4);              // heads of the unit: 0 .. hd_max
                 float fb[4];
 #pragma unroll
-                for (int hd = 0; hd < 4; ++hd) fb[hd] = __ldg(A.bias + (size_t)min(u * 4 + hd, H - 1) * A.nb + A.nb - 1);
+                for (int hd = 0; hd < 4; ++hd) fb[hd] = __ldg(bias_u + (size_t)min(hd, hd_max) * A.nb + A.nb - 1);
                 for (int n = n_lo; n < n_lo + cols; ++n) {
                     float acc[4][4];
 #pragma unroll
@@ -135,10 +154,6 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
                     const int slot = (j0 + n * 8 + g) % GA_PAGE;
                     auto krow = [&](int c) { return reinterpret_cast<const uint4*>(kp + (((size_t)max(page, 0) * A.G + c) * GA_PAGE + slot) * A.Dp); };
                     if constexpr (KEEP && SAMEC) {
-                        const uint4* kr = krow(u * 4 / R);
-                        uint4 kb[KS];
-#pragma unroll
-                        for (int s = 0; s < KS; ++s) kb[s] = 4 * s + t < nch ? kr[4 * s + t] : zero4;
 #pragma unroll
                         for (int s = 0; s < KS; ++s)
 #pragma unroll
@@ -148,6 +163,8 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
                                 fa::mma16816(acc[hd], f0, kb[s].x, kb[s].y);
                                 fa::mma16816(acc[hd], f1, kb[s].z, kb[s].w);
                             }
+                        if (n + 1 < n_lo + cols) fetch(step, n + 1);
+                        else if (step + 1 < s_hi) fetch(step + 1, n_lo);
                     } else {
                         for (int s = 0; s < ks_rt; ++s) {
                             const int ch = 4 * s + t;
@@ -172,20 +189,39 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
                             }
                         }
                     }
-                    // element e: query g + 8 (e / 2), key n * 8 + 2 t + e % 2
+                    // element e: query g + 8 (e / 2), key n * 8 + 2 t + e % 2.  The arguments of tanh of all sixteen scores are small
+                    // in nearly every case, and then one branch for the warp covers them.
+                    if (A.cap > 0.f) {
+                        float mx = 0.f;
+#pragma unroll
+                        for (int e = 0; e < 4; ++e)
+#pragma unroll
+                            for (int hd = 0; hd < 4; ++hd) { acc[hd][e] *= x_scale; mx = fmaxf(mx, fabsf(acc[hd][e])); }
+                        if (__any_sync(0xffffffffu, mx >= TANH_SERIES_MAX)) {
+#pragma unroll
+                            for (int e = 0; e < 4; ++e)
+#pragma unroll
+                                for (int hd = 0; hd < 4; ++hd) acc[hd][e] = tanh_any(acc[hd][e]);
+                        } else {
+#pragma unroll
+                            for (int e = 0; e < 4; ++e)
+#pragma unroll
+                                for (int hd = 0; hd < 4; ++hd) acc[hd][e] = tanh_series(acc[hd][e]);
+                        }
+                    }
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
                         const int i = g + (e >> 1) * 8, j = n * 8 + 2 * t + (e & 1), dist = q_pos + i - (j0 + j);
                         const bool ok = !edge || (page >= 0 && i < nq && dist >= 0 && dist < A.window);
-                        const int bi = min(max(dist, 0), A.nb - 1);
+                        float b[4] = {fb[0], fb[1], fb[2], fb[3]};
+                        if (!far) {
+                            const int bi = min(max(dist, 0), A.nb - 1);
+#pragma unroll
+                            for (int hd = 0; hd < 4; ++hd) b[hd] = __ldg(bias_u + (size_t)min(hd, hd_max) * A.nb + bi);
+                        }
                         float w[4];
 #pragma unroll
-                        for (int hd = 0; hd < 4; ++hd) {
-                            float s = acc[hd][e] * A.scale;
-                            if (A.cap > 0.f) s = soft_cap(s, A.cap, A.inv_cap);
-                            const float b = far ? fb[hd] : __ldg(A.bias + (size_t)min(u * 4 + hd, H - 1) * A.nb + bi);
-                            w[hd] = ok && u * 4 + hd < H ? sigmoid_w(s + b) : 0.f;
-                        }
+                        for (int hd = 0; hd < 4; ++hd) w[hd] = ok && hd <= hd_max ? sigmoid_ex2(-1.4426950408889634f * fmaf(acc[hd][e], y_scale, b[hd])) : 0.f;
                         uint4 o;
                         o.x = fa::pack_bf16(w[0], w[1]);
                         o.y = fa::pack_bf16(w[2], w[3]);
