@@ -1,4 +1,5 @@
-"""Command-line text generation from a GGUF file (or an Ollama model name).
+"""Command-line text generation from a GGUF file (or an Ollama model name), or from a directory with ``config.json`` and
+safetensors (the models of the batching engine: Hugging Face Llama, Kifusun).
 
     python -m prometorch_b200.generate MODEL [PROMPT] [--device cuda|cpu] [--greedy] [--max-tokens N] [--temp T]
         [--top-k K] [--top-p P] [--chat | --raw] [--info] [--tensors] [--profile] [--nprocs N]
@@ -18,6 +19,43 @@ import os
 import subprocess
 import sys
 import time
+
+
+def _generate_directory(a) -> int:
+    """A model directory: the batching engine (``serve/llm.py``) with one request; bf16 on the GPU, fp32 on the CPU."""
+    import torch
+    from .io.safetensors import load_checkpoint_dir
+    from .models.paged import read_config, resolve_architecture
+    from .serve.llm import GenerationConfig, LLMEngine
+    if a.info or a.tensors:
+        d = read_config(a.model)
+        if a.info:
+            print(f"model = {resolve_architecture(d).name!r}")
+            for k, v in d.items():
+                s = repr(v)
+                print(f"{k} = {s if len(s) < 120 else s[:117] + '...'}")
+        if a.tensors:
+            for name, t in load_checkpoint_dir(a.model).items():
+                print(f"{name:48s} {str(tuple(t.shape)):24s} {str(t.dtype).replace('torch.', ''):9s} {t.numel() * t.element_size()} B")
+        return 0
+    if a.nprocs > 1:
+        raise SystemExit("--nprocs: model directories run on one device")
+    use_cuda = (a.device in ("cuda", "gpu") or a.cuda) and torch.cuda.is_available()
+    t0 = time.time()
+    eng = LLMEngine(device="cuda" if use_cuda else "cpu", max_pages=256, max_active=1)
+    if not eng.load(a.model) or not eng.loaded:
+        raise SystemExit(f"{a.model}: no weights beside config.json")
+    print(f"[Model] {eng.model.architecture}, {eng.weights.num_parameters() / 1e6:.1f} M parameters, loaded in {time.time() - t0:.1f} s "
+          f"on {'CUDA' if use_cuda else 'CPU'}")
+    cfg = GenerationConfig(max_new_tokens=a.max_tokens, temperature=a.temp, top_k=a.top_k, top_p=a.top_p, repetition_penalty=a.repeat_penalty)
+    t1, n = time.time(), 0
+    for t in eng.stream(a.prompt if a.prompt is not None else "Hello, how are you?", cfg):
+        sys.stdout.write(eng.tokenizer.decode([t]))
+        sys.stdout.flush()
+        n += 1
+    dt = time.time() - t1
+    print(f"\n\n[Generate] {n} tokens in {dt:.2f}s ({n / max(dt, 1e-9):.1f} tok/s, prompt included)")
+    return 0
 
 
 def main(argv=None) -> int:
@@ -47,6 +85,10 @@ def main(argv=None) -> int:
     ap.add_argument("--master-addr", "--master_addr", default="127.0.0.1")
     ap.add_argument("--master-port", "--master_port", type=int, default=29500)
     a = ap.parse_args(argv)
+    if os.path.isfile(os.path.join(a.model, "config.json")):
+        if a.greedy:
+            a.temp, a.repeat_penalty = 0.0, 1.0
+        return _generate_directory(a)
     from .io.config import TransformerConfig
     from .io.gguf import GGUFReader
     from .io.ollama import resolve_model
