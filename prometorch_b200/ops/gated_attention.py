@@ -129,8 +129,8 @@ def head_norm_write(qkv: torch.Tensor, a: GatedAttention, q_weight: torch.Tensor
     q[..., :D] = norm(qs, q_weight).to(q.dtype)
     p = pos.long()
     pages = page_table[req.long(), p // PAGE].long()
-    k_pages[pages, :, p % PAGE, :D] = norm(ks, k_weight).to(k_pages.dtype)
-    v_pages[pages, :, p % PAGE, :Dv] = v.to(v_pages.dtype)
+    k_pages[pages, :, p % PAGE] = torch.nn.functional.pad(norm(ks, k_weight), (0, Dp - D)).to(k_pages.dtype)
+    v_pages[pages, :, p % PAGE] = torch.nn.functional.pad(v, (0, Dvp - Dv)).to(v_pages.dtype)
     return q
 
 
