@@ -19,6 +19,7 @@ namespace gp {
 
 constexpr int QT = 32;                 // queries per tile
 constexpr int KT = 32;                 // keys per step of the weights kernel
+constexpr float LOG2E = 1.4426950408889634f;
 constexpr int W_THREADS = 256, W_WARPS = 8;
 
 struct Tile { int tok0, pos0, count, req; };       // rows [tok0, tok0 + count) stand at pos0.. of the sequence in page-table row req
@@ -36,10 +37,10 @@ struct WeightsParams {
     GatedAttnParams A;
     const Tile* tiles;
     __nv_bfloat16* P;                  // [tiles][H][32][KW]
-    int KW, splits;
+    int KW, per;                       // key steps per CTA
 };
 
-// One CTA: 16 queries (half a tile) x the 32-key steps of its split, all heads.  A warp owns "units" of four consecutive heads.
+// One CTA: 16 queries (half a tile) x at most `per` 32-key steps, all heads.  A warp owns "units" of four consecutive heads.
 // Weights of a step in shared memory: row (query i, key j), 16-byte chunk per unit = {4 heads' high parts, 4 heads' low parts},
 // chunks XOR-swizzled so that both the stores below and ldmatrix spread over the banks.
 __device__ __forceinline__ uint32_t w_off(int i, int j, int chunk, int NC) {
@@ -80,8 +81,8 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
     const int half = blockIdx.y * 16;
     if (half >= T.count) return;
     const Band band = band_of(T, A.window);
-    const int steps = band.blocks * 2, per = (steps + P.splits - 1) / P.splits;
-    const int s_lo = blockIdx.z * per, s_hi = min(s_lo + per, steps);
+    const int steps = band.blocks * 2, s_lo = blockIdx.z * P.per, s_hi = min(s_lo + P.per, steps);
+    if (s_lo >= s_hi) return;
     const int nq = min(16, T.count - half), q_pos = T.pos0 + half;     // queries q_pos .. q_pos + nq - 1
     const int* table = A.page_table + (size_t)T.req * A.pt_stride;
     __nv_bfloat16* Pt = P.P + ((size_t)blockIdx.x * H * QT + half) * P.KW;
@@ -95,8 +96,16 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
     const __nv_bfloat16* q = (const __nv_bfloat16*)A.q + (size_t)(T.tok0 + half) * H * A.Dp;
     const __nv_bfloat16* kp = (const __nv_bfloat16*)A.k_pages;
     const uint4 zero4 = make_uint4(0, 0, 0, 0);
-    // score = y_scale * tanh(x_scale * dot), or scale * dot without a cap
-    const float x_scale = A.scale * A.inv_cap, y_scale = A.cap > 0.f ? A.cap : A.scale;
+    // -log2(e) cap tanh(x) = d (cf0 + cf1 d^2 + ...) with x = scale d / cap: the Taylor series of tanh through x^11, whose next term
+    // is below 2e-7 of the value for |x| < 0.4.  Without a cap, cf0 alone.
+    float cf[6];
+    const float xs = A.cap > 0.f ? A.scale * A.inv_cap : A.scale, dot_max = 0.4f / fabsf(xs);
+    {
+        const float a[6] = {1.f, -1.f / 3.f, 2.f / 15.f, -17.f / 315.f, 62.f / 2835.f, -1382.f / 155925.f};
+        float m = -LOG2E * (A.cap > 0.f ? A.cap : 1.f) * xs;
+#pragma unroll
+        for (int k = 0; k < 6; ++k) { cf[k] = a[k] * m; m *= xs * xs; }
+    }
     auto load_q = [&](int h, int row, int ch) {
         return (h < H && row < nq && ch < nch) ? *reinterpret_cast<const uint4*>(q + ((size_t)row * H + h) * A.Dp + ch * 8) : zero4;
     };
@@ -144,7 +153,7 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
                 const int hd_max = min(3, H - 1 - u * 4);              // heads of the unit: 0 .. hd_max
                 float fb[4];
 #pragma unroll
-                for (int hd = 0; hd < 4; ++hd) fb[hd] = __ldg(bias_u + (size_t)min(hd, hd_max) * A.nb + A.nb - 1);
+                for (int hd = 0; hd < 4; ++hd) fb[hd] = -LOG2E * __ldg(bias_u + (size_t)min(hd, hd_max) * A.nb + A.nb - 1);
                 for (int n = n_lo; n < n_lo + cols; ++n) {
                     float acc[4][4];
 #pragma unroll
@@ -189,46 +198,70 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
                             }
                         }
                     }
-                    // element e: query g + 8 (e / 2), key n * 8 + 2 t + e % 2.  The arguments of tanh of all sixteen scores are small
-                    // in nearly every case, and then one branch for the warp covers them.
+                    // element e: query g + 8 (e / 2), key n * 8 + 2 t + e % 2.  acc becomes -log2(e) times the capped, scaled score:
+                    // as a rule every |x| of the warp is small and an odd polynomial in the dot product itself is enough.
                     if (A.cap > 0.f) {
                         float mx = 0.f;
 #pragma unroll
-                        for (int e = 0; e < 4; ++e)
+                        for (int hd = 0; hd < 4; ++hd)
 #pragma unroll
-                            for (int hd = 0; hd < 4; ++hd) { acc[hd][e] *= x_scale; mx = fmaxf(mx, fabsf(acc[hd][e])); }
-                        if (__any_sync(0xffffffffu, mx >= TANH_SERIES_MAX)) {
+                            for (int e = 0; e < 4; ++e) mx = fmaxf(mx, fabsf(acc[hd][e]));
+                        if (__any_sync(0xffffffffu, mx >= dot_max)) {
 #pragma unroll
-                            for (int e = 0; e < 4; ++e)
+                            for (int hd = 0; hd < 4; ++hd)
 #pragma unroll
-                                for (int hd = 0; hd < 4; ++hd) acc[hd][e] = tanh_any(acc[hd][e]);
+                                for (int e = 0; e < 4; ++e) acc[hd][e] = -LOG2E * A.cap * tanh_any(acc[hd][e] * xs);
                         } else {
 #pragma unroll
-                            for (int e = 0; e < 4; ++e)
+                            for (int hd = 0; hd < 4; ++hd)
 #pragma unroll
-                                for (int hd = 0; hd < 4; ++hd) acc[hd][e] = tanh_series(acc[hd][e]);
+                                for (int e = 0; e < 4; ++e) {
+                                    const float d = acc[hd][e], v = d * d;
+                                    acc[hd][e] = d * fmaf(fmaf(fmaf(fmaf(fmaf(cf[5], v, cf[4]), v, cf[3]), v, cf[2]), v, cf[1]), v, cf[0]);
+                                }
+                        }
+                    } else {
+#pragma unroll
+                        for (int hd = 0; hd < 4; ++hd)
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) acc[hd][e] *= cf[0];
+                    }
+                    if (far) {
+#pragma unroll
+                        for (int hd = 0; hd < 4; ++hd)
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) acc[hd][e] = sigmoid_ex2(acc[hd][e] + fb[hd]);
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            const int bi = min(max(q_pos + g + (e >> 1) * 8 - (j0 + n * 8 + 2 * t + (e & 1)), 0), A.nb - 1);
+#pragma unroll
+                            for (int hd = 0; hd < 4; ++hd)
+                                acc[hd][e] = sigmoid_ex2(fmaf(-LOG2E, __ldg(bias_u + (size_t)min(hd, hd_max) * A.nb + bi), acc[hd][e]));
+                        }
+                    }
+                    if (edge) {
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            const int i = g + (e >> 1) * 8, dist = q_pos + i - (j0 + n * 8 + 2 * t + (e & 1));
+                            const bool ok = page >= 0 && i < nq && dist >= 0 && dist < A.window;
+#pragma unroll
+                            for (int hd = 0; hd < 4; ++hd) acc[hd][e] = ok ? acc[hd][e] : 0.f;
                         }
                     }
 #pragma unroll
+                    for (int hd = 1; hd < 4; ++hd)
+                        if (hd > hd_max)
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) acc[hd][e] = 0.f;
+#pragma unroll
                     for (int e = 0; e < 4; ++e) {
-                        const int i = g + (e >> 1) * 8, j = n * 8 + 2 * t + (e & 1), dist = q_pos + i - (j0 + j);
-                        const bool ok = !edge || (page >= 0 && i < nq && dist >= 0 && dist < A.window);
-                        float b[4] = {fb[0], fb[1], fb[2], fb[3]};
-                        if (!far) {
-                            const int bi = min(max(dist, 0), A.nb - 1);
-#pragma unroll
-                            for (int hd = 0; hd < 4; ++hd) b[hd] = __ldg(bias_u + (size_t)min(hd, hd_max) * A.nb + bi);
-                        }
-                        float w[4];
-#pragma unroll
-                        for (int hd = 0; hd < 4; ++hd) w[hd] = ok && hd <= hd_max ? sigmoid_ex2(-1.4426950408889634f * fmaf(acc[hd][e], y_scale, b[hd])) : 0.f;
+                        const int i = g + (e >> 1) * 8, j = n * 8 + 2 * t + (e & 1);
                         uint4 o;
-                        o.x = fa::pack_bf16(w[0], w[1]);
-                        o.y = fa::pack_bf16(w[2], w[3]);
-                        const float2 h0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&o.x));
-                        const float2 h1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&o.y));
-                        o.z = fa::pack_bf16(w[0] - h0.x, w[1] - h0.y);
-                        o.w = fa::pack_bf16(w[2] - h1.x, w[3] - h1.y);
+                        o.x = fa::pack_bf16(acc[0][e], acc[1][e]);
+                        o.y = fa::pack_bf16(acc[2][e], acc[3][e]);
+                        o.z = fa::pack_bf16(acc[0][e] - __uint_as_float(o.x << 16), acc[1][e] - __uint_as_float(o.x & 0xffff0000u));
+                        o.w = fa::pack_bf16(acc[2][e] - __uint_as_float(o.y << 16), acc[3][e] - __uint_as_float(o.y & 0xffff0000u));
                         *reinterpret_cast<uint4*>(buf + w_off(i, j, u, NC)) = o;
                     }
                 }
@@ -432,7 +465,7 @@ static int launch_weights(const WeightsParams& p, int tiles, cudaStream_t st) {
         PTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
         attr = true;
     }
-    PTB_CUDA_OK(ptb_launch(kern, dim3(tiles, 2, p.splits), dim3(W_THREADS), (size_t)smem, st, ptb_pdl_enabled(), p));
+    PTB_CUDA_OK(ptb_launch(kern, dim3(tiles, 2, (p.KW / KT + p.per - 1) / p.per), dim3(W_THREADS), (size_t)smem, st, ptb_pdl_enabled(), p));
     return 0;
 }
 template <int KS, bool KEEP, bool SAMEC>
@@ -469,14 +502,14 @@ PTB_API int ptb_gated_tiles_supported(int H, int G, int Dp, int Dvp) {
 
 // Query tiles of a prompt pass, bf16.  tiles: [n_tiles][4] int32 on the device: first row of q / out, its position, rows (<= 32), row
 // of the page table; a tile's rows stand at consecutive positions of one sequence whose keys and values are in the pages.
-// weights: scratch of n_tiles * H * 32 * KW bf16, KW (a multiple of 64) at least 64 times the most 64-key blocks a tile sees.
+// weights: scratch of n_tiles * H * 32 * KW bf16, KW (a multiple of 64) at least 64 times the most 64-key blocks a tile sees; per: 32-key steps a CTA of the weights kernel takes.
 // q [n, H, Dp], out [n, H Dv].
 PTB_API int ptb_gated_attn_tiles(const void* q, void* out, const int* tiles, int n_tiles, int H, int G, int Dp, int Dv, int Dvp,
                                  const int* page_table, int pt_stride, int n_pages, const void* k_pages, const void* v_pages, const float* bias,
-                                 int nb, const float* talk, int window, float scale, float cap, void* weights, int KW, int splits, int* status,
+                                 int nb, const float* talk, int window, float scale, float cap, void* weights, int KW, int per, int* status,
                                  cudaStream_t st) {
     if (n_tiles <= 0) return 0;
-    if (!ptb_gated_tiles_supported(H, G, Dp, Dvp) || nb < 1 || window < 1 || KW % 64 || splits < 1 || n_tiles > 65535) {
+    if (!ptb_gated_tiles_supported(H, G, Dp, Dvp) || nb < 1 || window < 1 || KW % 64 || per < 1 || n_tiles > 65535) {
         ptb_set_error("gated attention tiles: bad sizes (H %d, G %d, Dp %d, Dvp %d, KW %d, tiles %d)", H, G, Dp, Dvp, KW, n_tiles);
         return -1;
     }
@@ -485,7 +518,7 @@ PTB_API int ptb_gated_attn_tiles(const void* q, void* out, const int* tiles, int
     w.A.q = q; w.A.page_table = page_table; w.A.k_pages = k_pages; w.A.bias = bias; w.A.talk = talk; w.A.pt_stride = pt_stride; w.A.n_pages = n_pages;
     w.A.H = H; w.A.G = G; w.A.Dp = Dp; w.A.nb = nb; w.A.window = window; w.A.scale = scale; w.A.cap = cap; w.A.inv_cap = cap > 0.f ? 1.f / cap : 0.f;
     w.A.status = status;
-    w.tiles = (const gp::Tile*)tiles; w.P = (__nv_bfloat16*)weights; w.KW = KW; w.splits = splits;
+    w.tiles = (const gp::Tile*)tiles; w.P = (__nv_bfloat16*)weights; w.KW = KW; w.per = per;
     const int R = H / G, ks = (Dp + 31) / 32;
     const bool same = R % 4 == 0;
     int rc;

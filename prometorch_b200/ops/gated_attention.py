@@ -171,7 +171,8 @@ def gated_attention(q: torch.Tensor, a: GatedAttention, pos: torch.Tensor, req: 
 
 QUERY_TILE = 32                        # queries per tile of csrc/gated_prefill.cu
 TILES_FROM = 64                        # rows of a prompt pass from which the tile kernels are the better choice
-WEIGHTS_BYTES = 96 << 20               # scratch of the tile kernels per launch: it should stay in L2 between the two of them
+STEPS_PER_CTA = 9                      # 32-key steps of one CTA: short enough to balance bands of different lengths
+WEIGHTS_BYTES = 320 << 20              # scratch of the tile kernels per launch
 
 
 @dataclass
@@ -196,13 +197,8 @@ def tiles_supported(q: torch.Tensor, a: GatedAttention) -> bool:
     return q.is_cuda and q.dtype == torch.bfloat16 and bool(N.lib().ptb_gated_tiles_supported(a.heads, a.kv_heads, a.dim_stored, a.vdim_stored))
 
 
-def _tile_splits(halves: int, steps: int, sms: int) -> int:
-    """CTAs (one per SM) that share a half tile's key steps: the count with the shortest makespan, a CTA's start costing two steps."""
-    return min(range(1, max(1, min(steps, 16)) + 1), key=lambda s: (-(-halves * s // sms) * (-(-steps // s) + 2), s))
-
-
 def gated_attention_tiles(q: torch.Tensor, a: GatedAttention, tiles: PromptTiles, page_table: torch.Tensor, k_pages: torch.Tensor,
-                          v_pages: torch.Tensor, sms: int = 148) -> torch.Tensor:
+                          v_pages: torch.Tensor) -> torch.Tensor:
     """A prompt pass's rows against the pages, on the tensor cores (sizes: :func:`tiles_supported`)."""
     H, n, nt = a.heads, q.shape[0], len(tiles.host)
     out = torch.empty(n, H * a.vdim, dtype=q.dtype, device=q.device)
@@ -213,11 +209,10 @@ def gated_attention_tiles(q: torch.Tensor, a: GatedAttention, tiles: PromptTiles
     st = torch.cuda.current_stream(q.device).cuda_stream
     for lo in range(0, nt, step):
         m = min(step, nt - lo)
-        splits = _tile_splits(2 * m, KW // QUERY_TILE, sms)
         N.check(N.lib().ptb_gated_attn_tiles(q.data_ptr(), out.data_ptr(), tiles.device[lo:].data_ptr(), m, H, a.kv_heads, a.dim_stored, a.vdim,
                                              a.vdim_stored, page_table.data_ptr(), page_table.stride(0), k_pages.shape[0], k_pages.data_ptr(),
                                              v_pages.data_ptr(), a.bias.data_ptr(), a.bias.shape[1], N.ptr(a.talk), a.window, float(a.scale),
-                                             float(a.softcap), weights.data_ptr(), KW, splits, _status(q.device).data_ptr(), st), "gated_attn_tiles")
+                                             float(a.softcap), weights.data_ptr(), KW, STEPS_PER_CTA, _status(q.device).data_ptr(), st), "gated_attn_tiles")
     return out
 
 
