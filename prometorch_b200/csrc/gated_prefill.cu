@@ -13,6 +13,7 @@
 #include <algorithm>
 
 int ptb_make_tmap_bf16(CUtensorMap* map, const void* base, long long inner, long long outer, long long ld, int box_inner, int box_outer);
+int ptb_make_tmap_bf16_3d(CUtensorMap* map, const void* base, long long n0, long long n1, long long n2, int b0, int b1, int b2);
 
 namespace ptb {
 namespace gp {
@@ -31,6 +32,15 @@ __host__ __device__ __forceinline__ Band band_of(const Tile& t, int window) {
     b.k0 = (lo > 0 ? lo : 0) / 64 * 64;
     b.blocks = (t.pos0 + t.count - b.k0 + 63) / 64;
     return b;
+}
+
+// -log2(e) cap tanh(x) = d (cf0 + cf1 d^2 + ...) with x = xs d: the Taylor series of tanh through x^11, whose next term is below 2e-7
+// of the value for |x| < 0.4.  Without a cap, cf0 alone.
+__device__ __forceinline__ void tanh_poly(const GatedAttnParams& A, float xs, float* cf) {
+    const float a[6] = {1.f, -1.f / 3.f, 2.f / 15.f, -17.f / 315.f, 62.f / 2835.f, -1382.f / 155925.f};
+    float m = -LOG2E * (A.cap > 0.f ? A.cap : 1.f) * xs;
+#pragma unroll
+    for (int k = 0; k < 6; ++k) { cf[k] = a[k] * m; m *= xs * xs; }
 }
 
 struct WeightsParams {
@@ -96,16 +106,9 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
     const __nv_bfloat16* q = (const __nv_bfloat16*)A.q + (size_t)(T.tok0 + half) * H * A.Dp;
     const __nv_bfloat16* kp = (const __nv_bfloat16*)A.k_pages;
     const uint4 zero4 = make_uint4(0, 0, 0, 0);
-    // -log2(e) cap tanh(x) = d (cf0 + cf1 d^2 + ...) with x = scale d / cap: the Taylor series of tanh through x^11, whose next term
-    // is below 2e-7 of the value for |x| < 0.4.  Without a cap, cf0 alone.
     float cf[6];
     const float xs = A.cap > 0.f ? A.scale * A.inv_cap : A.scale, dot_max = 0.4f / fabsf(xs);
-    {
-        const float a[6] = {1.f, -1.f / 3.f, 2.f / 15.f, -17.f / 315.f, 62.f / 2835.f, -1382.f / 155925.f};
-        float m = -LOG2E * (A.cap > 0.f ? A.cap : 1.f) * xs;
-#pragma unroll
-        for (int k = 0; k < 6; ++k) { cf[k] = a[k] * m; m *= xs * xs; }
-    }
+    tanh_poly(A, xs, cf);
     auto load_q = [&](int h, int row, int ch) {
         return (h < H && row < nq && ch < nch) ? *reinterpret_cast<const uint4*>(q + ((size_t)row * H + h) * A.Dp + ch * 8) : zero4;
     };
@@ -335,6 +338,14 @@ __global__ void __launch_bounds__(W_THREADS, 1) gated_weights_kernel(const __gri
     }
 }
 
+}  // namespace gp
+}  // namespace ptb
+
+#include "gated_weights_sm100.cuh"
+
+namespace ptb {
+namespace gp {
+
 // ---------------------------------------------------------------------------------------------- O = P V
 constexpr int V_THREADS = 192, V_STAGES = 3;
 
@@ -503,10 +514,11 @@ PTB_API int ptb_gated_tiles_supported(int H, int G, int Dp, int Dvp) {
 // Query tiles of a prompt pass, bf16.  tiles: [n_tiles][4] int32 on the device: first row of q / out, its position, rows (<= 32), row
 // of the page table; a tile's rows stand at consecutive positions of one sequence whose keys and values are in the pages.
 // weights: scratch of n_tiles * H * 32 * KW bf16, KW (a multiple of 64) at least 64 times the most 64-key blocks a tile sees; per: 32-key steps a CTA of the weights kernel takes.
-// q [n, H, Dp], out [n, H Dv].
-PTB_API int ptb_gated_attn_tiles(const void* q, void* out, const int* tiles, int n_tiles, int H, int G, int Dp, int Dv, int Dvp,
+// tensor_cores: 1 takes the tcgen05 weights kernel where it fits, 0 the mma.sync one.
+// q [n_rows, H, Dp], out [n_rows, H Dv].
+PTB_API int ptb_gated_attn_tiles(const void* q, void* out, int n_rows, const int* tiles, int n_tiles, int H, int G, int Dp, int Dv, int Dvp,
                                  const int* page_table, int pt_stride, int n_pages, const void* k_pages, const void* v_pages, const float* bias,
-                                 int nb, const float* talk, int window, float scale, float cap, void* weights, int KW, int per, int* status,
+                                 int nb, const float* talk, int window, float scale, float cap, void* weights, int KW, int per, int tensor_cores, int* status,
                                  cudaStream_t st) {
     if (n_tiles <= 0) return 0;
     if (!ptb_gated_tiles_supported(H, G, Dp, Dvp) || nb < 1 || window < 1 || KW % 64 || per < 1 || n_tiles > 65535) {
@@ -522,7 +534,8 @@ PTB_API int ptb_gated_attn_tiles(const void* q, void* out, const int* tiles, int
     const int R = H / G, ks = (Dp + 31) / 32;
     const bool same = R % 4 == 0;
     int rc;
-    if (H > 32 || ks > 4) rc = gp::launch_weights_nk<1, false, false>(w, n_tiles, st);
+    if (tensor_cores && gp::tc_supported(w.A)) rc = gp::launch_tc_any(w, n_tiles, n_rows, std::max(1, per / 4), st);
+    else if (H > 32 || ks > 4) rc = gp::launch_weights_nk<1, false, false>(w, n_tiles, st);
     else if (!same) rc = ks <= 2 ? gp::launch_weights_nk<2, true, false>(w, n_tiles, st) : gp::launch_weights_nk<4, true, false>(w, n_tiles, st);
     else if (ks <= 2) rc = gp::launch_weights_nk<2, true, true>(w, n_tiles, st);
     else if (ks == 3) rc = gp::launch_weights_nk<3, true, true>(w, n_tiles, st);

@@ -42,6 +42,21 @@ int ptb_make_tmap_bf16(CUtensorMap* map, const void* base, long long inner, long
     return 0;
 }
 
+// 3-D bf16 tensor map of a contiguous [n2][n1][n0] tensor (n0 fastest); box sizes per dimension.
+int ptb_make_tmap_bf16_3d(CUtensorMap* map, const void* base, long long n0, long long n1, long long n2, int b0, int b1, int b2) {
+    EncodeTiledFn enc = get_encode();
+    if (!enc) { ptb_set_error("cuTensorMapEncodeTiled is not available (no CUDA driver?)"); return -1; }
+    if (((uintptr_t)base & 15) || ((n0 * 2) & 15)) { ptb_set_error("TMA operand needs a 16-byte aligned base and row pitch (n0=%lld)", n0); return -1; }
+    cuuint64_t dims[3] = {(cuuint64_t)n0, (cuuint64_t)n1, (cuuint64_t)n2};
+    cuuint64_t strides[2] = {(cuuint64_t)n0 * 2, (cuuint64_t)n0 * n1 * 2};
+    cuuint32_t box[3] = {(cuuint32_t)b0, (cuuint32_t)b1, (cuuint32_t)b2};
+    cuuint32_t estr[3] = {1, 1, 1};
+    CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) { ptb_set_error("cuTensorMapEncodeTiled failed with code %d", (int)r); return -1; }
+    return 0;
+}
+
 template <int BN, int STAGES, bool A_MN, bool B_MN>
 static int launch(const Operand& ta, const Operand& tb, const Params& p, int n_sm, cudaStream_t st) {
     auto kern = gemm_bf16_kernel<BN, STAGES, A_MN, B_MN>;

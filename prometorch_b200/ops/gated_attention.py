@@ -29,7 +29,7 @@ def _decls(L):
     L.ptb_gated_attn_rows.restype = ci
     L.ptb_gated_tiles_supported.argtypes = [ci, ci, ci, ci]
     L.ptb_gated_tiles_supported.restype = ci
-    L.ptb_gated_attn_tiles.argtypes = [vp, vp, vp, ci, ci, ci, ci, ci, ci, vp, ci, ci, vp, vp, vp, ci, vp, ci, cf, cf, vp, ci, ci, vp, vp]
+    L.ptb_gated_attn_tiles.argtypes = [vp, vp, ci, vp, ci, ci, ci, ci, ci, ci, vp, ci, ci, vp, vp, vp, ci, vp, ci, cf, cf, vp, ci, ci, ci, vp, vp]
     L.ptb_gated_attn_tiles.restype = ci
 
 
@@ -198,8 +198,9 @@ def tiles_supported(q: torch.Tensor, a: GatedAttention) -> bool:
 
 
 def gated_attention_tiles(q: torch.Tensor, a: GatedAttention, tiles: PromptTiles, page_table: torch.Tensor, k_pages: torch.Tensor,
-                          v_pages: torch.Tensor) -> torch.Tensor:
-    """A prompt pass's rows against the pages, on the tensor cores (sizes: :func:`tiles_supported`)."""
+                          v_pages: torch.Tensor, tensor_cores: bool = True) -> torch.Tensor:
+    """A prompt pass's rows against the pages, on the tensor cores (sizes: :func:`tiles_supported`).  ``tensor_cores``: the
+    scores and the head mixing on tcgen05 where its kernel takes the sizes, else on mma.sync."""
     H, n, nt = a.heads, q.shape[0], len(tiles.host)
     out = torch.empty(n, H * a.vdim, dtype=q.dtype, device=q.device)
     KW = tiles.width(a.window)
@@ -209,10 +210,10 @@ def gated_attention_tiles(q: torch.Tensor, a: GatedAttention, tiles: PromptTiles
     st = torch.cuda.current_stream(q.device).cuda_stream
     for lo in range(0, nt, step):
         m = min(step, nt - lo)
-        N.check(N.lib().ptb_gated_attn_tiles(q.data_ptr(), out.data_ptr(), tiles.device[lo:].data_ptr(), m, H, a.kv_heads, a.dim_stored, a.vdim,
+        N.check(N.lib().ptb_gated_attn_tiles(q.data_ptr(), out.data_ptr(), n, tiles.device[lo:].data_ptr(), m, H, a.kv_heads, a.dim_stored, a.vdim,
                                              a.vdim_stored, page_table.data_ptr(), page_table.stride(0), k_pages.shape[0], k_pages.data_ptr(),
                                              v_pages.data_ptr(), a.bias.data_ptr(), a.bias.shape[1], N.ptr(a.talk), a.window, float(a.scale),
-                                             float(a.softcap), weights.data_ptr(), KW, STEPS_PER_CTA, _status(q.device).data_ptr(), st), "gated_attn_tiles")
+                                             float(a.softcap), weights.data_ptr(), KW, STEPS_PER_CTA, int(tensor_cores), _status(q.device).data_ptr(), st), "gated_attn_tiles")
     return out
 
 

@@ -63,7 +63,10 @@ SHAPES = [dict(H=8, G=2, D=128, Dv=128, W=100, lens=[200, 300], starts=[0, 0]), 
           dict(H=12, G=12, D=64, Dv=64, W=33, lens=[90, 64], starts=[0, 1]), dict(H=5, G=1, D=80, Dv=100, W=50, lens=[90, 64], starts=[0, 1], talk=False),
           dict(H=40, G=8, D=64, Dv=128, W=90, lens=[90, 64], starts=[0, 1]), dict(H=64, G=8, D=96, Dv=96, W=90, lens=[120], starts=[0], cap=0.0),
           dict(H=8, G=4, D=256, Dv=256, W=90, lens=[120], starts=[3]), dict(H=3, G=3, D=16, Dv=64, W=1, lens=[70], starts=[0]),
-          dict(H=7, G=7, D=20, Dv=72, W=300, lens=[270], starts=[10]), dict(H=9, G=1, D=24, Dv=12, W=200, lens=[70], starts=[129])]
+          dict(H=7, G=7, D=20, Dv=72, W=300, lens=[270], starts=[10]), dict(H=9, G=1, D=24, Dv=12, W=200, lens=[70], starts=[129]),
+          dict(H=16, G=1, D=64, Dv=64, W=150, lens=[75, 33], starts=[300, 0]), dict(H=32, G=1, D=80, Dv=64, W=40, lens=[97], starts=[64]),
+          dict(H=8, G=4, D=96, Dv=64, W=257, lens=[300, 9], starts=[0, 257]), dict(H=24, G=6, D=128, Dv=64, W=500, lens=[200], starts=[450]),
+          dict(H=28, G=14, D=64, Dv=128, W=70, lens=[130], starts=[7], cap=0.0)]
 
 
 @pytest.mark.parametrize("shape", SHAPES, ids=lambda s: "h{H}g{G}d{D}v{Dv}w{W}".format(**s))
@@ -77,7 +80,8 @@ def test_attention_kernels(shape):
         assert rel(A.gated_attention(q, a, pos, req, table, k, v, splits, top), ref) < 4e-3
     if A.tiles_supported(q, a):
         tiles = A.PromptTiles.of(offs, shape["starts"], list(range(len(offs) - 1)), "cuda")
-        assert rel(A.gated_attention_tiles(q, a, tiles, table, k, v), ref) < 5e-3
+        for tc in (True, False):
+            assert rel(A.gated_attention_tiles(q, a, tiles, table, k, v, tensor_cores=tc), ref) < 5e-3
     P.check_status("cuda")
 
 
@@ -90,7 +94,8 @@ def test_large_scores(big):
     ref = A.gated_attention_reference(q.float(), a, pos, req, table, k.float(), v.float())
     assert rel(A.gated_attention(q.float(), a, pos, req, table, k.float(), v.float(), 1, 130), ref) < 2e-6
     assert rel(A.gated_attention(q, a, pos, req, table, k, v, 1, 130), ref) < 4e-3
-    assert rel(A.gated_attention_tiles(q, a, A.PromptTiles.of(offs, [0], [0], "cuda"), table, k, v), ref) < 5e-3
+    for tc in (True, False):
+        assert rel(A.gated_attention_tiles(q, a, A.PromptTiles.of(offs, [0], [0], "cuda"), table, k, v, tensor_cores=tc), ref) < 5e-3
 
 
 @pytest.mark.parametrize("W", [31, 32, 33, 64, 65, 128])
@@ -102,7 +107,8 @@ def test_window_edges(W):
     for j in (0, 31, 32, 63, 64, 100):
         v2 = v.clone()
         v2[table[0, j // 64], :, j % 64] += 200.0
-        for run in (lambda x: A.gated_attention(q, a, pos, req, table, k, x, 2, 230), lambda x: A.gated_attention_tiles(q, a, tiles, table, k, x)):
+        for run in (lambda x: A.gated_attention(q, a, pos, req, table, k, x, 2, 230), lambda x: A.gated_attention_tiles(q, a, tiles, table, k, x),
+                    lambda x: A.gated_attention_tiles(q, a, tiles, table, k, x, tensor_cores=False)):
             d = (run(v2).float() - run(v).float()).abs().amax(1)
             assert (d > 0.05).nonzero()[:, 0].tolist() == list(range(j, min(230, j + W)))
 
