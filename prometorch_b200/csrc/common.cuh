@@ -78,6 +78,18 @@ __device__ __forceinline__ bool mbar_try_wait(uint64_t* bar, uint32_t parity) {
         : "memory");
     return ok != 0;
 }
+// The same question without the hardware's suspension: for a thread that watches several barriers.
+__device__ __forceinline__ bool mbar_test_wait(uint64_t* bar, uint32_t parity) {
+    uint32_t ok;
+    asm volatile(
+        "{\n .reg .pred p;\n"
+        " mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n"
+        " selp.u32 %0, 1, 0, p;\n}"
+        : "=r"(ok)
+        : "r"(smem_u32(bar)), "r"(parity)
+        : "memory");
+    return ok != 0;
+}
 // Bounded wait.  Returns false (and records PTB_ERR_MBARRIER_TIMEOUT) if the phase did not complete within
 // `budget_ns` of wall-clock time (%globaltimer, read every 256 polls, so the budget does not depend on the SM clock).
 __device__ __forceinline__ bool mbar_wait(uint64_t* bar, uint32_t parity, int* status, uint64_t budget_ns = 2000000000ull) {

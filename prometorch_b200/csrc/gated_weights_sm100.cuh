@@ -137,7 +137,7 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
             mbar_expect_tx(q_full, (uint32_t)(H * NQ * chunks * 128));
             for (int c = 0; c < G; ++c)
                 for (int ch = 0; ch < chunks; ++ch) tma_load_3d(smem + (size_t)(c * chunks + ch) * N * 128, &tmQ, ch * 64, c * R, T.tok0 + q0, q_full);
-            int it = 0;
+            int s = 0, round = 0;
             for (int kt = 0; kt < nt && ok; ++kt) {
                 int page[2];
                 for (int b = 0; b < 2; ++b) {
@@ -149,12 +149,12 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
                     }
                 }
                 for (int c = 0; c < G && ok; ++c)
-                    for (int ch = 0; ch < chunks && ok; ++ch, ++it) {
-                        const int s = it % T_STAGES;
-                        if (it >= T_STAGES) ok = mbar_wait(&k_empty[s], (uint32_t)((it / T_STAGES - 1) & 1), A.status);
+                    for (int ch = 0; ch < chunks && ok; ++ch) {
+                        if (round > 0) ok = mbar_wait(&k_empty[s], (uint32_t)((round - 1) & 1), A.status);
                         if (!ok || *abort_flag) { ok = false; break; }
                         mbar_expect_tx(&k_full[s], 16384);
                         for (int b = 0; b < 2; ++b) tma_load_2d(sk + s * 16384 + b * 8192, &tmK, ch * 64, (page[b] * G + c) * GA_PAGE, &k_full[s]);
+                        if (++s == T_STAGES) { s = 0; ++round; }
                     }
             }
             if (!ok) *abort_flag = 1;
@@ -165,47 +165,54 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
             const uint32_t id_s = instr_desc(128, N, 0, 0), id_m = instr_desc(128, HP, 0, 0);
             bool ok = mbar_wait(q_full, 0, A.status);
             tc_fence_after();
-            int u = 0, ch = 0, it = 0, u_kt = 0, u_c = 0;               // next score block, its chunk, ring position
+            // next score block, its chunk, tile and key/value head, its columns; key ring position.  The loop of this one thread paces
+            // everything, so it keeps running counters instead of dividing.
+            int u = 0, ch = 0, u_kt = 0, u_c = 0, slot = 0, s = 0;
+            uint32_t s_par = 0, b_off = 0;
+            const uint32_t b_step = (uint32_t)(N * 128), k_base = smem_u32(sk), q_base = smem_u32(smem);
             int consumed = 0;                                           // tiles whose scores have been read
             int m_left = nt * nq, m_q = 0, wn[2] = {0, 0};              // mixing products still to issue, next query of the tile
             const int units = nt * G;
+            int free_until = TP.NU;                                     // blocks below this number have columns to go to
+            const uint64_t w_desc = smem_desc(smem_u32(sw), 16, 1024), t_desc = smem_desc(smem_u32(st), 16, 1024);
             uint64_t t0 = global_ns();
             uint32_t idle = 0;
             while (ok && (u < units || m_left > 0)) {
                 bool progress = false;
-                if (m_left > 0 && mbar_try_wait(&w_full[m_q & 1], (uint32_t)(wn[m_q & 1] & 1))) {
+                if (m_left > 0 && mbar_test_wait(&w_full[m_q & 1], (uint32_t)(wn[m_q & 1] & 1))) {
                     const int g = m_q & 1;
                     tc_fence_after();
-                    const uint32_t a0 = smem_u32(sw + g * 16384), b0 = smem_u32(st);
 #pragma unroll
-                    for (int k = 0; k < HP / 8; ++k)
-                        umma_bf16(tmem + D_COL + (uint32_t)(g * HP), smem_desc(a0 + k * 32, 16, 1024), smem_desc(b0 + k * 32, 16, 1024), id_m, k > 0 ? 1u : 0u);
+                    for (int k = 0; k < HP / 8; ++k) umma_bf16(tmem + D_COL + (uint32_t)(g * HP), w_desc + (uint64_t)(g * 1024) + 2 * k, t_desc + 2 * k, id_m, k > 0 ? 1u : 0u);
                     umma_commit(&d_full[g]);
                     ++wn[g];
                     --m_left;
                     if (++m_q == nq) m_q = 0;
                     progress = true;
                 } else if (u < units) {
-                    if (consumed < u_kt && mbar_try_wait(&s_empty[consumed & 1], (uint32_t)((consumed >> 1) & 1))) {
+                    if (consumed < u_kt && mbar_test_wait(&s_empty[consumed & 1], (uint32_t)((consumed >> 1) & 1))) {
                         tc_fence_after();
                         ++consumed;
+                        free_until += G;
                         progress = true;
                     }
                     // at most one tile ahead, and the block's columns are free
-                    if (u_kt <= consumed + 1 && (u < TP.NU || (u - TP.NU) / G < consumed) &&
-                        mbar_try_wait(&k_full[it % T_STAGES], (uint32_t)((it / T_STAGES) & 1))) {
+                    if (u_kt <= consumed + 1 && u < free_until && mbar_test_wait(&k_full[s], s_par)) {
                         tc_fence_after();
-                        const uint32_t a0 = smem_u32(sk + (it % T_STAGES) * 16384), b0 = smem_u32(smem) + (uint32_t)((u_c * chunks + ch) * N * 128);
-                        const uint32_t d = tmem + (uint32_t)((u % TP.NU) * N);
+                        const uint32_t d = tmem + (uint32_t)(slot * N);
+                        const uint64_t da = smem_desc(k_base + s * 16384, 16, 1024), db = smem_desc(q_base + b_off, 16, 1024);
 #pragma unroll
-                        for (int k = 0; k < 4; ++k) umma_bf16(d, smem_desc(a0 + k * 32, 16, 1024), smem_desc(b0 + k * 32, 16, 1024), id_s, (ch > 0 || k > 0) ? 1u : 0u);
-                        umma_commit(&k_empty[it % T_STAGES]);
-                        ++it;
+                        for (int k = 0; k < 4; ++k) umma_bf16(d, da + 2 * k, db + 2 * k, id_s, (ch > 0 || k > 0) ? 1u : 0u);   // 32 bytes further each
+                        umma_commit(&k_empty[s]);
+                        if (++s == T_STAGES) { s = 0; s_par ^= 1; }
+                        b_off += b_step;
                         if (++ch == chunks) {
                             ch = 0;
                             ++u;
+                            if (++slot == TP.NU) slot = 0;
                             if (++u_c == G) {
                                 u_c = 0;
+                                b_off = 0;
                                 umma_commit(&s_full[u_kt & 1]);
                                 ++u_kt;
                             }
@@ -233,6 +240,13 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         tanh_poly(A, xs, cf);
         __nv_bfloat16* Pt = P.P + ((size_t)blockIdx.x * H * QT + q0) * P.KW;
         uint8_t* wrow = sw + grp * 16384 + row * 128;
+        // where a read of RV heads starts: block of its key/value head and place in the group
+        int8_t rd_c[HP / RV];
+        int8_t rd_r[HP / RV];
+#pragma unroll
+        for (int i = 0; i < HP / RV; ++i) { rd_c[i] = (int8_t)(i * RV / R); rd_r[i] = (int8_t)(i * RV % R); }
+        const size_t h_step = (size_t)QT * P.KW;
+        int slot0 = -G;
         bool ok = true;
         int cnt = 0;
         __nv_bfloat16* pending = nullptr;                                // where this thread's mixed weights of the query before go
@@ -250,9 +264,10 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         };
         auto store_mixed = [&]() {
             if (!pending || !ok) return;
+            __nv_bfloat16* o = pending;
 #pragma unroll
-            for (int h = 0; h < HP; ++h)
-                if (h < H) pending[(size_t)h * QT * P.KW] = __float2bfloat16_rn(__uint_as_float(d[h]));
+            for (int h = 0; h < HP; ++h, o += h_step)
+                if (h < H) *o = __float2bfloat16_rn(__uint_as_float(d[h]));
         };
         for (int kt = 0; kt < nt && ok; ++kt) {
             if (!*abort_flag) ok = mbar_wait(&s_full[kt & 1], (uint32_t)((kt >> 1) & 1), A.status);
@@ -266,7 +281,15 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
                 const int page = table[col];
                 key_ok = page >= 0 && page < A.n_pages;
             }
-            const int slot0 = (kt * G) % TP.NU;
+            slot0 += G;
+            while (slot0 >= TP.NU) slot0 -= TP.NU;
+            int at_col[HP / RV];
+#pragma unroll
+            for (int i = 0; i < HP / RV; ++i) {
+                int slot = slot0 + rd_c[i];
+                while (slot >= TP.NU) slot -= TP.NU;
+                at_col[i] = slot * N + rd_r[i];
+            }
             if (grp >= nq) {
                 __syncwarp();
                 if (lane == 0) mbar_arrive(&s_empty[kt & 1]);
@@ -276,10 +299,7 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
 #pragma unroll
                 for (int h = 0; h < HP; h += RV) {
                     if (h < H) {
-                        const int c = h / R;
-                        int slot = slot0 + c;
-                        while (slot >= TP.NU) slot -= TP.NU;
-                        const uint32_t at = lane_addr + (uint32_t)(slot * N + q * R + h % R);
+                        const uint32_t at = lane_addr + (uint32_t)(at_col[h / RV] + q * R);
                         if constexpr (RV == 4) tmem_ld4(at, w + h);
                         else tmem_ld2(at, w + h);
                     } else {
