@@ -534,7 +534,7 @@ PTB_API int ptb_gated_attn_tiles(const void* q, void* out, int n_rows, const int
     const int R = H / G, ks = (Dp + 31) / 32;
     const bool same = R % 4 == 0;
     int rc;
-    if (tensor_cores && gp::tc_supported(w.A)) rc = gp::launch_tc_any(w, n_tiles, n_rows, std::max(1, per / 4), st);
+    if (tensor_cores && gp::tc_supported(w.A)) rc = gp::launch_tc_any(w, n_tiles, n_rows, st);
     else if (H > 32 || ks > 4) rc = gp::launch_weights_nk<1, false, false>(w, n_tiles, st);
     else if (!same) rc = ks <= 2 ? gp::launch_weights_nk<2, true, false>(w, n_tiles, st) : gp::launch_weights_nk<4, true, false>(w, n_tiles, st);
     else if (ks <= 2) rc = gp::launch_weights_nk<2, true, true>(w, n_tiles, st);

@@ -1,25 +1,28 @@
-// The mixed weights of gated attention (gated_prefill.cu) with both products on tcgen05, for designs of up to 32 heads.
+// The mixed weights of gated attention (gated_prefill.cu) with both products on tcgen05, for layers of up to 16 heads (with 32, a
+// thread's scores and weights of all heads no longer fit the registers of eighteen warps, and the mma.sync kernel is faster).
 //
 // One CTA: NQ queries x a run of 128-key tiles, all heads.  The queries stay in shared memory; keys stream through a TMA ring, 64 of
-// their elements at a time.  Ten warps:
-//   warp 8   TMA producer;
-//   warp 9   owns tensor memory and issues the MMAs from one event loop: S^T(c) = K_c Q_c^T for every key/value head c (rows: keys,
+// their elements at a time.  Eighteen warps:
+//   warp 16  TMA producer;
+//   warp 17  owns tensor memory and issues the MMAs from one event loop: S^T(c) = K_c Q_c^T for every key/value head c (rows: keys,
 //            columns: query-major, then the head's group) into a ring of column blocks that runs ahead into the next tile, and per
 //            query the mixing product D = W talk^T;
-//   warps 0-7  two groups of four.  A thread owns a key (its tensor-memory lane); for one query at a time it reads the scores of
+//   warps 0-15  four groups of four.  A thread owns a key (its tensor-memory lane); for one query at a time it reads the scores of
 //            all heads, forms the weights in fp32 and writes them, each as a high and a low bf16 part, into the 128-byte-swizzled
 //            row of its key: the A operand of the mixing product.  Then it reads the mixed weights of the query before and stores
-//            them.  The groups alternate the queries.
+//            them.  The groups take turns at the queries.
 // Every wait is bounded.
 #pragma once
 
 namespace ptb {
 namespace gp {
 
-constexpr int T_THREADS = 320, T_STAGES = 7, T_KEYS = 128;
+constexpr int T_PER = 5;              // 128-key tiles per CTA
+constexpr int T_GROUPS = 4, T_THREADS = T_GROUPS * 128 + 64, T_STAGES = 5, T_KEYS = 128;
+constexpr int T_TMA_WARP = T_GROUPS * 4, T_MMA_WARP = T_TMA_WARP + 1;
 
 struct TcParams {
-    WeightsParams W;                   // `per`: 128-key tiles per CTA
+    WeightsParams W;                   // `per`: 128-key tiles per CTA here
     int NU;                            // column blocks of the score ring
     int groups;                        // CTAs along a tile's queries
 };
@@ -55,14 +58,14 @@ struct TcSmem {
     __host__ __device__ TcSmem(int H, int NQ, int chunks, int HP) {
         k = H * NQ * chunks * 128;
         w = k + T_STAGES * 16384;
-        talk = w + 2 * 16384;
+        talk = w + T_GROUPS * 16384;
         far = talk + HP * 128;
         bar = far + 128;
         total = bar + 256 + 1024;
     }
 };
 
-// HP: heads padded to 16 or 32; RV: heads per tensor-memory read, a divisor of the group size (4 or 2); NQ: queries per CTA.
+// HP: heads padded to 16; RV: heads per tensor-memory read, a divisor of the group size (4 or 2); NQ: queries per CTA.
 template <int HP, int RV, int NQ>
 __global__ void __launch_bounds__(T_THREADS, 1)
 gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ TcParams TP) {
@@ -81,26 +84,27 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     uint64_t* q_full = bars;
     uint64_t* s_full = bars + 1;             // [2] by tile parity
     uint64_t* s_empty = bars + 3;            // [2]
-    uint64_t* w_full = bars + 5;             // [2] by group
-    uint64_t* d_full = bars + 7;             // [2]
-    uint64_t* k_full = bars + 9;             // [T_STAGES]
+    uint64_t* w_full = bars + 5;             // [T_GROUPS]
+    uint64_t* d_full = w_full + T_GROUPS;    // [T_GROUPS]
+    uint64_t* k_full = d_full + T_GROUPS;    // [T_STAGES]
     uint64_t* k_empty = k_full + T_STAGES;
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(k_empty + T_STAGES);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    constexpr uint32_t D_COL = 512 - 2 * HP;
+    constexpr uint32_t D_COL = 512 - T_GROUPS * HP;
 
     // constants: none of them is written by the kernel before
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
-        for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&s_empty[i], 8); mbar_init(&w_full[i], 4); mbar_init(&d_full[i], 1); }
+        for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&s_empty[i], T_GROUPS * 4); }
+        for (int i = 0; i < T_GROUPS; ++i) { mbar_init(&w_full[i], 4); mbar_init(&d_full[i], 1); }
         for (int s = 0; s < T_STAGES; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); }
         *abort_flag = 0;
         mbar_fence_init();
         prefetch_tmap(&tmQ);
         prefetch_tmap(&tmK);
     }
-    if (warp == 9) {
+    if (warp == T_MMA_WARP) {
         tmem_alloc(tmem_slot, 512);
         tmem_relinquish();
     }
@@ -130,7 +134,7 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     const int t_lo = blockIdx.z * P.per, t_hi = nq > 0 ? min(t_lo + P.per, (band.blocks + 1) / 2) : 0, nt = max(0, t_hi - t_lo);
     const int* table = A.page_table + (size_t)T.req * A.pt_stride;
 
-    if (warp == 8) {
+    if (warp == T_TMA_WARP) {
         // ------------------------------------------------------------------------ TMA producer
         if (lane == 0 && nt > 0) {
             bool ok = true;
@@ -159,7 +163,7 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
             }
             if (!ok) *abort_flag = 1;
         }
-    } else if (warp == 9) {
+    } else if (warp == T_MMA_WARP) {
         // ------------------------------------------------------------------------ MMA issuer
         if (lane == 0 && nt > 0) {
             const uint32_t id_s = instr_desc(128, N, 0, 0), id_m = instr_desc(128, HP, 0, 0);
@@ -171,7 +175,8 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
             uint32_t s_par = 0, b_off = 0;
             const uint32_t b_step = (uint32_t)(N * 128), k_base = smem_u32(sk), q_base = smem_u32(smem);
             int consumed = 0;                                           // tiles whose scores have been read
-            int m_left = nt * nq, m_q = 0, wn[2] = {0, 0};              // mixing products still to issue, next query of the tile
+            int m_left = nt * nq, m_q = 0;              // mixing products still to issue, next query of the tile
+            uint32_t w_par = 0;                                         // bit g: parity of group g's next weights
             const int units = nt * G;
             int free_until = TP.NU;                                     // blocks below this number have columns to go to
             const uint64_t w_desc = smem_desc(smem_u32(sw), 16, 1024), t_desc = smem_desc(smem_u32(st), 16, 1024);
@@ -179,13 +184,13 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
             uint32_t idle = 0;
             while (ok && (u < units || m_left > 0)) {
                 bool progress = false;
-                if (m_left > 0 && mbar_test_wait(&w_full[m_q & 1], (uint32_t)(wn[m_q & 1] & 1))) {
-                    const int g = m_q & 1;
+                if (m_left > 0 && mbar_test_wait(&w_full[m_q % T_GROUPS], (w_par >> (m_q % T_GROUPS)) & 1u)) {
+                    const int g = m_q % T_GROUPS;
                     tc_fence_after();
 #pragma unroll
                     for (int k = 0; k < HP / 8; ++k) umma_bf16(tmem + D_COL + (uint32_t)(g * HP), w_desc + (uint64_t)(g * 1024) + 2 * k, t_desc + 2 * k, id_m, k > 0 ? 1u : 0u);
                     umma_commit(&d_full[g]);
-                    ++wn[g];
+                    w_par ^= 1u << g;
                     --m_left;
                     if (++m_q == nq) m_q = 0;
                     progress = true;
@@ -233,7 +238,7 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         }
     } else {
         // ------------------------------------------------------------------------ weights
-        const int grp = warp >> 2, row = 32 * (warp & 3) + lane;         // query parity; key of the tile = tensor-memory lane
+        const int grp = warp >> 2, row = 32 * (warp & 3) + lane;         // key of the tile = tensor-memory lane
         const uint32_t lane_addr = tmem + ((uint32_t)(32 * (warp & 3)) << 16);
         float cf[6];
         const float xs = A.cap > 0.f ? A.scale * A.inv_cap : A.scale, dot_max = 0.4f / fabsf(xs);
@@ -250,24 +255,32 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         bool ok = true;
         int cnt = 0;
         __nv_bfloat16* pending = nullptr;                                // where this thread's mixed weights of the query before go
-        uint32_t d[HP];
+        uint32_t d[HP / 2];                                              // pairs of mixed weights, bf16
         auto read_mixed = [&]() {                                        // false: gave up
             if (ok && !*abort_flag) ok = mbar_wait(&d_full[grp], (uint32_t)((cnt - 1) & 1), A.status);
             else ok = false;
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) return;
             tc_fence_after();
-            if constexpr (HP == 32) tmem_ld32(lane_addr + D_COL + (uint32_t)(grp * HP), d);
-            else tmem_ld16(lane_addr + D_COL + (uint32_t)(grp * HP), d);
-            tmem_ld_wait();
+#pragma unroll
+            for (int b = 0; b < HP; b += 16) {
+                uint32_t r[16];
+                tmem_ld16(lane_addr + D_COL + (uint32_t)(grp * HP + b), r);
+                tmem_ld_wait();
+#pragma unroll
+                for (int i = 0; i < 8; ++i) d[b / 2 + i] = fa::pack_bf16(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1]));
+            }
             tc_fence_before();
         };
         auto store_mixed = [&]() {
             if (!pending || !ok) return;
-            __nv_bfloat16* o = pending;
+            uint16_t* o = reinterpret_cast<uint16_t*>(pending);
 #pragma unroll
-            for (int h = 0; h < HP; ++h, o += h_step)
-                if (h < H) *o = __float2bfloat16_rn(__uint_as_float(d[h]));
+            for (int h = 0; h < HP; h += 2, o += 2 * h_step)
+                if (h < H) {                                             // H is even: groups of two or more
+                    o[0] = (uint16_t)d[h / 2];
+                    o[h_step] = (uint16_t)(d[h / 2] >> 16);
+                }
         };
         for (int kt = 0; kt < nt && ok; ++kt) {
             if (!*abort_flag) ok = mbar_wait(&s_full[kt & 1], (uint32_t)((kt >> 1) & 1), A.status);
@@ -294,7 +307,7 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
                 __syncwarp();
                 if (lane == 0) mbar_arrive(&s_empty[kt & 1]);
             }
-            for (int q = grp; q < nq; q += 2) {
+            for (int q = grp; q < nq; q += T_GROUPS) {
                 float w[HP];
 #pragma unroll
                 for (int h = 0; h < HP; h += RV) {
@@ -308,7 +321,7 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
                     }
                 }
                 tmem_ld_wait();
-                if (q + 2 >= nq) {                                       // this warp has read all it needs of the tile
+                if (q + T_GROUPS >= nq) {                                       // this warp has read all it needs of the tile
                     tc_fence_before();
                     __syncwarp();
                     if (lane == 0) mbar_arrive(&s_empty[kt & 1]);
@@ -380,17 +393,17 @@ gated_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     // ---- teardown
     tc_fence_before();
     __syncthreads();
-    if (warp == 9) tmem_dealloc(tmem, 512);
+    if (warp == T_MMA_WARP) tmem_dealloc(tmem, 512);
 }
 
 template <int HP, int RV, int NQ>
-static int launch_tc(const WeightsParams& w, int tiles, int n_rows, int per, cudaStream_t st) {
+static int launch_tc(const WeightsParams& w, int tiles, int n_rows, cudaStream_t st) {
     const GatedAttnParams& A = w.A;
     const int R = A.H / A.G, N = R * NQ, chunks = (A.Dp + 63) / 64;
     TcParams p;
     p.W = w;
-    p.W.per = per;
-    p.NU = (512 - 2 * HP) / N;
+    p.W.per = T_PER;
+    p.NU = (512 - T_GROUPS * HP) / N;
     p.groups = QT / NQ;
     CUtensorMap mq, mk;
     if (ptb_make_tmap_bf16_3d(&mq, A.q, A.Dp, A.H, n_rows, 64, R, NQ)) return -1;
@@ -403,21 +416,19 @@ static int launch_tc(const WeightsParams& w, int tiles, int n_rows, int per, cud
     }
     const TcSmem L(A.H, NQ, chunks, HP);
     const int key_tiles = (w.KW + T_KEYS - 1) / T_KEYS;
-    PTB_CUDA_OK(ptb_launch(kern, dim3(tiles, p.groups, (key_tiles + per - 1) / per), dim3(T_THREADS), (size_t)L.total, st, ptb_pdl_enabled(), mq, mk, p));
+    PTB_CUDA_OK(ptb_launch(kern, dim3(tiles, p.groups, (key_tiles + T_PER - 1) / T_PER), dim3(T_THREADS), (size_t)L.total, st, ptb_pdl_enabled(), mq, mk, p));
     return 0;
 }
 
 // Sizes the tcgen05 kernel takes: whole groups of 2 or 4 heads per tensor-memory read, key vectors of 64 to 128 elements, and a ring
 // of score blocks that holds at least one tile.
 static bool tc_supported(const GatedAttnParams& A) {
-    const int R = A.H / A.G, NQ = A.H <= 16 ? 16 : 8, HP = A.H <= 16 ? 16 : 32, N = R * NQ;
-    if (A.H > 32 || A.Dp < 64 || A.Dp > 128 || (R != 2 && R % 4) || N % 16 || N > 256) return false;
-    return (512 - 2 * HP) / N >= A.G;
+    const int R = A.H / A.G, NQ = 16, N = R * NQ;
+    if (A.H > 16 || A.Dp < 64 || A.Dp > 128 || (R != 2 && R % 4) || N > 256) return false;
+    return (512 - T_GROUPS * 16) / N >= A.G;
 }
-static int launch_tc_any(const WeightsParams& w, int tiles, int n_rows, int per, cudaStream_t st) {
-    const bool two = w.A.H / w.A.G == 2;
-    if (w.A.H <= 16) return two ? launch_tc<16, 2, 16>(w, tiles, n_rows, per, st) : launch_tc<16, 4, 16>(w, tiles, n_rows, per, st);
-    return two ? launch_tc<32, 2, 8>(w, tiles, n_rows, per, st) : launch_tc<32, 4, 8>(w, tiles, n_rows, per, st);
+static int launch_tc_any(const WeightsParams& w, int tiles, int n_rows, cudaStream_t st) {
+    return w.A.H / w.A.G == 2 ? launch_tc<16, 2, 16>(w, tiles, n_rows, st) : launch_tc<16, 4, 16>(w, tiles, n_rows, st);
 }
 
 }  // namespace gp
