@@ -4,7 +4,7 @@ kernel of Llama with the fraction of the roofline both reach.
     python benchmarks/kifusun_bench.py [--sizes 1b,7b] [--windows 1024,4096] [--no-engine] [--no-kernels]      (or: python bench.py --model kifusun)
 
 Random bf16 weights, random prompts.  Engine: prompt passes and decode steps timed with CUDA events, the second of two identical
-rounds.  Kernels: a CUDA graph of launches over rotating inputs that together exceed L2, time per launch from the median of its
+repetitions.  Kernels: a CUDA graph of launches over rotating inputs that together exceed L2, time per launch from the median of its
 replays; `roof` is the slower of bytes over the measured copy bandwidth and FLOPs over the measured bf16 matrix throughput, and
 `frac` is roof / time.  One JSON object on the last line."""
 from __future__ import annotations
