@@ -225,6 +225,11 @@ __device__ __forceinline__ uint64_t global_ns() {
 }
 
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
+__device__ __forceinline__ float sigmoid(float x) { return 1.0f / (1.0f + __expf(-x)); }
+__device__ __forceinline__ float relu2(float x) {
+    x = fmaxf(x, 0.f);
+    return x * x;
+}
 __device__ __forceinline__ float gelu_tanh(float x) {
     // 0.5 x (1 + tanh(u)) = x * sigmoid(2 u): keeps its relative accuracy where 1 + tanh(u) cancels
     const float k2 = 2.0f * 0.7978845608028654f;

@@ -204,9 +204,9 @@ PTB_API int ptb_gemm_bf16_ex(void* const* a_ptrs, int a_shards, int a_shard_rows
                      out_shard_rows, M, N, K, bias, flags, status, n_sm, st, stage_a, stage_b, SplitK{1, 0, 0, 0});
 }
 
-// Sum the split-K partials, add the bias, apply GELU, round to bf16.  work: [splits][M][N] fp32; N a multiple of 4.
+// Sum the split-K partials, add the bias, apply the activation (1: GELU, 2: square of ReLU), round to bf16.  work: [splits][M][N] fp32; N a multiple of 4.
 __global__ void __launch_bounds__(256) splitk_reduce_kernel(const float* __restrict__ work, int splits, long long mn, int N,
-                                                            const float* __restrict__ bias, int gelu, __nv_bfloat16* __restrict__ C,
+                                                            const float* __restrict__ bias, int act, __nv_bfloat16* __restrict__ C,
                                                             long long ldc) {
     pdl_wait();
     pdl_launch_dependents();
@@ -220,7 +220,8 @@ __global__ void __launch_bounds__(256) splitk_reduce_kernel(const float* __restr
     const long long row = i4 / N;
     const int col = (int)(i4 - row * N);
     if (bias) { acc.x += bias[col]; acc.y += bias[col + 1]; acc.z += bias[col + 2]; acc.w += bias[col + 3]; }
-    if (gelu) { acc.x = gelu_tanh(acc.x); acc.y = gelu_tanh(acc.y); acc.z = gelu_tanh(acc.z); acc.w = gelu_tanh(acc.w); }
+    if (act == 1) { acc.x = gelu_tanh(acc.x); acc.y = gelu_tanh(acc.y); acc.z = gelu_tanh(acc.z); acc.w = gelu_tanh(acc.w); }
+    else if (act == 2) { acc.x = relu2(acc.x); acc.y = relu2(acc.y); acc.z = relu2(acc.z); acc.w = relu2(acc.w); }
     __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(C + row * ldc + col);
     o[0] = __floats2bfloat162_rn(acc.x, acc.y);
     o[1] = __floats2bfloat162_rn(acc.z, acc.w);
@@ -428,16 +429,16 @@ static int skinny_partials(const void* A, long long lda, const void* B, long lon
     return 0;
 }
 
-// Skinny GEMM (M <= 128), K-major operands: C[M,N] bf16 = A[M,K] B[N,K]^T (+ bias, GELU) with `splits` K-splits whose
+// Skinny GEMM (M <= 128), K-major operands: C[M,N] bf16 = A[M,K] B[N,K]^T (+ bias, then act: 0 none, 1 GELU, 2 square of ReLU) with `splits` K-splits whose
 // fp32 partials go through `work` ([splits][M][N] floats) and one reduce launch.  N must be a multiple of 4.
 PTB_API int ptb_gemm_bf16_splitk(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc, int M, int N, int K,
-                                 const float* bias, int gelu, int splits, float* work, int* status, int n_sm, cudaStream_t st) {
+                                 const float* bias, int act, int splits, float* work, int* status, int n_sm, cudaStream_t st) {
     if (M <= 0 || N <= 0 || K <= 0) return 0;
     int real = 0;
     if (skinny_partials(A, lda, B, ldb, M, N, K, splits, work, status, n_sm, st, &real)) return -1;
     const long long mn = (long long)M * N;
     PTB_CUDA_OK(ptb_launch(splitk_reduce_kernel, dim3((unsigned)((mn / 4 + 255) / 256)), dim3(256), 0, st, ptb_pdl_enabled(), work, real, mn, N, bias,
-                           gelu, (__nv_bfloat16*)C, ldc));
+                           act, (__nv_bfloat16*)C, ldc));
     PTB_CUDA_OK(cudaGetLastError());
     return 0;
 }
@@ -512,7 +513,7 @@ PTB_API int ptb_gemm_bf16_splitk_gated(const void* A, long long lda, const void*
 // C[M,N] (+)= op(A) op(B)^T with bf16 operands and fp32 accumulation, all operands local.
 //   a_mn == 0: A is [M, K] row-major (pitch lda);  a_mn == 1: A is stored as [K, M] row-major.
 //   b_mn == 0: B is [N, K] row-major (pitch ldb);  b_mn == 1: B is stored as [K, N] row-major.
-//   flags: EPI_BIAS | EPI_ACCUM | EPI_OUT_F32 | EPI_GELU.  status: device int, set non-zero if a wait timed out.
+//   flags: EPI_BIAS | EPI_ACCUM | EPI_OUT_F32 | EPI_GELU | EPI_RELU2.  status: device int, set non-zero if a wait timed out.
 PTB_API int ptb_gemm_bf16(const void* A, long long lda, int a_mn, const void* B, long long ldb, int b_mn, void* C, long long ldc,
                           int M, int N, int K, const float* bias, int flags, int* status, int n_sm, cudaStream_t st) {
     void* ap[1] = {const_cast<void*>(A)};

@@ -28,6 +28,7 @@ constexpr int MAX_SHARDS = 8;
 
 enum EpiFlags : int { EPI_BIAS = 1, EPI_ACCUM = 2, EPI_OUT_F32 = 4, EPI_GELU = 8, EPI_SCATTER_ADD = 16, EPI_SCATTER_STORE = 32,
                       EPI_TRANS = 64 };   // EPI_TRANS: element (row, col) is stored at C[col * ldc + row] (fp32 only)
+constexpr int EPI_RELU2 = 128;        // the square of ReLU
 
 // An operand whose stored matrix is split by rows over up to eight GPUs (each piece in that GPU's
 // memory, mapped here): piece r holds stored rows [r*shard_rows, (r+1)*shard_rows).  The producer warp
@@ -390,6 +391,10 @@ gemm_bf16_kernel(const __grid_constant__ Operand opA, const __grid_constant__ Op
                     if (P.flags & EPI_GELU) {
 #pragma unroll
                         for (int j = 0; j < 32; ++j) v[j] = gelu_tanh(v[j]);
+                    }
+                    if (P.flags & EPI_RELU2) {
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) v[j] = relu2(v[j]);
                     }
                     if (P.flags & EPI_TRANS) {
                         // swapped operands (rows = output features, columns = tokens): a warp's 32 lanes hold 32

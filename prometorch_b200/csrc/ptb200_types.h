@@ -63,3 +63,27 @@ typedef struct PtbSampleRequest {
     int n_hist, hist_cap, top_k, pad;
     float repeat_penalty, temperature, top_p, u;
 } PtbSampleRequest;
+
+// A recurrent layer over the rows of a batch (recurrence.cuh has the equations).
+typedef struct PtbRecurrence {
+    const void* x;          // [n] rows of pitch ld, bf16 or fp32: q [G D], k [G D], v [H Dv] at the three columns
+    long long ld;
+    int q_col, k_col, v_col;
+    int silu;               // decay attention: q, k and v pass SiLU first
+    int delta;              // 1: gated delta rule; 0: decay attention (G == H)
+    int bf16;
+    const void* beta;       // delta: [n][H] of pitch ld_beta in the type of x, before the sigmoid
+    long long ld_beta;
+    const float* a;         // delta: [n][H D] of pitch ld_a
+    long long ld_a;
+    const float* decay;     // [H]: the decay, or exp(A_log)
+    const float* dt_bias;   // delta: [H D]
+    float* state;           // [slots][H][D][Dv]
+    int slots, n, H, G, D, Dv;
+    const void* seqs;       // [n_seqs] int4 (first row, rows, position of the first, slot); null: one token per row
+    int n_seqs, pos_stride, req_stride, pad;
+    const int* pos;         // [n] of pos_stride
+    const int* req;         // [n] of req_stride: slots
+    float* out;             // [n][H Dv]
+    int* status;
+} PtbRecurrence;

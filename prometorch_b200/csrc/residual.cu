@@ -1,6 +1,8 @@
 // Kernels around an fp32 residual stream, for decoders that keep the sum of their sublayers in 32-bit while the matrix
 // products run on bf16 copies:
 //   embed_residual_kernel   x = table[id] * scale (fp32) and its copy in the compute type;
+//   residual_norm_kernel    x += the sum of one or two sublayer outputs (each RMS-normed first if it has a weight; bf16, fp32 or
+//                           split-K partials), then h = rmsnorm(x) * w for the next sublayer;
 //   post_norm_add_kernel    x += rmsnorm(y) * g: the norm sits on a sublayer's output, before the sum;
 //   row_norm_kernel         rmsnorm of chosen rows of x, in the compute type (the model's last norm).
 // A norm's weight is a vector, a single number, or both.  T is the compute type (bf16 or float); with float the copy is x itself
@@ -130,9 +132,151 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const float* __res
     for (int c = threadIdx.x; c < W; c += RS_THREADS) from_f(out + o * W + c, xr[c] * rs * (w ? w[c] : 1.f));
 }
 
+// A sublayer's output on its way into the stream: y = sum over `splits` partials (pitch ld), times g, and w / rms(y) if there is a w.
+struct Branch {
+    const void* y;                     // null: absent
+    int f32, splits;
+    long long stride, ld;
+    const float* w;
+    float g;
+};
+template <int V> struct Row { float v[V]; };
+template <int V>
+__device__ __forceinline__ Row<V> branch_load(const Branch& B, size_t row, int c) {
+    Row<V> r;
+    if (B.f32) {
+        const float* p = (const float*)B.y + row * B.ld + c;
+        if constexpr (V == 4) { const float4 a = load4<float>(p); r.v[0] = a.x; r.v[1] = a.y; r.v[2] = a.z; r.v[3] = a.w; }
+        else r.v[0] = *p;
+        for (int s = 1; s < B.splits; ++s) {
+            p += B.stride;
+            if constexpr (V == 4) { const float4 a = load4<float>(p); r.v[0] += a.x; r.v[1] += a.y; r.v[2] += a.z; r.v[3] += a.w; }
+            else r.v[0] += *p;
+        }
+    } else {
+        const __nv_bfloat16* p = (const __nv_bfloat16*)B.y + row * B.ld + c;
+        if constexpr (V == 4) { const float4 a = load4<__nv_bfloat16>(p); r.v[0] = a.x; r.v[1] = a.y; r.v[2] = a.z; r.v[3] = a.w; }
+        else r.v[0] = to_f(*p);
+    }
+    return r;
+}
+
+// One CTA per row.  A thread keeps NK groups of V elements of x and of both branches in registers; wider rows are read again.
+template <typename T, int V, int NK, int NB>
+__global__ void __launch_bounds__(RS_THREADS) residual_norm_kernel(const Branch A, const Branch B, float eps, float* __restrict__ x,
+                                                                   const float* __restrict__ w, T* __restrict__ out, int W) {
+    __shared__ float red[4][32];
+    pdl_wait();
+    pdl_launch_dependents();
+    const size_t row = blockIdx.x;
+    float* xr = x + row * W;
+    const int nc = W / V, kept = NK * RS_THREADS;
+    Row<V> a[NK], b[NB == 2 ? NK : 1], xs[NK];
+    float sa = 0.f, sb = 0.f;
+#pragma unroll
+    for (int k = 0; k < NK; ++k) {
+        const int c = k * RS_THREADS + threadIdx.x;
+        if (c < nc) {
+            a[k] = branch_load<V>(A, row, c * V);
+            if constexpr (NB == 2) b[k] = branch_load<V>(B, row, c * V);
+            if constexpr (V == 4) { const float4 t = load4<float>(xr + c * 4); xs[k].v[0] = t.x; xs[k].v[1] = t.y; xs[k].v[2] = t.z; xs[k].v[3] = t.w; }
+            else xs[k].v[0] = xr[c];
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+                sa += a[k].v[e] * a[k].v[e];
+                if constexpr (NB == 2) sb += b[k].v[e] * b[k].v[e];
+            }
+        }
+    }
+    for (int c = kept + threadIdx.x; c < nc; c += RS_THREADS) {
+        const Row<V> r = branch_load<V>(A, row, c * V);
+#pragma unroll
+        for (int e = 0; e < V; ++e) sa += r.v[e] * r.v[e];
+        if constexpr (NB == 2) {
+            const Row<V> q = branch_load<V>(B, row, c * V);
+#pragma unroll
+            for (int e = 0; e < V; ++e) sb += q.v[e] * q.v[e];
+        }
+    }
+    float ra = A.g, rb = B.g;
+    if (A.w) ra *= rsqrtf(cta_sum(sa, red[0]) / (float)W + eps);
+    if (NB == 2 && B.w) rb *= rsqrtf(cta_sum(sb, red[1]) / (float)W + eps);
+    float ss = 0.f;
+    auto sum = [&](int c, const Row<V>& p, const Row<V>& q, Row<V>& r) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            r.v[e] += p.v[e] * ra * (A.w ? A.w[c * V + e] : 1.f);
+            if constexpr (NB == 2) r.v[e] += q.v[e] * rb * (B.w ? B.w[c * V + e] : 1.f);
+            ss += r.v[e] * r.v[e];
+        }
+        if constexpr (V == 4) store4(xr + c * 4, make_float4(r.v[0], r.v[1], r.v[2], r.v[3]));
+        else xr[c] = r.v[0];
+    };
+#pragma unroll
+    for (int k = 0; k < NK; ++k) {
+        const int c = k * RS_THREADS + threadIdx.x;
+        if (c < nc) sum(c, a[k], b[NB == 2 ? k : 0], xs[k]);
+    }
+    for (int c = kept + threadIdx.x; c < nc; c += RS_THREADS) {
+        Row<V> p = branch_load<V>(A, row, c * V), q = p, r;
+        if constexpr (NB == 2) q = branch_load<V>(B, row, c * V);
+#pragma unroll
+        for (int e = 0; e < V; ++e) r.v[e] = xr[c * V + e];
+        sum(c, p, q, r);
+    }
+    if (!w) return;
+    const float rs = rsqrtf(cta_sum(ss, red[2]) / (float)W + eps);
+    T* o = out + row * W;
+    auto put = [&](int c, const Row<V>& r) {
+        if constexpr (V == 4) {
+            const float4 m = *reinterpret_cast<const float4*>(w + c * 4);
+            store4(o + c * 4, make_float4(r.v[0] * rs * m.x, r.v[1] * rs * m.y, r.v[2] * rs * m.z, r.v[3] * rs * m.w));
+        } else from_f(o + c, r.v[0] * rs * w[c]);
+    };
+#pragma unroll
+    for (int k = 0; k < NK; ++k) {
+        const int c = k * RS_THREADS + threadIdx.x;
+        if (c < nc) put(c, xs[k]);
+    }
+    for (int c = kept + threadIdx.x; c < nc; c += RS_THREADS) {
+        Row<V> r;
+#pragma unroll
+        for (int e = 0; e < V; ++e) r.v[e] = xr[c * V + e];
+        put(c, r);
+    }
+}
+
+template <typename T, int NB>
+static cudaError_t residual_norm_launch(const Branch& A, const Branch& B, float eps, float* x, const float* w, void* out, int n, int W, bool vec,
+                                        cudaStream_t st) {
+    auto go = [&](auto k) { return ptb_launch(k, dim3(n), dim3(RS_THREADS), 0, st, ptb_pdl_enabled(), A, B, eps, x, w, (T*)out, W); };
+    if (!vec) return go(residual_norm_kernel<T, 1, 4, NB>);
+    const int nk = (W / 4 + RS_THREADS - 1) / RS_THREADS;
+    if (nk <= 1) return go(residual_norm_kernel<T, 4, 1, NB>);
+    if (nk <= 2) return go(residual_norm_kernel<T, 4, 2, NB>);
+    return go(residual_norm_kernel<T, 4, 4, NB>);
+}
+
 }  // namespace ptb
 
 using namespace ptb;
+
+// x [n, W] fp32 += branch a (+ branch b, absent with yb null); h [n, W] (bf16 or fp32) = x / rms(x) * w unless w is null.  A branch: y in
+// bf16 (f32 = 0) or as the sum of `splits` fp32 matrices `stride` apart, row pitch ld; times g; RMS-normed with the fp32 weight w[W]
+// when that is given.  eps sits inside every root.
+PTB_API int ptb_residual_norm(float* x, const void* ya, int f32a, int splits_a, long long stride_a, long long ld_a, const float* wa, float ga,
+                              const void* yb, int f32b, int splits_b, long long stride_b, long long ld_b, const float* wb, float gb, float eps,
+                              const float* w, void* h, int n, int W, int bf16, cudaStream_t st) {
+    if (n <= 0) return 0;
+    const Branch A{ya, f32a, splits_a, stride_a, ld_a, wa, ga}, B{yb, f32b, splits_b, stride_b, ld_b, wb, gb};
+    const uintptr_t bases = (uintptr_t)x | (uintptr_t)ya | (uintptr_t)yb | (uintptr_t)wa | (uintptr_t)wb | (uintptr_t)w | (uintptr_t)h;
+    const bool vec = W % 4 == 0 && (bases & 15) == 0 && ld_a % 4 == 0 && ld_b % 4 == 0 && stride_a % 4 == 0 && stride_b % 4 == 0;
+    if (!ya || (splits_a > 1 && !f32a) || (splits_b > 1 && !f32b)) { ptb_set_error("residual_norm: partials are fp32, and the first branch is there"); return -1; }
+    if (bf16) PTB_CUDA_OK((yb ? residual_norm_launch<__nv_bfloat16, 2> : residual_norm_launch<__nv_bfloat16, 1>)(A, B, eps, x, w, h, n, W, vec, st));
+    else PTB_CUDA_OK((yb ? residual_norm_launch<float, 2> : residual_norm_launch<float, 1>)(A, B, eps, x, w, h, n, W, vec, st));
+    PTB_CUDA_OK(cudaGetLastError());
+    return 0;
+}
 
 // x [n, W] fp32 = table[ids[i * id_stride]] * scale; xb: its bf16 copy (bf16 != 0; the table has the same type).
 PTB_API int ptb_embed_residual(const int* ids, int id_stride, const void* table, int V, int W, float scale, int n, float* x, void* xb,

@@ -1,0 +1,459 @@
+// Row kernels of window attention (window_attn.cuh):
+//   proj_norm_write_kernel   after the packed projection: RMS norm of the whole q and k rows, page write;
+//   window_rows_mma_kernel   bf16, one CTA per (split of the keys, kv head, row).  Scores straight from the pages on the tensor cores,
+//                            values on their way to shared memory meanwhile; a weight enters the value product as the sum of two
+//                            bf16 numbers in the two halves of the 16-row operand;
+//   window_rows_f32_kernel   the same in true fp32 arithmetic (FMA);
+//   window_merge_kernel      joins the splits, the sink and the gate.
+// Page ids, positions and page-table columns are checked against their extents; a bad one sets PTB_ERR_BOUNDS and its key counts
+// as invisible.
+#include "window_attn.cuh"
+#include "flash_attn.cuh"
+#include <algorithm>
+
+namespace ptb {
+
+template <typename T> __device__ __forceinline__ float wa_f(T v);
+template <> __device__ __forceinline__ float wa_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ float wa_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T wa_t(float v);
+template <> __device__ __forceinline__ float wa_t<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 wa_t<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+// ---------------------------------------------------------------------------------------------- norm + page write
+struct ProjNormParams {
+    const void* x;
+    long long ld;
+    int q_col, k_col, v_col;
+    void* q_out;                       // [n, H, Dp], the pad filled with zeros
+    void* k_pages;
+    void* v_pages;
+    const float* qw;                   // [H D]
+    const float* kw;                   // [G D]
+    const int* pos;
+    const int* req;
+    const int* page_table;
+    int pos_stride, req_stride, pt_stride, n_pages;
+    int H, G, D, Dp, Dv, Dvp;
+    float eps;
+    int* status;
+};
+
+constexpr int PN_THREADS = 256;
+
+// E elements per access: 8 where sizes and columns are multiples of eight, else 1.  One CTA per row.
+template <typename T, int E>
+__global__ void __launch_bounds__(PN_THREADS) proj_norm_write_kernel(const __grid_constant__ ProjNormParams P) {
+    __shared__ float red[2][PN_THREADS / 32];
+    pdl_wait();
+    pdl_launch_dependents();
+    const size_t i = blockIdx.x;
+    const int pos = P.pos[i * P.pos_stride], col = pos / WA_PAGE, slot = pos % WA_PAGE;
+    int page = -1;
+    if (pos >= 0 && col < P.pt_stride) page = P.page_table[(size_t)P.req[i * P.req_stride] * P.pt_stride + col];
+    if (page < 0 || page >= P.n_pages) {
+        if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+        page = -1;
+    }
+    const T* row = (const T*)P.x + i * P.ld;
+    struct Vec { float v[E]; };
+    auto load = [&](const T* p) {
+        Vec r;
+        if constexpr (E == 8 && sizeof(T) == 2) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(p);
+            const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) { const float2 f = __bfloat1622float2(h[e]); r.v[2 * e] = f.x; r.v[2 * e + 1] = f.y; }
+        } else {
+#pragma unroll
+            for (int e = 0; e < E; ++e) r.v[e] = wa_f<T>(p[e]);
+        }
+        return r;
+    };
+    auto store = [&](T* p, const Vec& r) {
+        if constexpr (E == 8 && sizeof(T) == 2) {
+            uint4 raw;
+            __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) h[e] = __floats2bfloat162_rn(r.v[2 * e], r.v[2 * e + 1]);
+            *reinterpret_cast<uint4*>(p) = raw;
+        } else {
+#pragma unroll
+            for (int e = 0; e < E; ++e) p[e] = wa_t<T>(r.v[e]);
+        }
+    };
+    float sq = 0.f, sk = 0.f;
+    for (int c = threadIdx.x * E; c < P.H * P.D; c += PN_THREADS * E) {
+        const Vec f = load(row + P.q_col + c);
+#pragma unroll
+        for (int e = 0; e < E; ++e) sq += f.v[e] * f.v[e];
+    }
+    for (int c = threadIdx.x * E; c < P.G * P.D; c += PN_THREADS * E) {
+        const Vec f = load(row + P.k_col + c);
+#pragma unroll
+        for (int e = 0; e < E; ++e) sk += f.v[e] * f.v[e];
+    }
+    sq = warp_sum(sq); sk = warp_sum(sk);
+    if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sq; red[1][threadIdx.x >> 5] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < PN_THREADS / 32; ++w) { sq += red[0][w]; sk += red[1][w]; }
+    const float rq = rsqrtf(sq / (float)(P.H * P.D) + P.eps), rk = rsqrtf(sk / (float)(P.G * P.D) + P.eps);
+    // heads of `width` columns from src to heads of `padded` elements `pitch` apart
+    auto put = [&](const T* src, int heads, int width, int padded, T* dst, size_t pitch, const float* w, float rs) {
+        for (int c = threadIdx.x * E; c < heads * padded; c += PN_THREADS * E) {
+            const int h = c / padded, d = c % padded;
+            Vec f;
+#pragma unroll
+            for (int e = 0; e < E; ++e) f.v[e] = 0.f;
+            if (d < width) {
+                f = load(src + h * width + d);
+                if (w) {
+#pragma unroll
+                    for (int e = 0; e < E; ++e) f.v[e] *= rs * w[h * width + d + e];
+                }
+            }
+            store(dst + h * pitch + d, f);
+        }
+    };
+    put(row + P.q_col, P.H, P.D, P.Dp, (T*)P.q_out + i * P.H * P.Dp, P.Dp, P.qw, rq);
+    if (page < 0) return;
+    put(row + P.k_col, P.G, P.D, P.Dp, (T*)P.k_pages + ((size_t)page * P.G * WA_PAGE + slot) * P.Dp, (size_t)WA_PAGE * P.Dp, P.kw, rk);
+    put(row + P.v_col, P.G, P.Dv, P.Dvp, (T*)P.v_pages + ((size_t)page * P.G * WA_PAGE + slot) * P.Dvp, (size_t)WA_PAGE * P.Dvp, nullptr, 1.f);
+}
+
+// ---------------------------------------------------------------------------------------------- one query row
+// The cache slots (page * 64 + place, or -1) of the keys of split `split` of row `i`; returns their number.
+__device__ __forceinline__ int row_keys(const WindowAttnParams& P, int i, int split, int* krow) {
+    const int pos = P.pos[(size_t)i * P.pos_stride];
+    const Seen s = seen_by(pos, P.window, P.keep);
+    int per = (s.count + P.nsplit - 1) / P.nsplit;
+    if (pos < 0 || per > P.kcap) {                     // the host sizes the splits for the row that sees most
+        if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+        per = min(per, P.kcap);
+    }
+    const int e0 = split * per, nk = max(0, min(per, s.count - e0));
+    const int* table = P.page_table + (size_t)P.req[(size_t)i * P.req_stride] * P.pt_stride;
+    for (int e = threadIdx.x; e < P.kcap; e += blockDim.x) {
+        int v = -1;
+        if (e < nk) {
+            const int j = e0 + e < s.kept ? e0 + e : s.lo + e0 + e - s.kept, col = j / WA_PAGE;
+            const int page = col < P.pt_stride ? table[col] : -1;
+            if (page >= 0 && page < P.n_pages) v = page * WA_PAGE + j % WA_PAGE;
+            else if (P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+        }
+        krow[e] = v;
+    }
+    return nk;
+}
+__device__ __forceinline__ size_t cache_row(int krow, int G, int g) { return ((size_t)(krow / WA_PAGE) * G + g) * WA_PAGE + krow % WA_PAGE; }
+
+// Factor of a head's sum given its largest (log2) score and total: the sink joins the denominator, the gate multiplies.
+template <typename T>
+__device__ __forceinline__ float finish_factor(const WindowAttnParams& P, size_t i, int h, float m, float l) {
+    float M = m, f = 1.f;
+    if (P.sink) {
+        const float s = P.sink[h] * WA_LOG2E;
+        M = fmaxf(m, s);
+        f = m == -INFINITY ? 0.f : exp2f(m - M);
+        l = l * f + exp2f(s - M);
+    }
+    f = l > 0.f ? f / l : 0.f;
+    if (P.gate) f *= sigmoid(wa_f<T>(((const T*)P.gate)[i * P.gate_ld + h]));
+    return f;
+}
+
+constexpr int WR_THREADS = 128, WR_WARPS = 4;
+
+struct WindowSmem {
+    int v, q, w, hi, lo, ml, krow, pitch, ldw, ldh, total;      // byte offsets; pitches in bytes (v) and elements
+    __host__ __device__ WindowSmem(int R8, int Dp, int Dvp, int kcap, bool mma) {
+        pitch = Dvp * 2 + 16; ldw = kcap + 1; ldh = kcap + 8;
+        v = 0;
+        q = mma ? kcap * pitch : 0;
+        w = q + R8 * Dp * (mma ? 2 : 4);
+        hi = (w + R8 * ldw * 4 + 15) & ~15;
+        lo = hi + (mma ? R8 * ldh * 2 : 0);
+        ml = lo + (mma ? R8 * ldh * 2 : 0);
+        krow = ml + R8 * 8;
+        total = krow + kcap * 4;
+    }
+};
+
+__global__ void __launch_bounds__(WR_THREADS) window_rows_mma_kernel(const __grid_constant__ WindowAttnParams P) {
+    extern __shared__ __align__(16) unsigned char smem[];
+    const int R = P.H / P.G, RB = (R + 7) / 8, R8 = RB * 8;
+    const WindowSmem L(R8, P.Dp, P.Dvp, P.kcap, true);
+    __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem + L.q);
+    float* w_s = reinterpret_cast<float*>(smem + L.w);
+    __nv_bfloat16* hi_s = reinterpret_cast<__nv_bfloat16*>(smem + L.hi);
+    __nv_bfloat16* lo_s = reinterpret_cast<__nv_bfloat16*>(smem + L.lo);
+    float2* ml_s = reinterpret_cast<float2*>(smem + L.ml);
+    int* krow = reinterpret_cast<int*>(smem + L.krow);
+    const int split = blockIdx.x, c = blockIdx.y, i = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int nk = row_keys(P, i, split, krow);
+    {
+        const uint4* src = reinterpret_cast<const uint4*>((const __nv_bfloat16*)P.q + ((size_t)i * P.H + c * R) * P.Dp);
+        uint4* dst = reinterpret_cast<uint4*>(q_s);
+        for (int e = threadIdx.x; e < R8 * P.Dp / 8; e += WR_THREADS) dst[e] = e < R * P.Dp / 8 ? src[e] : make_uint4(0, 0, 0, 0);
+    }
+    __syncthreads();
+    const int kgroups = (nk + 15) / 16;
+    {                                                  // the values, while the scores are formed
+        const int vch = P.Dvp / 8;
+        const uint32_t v0 = smem_u32(smem + L.v);
+        for (int e = threadIdx.x; e < kgroups * 16 * vch; e += WR_THREADS) {
+            const int r = e / vch, ch = e % vch, kr = krow[r];
+            fa::cp_async16(v0 + (uint32_t)(r * L.pitch + ch * 16), (const __nv_bfloat16*)P.v_pages + (kr >= 0 ? cache_row(kr, P.G, c) * P.Dvp + ch * 8 : 0), kr >= 0);
+        }
+        fa::cp_async_commit();
+    }
+    // a lane's 16 bytes serve as its elements of two k16 steps of both operands, so the order inside a 32-element group cancels
+    const uint4 zero4 = make_uint4(0, 0, 0, 0);
+    const __nv_bfloat16* kp = (const __nv_bfloat16*)P.k_pages;
+    const int nch = P.Dp / 8;
+    for (int u = warp; u < RB * kgroups; u += WR_WARPS) {
+        const int kg = u % kgroups, rb = u / kgroups;
+        const int r0 = krow[kg * 16 + g], r1 = krow[kg * 16 + g + 8];
+        const uint4* k0 = reinterpret_cast<const uint4*>(kp + cache_row(max(r0, 0), P.G, c) * P.Dp);
+        const uint4* k1 = reinterpret_cast<const uint4*>(kp + cache_row(max(r1, 0), P.G, c) * P.Dp);
+        const uint4* qv = reinterpret_cast<const uint4*>(q_s + (size_t)(rb * 8 + g) * P.Dp);
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int b0 = 0; b0 < nch; b0 += 16) {
+            uint4 a[4], b[4];
+#pragma unroll
+            for (int s = 0; s < 4; ++s) {
+                const int ch = b0 + s * 4 + t;
+                a[s] = (ch < nch && r0 >= 0) ? k0[ch] : zero4;
+                b[s] = (ch < nch && r1 >= 0) ? k1[ch] : zero4;
+            }
+#pragma unroll
+            for (int s = 0; s < 4; ++s) {
+                const int ch = b0 + s * 4 + t;
+                if (b0 + s * 4 < nch) {
+                    const uint4 q4 = ch < nch ? qv[ch] : zero4;
+                    const uint32_t f0[4] = {a[s].x, b[s].x, a[s].y, b[s].y}, f1[4] = {a[s].z, b[s].z, a[s].w, b[s].w};
+                    fa::mma16816(acc, f0, q4.x, q4.y);
+                    fa::mma16816(acc, f1, q4.z, q4.w);
+                }
+            }
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+            w_s[(rb * 8 + 2 * t + (e & 1)) * L.ldw + kg * 16 + g + (e >> 1) * 8] = ((e >> 1) ? r1 : r0) >= 0 ? acc[e] * P.scale_log2 : -INFINITY;
+    }
+    __syncthreads();
+    for (int h = warp; h < R8; h += WR_WARPS) {
+        float m = -INFINITY, l = 0.f;
+        for (int j = lane; j < kgroups * 16; j += 32) m = fmaxf(m, w_s[h * L.ldw + j]);
+        m = warp_max(m);
+        const float base = m == -INFINITY ? 0.f : m;
+        for (int j = lane; j < kgroups * 16; j += 32) {
+            const float p = h < R ? exp2f(w_s[h * L.ldw + j] - base) : 0.f;
+            const __nv_bfloat16 hi = __float2bfloat16_rn(p);
+            hi_s[h * L.ldh + j] = hi;
+            lo_s[h * L.ldh + j] = __float2bfloat16_rn(p - __bfloat162float(hi));
+            l += p;
+        }
+        l = warp_sum(l);
+        if (lane == 0) ml_s[h] = make_float2(m, l);
+    }
+    fa::cp_async_wait<0>();
+    __syncthreads();
+    // rows 0-7 of the left operand carry the high halves of eight heads' weights, rows 8-15 the low halves; columns are values
+    const uint32_t v0 = smem_u32(smem + L.v);
+    const int DC = (P.Dvp + 31) / 32;
+    for (int u = warp; u < RB * DC; u += WR_WARPS) {
+        const int dc = u % DC, rb = u / DC;
+        const bool two = dc * 32 + 16 < P.Dvp;         // Dvp is a multiple of 16
+        const __nv_bfloat16* hi_r = hi_s + (rb * 8 + g) * L.ldh + 2 * t;
+        const __nv_bfloat16* lo_r = lo_s + (rb * 8 + g) * L.ldh + 2 * t;
+        float acc[4][4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) acc[e][k] = 0.f;
+        for (int kg = 0; kg < kgroups; ++kg) {
+            uint32_t a[4];
+            a[0] = *reinterpret_cast<const uint32_t*>(hi_r + kg * 16);
+            a[1] = *reinterpret_cast<const uint32_t*>(lo_r + kg * 16);
+            a[2] = *reinterpret_cast<const uint32_t*>(hi_r + kg * 16 + 8);
+            a[3] = *reinterpret_cast<const uint32_t*>(lo_r + kg * 16 + 8);
+            const uint32_t at = v0 + (uint32_t)((kg * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * L.pitch + (dc * 4 + (lane >> 4)) * 16);
+            uint32_t b[4];
+            fa::ldsm4_t(at, b[0], b[1], b[2], b[3]);
+            fa::mma16816(acc[0], a, b[0], b[1]);
+            fa::mma16816(acc[1], a, b[2], b[3]);
+            if (two) {
+                fa::ldsm4_t(at + 32, b[0], b[1], b[2], b[3]);
+                fa::mma16816(acc[2], a, b[0], b[1]);
+                fa::mma16816(acc[3], a, b[2], b[3]);
+            }
+        }
+        const int hl = rb * 8 + g, h = c * R + hl;
+        if (hl >= R) continue;
+        const float2 ml = ml_s[hl];
+        const float f = P.nsplit > 1 ? 1.f : finish_factor<__nv_bfloat16>(P, i, h, ml.x, ml.y);
+        float* wk = P.work + (((size_t)i * P.nsplit + split) * P.H + h) * (P.Dvp + 2);
+        __nv_bfloat16* o = (__nv_bfloat16*)P.out + ((size_t)i * P.H + h) * P.Dv;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int d = dc * 32 + e * 8 + 2 * t;
+            const float x = acc[e][0] + acc[e][2], y = acc[e][1] + acc[e][3];
+            if (P.nsplit > 1) {
+                if (d < P.Dvp) *reinterpret_cast<float2*>(wk + d) = make_float2(x, y);
+            } else {
+                if (d < P.Dv) o[d] = __float2bfloat16_rn(x * f);
+                if (d + 1 < P.Dv) o[d + 1] = __float2bfloat16_rn(y * f);
+            }
+        }
+        if (P.nsplit > 1 && dc == 0 && t == 0) *reinterpret_cast<float2*>(wk + P.Dvp) = ml;
+    }
+}
+
+__global__ void __launch_bounds__(WR_THREADS) window_rows_f32_kernel(const __grid_constant__ WindowAttnParams P) {
+    extern __shared__ __align__(16) unsigned char smem[];
+    const int R = P.H / P.G, R8 = (R + 7) / 8 * 8;
+    const WindowSmem L(R8, P.Dp, P.Dvp, P.kcap, false);
+    float* q_s = reinterpret_cast<float*>(smem + L.q);
+    float* w_s = reinterpret_cast<float*>(smem + L.w);
+    float2* ml_s = reinterpret_cast<float2*>(smem + L.ml);
+    int* krow = reinterpret_cast<int*>(smem + L.krow);
+    const int split = blockIdx.x, c = blockIdx.y, i = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int nk = row_keys(P, i, split, krow);
+    for (int e = threadIdx.x; e < R * P.Dp; e += WR_THREADS) q_s[e] = ((const float*)P.q)[((size_t)i * P.H + c * R) * P.Dp + e];
+    __syncthreads();
+    for (int e = threadIdx.x; e < R * nk; e += WR_THREADS) {
+        const int h = e / nk, j = e % nk, r = krow[j];
+        float s = -INFINITY;
+        if (r >= 0) {
+            const float4* k4 = reinterpret_cast<const float4*>((const float*)P.k_pages + cache_row(r, P.G, c) * P.Dp);
+            const float4* q4 = reinterpret_cast<const float4*>(q_s + (size_t)h * P.Dp);
+            float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int d = 0; d < P.Dp / 4; ++d) {
+                const float4 x = k4[d], y = q4[d];
+                a.x = fmaf(x.x, y.x, a.x); a.y = fmaf(x.y, y.y, a.y); a.z = fmaf(x.z, y.z, a.z); a.w = fmaf(x.w, y.w, a.w);
+            }
+            s = ((a.x + a.y) + (a.z + a.w)) * P.scale_log2;
+        }
+        w_s[h * L.ldw + j] = s;
+    }
+    __syncthreads();
+    for (int h = warp; h < R; h += WR_WARPS) {
+        float m = -INFINITY, l = 0.f;
+        for (int j = lane; j < nk; j += 32) m = fmaxf(m, w_s[h * L.ldw + j]);
+        m = warp_max(m);
+        for (int j = lane; j < nk; j += 32) {
+            const float p = exp2f(w_s[h * L.ldw + j] - (m == -INFINITY ? 0.f : m));
+            w_s[h * L.ldw + j] = p;
+            l += p;
+        }
+        l = warp_sum(l);
+        if (lane == 0) ml_s[h] = make_float2(m, l);
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < R * P.Dvp; e += WR_THREADS) {
+        const int hl = e / P.Dvp, d = e % P.Dvp, h = c * R + hl;
+        float a = 0.f;
+        for (int j = 0; j < nk; ++j)
+            if (krow[j] >= 0) a = fmaf(w_s[hl * L.ldw + j], ((const float*)P.v_pages)[cache_row(krow[j], P.G, c) * P.Dvp + d], a);
+        const float2 ml = ml_s[hl];
+        float* wk = P.work + (((size_t)i * P.nsplit + split) * P.H + h) * (P.Dvp + 2);
+        if (P.nsplit > 1) {
+            wk[d] = a;
+            if (d == 0) *reinterpret_cast<float2*>(wk + P.Dvp) = ml;
+        } else if (d < P.Dv) ((float*)P.out)[((size_t)i * P.H + h) * P.Dv + d] = a * finish_factor<float>(P, i, h, ml.x, ml.y);
+    }
+}
+
+// One CTA per (head, row).
+template <typename T>
+__global__ void __launch_bounds__(128) window_merge_kernel(const __grid_constant__ WindowAttnParams P) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int h = blockIdx.x;
+    const size_t i = blockIdx.y, pitch = (size_t)P.H * (P.Dvp + 2);
+    const float* wk = P.work + i * P.nsplit * pitch + (size_t)h * (P.Dvp + 2);
+    float M = -INFINITY, l = 0.f;
+    for (int s = 0; s < P.nsplit; ++s) M = fmaxf(M, wk[s * pitch + P.Dvp]);
+    const float base = M == -INFINITY ? 0.f : M;
+    for (int s = 0; s < P.nsplit; ++s) l += wk[s * pitch + P.Dvp + 1] * exp2f(wk[s * pitch + P.Dvp] - base);
+    const float f = finish_factor<T>(P, i, h, M, l);
+    for (int d = threadIdx.x; d < P.Dv; d += blockDim.x) {
+        float a = 0.f;
+#pragma unroll 4
+        for (int s = 0; s < P.nsplit; ++s) a += wk[s * pitch + d] * exp2f(wk[s * pitch + P.Dvp] - base);
+        ((T*)P.out)[(i * P.H + h) * P.Dv + d] = wa_t<T>(a * f);
+    }
+}
+
+}  // namespace ptb
+
+using namespace ptb;
+
+// After the packed projection x [n, *] (pitch ld; q, k and v rows at the three columns): q_out [n, H, Dp] = q / rms(q) * qw over all H D
+// columns together; k, normed over its G D columns with kw, and v go to the page slot of (req, pos).  Dp, Dvp: sizes as stored,
+// multiples of 16; the pad is zero.
+PTB_API int ptb_proj_norm_write(const void* x, long long ld, int q_col, int k_col, int v_col, void* q_out, void* k_pages, void* v_pages,
+                                const float* qw, const float* kw, const int* pos, int pos_stride, const int* req, int req_stride,
+                                const int* page_table, int pt_stride, int n_pages, int n, int H, int G, int D, int Dp, int Dv, int Dvp, float eps,
+                                int* status, int bf16, cudaStream_t st) {
+    if (n <= 0) return 0;
+    if (H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || Dp % 16 || Dvp % 16 || Dp < D || Dvp < Dv) {
+        ptb_set_error("proj_norm_write: bad sizes (H %d, G %d, D %d/%d, Dv %d/%d)", H, G, D, Dp, Dv, Dvp);
+        return -1;
+    }
+    ProjNormParams p{x, ld, q_col, k_col, v_col, q_out, k_pages, v_pages, qw, kw, pos, req, page_table, pos_stride, req_stride, pt_stride, n_pages,
+                     H, G, D, Dp, Dv, Dvp, eps, status};
+    const bool vec = D % 8 == 0 && Dv % 8 == 0 && ld % 8 == 0 && q_col % 8 == 0 && k_col % 8 == 0 && v_col % 8 == 0 && ((uintptr_t)x & 15) == 0;
+    const bool pdl = ptb_pdl_enabled();
+    if (bf16) PTB_CUDA_OK(ptb_launch(vec ? proj_norm_write_kernel<__nv_bfloat16, 8> : proj_norm_write_kernel<__nv_bfloat16, 1>, dim3(n), dim3(PN_THREADS), 0, st, pdl, p));
+    else PTB_CUDA_OK(ptb_launch(proj_norm_write_kernel<float, 1>, dim3(n), dim3(PN_THREADS), 0, st, pdl, p));
+    PTB_CUDA_OK(cudaGetLastError());
+    return 0;
+}
+
+// Floats of workspace the row kernels need for `nsplit` > 1.
+PTB_API long long ptb_window_rows_work_floats(int n, int H, int Dvp, int nsplit) { return nsplit > 1 ? (long long)n * nsplit * H * (Dvp + 2) : 0; }
+
+// Query rows q [n, H, Dp], each at its own position of its own sequence, against the cached keys it sees.  max_keys: the most keys any
+// row sees; nsplit CTAs share a row's keys (at most WA_KEYS each).  out [n, H Dv] in the type of q.
+PTB_API int ptb_window_attn_rows(const void* q, void* out, int n, int H, int G, int Dp, int Dv, int Dvp, const int* pos, int pos_stride,
+                                 const int* req, int req_stride, const int* page_table, int pt_stride, int n_pages, const void* k_pages,
+                                 const void* v_pages, const float* sink, const void* gate, long long gate_ld, int window, int keep, float scale,
+                                 int max_keys, float* work, int nsplit, int* status, int bf16, cudaStream_t st) {
+    if (n <= 0) return 0;
+    if (G <= 0 || H % G || Dp % 16 || Dvp % 16 || window < 1 || keep < 0 || G > 65535) {
+        ptb_set_error("window attention: bad sizes (H %d, G %d, Dp %d, Dvp %d, window %d, keep %d)", H, G, Dp, Dvp, window, keep);
+        return -1;
+    }
+    const int per = (std::max(1, max_keys) + nsplit - 1) / std::max(1, nsplit);
+    if (nsplit < 1 || per > WA_KEYS || (nsplit > 1 && !work)) {
+        ptb_set_error("window attention: %d splits for %d keys (at most %d keys per split, workspace needed above one)", nsplit, max_keys, WA_KEYS);
+        return -1;
+    }
+    if (n > 65535) { ptb_set_error("window attention: %d rows in one launch", n); return -1; }
+    WindowAttnParams p;
+    p.q = q; p.out = out; p.work = work; p.pos = pos; p.req = req; p.page_table = page_table; p.k_pages = k_pages; p.v_pages = v_pages;
+    p.sink = sink; p.gate = gate; p.gate_ld = gate_ld; p.pos_stride = pos_stride; p.req_stride = req_stride; p.pt_stride = pt_stride;
+    p.n_pages = n_pages; p.n = n; p.H = H; p.G = G; p.Dp = Dp; p.Dv = Dv; p.Dvp = Dvp; p.window = window; p.keep = keep; p.nsplit = nsplit;
+    p.kcap = (per + 15) & ~15; p.scale_log2 = scale * WA_LOG2E; p.status = status;
+    const int R8 = (H / G + 7) / 8 * 8;
+    const WindowSmem L(R8, Dp, Dvp, p.kcap, bf16 != 0);
+    if (L.total > 227 * 1024) { ptb_set_error("window attention: %d heads of %d need %d bytes of shared memory", H / G, Dp, L.total); return -1; }
+    auto kern = bf16 ? window_rows_mma_kernel : window_rows_f32_kernel;
+    if (L.total > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    const bool pdl = ptb_pdl_enabled();
+    PTB_CUDA_OK(ptb_launch(kern, dim3(nsplit, G, n), dim3(WR_THREADS), (size_t)L.total, st, pdl, p));
+    if (nsplit > 1) {
+        if (bf16) PTB_CUDA_OK(ptb_launch(window_merge_kernel<__nv_bfloat16>, dim3(H, n), dim3(128), 0, st, pdl, p));
+        else PTB_CUDA_OK(ptb_launch(window_merge_kernel<float>, dim3(H, n), dim3(128), 0, st, pdl, p));
+    }
+    PTB_CUDA_OK(cudaGetLastError());
+    return 0;
+}

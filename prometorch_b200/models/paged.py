@@ -1,7 +1,7 @@
 """What the batching engine (``serve/llm.py``) asks of a model, and the registry that finds the model for a ``config.json``.
 
-The engine owns requests, the page table, the page pool, CUDA graphs and sampling.  A model owns its weights and the device work
-of two passes over the engine's paged cache: a prompt pass (many tokens of several sequences) and a decode pass (one token per
+The engine owns requests, the page table, the page pool, recurrent states, CUDA graphs and sampling.  A model owns its weights and
+the device work of two passes over the engine's cache: a prompt pass (many tokens of several sequences) and a decode pass (one token per
 batch row).  A new design is a :class:`PagedModel` with a configuration and a weights class, registered under the name its
 ``config.json`` carries."""
 from __future__ import annotations
@@ -30,10 +30,41 @@ class PromptBatch:
         return [b - a for a, b in zip(self.offs, self.offs[1:])]
 
 
+class RowPack:
+    """Matrices that read the same input, stacked by rows into one: ``sizes`` maps names to row counts.  Every part starts at a
+    multiple of eight rows and the whole has one (what the projection kernel and 16-byte loads of its output ask for); the gaps
+    are zeros.  ``at[name]``: a part's first column in the product."""
+
+    def __init__(self, sizes: Dict[str, int]):
+        self.sizes, self.at, self.rows = dict(sizes), {}, 0
+        for n, k in sizes.items():
+            self.at[n] = self.rows
+            self.rows += self.up(k)
+
+    @staticmethod
+    def up(n: int) -> int:
+        return -(-n // 8) * 8
+
+    @staticmethod
+    def pad(t: torch.Tensor) -> torch.Tensor:
+        """``t`` with rows of zeros up to a multiple of eight."""
+        more = RowPack.up(t.shape[0]) - t.shape[0]
+        return torch.cat([t, t.new_zeros((more,) + tuple(t.shape[1:]))]) if more else t.contiguous()
+
+    def pack(self, parts: Dict[str, torch.Tensor]) -> torch.Tensor:
+        return torch.cat([self.pad(parts[n]) for n in self.sizes])
+
+    def cols(self, product: torch.Tensor, name: str, padded: bool = False) -> torch.Tensor:
+        """A part's columns of ``product [n, rows]`` (a view); ``padded``: up to the next multiple of eight."""
+        k = self.sizes[name]
+        return product[:, self.at[name]:self.at[name] + (self.up(k) if padded else k)]
+
+
 class PagedModel:
     """Base class: ``cfg`` must have ``vocab_size``, ``max_position_embeddings``, ``bos_token_id`` and ``eos_token_id``."""
     architecture = ""
     continues_prompts = False          # whether a prompt pass may start behind cached tokens
+    rewinds = True                     # whether a decoded token can be taken back by decoding another one at its position
 
     def __init__(self, weights, device, dtype):
         self.cfg = weights.cfg
@@ -43,6 +74,15 @@ class PagedModel:
     def kv_shapes(self) -> List[Tuple[int, int, int]]:
         """(kv heads, key size, value size) of every layer's cache, in elements as stored."""
         raise NotImplementedError
+
+    def state_shapes(self) -> List[Dict[str, Tuple[tuple, torch.dtype]]]:
+        """What each layer keeps per sequence besides pages: name -> (shape, dtype).  The engine holds one slot of it per page-table
+        row; a pass whose first token stands at position 0 takes the slot's content as zero."""
+        return [{} for _ in self.kv_shapes()]
+
+    def kept_tokens(self) -> int:
+        """How many of a sequence's first tokens stay readable whatever :meth:`cache_window` says."""
+        return 0
 
     def cache_window(self) -> Optional[int]:
         """How many of the latest tokens any layer can still read (None: all of them).  Pages that lie behind go back to the
@@ -80,7 +120,7 @@ def register_model(config: type, weights: type, model: type, *names: str) -> Non
 
 
 def _ensure_builtin():
-    from . import kifusun, llama_paged  # noqa: F401  (they register themselves)
+    from . import gelutar, kifusun, llama_paged  # noqa: F401  (they register themselves)
 
 
 def known_models() -> List[str]:

@@ -15,7 +15,7 @@ import torch
 
 from .. import _native as N
 
-EPI_BIAS, EPI_ACCUM, EPI_OUT_F32, EPI_GELU, EPI_SCATTER_ADD, EPI_SCATTER_STORE = 1, 2, 4, 8, 16, 32
+EPI_BIAS, EPI_ACCUM, EPI_OUT_F32, EPI_GELU, EPI_SCATTER_ADD, EPI_SCATTER_STORE, EPI_RELU2 = 1, 2, 4, 8, 16, 32, 128
 
 
 @N.register_decls
@@ -72,8 +72,9 @@ def _rowmajor(t):
 
 
 def gemm_bf16(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = False, out: Optional[torch.Tensor] = None,
-              bias: Optional[torch.Tensor] = None, accumulate: bool = False, out_dtype=torch.bfloat16, gelu: bool = False):
-    """``C[M,N] (+)= A B^T``.  ``a``: ``[M,K]`` (or ``[K,M]`` with ``a_mn``); ``b``: ``[N,K]`` (or ``[K,N]`` with ``b_mn``)."""
+              bias: Optional[torch.Tensor] = None, accumulate: bool = False, out_dtype=torch.bfloat16, gelu: bool = False,
+              relu2: bool = False):
+    """``C[M,N] (+)= A B^T``, optionally through tanh-GELU or the square of ReLU.  ``a``: ``[M,K]`` (or ``[K,M]`` with ``a_mn``); ``b``: ``[N,K]`` (or ``[K,N]`` with ``b_mn``)."""
     a, b = _rowmajor(a), _rowmajor(b)
     if a.dtype != torch.bfloat16 or b.dtype != torch.bfloat16 or not a.is_cuda:
         raise TypeError("gemm_bf16 takes CUDA bf16 operands")
@@ -92,11 +93,11 @@ def gemm_bf16(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: boo
             work = torch.empty(splits * M * Nn, dtype=torch.float32, device=a.device)
             st = torch.cuda.current_stream(a.device).cuda_stream
             N.check(N.lib().ptb_gemm_bf16_splitk(a.data_ptr(), a.stride(0), b.data_ptr(), b.stride(0), out.data_ptr(), out.stride(0), M, Nn,
-                                                 K, N.ptr(bias.float().contiguous() if bias is not None else None), int(gelu), splits,
+                                                 K, N.ptr(bias.float().contiguous() if bias is not None else None), 2 if relu2 else int(gelu), splits,
                                                  work.data_ptr(), _status(a.device).data_ptr(), 0, st), "gemm_bf16_splitk")
             return out
     flags = (EPI_BIAS if bias is not None else 0) | (EPI_ACCUM if accumulate else 0) | \
-        (EPI_OUT_F32 if out.dtype == torch.float32 else 0) | (EPI_GELU if gelu else 0)
+        (EPI_OUT_F32 if out.dtype == torch.float32 else 0) | (EPI_GELU if gelu else 0) | (EPI_RELU2 if relu2 else 0)
     if bias is not None:
         bias = bias.float().contiguous()
     st = torch.cuda.current_stream(a.device).cuda_stream
@@ -138,6 +139,13 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] =
     if x.is_cuda and x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and x.shape[-1] % 8 == 0 and weight.shape[0] % 8 == 0:
         return _Linear.apply(x, weight, bias)
     return torch.nn.functional.linear(x, weight, bias)
+
+
+def linear_relu2(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """``relu(x W^T)^2`` (inference path, no autograd); on the tcgen05 kernel the activation runs in its epilogue."""
+    if x.is_cuda and x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and x.shape[-1] % 8 == 0 and weight.shape[0] % 8 == 0:
+        return gemm_bf16(x, weight, relu2=True)
+    return torch.relu(torch.nn.functional.linear(x, weight)).square()
 
 
 def _skinny_splits(x: torch.Tensor, w: torch.Tensor) -> int:

@@ -1,0 +1,192 @@
+"""Softmax attention over the paged cache inside a sliding window (csrc/window_attn.cu, csrc/window_attn_sm100.cu), with what designs
+add to it: the first tokens of a sequence stay visible, a learned sink joins every head's denominator, a gate scales every head's
+output.
+
+:class:`WindowAttention` holds what a layer fixes; :func:`proj_norm_write` normalises the whole q and k projections of new tokens
+and fills the pages; :func:`window_attention` runs query rows at given positions against the pages, :func:`window_attention_tiles`
+the many rows of a prompt.  CUDA tensors run the kernels, CPU tensors the plain math."""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass
+from typing import List, Optional, Tuple
+
+import torch
+
+from .. import _native as N
+from .paged import PAGE, _status
+
+KEYS_PER_CTA = 128                     # WA_KEYS of csrc/window_attn.cuh
+UNBOUNDED = 1 << 30                    # a window that never ends
+
+
+@N.register_decls
+def _decls(L):
+    vp, ci, cf, ll = C.c_void_p, C.c_int, C.c_float, C.c_longlong
+    L.ptb_proj_norm_write.argtypes = [vp, ll, ci, ci, ci, vp, vp, vp, vp, vp, vp, ci, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, ci, cf, vp, ci, vp]
+    L.ptb_proj_norm_write.restype = ci
+    L.ptb_window_rows_work_floats.argtypes = [ci, ci, ci, ci]
+    L.ptb_window_rows_work_floats.restype = ll
+    L.ptb_window_attn_rows.argtypes = [vp, vp, ci, ci, ci, ci, ci, ci, vp, ci, vp, ci, vp, ci, ci, vp, vp, vp, vp, ll, ci, ci, cf, ci, vp, ci, vp, ci, vp]
+    L.ptb_window_attn_rows.restype = ci
+    if not hasattr(L, 'ptb_window_attn_tiles'): return  # TMP
+    L.ptb_window_attn_tiles.argtypes = [vp, vp, ci, vp, ci, ci, ci, ci, ci, ci, vp, ci, ci, vp, vp, vp, vp, ll, ci, ci, cf, vp, vp]
+    L.ptb_window_attn_tiles.restype = ci
+
+
+def stored(size: int) -> int:
+    """Size of a head's vector as the cache stores it: the kernels address 16-element groups."""
+    return (size + 15) // 16 * 16
+
+
+@dataclass
+class WindowAttention:
+    heads: int
+    kv_heads: int
+    dim: int                           # query / key size per head
+    vdim: int                          # value size per head
+    window: int                        # a query sees itself and the window - 1 tokens before it
+    keep: int                          # ... and the first `keep` tokens of its sequence
+    scale: float
+    sink: Optional[torch.Tensor] = None      # [heads] fp32: exp(sink) joins the denominator
+
+    @property
+    def dim_stored(self) -> int:
+        return stored(self.dim)
+
+    @property
+    def vdim_stored(self) -> int:
+        return stored(self.vdim)
+
+    def most_keys(self, max_len: int) -> int:
+        """The most keys a row at a position below ``max_len`` sees."""
+        return max(1, min(max_len, self.window + self.keep))
+
+
+def proj_norm_write(p: torch.Tensor, cols: Tuple[int, int, int], a: WindowAttention, q_weight: torch.Tensor, k_weight: torch.Tensor, eps: float,
+                    pos: torch.Tensor, req: torch.Tensor, page_table: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor) -> torch.Tensor:
+    """``p [n, *]``: a packed projection whose q, k and v rows start at the columns ``cols``.  q ``[n, H, stored dim]`` after an RMS
+    norm over all its heads together (fp32 weight ``[H dim]``); k, normed the same way, and v go to the page slot of
+    ``(req[i], pos[i])``.  ``pos`` / ``req``: int32 vectors of any stride."""
+    n, H, G, D, Dv, Dp, Dvp = p.shape[0], a.heads, a.kv_heads, a.dim, a.vdim, a.dim_stored, a.vdim_stored
+    q = torch.empty(n, H, Dp, dtype=p.dtype, device=p.device)
+    if p.is_cuda:
+        if p.dtype not in (torch.bfloat16, torch.float32):
+            raise TypeError(f"proj_norm_write takes bf16 or fp32, got {p.dtype}")
+        assert p.stride(1) == 1 and pos.dtype == req.dtype == page_table.dtype == torch.int32
+        st = torch.cuda.current_stream(p.device).cuda_stream
+        N.check(N.lib().ptb_proj_norm_write(p.data_ptr(), p.stride(0), *cols, q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), q_weight.data_ptr(),
+                                            k_weight.data_ptr(), pos.data_ptr(), pos.stride(0), req.data_ptr(), req.stride(0), page_table.data_ptr(),
+                                            page_table.stride(0), k_pages.shape[0], n, H, G, D, Dp, Dv, Dvp, float(eps), _status(p.device).data_ptr(),
+                                            int(p.dtype == torch.bfloat16), st), "proj_norm_write")
+        return q
+    x = p.float()
+
+    def norm(at, heads, w):
+        t = x[:, at:at + heads * D]
+        return (t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * w).reshape(n, heads, D)
+    q.zero_()
+    q[..., :D] = norm(cols[0], H, q_weight).to(q.dtype)
+    at = pos.long()
+    pages = page_table[req.long(), at // PAGE].long()
+    k_pages[pages, :, at % PAGE] = torch.nn.functional.pad(norm(cols[1], G, k_weight), (0, Dp - D)).to(k_pages.dtype)
+    v_pages[pages, :, at % PAGE] = torch.nn.functional.pad(x[:, cols[2]:cols[2] + G * Dv].reshape(n, G, Dv), (0, Dvp - Dv)).to(v_pages.dtype)
+    return q
+
+
+def pick_splits(rows: int, kv_heads: int, keys: int, sms: int = 148) -> int:
+    """CTAs that share a row's keys: as many as bring the grid to about four per SM while a CTA keeps 32 keys, and at least as many
+    as the kernel's limit of keys per CTA asks for.  The number of keys is rounded up to a power of two so that the choice (part of
+    a CUDA graph's key) changes rarely as a context grows."""
+    bucket = 32
+    while bucket < keys:
+        bucket *= 2
+    need = (bucket + KEYS_PER_CTA - 1) // KEYS_PER_CTA
+    return int(max(need, min(bucket // 32, -(-4 * sms // max(1, rows * kv_heads)))))
+
+
+def window_attention(q: torch.Tensor, a: WindowAttention, pos: torch.Tensor, req: torch.Tensor, page_table: torch.Tensor, k_pages: torch.Tensor,
+                     v_pages: torch.Tensor, nsplit: int, max_len: int, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Rows ``q [n, H, stored dim]`` at ``pos`` of the sequences in page-table rows ``req``, against their cached tokens (their own
+    included).  ``max_len``: no row's position is at or past it.  ``gate [n, H]`` (any row pitch): its sigmoid scales the heads.
+    Returns ``[n, H vdim]``."""
+    n, H, G = q.shape[0], a.heads, a.kv_heads
+    if not q.is_cuda:
+        return window_attention_reference(q, a, pos, req, page_table, k_pages, v_pages, gate)
+    out = torch.empty(n, H * a.vdim, dtype=q.dtype, device=q.device)
+    st = torch.cuda.current_stream(q.device).cuda_stream
+    per_row = int(N.lib().ptb_window_rows_work_floats(1, H, a.vdim_stored, nsplit))
+    step = n if nsplit == 1 else max(1, min(n, (256 << 20) // max(1, 4 * per_row)))       # bound the workspace
+    step = min(step, 65535)
+    work = torch.empty(step * per_row, dtype=torch.float32, device=q.device) if nsplit > 1 else None
+    for lo in range(0, n, step):
+        m = min(step, n - lo)
+        N.check(N.lib().ptb_window_attn_rows(q[lo:].data_ptr(), out[lo:].data_ptr(), m, H, G, a.dim_stored, a.vdim, a.vdim_stored, pos[lo:].data_ptr(),
+                                             pos.stride(0), req[lo:].data_ptr(), req.stride(0), page_table.data_ptr(), page_table.stride(0),
+                                             k_pages.shape[0], k_pages.data_ptr(), v_pages.data_ptr(), N.ptr(a.sink),
+                                             gate[lo:].data_ptr() if gate is not None else 0, gate.stride(0) if gate is not None else 0, a.window, a.keep,
+                                             float(a.scale), a.most_keys(max_len), N.ptr(work), nsplit, _status(q.device).data_ptr(),
+                                             int(q.dtype == torch.bfloat16), st), "window_attn_rows")
+    return out
+
+
+QUERY_TILE = 128                       # queries per tile of csrc/window_attn_sm100.cu
+TILES_FROM = 16                        # rows of a prompt pass from which the tile kernel is the better choice
+
+
+@dataclass
+class PromptTiles:
+    """The query tiles of a prompt pass: on the device ``[tiles, 4]`` int32 (first row, its position, rows, page-table row), tiles
+    with many keys first."""
+    host: List[Tuple[int, int, int, int]]
+    device: torch.Tensor
+
+    @classmethod
+    def of(cls, offs: List[int], starts: List[int], rows: List[int], device) -> "PromptTiles":
+        host = [(lo + i, at + i, min(QUERY_TILE, hi - lo - i), r) for lo, hi, at, r in zip(offs, offs[1:], starts, rows)
+                for i in range(0, hi - lo, QUERY_TILE)]
+        host.sort(key=lambda t: -t[1])
+        return cls(host, torch.tensor(host, dtype=torch.int32).to(device))
+
+
+def tiles_supported(q: torch.Tensor, a: WindowAttention) -> bool:
+    return hasattr(N.lib(), 'ptb_window_attn_tiles') and q.is_cuda and q.dtype == torch.bfloat16 and a.dim_stored <= 128 and a.vdim_stored <= 128
+
+
+def window_attention_tiles(q: torch.Tensor, a: WindowAttention, tiles: PromptTiles, page_table: torch.Tensor, k_pages: torch.Tensor,
+                           v_pages: torch.Tensor, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """A prompt pass's rows against the pages, both products on tcgen05 (sizes: :func:`tiles_supported`)."""
+    H, n, nt = a.heads, q.shape[0], len(tiles.host)
+    out = torch.empty(n, H * a.vdim, dtype=q.dtype, device=q.device)
+    st = torch.cuda.current_stream(q.device).cuda_stream
+    N.check(N.lib().ptb_window_attn_tiles(q.data_ptr(), out.data_ptr(), n, tiles.device.data_ptr(), nt, H, a.kv_heads, a.dim_stored, a.vdim, a.vdim_stored,
+                                          page_table.data_ptr(), page_table.stride(0), k_pages.shape[0], k_pages.data_ptr(), v_pages.data_ptr(),
+                                          N.ptr(a.sink), N.ptr(gate), gate.stride(0) if gate is not None else 0, a.window, a.keep, float(a.scale),
+                                          _status(q.device).data_ptr(), st), "window_attn_tiles")
+    return out
+
+
+def window_attention_reference(q, a: WindowAttention, pos, req, page_table, k_pages, v_pages, gate=None) -> torch.Tensor:
+    """The same in plain fp32 math, sequence by sequence (CPU path).  Pages between the kept tokens and the first window are gone."""
+    n, H, G, D, Dv = q.shape[0], a.heads, a.kv_heads, a.dim, a.vdim
+    out = torch.zeros(n, H * Dv, dtype=q.dtype, device=q.device)
+    R = H // G
+    for r in torch.unique(req).tolist():
+        rows = (req == r).nonzero()[:, 0]
+        p = pos[rows].long()
+        top, first = int(p.max()) + 1, max(0, int(p.min()) - a.window + 1)
+        j = torch.cat([torch.arange(0, min(a.keep, first)), torch.arange(first, top)]).to(q.device)
+        pages = page_table[r, j // PAGE].long()
+        k = k_pages[pages, :, j % PAGE].float()[..., :D].transpose(0, 1).repeat_interleave(R, 0)          # [H, keys, D]
+        v = v_pages[pages, :, j % PAGE].float()[..., :Dv].transpose(0, 1).repeat_interleave(R, 0)
+        dist = p[:, None] - j[None, :]
+        s = torch.einsum("nhd,hjd->hnj", q[rows][..., :D].float(), k) * a.scale
+        s = s.masked_fill(~((dist >= 0) & ((dist < a.window) | (j[None, :] < a.keep))), float("-inf"))
+        if a.sink is not None:
+            s = torch.cat([s, a.sink.float()[:, None, None].expand(H, len(rows), 1)], -1)
+        w = torch.softmax(s, -1)[..., :len(j)]
+        o = torch.einsum("hnj,hjd->nhd", w, v)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[rows].float())[..., None]
+        out[rows] = o.reshape(len(rows), H * Dv).to(q.dtype)
+    return out

@@ -1,5 +1,5 @@
 """Continuous-batching engine with a paged KV cache for the models registered in ``models/paged.py`` (Hugging Face Llama
-checkpoints, Kifusun).
+checkpoints, Kifusun, Gelutar).
 
 Same public surface as the reference's ``LLMEngine`` (torch/serve/llm.h:33-57 for the request types, :299-334 for the
 64-token page pool, :352-437 for ``load / set_weights / generate / submit_request / step / poll_responses``).  The
@@ -11,7 +11,8 @@ reference walks its active requests one after another on the CPU; here one ``ste
   attention kernel reads each request's pages through the page table, and the sampler picks the next ids on the device.
 
 Pages come from one pool shared by all requests and go back to it when a request finishes, or earlier when every layer of
-the model has a window and the page lies behind all of them.  ``feed`` runs given ids through the same passes and returns
+the model has a window and the page lies behind all of them.  What a recurrent layer carries from token to token lives in a slot per
+page-table row beside the pages.  ``feed`` runs given ids through the same passes and returns
 logits (scoring, replay).  CPU tensors take the
 plain torch path of every op, which is how the scheduling logic is tested without a GPU.
 """
@@ -103,19 +104,21 @@ class PagedKVCache:
     """One pool of 64-token pages shared by all requests; a page id addresses the same slot in every layer."""
 
     def __init__(self, num_layers: int, num_kv_heads: int, head_dim: int, max_pages: int, device, dtype, spare: bool = False,
-                 shapes: Optional[List[tuple]] = None):
-        """``shapes``: (kv heads, key size, value size) per layer, for models whose layers differ."""
+                 shapes: Optional[List[tuple]] = None, states: Optional[List[dict]] = None, slots: int = 0):
+        """``shapes``: (kv heads, key size, value size) per layer, for models whose layers differ.  ``states``: per layer, name ->
+        (shape, dtype) of what a sequence carries besides its pages; ``slots`` of each are held."""
         n = max_pages + (1 if spare else 0)                # the spare page (id max_pages) is never handed out
         shapes = shapes if shapes is not None else [(num_kv_heads, head_dim, head_dim)] * num_layers
         self.k = [torch.zeros(n, hk, PAGE, dk, device=device, dtype=dtype) for hk, dk, _ in shapes]
         self.v = [torch.zeros(n, hk, PAGE, dv, device=device, dtype=dtype) for hk, _, dv in shapes]
+        self.state = [{k: torch.zeros((slots,) + tuple(shape), device=device, dtype=dt) for k, (shape, dt) in d.items()} for d in states or [{}] * len(shapes)]
         self.max_pages = max_pages
         self.spare_page = max_pages if spare else -1
         self.free_pages: Deque[int] = collections.deque(range(max_pages))
 
     @classmethod
-    def for_model(cls, model: PagedModel, max_pages: int, device, dtype) -> "PagedKVCache":
-        return cls(0, 0, 0, max_pages, device, dtype, spare=True, shapes=model.kv_shapes())
+    def for_model(cls, model: PagedModel, max_pages: int, device, dtype, slots: int = 1) -> "PagedKVCache":
+        return cls(0, 0, 0, max_pages, device, dtype, spare=True, shapes=model.kv_shapes(), states=model.state_shapes(), slots=slots)
 
     def alloc_page(self) -> int:
         return self.free_pages.popleft() if self.free_pages else -1
@@ -174,7 +177,7 @@ class LLMEngine:
         self.launch_log: List[int] = []          # batch size of every decode pass (tests and metrics read it)
         self.use_graphs = use_graphs
         self._graphs: Dict[tuple, tuple] = {}
-        # speculative decoding for greedy requests: up to `spec_tokens` ids proposed by an n-gram look-up in the request's
+        # speculative decoding for greedy requests of models that can take a token back: up to `spec_tokens` ids proposed by an n-gram look-up in the request's
         # own history are verified in the same decode pass (one extra batch row per proposed id)
         self.spec_tokens = spec_tokens
         self.max_prompt_tokens = 16384           # tokens of new requests that share one prompt pass
@@ -203,9 +206,9 @@ class LLMEngine:
         self.cfg = w.cfg
         self.model = entry_of(w.cfg).model(w, self.device, self.dtype)
         c = self.cfg
-        self.kv = PagedKVCache.for_model(self.model, self.max_pages, self.device, self.dtype)
+        self.kv = PagedKVCache.for_model(self.model, self.max_pages, self.device, self.dtype, self.max_active + 1)
         self.pt_stride = (c.max_position_embeddings + PAGE - 1) // PAGE
-        # one row per active request plus a spare one whose single page absorbs the writes of padding rows
+        # one row (and one state slot) per active request plus a spare one whose single page absorbs the writes of padding rows
         self.page_table = torch.zeros(self.max_active + 1, self.pt_stride, dtype=torch.int32, device=self.device)
         self.page_table[self.max_active].fill_(self.kv.spare_page)
         self.free_rows = list(range(self.max_active))
@@ -369,7 +372,7 @@ class LLMEngine:
                 s.prefill_done = True
                 self._emit(s, self._sample([s], logits[i:i + 1])[0])
         running = [s for s in running if self._ensure_pages(s, s.kv_position) or self._finish(s)]
-        if running and self.spec_tokens > 0:
+        if running and self.spec_tokens > 0 and self.model.rewinds:
             self._step_speculative(running)
         elif running:                                          # one batched decode pass for everyone else
             logits = self._forward_decode(running)
@@ -490,7 +493,8 @@ class LLMEngine:
         if window is None:
             return
         keep = max(0, s.kv_position - window + 1) // PAGE             # first page that is still in a window
-        for i in range(s.passed, min(keep, len(s.pages))):
+        held = -(-self.model.kept_tokens() // PAGE)                   # leading pages that are never given back
+        for i in range(max(s.passed, held), min(keep, len(s.pages))):
             self.kv.free_page(s.pages[i])
             s.pages[i] = -1
         s.passed = max(s.passed, min(keep, len(s.pages)))
@@ -601,16 +605,17 @@ class LLMEngine:
         rows += [[0, 0, self.max_active, 1]] * (Bb - B)        # padding: the spare row of the page table
         key = (Bb, nsplit)
         if key not in self._graphs:
-            self._graphs[key] = self._capture(Bb, nsplit, rows)
+            self._graphs[key] = self._capture(Bb, nsplit)
         graph, meta_dev, meta_host, logits = self._graphs[key]
         meta_host.copy_(torch.tensor(rows, dtype=torch.int32))
         meta_dev.copy_(meta_host, non_blocking=True)
         graph.replay()
         return logits[:B]
 
-    def _capture(self, Bb: int, nsplit: int, rows):
+    def _capture(self, Bb: int, nsplit: int):
+        """The warm-up pass runs on padding rows alone: it must not advance a live sequence's recurrent state."""
         dev = self.device
-        meta_host = torch.tensor(rows, dtype=torch.int32).pin_memory()
+        meta_host = torch.tensor([[0, 0, self.max_active, 1]] * Bb, dtype=torch.int32).pin_memory()
         meta_dev = meta_host.to(dev)
         side = torch.cuda.Stream(device=dev)
         side.wait_stream(torch.cuda.current_stream(dev))
