@@ -86,4 +86,7 @@ typedef struct PtbRecurrence {
     const int* req;         // [n] of req_stride: slots
     float* out;             // [n][H Dv]
     int* status;
+    const void* chunks;     // the matrix form: [n_chunks] int4 (first row, rows <= 64, sequence, 0), sequence by sequence
+    const int* first_chunk; // [n_seqs]
+    int n_chunks, pad2;
 } PtbRecurrence;

@@ -1,0 +1,727 @@
+// The recurrent layers of recurrence.cuh over prompts in matrix form, bf16 inputs.  A sequence is cut into chunks of 64 tokens.  With G_i
+// the product of the decays of the chunk's tokens up to i (per key channel for the delta rule, a power of the head's decay otherwise)
+// and S the state before the chunk,
+//     o_i = (q_i G_i)^T S + sum_{j<=i} A_ij u_j,     A_ij = q_i . (k_j G_i / G_j)
+//     S'  = G_end S + sum_j (k_j G_end / G_j) u_j^T
+// where u is v for decay attention.  For the delta rule (1 + B) u = beta (v - (k G)^T S) with B_ij = beta_i k_i . (k_j G_i / G_j) for
+// j < i (a unit lower triangular system, the UT transform of delta-rule attention), hence u = U - W S with U = (1 + B)^-1 beta v and
+// W = (1 + B)^-1 beta (k G).  Two kernels:
+//   delta_chunk_kernel / decay_chunk_kernel   everything that does not depend on S, all chunks at once, into a workspace;
+//   chunk_state_kernel                        walks a sequence's chunks for a slice of value columns; S stays in registers.
+// Quotients of decays are never formed from products that could overflow: across blocks of 16 tokens both factors refer to the block
+// border between the two tokens and are at most 1, inside a block the exponent of every pair is taken directly.
+// Products run on the tensor cores with every fp32 operand split into two bf16 numbers (three products: 16 bits of both operands).
+#include "recurrence.cuh"
+#include "flash_attn.cuh"
+#include <algorithm>
+
+namespace ptb {
+namespace rc {
+
+constexpr int CH = 64, THREADS = 256, WARPS = 8;
+constexpr float LOG2E = 1.4426950408889634f;
+
+// Workspace of one (chunk, head): bf16 tiles in the swizzled order of fa::tile_off, high parts then low parts.
+template <int DT>
+struct Work {
+    static constexpr int TILE = CH * DT * 2, ATILE = CH * CH * 2;
+    static constexpr int W = 0, Q = 2 * TILE, K = 4 * TILE, A = 6 * TILE, G = A + 2 * ATILE, U = G + DT * 4;      // byte offsets
+    static __host__ __device__ size_t bytes(int Dvp) { return (size_t)U + (size_t)CH * Dvp * 4; }
+};
+
+struct Params {
+    PtbRecurrence P;
+    unsigned char* work;
+    size_t stride;                     // bytes per (chunk, head)
+    int Dvp;                           // value columns rounded up to 32
+    int vec;                           // 16-byte loads of x rows
+};
+
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    const float2 f = __bfloat1622float2(h);
+    const __nv_bfloat162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
+    hi = *reinterpret_cast<const uint32_t*>(&h);
+    lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+__device__ __forceinline__ float2 unpack(uint32_t v) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v)); }
+// d += a b for operands given as high and low parts
+__device__ __forceinline__ void mma3(float* d, const uint32_t* ah, const uint32_t* al, uint32_t bh0, uint32_t bh1, uint32_t bl0, uint32_t bl1) {
+    fa::mma16816(d, al, bh0, bh1);
+    fa::mma16816(d, ah, bl0, bl1);
+    fa::mma16816(d, ah, bh0, bh1);
+}
+// Store columns col, col + 1 (col even) of row r of a high and a low tile.
+template <int DT>
+__device__ __forceinline__ void store_split(unsigned char* hi, unsigned char* lo, int r, int col, float a, float b) {
+    uint32_t h, l;
+    split2(a, b, h, l);
+    const uint32_t off = fa::tile_off<DT>(r, col >> 3) + (col & 7) * 2;
+    *reinterpret_cast<uint32_t*>(hi + off) = h;
+    *reinterpret_cast<uint32_t*>(lo + off) = l;
+}
+// Eight columns at once (col a multiple of eight).
+template <int DT>
+__device__ __forceinline__ void store_split8(unsigned char* hi, unsigned char* lo, int r, int col, const float* f) {
+    uint4 h, l;
+    split2(f[0], f[1], h.x, l.x); split2(f[2], f[3], h.y, l.y); split2(f[4], f[5], h.z, l.z); split2(f[6], f[7], h.w, l.w);
+    const uint32_t off = fa::tile_off<DT>(r, col >> 3);
+    *reinterpret_cast<uint4*>(hi + off) = h;
+    *reinterpret_cast<uint4*>(lo + off) = l;
+}
+
+// Rows of x (columns col .. col + width) of a chunk into a bf16 tile of `pitch` elements per row, zeros past the rows and the width.
+__device__ __forceinline__ void load_rows(const PtbRecurrence& P, bool vec, int row0, int count, int col, int width, int padded, __nv_bfloat16* dst, int pitch) {
+    const __nv_bfloat16* x = (const __nv_bfloat16*)P.x;
+    const int ch = padded / 8;
+    for (int e = threadIdx.x; e < CH * ch; e += THREADS) {
+        const int r = e / ch, c = (e % ch) * 8;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (r < count && c < width) {
+            const __nv_bfloat16* s = x + (size_t)(row0 + r) * P.ld + col + c;
+            if (vec) v = *reinterpret_cast<const uint4*>(s);
+            else {
+                __nv_bfloat16* b = reinterpret_cast<__nv_bfloat16*>(&v);
+                for (int k = 0; k < 8 && c + k < width; ++k) b[k] = s[k];
+            }
+        }
+        *reinterpret_cast<uint4*>(dst + r * pitch + c) = v;
+    }
+}
+
+// ---------------------------------------------------------------------------------------------- delta rule, one chunk
+template <int DT>
+struct DeltaSmem {
+    static constexpr int PB = DT + 8;                  // pitch of the bf16 tiles
+    static constexpr int PG = DT + 8;                  // pitch of the decays (floats)
+    static constexpr int PA = CH + 4;                  // pitch of the 64 x 64 matrices (floats)
+    static constexpr int Q = 0, K = Q + CH * PB * 2, G = K + CH * PB * 2, E = G + CH * PG * 4, AQ = E + 4 * DT * 4, AK = AQ + CH * PA * 4;
+    static constexpr int TH = AK + CH * PA * 4, TL = TH + CH * CH * 2, TMP = TL + CH * CH * 2, ROW = TMP + 16 * 52 * 4, V = ROW + 3 * CH * 4 + 16;
+    static __host__ __device__ int total(int Dvp) { return V + CH * (Dvp + 8) * 2; }
+};
+
+template <int DT>
+__global__ void __launch_bounds__(THREADS) delta_chunk_kernel(const __grid_constant__ Params W) {
+    using S = DeltaSmem<DT>;
+    using L = Work<DT>;
+    extern __shared__ __align__(128) unsigned char smem[];
+    __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem + S::Q);
+    __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem + S::K);
+    __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(smem + S::V);
+    float* G_s = reinterpret_cast<float*>(smem + S::G);            // log2 of the product of decays up to and with a token
+    float* E_s = reinterpret_cast<float*>(smem + S::E);            // ... of a whole block of 16
+    float* aq = reinterpret_cast<float*>(smem + S::AQ);            // q . k, then the inverse
+    float* ak = reinterpret_cast<float*>(smem + S::AK);            // B
+    float* tmp = reinterpret_cast<float*>(smem + S::TMP);
+    float* qn = reinterpret_cast<float*>(smem + S::ROW);
+    float* kn = qn + CH;
+    float* bt = kn + CH;
+    int* next_unit = reinterpret_cast<int*>(bt + CH);
+    const PtbRecurrence& P = W.P;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int h = blockIdx.y, D = P.D, Dv = P.Dv, hk = h / (P.H / P.G), PV = W.Dvp + 8;
+    const int4 chunk = reinterpret_cast<const int4*>(P.chunks)[blockIdx.x];
+    const int row0 = chunk.x, cnt = chunk.y;
+    if (row0 < 0 || cnt < 1 || cnt > CH || row0 + cnt > P.n) {
+        if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+        return;
+    }
+    unsigned char* out = W.work + ((size_t)blockIdx.x * P.H + h) * W.stride;
+    load_rows(P, W.vec, row0, cnt, P.q_col + hk * D, D, DT, q_s, S::PB);
+    load_rows(P, W.vec, row0, cnt, P.k_col + hk * D, D, DT, k_s, S::PB);
+    load_rows(P, W.vec, row0, cnt, P.v_col + h * Dv, Dv, W.Dvp, v_s, PV);
+    const float rate = P.decay[h] * LOG2E;
+    for (int e = threadIdx.x; e < CH * DT; e += THREADS) {
+        const int r = e / DT, d = e % DT;
+        G_s[r * S::PG + d] = r < cnt && d < D ? fmaxf(-150.f, delta_log_decay(P.a[(size_t)(row0 + r) * P.ld_a + h * D + d], P.dt_bias[h * D + d], rate)) : 0.f;      // 2^-150 is 0
+    }
+    if (threadIdx.x < CH)
+        bt[threadIdx.x] = threadIdx.x < cnt ? sigmoid(__bfloat162float(((const __nv_bfloat16*)P.beta)[(size_t)(row0 + threadIdx.x) * P.ld_beta + h])) : 0.f;
+    if (threadIdx.x == 0) *next_unit = WARPS;
+    __syncthreads();
+    for (int r = warp; r < CH; r += WARPS) {
+        float a = 0.f, b = 0.f;
+        for (int d = lane * 2; d < DT; d += 64) {
+            const float2 x = unpack(*reinterpret_cast<const uint32_t*>(q_s + r * S::PB + d)), y = unpack(*reinterpret_cast<const uint32_t*>(k_s + r * S::PB + d));
+            a += x.x * x.x + x.y * x.y;
+            b += y.x * y.x + y.y * y.y;
+        }
+        a = warp_sum(a); b = warp_sum(b);
+        if (lane == 0) { qn[r] = rsqrtf(a + UNIT_EPS) * rsqrtf((float)D); kn[r] = rsqrtf(b + UNIT_EPS); }
+    }
+    for (int e = threadIdx.x; e < 4 * DT; e += THREADS) {          // running sums inside the blocks of 16
+        const int s = e / DT, d = e % DT;
+        float acc = 0.f;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            float* p = G_s + (s * 16 + i) * S::PG + d;
+            acc += *p;
+            *p = acc;
+        }
+        E_s[s * DT + d] = acc;
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < 3 * DT; e += THREADS) {          // ... and what lies before the block
+        const int s = e / DT + 1, d = e % DT;
+        float base = 0.f;
+        for (int r = 0; r < s; ++r) base += E_s[r * DT + d];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) G_s[(s * 16 + i) * S::PG + d] += base;
+    }
+    for (int e = threadIdx.x; e < CH * S::PA; e += THREADS) { aq[e] = 0.f; ak[e] = 0.f; }
+    __syncthreads();
+    // ---- q . k and k . k under the decays: units 0-5 are blocks of 16 x 16 below the diagonal on the tensor cores, the rest 32 pairs each
+    // of the diagonal blocks
+    for (int unit = warp; unit < 6 + 17;) {
+        if (unit < 6) {
+            const int s = unit < 1 ? 1 : unit < 3 ? 2 : 3, r = unit - (s == 1 ? 0 : s == 2 ? 1 : 3);
+            const float* base = G_s + (s * 16 - 1) * S::PG;        // both factors refer to the end of the block before s
+            float cq[2][4], ck[2][4];
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) cq[n][e] = ck[n][e] = 0.f;
+#pragma unroll 2
+            for (int ks = 0; ks < DT / 16; ++ks) {
+                uint32_t qh[4], ql[4], kh[4], kl[4];
+                float2 b2[2];
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {                      // row g + 8 (u & 1), columns 2t + 8 (u >> 1)
+                    const int i = s * 16 + g + 8 * (u & 1), d = ks * 16 + 2 * t + 8 * (u >> 1);
+                    if ((u & 1) == 0) b2[u >> 1] = *reinterpret_cast<const float2*>(base + d);
+                    const float2 G = *reinterpret_cast<const float2*>(G_s + i * S::PG + d);
+                    const float ex = exp2f(G.x - b2[u >> 1].x), ey = exp2f(G.y - b2[u >> 1].y);
+                    const float2 q = unpack(*reinterpret_cast<const uint32_t*>(q_s + i * S::PB + d)), k = unpack(*reinterpret_cast<const uint32_t*>(k_s + i * S::PB + d));
+                    split2(q.x * ex, q.y * ey, qh[u], ql[u]);
+                    split2(k.x * ex, k.y * ey, kh[u], kl[u]);
+                }
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+                    const int j = r * 16 + n * 8 + g;
+                    uint32_t bh[2], bl[2];
+#pragma unroll
+                    for (int u = 0; u < 2; ++u) {
+                        const int d = ks * 16 + 2 * t + 8 * u;
+                        const float2 G = *reinterpret_cast<const float2*>(G_s + j * S::PG + d);
+                        const float2 k = unpack(*reinterpret_cast<const uint32_t*>(k_s + j * S::PB + d));
+                        split2(k.x * exp2f(b2[u].x - G.x), k.y * exp2f(b2[u].y - G.y), bh[u], bl[u]);
+                    }
+                    mma3(cq[n], qh, ql, bh[0], bh[1], bl[0], bl[1]);
+                    mma3(ck[n], kh, kl, bh[0], bh[1], bl[0], bl[1]);
+                }
+            }
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int i = s * 16 + g + 8 * (e >> 1), j = r * 16 + n * 8 + 2 * t + (e & 1);
+                    aq[i * S::PA + j] = cq[n][e] * qn[i] * kn[j];
+                    ak[i * S::PA + j] = ck[n][e] * kn[i] * kn[j] * bt[i];
+                }
+        } else {
+            const int p = (unit - 6) * 32 + lane, s = p / 136, m = p % 136;
+            int a = (int)((sqrtf(8.f * m + 1.f) - 1.f) * 0.5f);
+            while (a * (a + 1) / 2 > m) --a;
+            while ((a + 1) * (a + 2) / 2 <= m) ++a;
+            const int i = s * 16 + a, j = s * 16 + m - a * (a + 1) / 2;
+            const float* Gi = G_s + i * S::PG;
+            const float* Gj = G_s + j * S::PG;
+            float sq = 0.f, sk = 0.f;
+            for (int d = 0; d < DT; d += 4) {
+                const float4 x = *reinterpret_cast<const float4*>(Gi + d), y = *reinterpret_cast<const float4*>(Gj + d);
+                const uint2 qr = *reinterpret_cast<const uint2*>(q_s + i * S::PB + d), kr = *reinterpret_cast<const uint2*>(k_s + i * S::PB + d);
+                const uint2 jr = *reinterpret_cast<const uint2*>(k_s + j * S::PB + d);
+                const float2 q0 = unpack(qr.x), q1 = unpack(qr.y), k0 = unpack(kr.x), k1 = unpack(kr.y), j0 = unpack(jr.x), j1 = unpack(jr.y);
+                const float e0 = j0.x * exp2f(x.x - y.x), e1 = j0.y * exp2f(x.y - y.y), e2 = j1.x * exp2f(x.z - y.z), e3 = j1.y * exp2f(x.w - y.w);
+                sq = fmaf(q0.x, e0, fmaf(q0.y, e1, fmaf(q1.x, e2, fmaf(q1.y, e3, sq))));
+                sk = fmaf(k0.x, e0, fmaf(k0.y, e1, fmaf(k1.x, e2, fmaf(k1.y, e3, sk))));
+            }
+            aq[i * S::PA + j] = sq * qn[i] * kn[j];
+            if (i != j) ak[i * S::PA + j] = sk * kn[i] * kn[j] * bt[i];
+        }
+        if (lane == 0) unit = atomicAdd(next_unit, 1);
+        unit = __shfl_sync(0xffffffffu, unit, 0);
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < CH * CH / 8; e += THREADS) {
+        const int r = e / 8, c = (e % 8) * 8;
+        store_split8<CH>(out + L::A, out + L::A + L::ATILE, r, c, aq + r * S::PA + c);
+    }
+    __syncthreads();
+    // ---- (1 + B)^-1 over aq: the diagonal blocks by substitution (a lane owns a column), then block row after block row
+    if (warp < 4 && lane < 16) {
+        float x[16];
+        const float* b = ak + warp * 16 * S::PA + warp * 16;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            float v = i == lane ? 1.f : 0.f;
+#pragma unroll
+            for (int m = 0; m < i; ++m) v = fmaf(-b[i * S::PA + m], x[m], v);
+            x[i] = v;
+        }
+#pragma unroll
+        for (int i = 0; i < 16; ++i) aq[(warp * 16 + i) * S::PA + warp * 16 + lane] = x[i];
+    }
+    __syncthreads();
+    for (int s = 1; s < 4; ++s) {
+        const int i = threadIdx.x >> 4, c = threadIdx.x & 15;
+        for (int r = 0; r < s; ++r) {
+            float v = 0.f;
+            for (int m = r * 16; m < s * 16; ++m) v = fmaf(ak[(s * 16 + i) * S::PA + m], aq[m * S::PA + r * 16 + c], v);
+            tmp[i * 52 + r * 16 + c] = v;
+        }
+        __syncthreads();
+        for (int r = 0; r < s; ++r) {
+            float v = 0.f;
+#pragma unroll
+            for (int m = 0; m < 16; ++m) v = fmaf(aq[(s * 16 + i) * S::PA + s * 16 + m], tmp[m * 52 + r * 16 + c], v);
+            aq[(s * 16 + i) * S::PA + r * 16 + c] = -v;
+        }
+        __syncthreads();
+    }
+    for (int e = threadIdx.x; e < CH * CH / 8; e += THREADS) {     // times beta, split
+        const int r = e / 8, c = (e % 8) * 8;
+        float f[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) f[k] = c + k <= r ? aq[r * S::PA + c + k] * bt[c + k] : 0.f;
+        store_split8<CH>(smem + S::TH, smem + S::TL, r, c, f);
+    }
+    __syncthreads();
+    // ---- W and U: units of 16 columns
+    const uint32_t th = smem_u32(smem + S::TH), tl = smem_u32(smem + S::TL);
+    for (int unit = warp; unit < DT / 16 + W.Dvp / 16; unit += WARPS) {
+        const bool is_w = unit < DT / 16;
+        const int n0 = (is_w ? unit : unit - DT / 16) * 16;
+        uint32_t bh[4][4], bl[4][4];
+        if (is_w) {
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks)
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {                      // n-block u >> 1, rows 2t, 2t + 1 (+ 8 for odd u)
+                    const int j = ks * 16 + 2 * t + 8 * (u & 1), d = n0 + g + 8 * (u >> 1);
+                    const float a = __bfloat162float(k_s[j * S::PB + d]) * kn[j] * exp2f(G_s[j * S::PG + d]);
+                    const float b = __bfloat162float(k_s[(j + 1) * S::PB + d]) * kn[j + 1] * exp2f(G_s[(j + 1) * S::PG + d]);
+                    split2(a, b, bh[ks][u], bl[ks][u]);
+                }
+        } else {
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks)
+                fa::ldsm4_t(smem_u32(v_s + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PV + n0 + (lane >> 4) * 8), bh[ks][0], bh[ks][1], bh[ks][2], bh[ks][3]);
+        }
+#pragma unroll
+        for (int rb = 0; rb < 4; ++rb) {
+            float c[2][4];
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) c[n][e] = 0.f;
+#pragma unroll
+            for (int ks = 0; ks <= rb; ++ks) {
+                uint32_t ah[4], al[4];
+                fa::load_a<CH>(th, rb * 16, ks, ah);
+                fa::load_a<CH>(tl, rb * 16, ks, al);
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+                    if (is_w) mma3(c[n], ah, al, bh[ks][2 * n], bh[ks][2 * n + 1], bl[ks][2 * n], bl[ks][2 * n + 1]);
+                    else {
+                        fa::mma16816(c[n], al, bh[ks][2 * n], bh[ks][2 * n + 1]);
+                        fa::mma16816(c[n], ah, bh[ks][2 * n], bh[ks][2 * n + 1]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int r = rb * 16 + g + 8 * e, col = n0 + n * 8 + 2 * t;
+                    if (is_w) store_split<DT>(out + L::W, out + L::W + L::TILE, r, col, c[n][2 * e], c[n][2 * e + 1]);
+                    else *reinterpret_cast<float2*>(out + L::U + ((size_t)r * W.Dvp + col) * 4) = make_float2(c[n][2 * e], c[n][2 * e + 1]);
+                }
+        }
+    }
+    // ---- q G, k G_end / G and G_end
+    const float* Ge = G_s + (CH - 1) * S::PG;
+    for (int e = threadIdx.x; e < CH * DT / 8; e += THREADS) {
+        const int r = e / (DT / 8), d = (e % (DT / 8)) * 8;
+        float fq[8], fk[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+            const float G = G_s[r * S::PG + d + k];
+            fq[k] = __bfloat162float(q_s[r * S::PB + d + k]) * qn[r] * exp2f(G);
+            fk[k] = __bfloat162float(k_s[r * S::PB + d + k]) * kn[r] * exp2f(Ge[d + k] - G);
+        }
+        store_split8<DT>(out + L::Q, out + L::Q + L::TILE, r, d, fq);
+        store_split8<DT>(out + L::K, out + L::K + L::TILE, r, d, fk);
+    }
+    for (int d = threadIdx.x; d < DT; d += THREADS) reinterpret_cast<float*>(out + L::G)[d] = exp2f(Ge[d]);
+}
+
+// ---------------------------------------------------------------------------------------------- fixed decay, one chunk
+template <int DT>
+__global__ void __launch_bounds__(THREADS) decay_chunk_kernel(const __grid_constant__ Params W) {
+    using L = Work<DT>;
+    extern __shared__ __align__(128) unsigned char smem[];
+    __shared__ float pw[CH + 1];                       // powers of the decay
+    unsigned char *qh = smem, *ql = smem + L::TILE, *kh = smem + 2 * L::TILE, *kl = smem + 3 * L::TILE;
+    const PtbRecurrence& P = W.P;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int h = blockIdx.y, D = P.D;
+    const int4 chunk = reinterpret_cast<const int4*>(P.chunks)[blockIdx.x];
+    const int row0 = chunk.x, cnt = chunk.y;
+    if (row0 < 0 || cnt < 1 || cnt > CH || row0 + cnt > P.n) {
+        if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+        return;
+    }
+    unsigned char* out = W.work + ((size_t)blockIdx.x * P.H + h) * W.stride;
+    if (warp == 0) {                                   // pw[i] = decay^i: by products over the lanes, then one more step for 32 .. 64
+        const float a = P.decay[h];
+        float p = lane == 0 ? 1.f : a;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) { const float q = __shfl_up_sync(0xffffffffu, p, o); if (lane >= o) p *= q; }
+        const float p32 = __shfl_sync(0xffffffffu, p, 31) * a;
+        pw[lane] = p;
+        pw[32 + lane] = p * p32;
+        if (lane == 31) pw[64] = p32 * p32;
+    }
+    __syncthreads();
+    const __nv_bfloat16* x = (const __nv_bfloat16*)P.x;
+    for (int e = threadIdx.x; e < CH * DT / 8; e += THREADS) {
+        const int r = e / (DT / 8), d = (e % (DT / 8)) * 8;
+        float fq[8], fk[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) fq[k] = fk[k] = 0.f;
+        if (r < cnt && d < D) {
+            const __nv_bfloat16* q = x + (size_t)(row0 + r) * P.ld + P.q_col + h * D + d;
+            const __nv_bfloat16* kk = x + (size_t)(row0 + r) * P.ld + P.k_col + h * D + d;
+            if (W.vec) {
+                const uint4 a = *reinterpret_cast<const uint4*>(q), b = *reinterpret_cast<const uint4*>(kk);
+                const uint32_t *ap = reinterpret_cast<const uint32_t*>(&a), *bp = reinterpret_cast<const uint32_t*>(&b);
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    const float2 f = unpack(ap[k]), s = unpack(bp[k]);
+                    fq[2 * k] = f.x; fq[2 * k + 1] = f.y; fk[2 * k] = s.x; fk[2 * k + 1] = s.y;
+                }
+            } else
+                for (int k = 0; k < 8 && d + k < D; ++k) { fq[k] = __bfloat162float(q[k]); fk[k] = __bfloat162float(kk[k]); }
+            if (P.silu)
+#pragma unroll
+                for (int k = 0; k < 8; ++k) { fq[k] = silu(fq[k]); fk[k] = silu(fk[k]); }
+        }
+        store_split8<DT>(qh, ql, r, d, fq);
+        store_split8<DT>(kh, kl, r, d, fk);
+        const float a = pw[r + 1], b = r < cnt ? pw[cnt - 1 - r] : 0.f;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) { fq[k] *= a; fk[k] *= b; }
+        store_split8<DT>(out + L::Q, out + L::Q + L::TILE, r, d, fq);
+        store_split8<DT>(out + L::K, out + L::K + L::TILE, r, d, fk);
+    }
+    __syncthreads();
+    const uint32_t a_h = smem_u32(qh), a_l = smem_u32(ql), b_h = smem_u32(kh), b_l = smem_u32(kl);
+    for (int unit = warp; unit < 16; unit += WARPS) {              // 16 x 16 blocks; those above the diagonal are zeros
+        const int s = unit >> 2, r = unit & 3;
+        float c[2][4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) c[n][e] = 0.f;
+        if (r <= s)
+#pragma unroll 2
+            for (int ks = 0; ks < DT / 16; ++ks) {
+                uint32_t ah[4], al[4], bh[4], bl[4];
+                fa::load_a<DT>(a_h, s * 16, ks, ah);
+                fa::load_a<DT>(a_l, s * 16, ks, al);
+                fa::load_b<DT>(b_h, r * 16, ks, bh);
+                fa::load_b<DT>(b_l, r * 16, ks, bl);
+                mma3(c[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
+                mma3(c[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+            }
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int i = s * 16 + g + 8 * e, j = r * 16 + n * 8 + 2 * t;
+                store_split<CH>(out + L::A, out + L::A + L::ATILE, i, j, j <= i ? c[n][2 * e] * pw[i - j] : 0.f, j + 1 <= i ? c[n][2 * e + 1] * pw[i - j - 1] : 0.f);
+            }
+    }
+    for (int d = threadIdx.x; d < DT; d += THREADS) reinterpret_cast<float*>(out + L::G)[d] = pw[cnt];
+}
+
+// ---------------------------------------------------------------------------------------------- the walk over a sequence's chunks
+template <int DT, int VS>
+struct StateSmem {
+    using L = Work<DT>;
+    static constexpr int WQ = 0, KA = 4 * L::TILE, SH = KA + 2 * L::TILE + 2 * L::ATILE, SL = SH + VS * DT * 2, UH = SL + VS * DT * 2, UL = UH + VS * CH * 2;
+    static constexpr int BAR = UL + VS * CH * 2, TOTAL = BAR + 64;
+};
+
+// One CTA per (VS value columns, head, sequence), eight warps.  Of a chunk, warps 0-3 form u (64 rows) and then the new state, warps 4-7
+// the read-out; the state lives transposed, [value][key channel], in the accumulators of warps 0-3 and as two bf16 tiles in shared
+// memory for the products that read it.  Tiles arrive by bulk copies: those of a chunk's first half while the chunk before finishes.
+template <int DT, int VS, bool DELTA>
+__global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_constant__ Params W) {
+    using L = Work<DT>;
+    using S = StateSmem<DT, VS>;
+    constexpr int NT = DT / 32, MT = VS / 16, NB = VS / 8;         // state tiles of a warp: MT x NT of 16 x 8
+    extern __shared__ __align__(128) unsigned char smem[];
+    uint64_t* bar = reinterpret_cast<uint64_t*>(smem + S::BAR);    // 0: W and q tiles, 1: k and A tiles
+    const PtbRecurrence& P = W.P;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    if (threadIdx.x == 0) {
+        mbar_init(&bar[0], 1);
+        mbar_init(&bar[1], 1);
+        mbar_fence_init();
+    }
+    __syncthreads();
+    pdl_wait();
+    pdl_launch_dependents();
+    const int h = blockIdx.y, v0 = blockIdx.x * VS, D = P.D, Dv = P.Dv;
+    const Span sp = span_of(P, blockIdx.z);
+    if (sp.slot < 0 || sp.count == 0) return;
+    const int first = P.first_chunk[blockIdx.z], chunks = (sp.count + CH - 1) / CH;
+    if (first < 0 || first + chunks > P.n_chunks) {
+        if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+        return;
+    }
+    auto tiles = [&](int c) { return W.work + ((size_t)(first + c) * P.H + h) * W.stride; };
+    auto load_wq = [&](int c) {
+        constexpr uint32_t bytes = (DELTA ? 4 : 2) * L::TILE;
+        mbar_expect_tx(&bar[0], bytes);
+        bulk_g2s(smem + S::WQ + (DELTA ? 0 : 2 * L::TILE), tiles(c) + (DELTA ? L::W : L::Q), bytes, &bar[0]);
+    };
+    auto load_ka = [&](int c) {
+        constexpr uint32_t bytes = 2 * L::TILE + 2 * L::ATILE;
+        mbar_expect_tx(&bar[1], bytes);
+        bulk_g2s(smem + S::KA, tiles(c) + L::K, bytes, &bar[1]);
+    };
+    if (threadIdx.x == 0) { load_wq(0); load_ka(0); }
+    const uint32_t wh = smem_u32(smem + S::WQ), qh = wh + 2 * L::TILE, kh = smem_u32(smem + S::KA), ah = kh + 2 * L::TILE;
+    const uint32_t sh = smem_u32(smem + S::SH), sl = smem_u32(smem + S::SL), uh = smem_u32(smem + S::UH), ul = smem_u32(smem + S::UL);
+    const bool owner = warp < 4;                       // of the state channels d0 .. d0 + DT / 4
+    const int wr = (warp & 3) * 16, d0 = (warp & 3) * (DT / 4);
+    float* st = P.state + (((size_t)sp.slot * P.H + h) * D) * Dv;
+    float X[MT][NT][4];                                // S^T: row v0 + 16 m + g (+ 8), column d0 + 8 n + 2t (+ 1)
+    auto each_state = [&](auto f) {
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int n = 0; n < NT; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) f(X[m][n][e], v0 + m * 16 + g + 8 * (e >> 1), d0 + n * 8 + 2 * t + (e & 1));
+    };
+    auto publish = [&]() {
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int n = 0; n < NT; ++n)
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+                    store_split<DT>(smem + S::SH, smem + S::SL, m * 16 + g + 8 * e, d0 + n * 8 + 2 * t, X[m][n][2 * e], X[m][n][2 * e + 1]);
+    };
+    if (owner) {
+        each_state([&](float& x, int v, int d) { x = sp.pos0 > 0 && v < Dv && d < D ? st[(size_t)d * Dv + v] : 0.f; });
+        publish();
+    }
+    __syncthreads();
+    bool ok = true;
+    for (int c = 0; c < chunks; ++c) {
+        const int row0 = sp.row0 + c * CH, cnt = min(CH, sp.count - c * CH);
+        const unsigned char* tile = tiles(c);
+        float acc[NB][4], ge[NT][2];
+#pragma unroll
+        for (int n = 0; n < NB; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
+        float2 base[NB][2];                            // U (delta) or v of rows wr + g, wr + g + 8
+        if (owner) {
+#pragma unroll
+            for (int n = 0; n < NT; ++n) {
+                const float2 f = *reinterpret_cast<const float2*>(tile + L::G + (d0 + n * 8 + 2 * t) * 4);
+                ge[n][0] = f.x; ge[n][1] = f.y;
+            }
+#pragma unroll
+            for (int n = 0; n < NB; ++n)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int r = wr + g + 8 * e, v = v0 + n * 8 + 2 * t;
+                    if constexpr (DELTA) base[n][e] = *reinterpret_cast<const float2*>(tile + L::U + ((size_t)r * W.Dvp + v) * 4);
+                    else {
+                        float2 f = make_float2(0.f, 0.f);
+                        if (r < cnt) {
+                            const __nv_bfloat16* x = (const __nv_bfloat16*)P.x + (size_t)(row0 + r) * P.ld + P.v_col + (size_t)h * Dv + v;
+                            if (v < Dv) f.x = __bfloat162float(x[0]);
+                            if (v + 1 < Dv) f.y = __bfloat162float(x[1]);
+                            if (P.silu) { f.x = silu(f.x); f.y = silu(f.y); }
+                        }
+                        base[n][e] = f;
+                    }
+                }
+        }
+        if (ok) ok = mbar_wait(&bar[0], (uint32_t)(c & 1), P.status);
+        if (DELTA || !owner) {                         // W S (warps 0-3) or (q G) S (warps 4-7): 16 rows each
+            const uint32_t th = owner ? wh : qh, tl = th + L::TILE;
+#pragma unroll 2
+            for (int ks = 0; ks < DT / 16; ++ks) {
+                uint32_t a[4], b[4];
+                fa::load_a<DT>(th, wr, ks, a);
+                fa::load_a<DT>(tl, wr, ks, b);
+#pragma unroll
+                for (int n = 0; n < MT; ++n) {
+                    uint32_t bh[4], bl[4];
+                    fa::load_b<DT>(sh, n * 16, ks, bh);
+                    fa::load_b<DT>(sl, n * 16, ks, bl);
+                    mma3(acc[2 * n], a, b, bh[0], bh[1], bl[0], bl[1]);
+                    mma3(acc[2 * n + 1], a, b, bh[2], bh[3], bl[2], bl[3]);
+                }
+            }
+        }
+        if (owner) {                                   // u^T, split
+#pragma unroll
+            for (int n = 0; n < NB; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float2 f = base[n][e >> 1];
+                    const float u = ((e & 1) ? f.y : f.x) - acc[n][e];
+                    const int v = n * 8 + 2 * t + (e & 1), r = wr + g + 8 * (e >> 1);
+                    const __nv_bfloat16 hi = __float2bfloat16_rn(u);
+                    const uint32_t off = fa::tile_off<CH>(v, r >> 3) + (r & 7) * 2;
+                    *reinterpret_cast<__nv_bfloat16*>(smem + S::UH + off) = hi;
+                    *reinterpret_cast<__nv_bfloat16*>(smem + S::UL + off) = __float2bfloat16_rn(u - __bfloat162float(hi));
+                }
+        }
+        __syncthreads();                               // u is there; W, q and the state tiles have been read
+        if (threadIdx.x == 0 && c + 1 < chunks && ok) load_wq(c + 1);
+        if (ok) ok = mbar_wait(&bar[1], (uint32_t)(c & 1), P.status);
+        if (owner) {
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int n = 0; n < NT; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) X[m][n][e] *= ge[n][e & 1];
+#pragma unroll
+            for (int ks = 0; ks < CH / 16; ++ks) {
+                uint32_t bh[NT / 2][4], bl[NT / 2][4];
+#pragma unroll
+                for (int n = 0; n < NT / 2; ++n) {
+                    fa::load_b_t<DT>(kh, ks * 16, d0 / 8 + 2 * n, bh[n]);
+                    fa::load_b_t<DT>(kh + L::TILE, ks * 16, d0 / 8 + 2 * n, bl[n]);
+                }
+#pragma unroll
+                for (int m = 0; m < MT; ++m) {
+                    uint32_t a[4], b[4];
+                    fa::load_a<CH>(uh, m * 16, ks, a);
+                    fa::load_a<CH>(ul, m * 16, ks, b);
+#pragma unroll
+                    for (int n = 0; n < NT / 2; ++n) {
+                        mma3(X[m][2 * n], a, b, bh[n][0], bh[n][1], bl[n][0], bl[n][1]);
+                        mma3(X[m][2 * n + 1], a, b, bh[n][2], bh[n][3], bl[n][2], bl[n][3]);
+                    }
+                }
+            }
+            publish();
+        } else {
+            for (int ks = 0; ks <= wr / 16; ++ks) {
+                uint32_t a[4], b[4];
+                fa::load_a<CH>(ah, wr, ks, a);
+                fa::load_a<CH>(ah + L::ATILE, wr, ks, b);
+#pragma unroll
+                for (int n = 0; n < MT; ++n) {
+                    uint32_t bh[4], bl[4];
+                    fa::load_b<CH>(uh, n * 16, ks, bh);
+                    fa::load_b<CH>(ul, n * 16, ks, bl);
+                    mma3(acc[2 * n], a, b, bh[0], bh[1], bl[0], bl[1]);
+                    mma3(acc[2 * n + 1], a, b, bh[2], bh[3], bl[2], bl[3]);
+                }
+            }
+#pragma unroll
+            for (int n = 0; n < NB; ++n)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int r = wr + g + 8 * e, v = v0 + n * 8 + 2 * t;
+                    float* o = P.out + (size_t)(row0 + r) * P.H * Dv + (size_t)h * Dv + v;
+                    if (r >= cnt) continue;
+                    if (v + 1 < Dv && (Dv & 1) == 0) *reinterpret_cast<float2*>(o) = make_float2(acc[n][2 * e], acc[n][2 * e + 1]);
+                    else {
+                        if (v < Dv) o[0] = acc[n][2 * e];
+                        if (v + 1 < Dv) o[1] = acc[n][2 * e + 1];
+                    }
+                }
+        }
+        __syncthreads();                               // the new state is there; k, A and u have been read
+        if (threadIdx.x == 0 && c + 1 < chunks && ok) load_ka(c + 1);
+    }
+    if (owner) each_state([&](float& x, int v, int d) { if (ok && v < Dv && d < D) st[(size_t)d * Dv + v] = x; });
+}
+
+template <int DT, int VS>
+static int launch_state(const Params& p, cudaStream_t st) {
+    const dim3 grid((p.P.Dv + VS - 1) / VS, p.P.H, p.P.n_seqs);
+    auto kern = p.P.delta ? chunk_state_kernel<DT, VS, true> : chunk_state_kernel<DT, VS, false>;
+    constexpr int smem = StateSmem<DT, VS>::TOTAL;
+    PTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    PTB_CUDA_OK(ptb_launch(kern, grid, dim3(THREADS), (size_t)smem, st, ptb_pdl_enabled(), p));
+    return 0;
+}
+
+template <int DT>
+static int launch(Params p, cudaStream_t st) {
+    const dim3 grid(p.P.n_chunks, p.P.H);
+    const bool pdl = ptb_pdl_enabled();
+    if (p.P.delta) {
+        const int smem = DeltaSmem<DT>::total(p.Dvp);
+        PTB_CUDA_OK(cudaFuncSetAttribute(delta_chunk_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+        PTB_CUDA_OK(ptb_launch(delta_chunk_kernel<DT>, grid, dim3(THREADS), (size_t)smem, st, pdl, p));
+    } else {
+        constexpr int smem = 4 * Work<DT>::TILE;
+        PTB_CUDA_OK(cudaFuncSetAttribute(decay_chunk_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+        PTB_CUDA_OK(ptb_launch(decay_chunk_kernel<DT>, grid, dim3(THREADS), (size_t)smem, st, pdl, p));
+    }
+    // few CTAs: narrow slices, so that more of them share the walk
+    const long long wide = (long long)((p.P.Dv + 31) / 32) * p.P.H * p.P.n_seqs;
+    if (wide < 56 ? launch_state<DT, 16>(p, st) : launch_state<DT, 32>(p, st)) return -1;
+    PTB_CUDA_OK(cudaGetLastError());
+    return 0;
+}
+
+}  // namespace rc
+
+int recurrence_check(const PtbRecurrence& p);
+
+static size_t chunk_bytes(const PtbRecurrence& p) {
+    const int Dvp = (p.Dv + 31) / 32 * 32;
+    return p.D <= 64 ? rc::Work<64>::bytes(Dvp) : rc::Work<128>::bytes(Dvp);
+}
+
+}  // namespace ptb
+
+using namespace ptb;
+
+// Bytes of workspace of ptb_recurrence_chunked, or -1 for sizes it does not take (bf16, D and Dv up to 128).
+PTB_API long long ptb_recurrence_chunked_bytes(const PtbRecurrence* args) {
+    const PtbRecurrence& p = *args;
+    if (!p.bf16 || p.D > 128 || p.Dv > 128 || p.n_chunks < 1) return -1;
+    return (long long)chunk_bytes(p) * p.n_chunks * p.H;
+}
+
+// ptb_recurrence for a prompt pass, in chunks of 64 rows; see PtbRecurrence.
+PTB_API int ptb_recurrence_chunked(const PtbRecurrence* args, void* work, long long bytes, cudaStream_t st) {
+    if (args->n <= 0 || args->n_seqs <= 0) return 0;
+    if (recurrence_check(*args)) return -1;
+    const long long need = ptb_recurrence_chunked_bytes(args);
+    if (need < 0 || bytes < need || !args->seqs || !args->chunks || !args->first_chunk || ((uintptr_t)work & 127)) {
+        ptb_set_error("recurrence_chunked: sizes (D %d, Dv %d), workspace (%lld of %lld bytes) or chunk table", args->D, args->Dv, bytes, need);
+        return -1;
+    }
+    rc::Params p;
+    p.P = *args;
+    p.work = (unsigned char*)work;
+    p.stride = chunk_bytes(*args);
+    p.Dvp = (args->Dv + 31) / 32 * 32;
+    p.vec = args->D % 8 == 0 && args->Dv % 8 == 0 && args->ld % 8 == 0 && args->q_col % 8 == 0 && args->k_col % 8 == 0 && args->v_col % 8 == 0 &&
+            ((uintptr_t)args->x & 15) == 0;
+    return args->D <= 64 ? rc::launch<64>(p, st) : rc::launch<128>(p, st);
+}

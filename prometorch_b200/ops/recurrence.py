@@ -24,7 +24,8 @@ class RecurrenceArgs(C.Structure):
                 ("decay", C.c_void_p), ("dt_bias", C.c_void_p),
                 ("state", C.c_void_p), ("slots", C.c_int), ("n", C.c_int), ("H", C.c_int), ("G", C.c_int), ("D", C.c_int), ("Dv", C.c_int),
                 ("seqs", C.c_void_p), ("n_seqs", C.c_int), ("pos_stride", C.c_int), ("req_stride", C.c_int), ("pad", C.c_int),
-                ("pos", C.c_void_p), ("req", C.c_void_p), ("out", C.c_void_p), ("status", C.c_void_p)]
+                ("pos", C.c_void_p), ("req", C.c_void_p), ("out", C.c_void_p), ("status", C.c_void_p),
+                ("chunks", C.c_void_p), ("first_chunk", C.c_void_p), ("n_chunks", C.c_int), ("pad2", C.c_int)]
 
 
 @N.register_decls
@@ -36,23 +37,34 @@ def _decls(L):
     L.ptb_recurrence.restype = ci
     L.ptb_group_norm_gate.argtypes = [vp, vp, vp, ci, ll, vp, ci, ci, ci, cf, ci, vp]
     L.ptb_group_norm_gate.restype = ci
-    if not hasattr(L, 'ptb_recurrence_chunked'): return  # TMP
-    L.ptb_recurrence_chunked.argtypes = [C.POINTER(RecurrenceArgs), ci, vp, ll, vp]
+    L.ptb_recurrence_chunked.argtypes = [C.POINTER(RecurrenceArgs), vp, ll, vp]
     L.ptb_recurrence_chunked.restype = ci
-    L.ptb_recurrence_chunked_bytes.argtypes = [C.POINTER(RecurrenceArgs), ci]
+    L.ptb_recurrence_chunked_bytes.argtypes = [C.POINTER(RecurrenceArgs)]
     L.ptb_recurrence_chunked_bytes.restype = ll
+
+
+CHUNK = 64                             # rows of a chunk of csrc/recurrence_chunk.cu
+CHUNKED_FROM = 32                      # longest sequence of a prompt pass from which it runs in chunks
 
 
 @dataclass
 class Sequences:
-    """The sequences of a prompt pass: on the device ``[sequences, 4]`` int32 (first row, rows, position of the first, slot)."""
+    """The sequences of a prompt pass: on the device ``[sequences, 4]`` int32 (first row, rows, position of the first, slot), and
+    their cut into chunks for the matrix form: ``[chunks, 4]`` (first row, rows, sequence, unused) and every sequence's first chunk."""
     host: List[Tuple[int, int, int, int]]
     device: torch.Tensor
+    chunks: Optional[torch.Tensor] = None
+    first_chunk: Optional[torch.Tensor] = None
 
     @classmethod
     def of(cls, offs: List[int], starts: List[int], rows: List[int], device) -> "Sequences":
         host = [(lo, hi - lo, at, r) for lo, hi, at, r in zip(offs, offs[1:], starts, rows)]
-        return cls(host, torch.tensor(host, dtype=torch.int32).to(device))
+        chunks, first = [], []
+        for i, (lo, n, _, _) in enumerate(host):
+            first.append(len(chunks))
+            chunks += [(lo + j, min(CHUNK, n - j), i, 0) for j in range(0, n, CHUNK)]
+        up = lambda t: torch.tensor(t, dtype=torch.int32).to(device)
+        return cls(host, up(host), up(chunks), up(first))
 
     @classmethod
     def of_rows(cls, pos: torch.Tensor, req: torch.Tensor) -> "Sequences":
@@ -87,7 +99,8 @@ def short_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, pos: 
                                        len(seqs.host) if seqs else 0, _status(x.device).data_ptr(), int(x.dtype == torch.bfloat16), _st(x)), "short_conv")
         return out
     for lo, count, at, slot in (seqs or Sequences.of_rows(pos, req)).host:
-        before = state[slot].float() if at > 0 else torch.zeros(taps - 1, Ch)
+        before = state[slot].float()
+        before[:max(0, taps - 1 - at)] = 0                      # rows from before position 0
         full = torch.cat([before, x[lo:lo + count].float()])
         y = sum(full[i:i + count] * weight[i].float() for i in range(taps))
         out[lo:lo + count] = torch.nn.functional.silu(y).to(out.dtype)
@@ -122,24 +135,20 @@ def _unit(x):
     return x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6)
 
 
-CHUNKED_FROM = 32                      # tokens of a sequence from which a prompt pass runs in chunks
-
-
 def _run(args: RecurrenceArgs, x: torch.Tensor, seqs: Optional[Sequences], pos, req, state: torch.Tensor, out: torch.Tensor, chunked: Optional[bool]):
     args.x, args.ld, args.bf16 = x.data_ptr(), x.stride(0), int(x.dtype == torch.bfloat16)
     args.state, args.slots, args.n, args.out, args.status = state.data_ptr(), state.shape[0], x.shape[0], out.data_ptr(), _status(x.device).data_ptr()
     args.pos, args.pos_stride, args.req, args.req_stride = pos.data_ptr(), pos.stride(0), req.data_ptr(), req.stride(0)
     if seqs is not None:
         args.seqs, args.n_seqs = seqs.device.data_ptr(), len(seqs.host)
-        longest = max(c for _, c, _, _ in seqs.host)
+        args.chunks, args.n_chunks, args.first_chunk = seqs.chunks.data_ptr(), seqs.chunks.shape[0], seqs.first_chunk.data_ptr()
         if chunked is None:
-            chunked = x.dtype == torch.bfloat16 and longest >= CHUNKED_FROM and hasattr(N.lib(), 'ptb_recurrence_chunked')
-        if chunked:
-            size = int(N.lib().ptb_recurrence_chunked_bytes(C.byref(args), longest))
-            if size >= 0:                                      # -1: sizes the chunk kernels do not take
-                work = torch.empty(max(1, size), dtype=torch.uint8, device=x.device)
-                N.check(N.lib().ptb_recurrence_chunked(C.byref(args), longest, work.data_ptr(), size, _st(x)), "recurrence_chunked")
-                return
+            chunked = x.dtype == torch.bfloat16 and max(c for _, c, _, _ in seqs.host) >= CHUNKED_FROM
+        size = int(N.lib().ptb_recurrence_chunked_bytes(C.byref(args))) if chunked else -1
+        if size > 0:                                           # -1: sizes the chunk kernels do not take
+            work = torch.empty(size, dtype=torch.uint8, device=x.device)
+            N.check(N.lib().ptb_recurrence_chunked(C.byref(args), work.data_ptr(), size, _st(x)), "recurrence_chunked")
+            return
     N.check(N.lib().ptb_recurrence(C.byref(args), _st(x)), "recurrence")
 
 

@@ -29,7 +29,6 @@ def _decls(L):
     L.ptb_window_rows_work_floats.restype = ll
     L.ptb_window_attn_rows.argtypes = [vp, vp, ci, ci, ci, ci, ci, ci, vp, ci, vp, ci, vp, ci, ci, vp, vp, vp, vp, ll, ci, ci, cf, ci, vp, ci, vp, ci, vp]
     L.ptb_window_attn_rows.restype = ci
-    if not hasattr(L, 'ptb_window_attn_tiles'): return  # TMP
     L.ptb_window_attn_tiles.argtypes = [vp, vp, ci, vp, ci, ci, ci, ci, ci, ci, vp, ci, ci, vp, vp, vp, vp, ll, ci, ci, cf, vp, vp]
     L.ptb_window_attn_tiles.restype = ci
 
@@ -150,7 +149,7 @@ class PromptTiles:
 
 
 def tiles_supported(q: torch.Tensor, a: WindowAttention) -> bool:
-    return hasattr(N.lib(), 'ptb_window_attn_tiles') and q.is_cuda and q.dtype == torch.bfloat16 and a.dim_stored <= 128 and a.vdim_stored <= 128
+    return q.is_cuda and q.dtype == torch.bfloat16 and a.dim_stored <= 128 and a.vdim_stored <= 128
 
 
 def window_attention_tiles(q: torch.Tensor, a: WindowAttention, tiles: PromptTiles, page_table: torch.Tensor, k_pages: torch.Tensor,
