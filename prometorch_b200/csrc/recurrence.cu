@@ -68,7 +68,7 @@ __device__ __forceinline__ void st_elems(T* p, const Elems<T, E>& r) {
     }
 }
 
-constexpr int CONV_TOKENS = 4;         // consecutive rows of one thread of a prompt pass
+constexpr int CONV_TOKENS = 16;        // consecutive rows of one thread of a prompt pass
 
 // Inputs of the channels c.. that lie `m` tokens before row i (m <= taps - 1), of which `in_batch` are rows of the batch.
 template <typename T, int E>
@@ -79,6 +79,53 @@ __device__ __forceinline__ Elems<T, E> conv_input(const ConvParams& P, int i, in
     for (int e = 0; e < E; ++e) z.v[e] = 0.f;
     if (pos - m < 0 || slot < 0) return z;
     return ld_elems<T, E>((const T*)P.state + ((size_t)slot * (P.taps - 1) + (P.taps - 1 - (m - in_batch))) * P.C + c);
+}
+
+// A prompt pass with a fixed number of taps: weights and the last inputs stay in registers while a thread walks its rows.
+template <typename T, int E, int TAPS>
+__global__ void __launch_bounds__(256) short_conv_taps_kernel(const __grid_constant__ ConvParams P) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * E;
+    if (c >= P.C) return;
+    const int lo = blockIdx.y * CONV_TOKENS, hi = min(lo + CONV_TOKENS, P.n);
+    Elems<float, E> w[TAPS], x[TAPS];                  // x[m]: the input m tokens back
+#pragma unroll
+    for (int m = 0; m < TAPS; ++m) w[m] = ld_elems<float, E>(P.w + (size_t)(TAPS - 1 - m) * P.C + c);
+    int before = -1;                                   // slot of the row before
+#pragma unroll 4
+    for (int i = lo; i < hi; ++i) {
+        int slot = P.req[(size_t)i * P.req_stride];
+        const Elems<T, E> now = ld_elems<T, E>((const T*)P.x + (size_t)i * P.ld + c);
+        if (slot < 0 || slot >= P.slots) {
+            if (P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+            slot = -1;
+        }
+        if (i == lo || slot != before) {               // a sequence starts here, or this thread's rows do
+            const int pos = P.pos[(size_t)i * P.pos_stride];
+            int in_batch = 0;
+            while (in_batch < TAPS - 1 && i - in_batch - 1 >= 0 && P.req[(size_t)(i - in_batch - 1) * P.req_stride] == slot) ++in_batch;
+#pragma unroll
+            for (int m = 1; m < TAPS; ++m) {
+                const Elems<T, E> v = conv_input<T, E>(P, i, m, in_batch, pos, slot, c);
+#pragma unroll
+                for (int e = 0; e < E; ++e) x[m].v[e] = v.v[e];
+            }
+            before = slot;
+        }
+        Elems<T, E> acc;
+#pragma unroll
+        for (int e = 0; e < E; ++e) {
+            x[0].v[e] = now.v[e];
+            float a = x[TAPS - 1].v[e] * w[TAPS - 1].v[e];
+#pragma unroll
+            for (int m = TAPS - 2; m >= 0; --m) a = fmaf(x[m].v[e], w[m].v[e], a);
+            acc.v[e] = silu(a);
+#pragma unroll
+            for (int m = TAPS - 1; m > 0; --m) x[m].v[e] = x[m - 1].v[e];
+        }
+        st_elems<T, E>((T*)P.out + (size_t)i * P.C + c, acc);
+    }
 }
 
 template <typename T, int E>
@@ -354,7 +401,10 @@ PTB_API int ptb_short_conv(const void* x, long long ld, const float* w, int C, i
     const int lanes = vec ? C / 8 : C, threads = lanes >= 256 ? 256 : (lanes + 31) / 32 * 32;
     const dim3 grid((lanes + threads - 1) / threads, (unsigned)rows);
     const bool pdl = ptb_pdl_enabled();
-    if (bf16) PTB_CUDA_OK(ptb_launch(vec ? short_conv_kernel<__nv_bfloat16, 8> : short_conv_kernel<__nv_bfloat16, 1>, grid, dim3(threads), 0, st, pdl, p));
+    if (bf16 && vec && seqs && taps >= 2 && taps <= 4)
+        PTB_CUDA_OK(ptb_launch(taps == 2 ? short_conv_taps_kernel<__nv_bfloat16, 8, 2> : taps == 3 ? short_conv_taps_kernel<__nv_bfloat16, 8, 3> : short_conv_taps_kernel<__nv_bfloat16, 8, 4>,
+                               grid, dim3(threads), 0, st, pdl, p));
+    else if (bf16) PTB_CUDA_OK(ptb_launch(vec ? short_conv_kernel<__nv_bfloat16, 8> : short_conv_kernel<__nv_bfloat16, 1>, grid, dim3(threads), 0, st, pdl, p));
     else PTB_CUDA_OK(ptb_launch(vec ? short_conv_kernel<float, 8> : short_conv_kernel<float, 1>, grid, dim3(threads), 0, st, pdl, p));
     if (seqs && taps > 1) {
         const dim3 tail((C + 255) / 256, n_seqs);

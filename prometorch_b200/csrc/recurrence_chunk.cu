@@ -34,7 +34,7 @@ struct Params {
     unsigned char* work;
     size_t stride;                     // bytes per (chunk, head)
     int Dvp;                           // value columns rounded up to 32
-    int vec;                           // 16-byte loads of x rows
+    int vec, vec_a;                    // 16-byte loads of x rows, of a
 };
 
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
@@ -70,22 +70,23 @@ __device__ __forceinline__ void store_split8(unsigned char* hi, unsigned char* l
     *reinterpret_cast<uint4*>(lo + off) = l;
 }
 
-// Rows of x (columns col .. col + width) of a chunk into a bf16 tile of `pitch` elements per row, zeros past the rows and the width.
+// Rows of x (columns col .. col + width) of a chunk on their way into a bf16 tile of `pitch` elements per row, zeros past the rows and
+// the width (cp.async where `vec` says that rows are 16-byte aligned; the caller commits and waits).
 __device__ __forceinline__ void load_rows(const PtbRecurrence& P, bool vec, int row0, int count, int col, int width, int padded, __nv_bfloat16* dst, int pitch) {
     const __nv_bfloat16* x = (const __nv_bfloat16*)P.x;
     const int ch = padded / 8;
     for (int e = threadIdx.x; e < CH * ch; e += THREADS) {
         const int r = e / ch, c = (e % ch) * 8;
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (r < count && c < width) {
-            const __nv_bfloat16* s = x + (size_t)(row0 + r) * P.ld + col + c;
-            if (vec) v = *reinterpret_cast<const uint4*>(s);
-            else {
-                __nv_bfloat16* b = reinterpret_cast<__nv_bfloat16*>(&v);
+        const bool live = r < count && c < width;
+        const __nv_bfloat16* s = x + (size_t)(row0 + (live ? r : 0)) * P.ld + col + (live ? c : 0);
+        if (vec) fa::cp_async16(smem_u32(dst + r * pitch + c), s, live);
+        else {
+            uint4 v = make_uint4(0, 0, 0, 0);
+            __nv_bfloat16* b = reinterpret_cast<__nv_bfloat16*>(&v);
+            if (live)
                 for (int k = 0; k < 8 && c + k < width; ++k) b[k] = s[k];
-            }
+            *reinterpret_cast<uint4*>(dst + r * pitch + c) = v;
         }
-        *reinterpret_cast<uint4*>(dst + r * pitch + c) = v;
     }
 }
 
@@ -95,23 +96,22 @@ struct DeltaSmem {
     static constexpr int PB = DT + 8;                  // pitch of the bf16 tiles
     static constexpr int PG = DT + 8;                  // pitch of the decays (floats)
     static constexpr int PA = CH + 4;                  // pitch of the 64 x 64 matrices (floats)
-    static constexpr int Q = 0, K = Q + CH * PB * 2, G = K + CH * PB * 2, E = G + CH * PG * 4, AQ = E + 4 * DT * 4, AK = AQ + CH * PA * 4;
-    static constexpr int TH = AK + CH * PA * 4, TL = TH + CH * CH * 2, TMP = TL + CH * CH * 2, ROW = TMP + 16 * 52 * 4, V = ROW + 3 * CH * 4 + 16;
-    static __host__ __device__ int total(int Dvp) { return V + CH * (Dvp + 8) * 2; }
+    static constexpr int K = 0, G = K + CH * PB * 2, E = G + CH * PG * 4, A = E + 4 * DT * 4, TH = A + CH * PA * 4, TL = TH + CH * CH * 2;
+    static constexpr int TMP = TL + CH * CH * 2, ROW = TMP + 16 * 52 * 4, Q = ROW + 3 * CH * 4 + 16;      // q, and v once q is done with
+    static __host__ __device__ int total(int Dvp) { return Q + CH * (Dvp > DT ? Dvp + 8 : PB) * 2; }
 };
 
 template <int DT>
-__global__ void __launch_bounds__(THREADS) delta_chunk_kernel(const __grid_constant__ Params W) {
+__global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_constant__ Params W) {
     using S = DeltaSmem<DT>;
     using L = Work<DT>;
     extern __shared__ __align__(128) unsigned char smem[];
     __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem + S::Q);
     __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem + S::K);
-    __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(smem + S::V);
+    __nv_bfloat16* v_s = q_s;
     float* G_s = reinterpret_cast<float*>(smem + S::G);            // log2 of the product of decays up to and with a token
     float* E_s = reinterpret_cast<float*>(smem + S::E);            // ... of a whole block of 16
-    float* aq = reinterpret_cast<float*>(smem + S::AQ);            // q . k, then the inverse
-    float* ak = reinterpret_cast<float*>(smem + S::AK);            // B
+    float* ak = reinterpret_cast<float*>(smem + S::A);             // B, then (1 + B)^-1 in its place
     float* tmp = reinterpret_cast<float*>(smem + S::TMP);
     float* qn = reinterpret_cast<float*>(smem + S::ROW);
     float* kn = qn + CH;
@@ -131,15 +131,34 @@ __global__ void __launch_bounds__(THREADS) delta_chunk_kernel(const __grid_const
     unsigned char* out = W.work + ((size_t)blockIdx.x * P.H + h) * W.stride;
     load_rows(P, W.vec, row0, cnt, P.q_col + hk * D, D, DT, q_s, S::PB);
     load_rows(P, W.vec, row0, cnt, P.k_col + hk * D, D, DT, k_s, S::PB);
-    load_rows(P, W.vec, row0, cnt, P.v_col + h * Dv, Dv, W.Dvp, v_s, PV);
+    if (W.vec_a) {
+        for (int e = threadIdx.x; e < CH * DT / 4; e += THREADS) {
+            const int r = e / (DT / 4), d = e % (DT / 4) * 4;
+            const bool live = r < cnt && d < D;
+            fa::cp_async16(smem_u32(G_s + r * S::PG + d), P.a + (live ? (size_t)(row0 + r) * P.ld_a + h * D + d : 0), live);
+        }
+    } else
+        for (int e = threadIdx.x; e < CH * DT; e += THREADS) {
+            const int r = e / DT, d = e % DT;
+            G_s[r * S::PG + d] = r < cnt && d < D ? P.a[(size_t)(row0 + r) * P.ld_a + h * D + d] : 0.f;
+        }
+    fa::cp_async_commit();
     const float rate = P.decay[h] * LOG2E;
-    for (int e = threadIdx.x; e < CH * DT; e += THREADS) {
-        const int r = e / DT, d = e % DT;
-        G_s[r * S::PG + d] = r < cnt && d < D ? fmaxf(-150.f, delta_log_decay(P.a[(size_t)(row0 + r) * P.ld_a + h * D + d], P.dt_bias[h * D + d], rate)) : 0.f;      // 2^-150 is 0
-    }
     if (threadIdx.x < CH)
         bt[threadIdx.x] = threadIdx.x < cnt ? sigmoid(__bfloat162float(((const __nv_bfloat16*)P.beta)[(size_t)(row0 + threadIdx.x) * P.ld_beta + h])) : 0.f;
     if (threadIdx.x == 0) *next_unit = WARPS;
+    for (int e = threadIdx.x; e < CH * S::PA; e += THREADS) ak[e] = 0.f;
+    {                                                  // the half of the q . k tiles that stays zero
+        constexpr int above = 8 * 7 / 2;               // 8 x 8 blocks above the diagonal
+        for (int e = threadIdx.x; e < above * 8; e += THREADS) {
+            int b = e / 8, r = 0;
+            while (b >= 7 - r) { b -= 7 - r; ++r; }
+            const uint32_t off = fa::tile_off<CH>(r * 8 + e % 8, r + 1 + b);
+            *reinterpret_cast<uint4*>(out + L::A + off) = make_uint4(0, 0, 0, 0);
+            *reinterpret_cast<uint4*>(out + L::A + L::ATILE + off) = make_uint4(0, 0, 0, 0);
+        }
+    }
+    fa::cp_async_wait<0>();
     __syncthreads();
     for (int r = warp; r < CH; r += WARPS) {
         float a = 0.f, b = 0.f;
@@ -151,13 +170,14 @@ __global__ void __launch_bounds__(THREADS) delta_chunk_kernel(const __grid_const
         a = warp_sum(a); b = warp_sum(b);
         if (lane == 0) { qn[r] = rsqrtf(a + UNIT_EPS) * rsqrtf((float)D); kn[r] = rsqrtf(b + UNIT_EPS); }
     }
-    for (int e = threadIdx.x; e < 4 * DT; e += THREADS) {          // running sums inside the blocks of 16
+    for (int e = threadIdx.x; e < 4 * DT; e += THREADS) {          // decays (2^-150 is 0) and their running sums inside the blocks of 16
         const int s = e / DT, d = e % DT;
+        const float dt = d < D ? P.dt_bias[h * D + d] : 0.f;
         float acc = 0.f;
-#pragma unroll
+#pragma unroll 4
         for (int i = 0; i < 16; ++i) {
             float* p = G_s + (s * 16 + i) * S::PG + d;
-            acc += *p;
+            acc += s * 16 + i < cnt && d < D ? fmaxf(-150.f, delta_log_decay(*p, dt, rate)) : 0.f;
             *p = acc;
         }
         E_s[s * DT + d] = acc;
@@ -170,8 +190,26 @@ __global__ void __launch_bounds__(THREADS) delta_chunk_kernel(const __grid_const
 #pragma unroll
         for (int i = 0; i < 16; ++i) G_s[(s * 16 + i) * S::PG + d] += base;
     }
-    for (int e = threadIdx.x; e < CH * S::PA; e += THREADS) { aq[e] = 0.f; ak[e] = 0.f; }
     __syncthreads();
+    // ---- q G, k G_end / G and G_end
+    const float* Ge = G_s + (CH - 1) * S::PG;
+    for (int e = threadIdx.x; e < CH * DT / 8; e += THREADS) {
+        const int r = e / (DT / 8), d = (e % (DT / 8)) * 8;
+        const uint4 qr = *reinterpret_cast<const uint4*>(q_s + r * S::PB + d), kr = *reinterpret_cast<const uint4*>(k_s + r * S::PB + d);
+        const uint32_t *qp = reinterpret_cast<const uint32_t*>(&qr), *kp = reinterpret_cast<const uint32_t*>(&kr);
+        const float a = qn[r], b = kn[r];
+        float fq[8], fk[8];
+#pragma unroll
+        for (int k = 0; k < 8; k += 4) {
+            const float4 G = *reinterpret_cast<const float4*>(G_s + r * S::PG + d + k), E = *reinterpret_cast<const float4*>(Ge + d + k);
+            const float2 q0 = unpack(qp[k / 2]), q1 = unpack(qp[k / 2 + 1]), k0 = unpack(kp[k / 2]), k1 = unpack(kp[k / 2 + 1]);
+            fq[k] = q0.x * a * exp2f(G.x); fq[k + 1] = q0.y * a * exp2f(G.y); fq[k + 2] = q1.x * a * exp2f(G.z); fq[k + 3] = q1.y * a * exp2f(G.w);
+            fk[k] = k0.x * b * exp2f(E.x - G.x); fk[k + 1] = k0.y * b * exp2f(E.y - G.y); fk[k + 2] = k1.x * b * exp2f(E.z - G.z); fk[k + 3] = k1.y * b * exp2f(E.w - G.w);
+        }
+        store_split8<DT>(out + L::Q, out + L::Q + L::TILE, r, d, fq);
+        store_split8<DT>(out + L::K, out + L::K + L::TILE, r, d, fk);
+    }
+    for (int d = threadIdx.x; d < DT; d += THREADS) reinterpret_cast<float*>(out + L::G)[d] = exp2f(Ge[d]);
     // ---- q . k and k . k under the decays: units 0-5 are blocks of 16 x 16 below the diagonal on the tensor cores, the rest 32 pairs each
     // of the diagonal blocks
     for (int unit = warp; unit < 6 + 17;) {
@@ -215,10 +253,11 @@ __global__ void __launch_bounds__(THREADS) delta_chunk_kernel(const __grid_const
 #pragma unroll
             for (int n = 0; n < 2; ++n)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int i = s * 16 + g + 8 * (e >> 1), j = r * 16 + n * 8 + 2 * t + (e & 1);
-                    aq[i * S::PA + j] = cq[n][e] * qn[i] * kn[j];
-                    ak[i * S::PA + j] = ck[n][e] * kn[i] * kn[j] * bt[i];
+                for (int e = 0; e < 2; ++e) {
+                    const int i = s * 16 + g + 8 * e, j = r * 16 + n * 8 + 2 * t;
+                    const float a = qn[i], b = kn[i] * bt[i], k0 = kn[j], k1 = kn[j + 1];
+                    store_split<CH>(out + L::A, out + L::A + L::ATILE, i, j, cq[n][2 * e] * a * k0, cq[n][2 * e + 1] * a * k1);
+                    *reinterpret_cast<float2*>(ak + i * S::PA + j) = make_float2(ck[n][2 * e] * b * k0, ck[n][2 * e + 1] * b * k1);
                 }
         } else {
             const int p = (unit - 6) * 32 + lane, s = p / 136, m = p % 136;
@@ -238,46 +277,62 @@ __global__ void __launch_bounds__(THREADS) delta_chunk_kernel(const __grid_const
                 sq = fmaf(q0.x, e0, fmaf(q0.y, e1, fmaf(q1.x, e2, fmaf(q1.y, e3, sq))));
                 sk = fmaf(k0.x, e0, fmaf(k0.y, e1, fmaf(k1.x, e2, fmaf(k1.y, e3, sk))));
             }
-            aq[i * S::PA + j] = sq * qn[i] * kn[j];
+            const float f = sq * qn[i] * kn[j];
+            const __nv_bfloat16 hi = __float2bfloat16_rn(f);
+            const uint32_t off = fa::tile_off<CH>(i, j >> 3) + (j & 7) * 2;
+            *reinterpret_cast<__nv_bfloat16*>(out + L::A + off) = hi;
+            *reinterpret_cast<__nv_bfloat16*>(out + L::A + L::ATILE + off) = __float2bfloat16_rn(f - __bfloat162float(hi));
             if (i != j) ak[i * S::PA + j] = sk * kn[i] * kn[j] * bt[i];
+            // the tiles' 8 x 8 blocks on the diagonal: what lies above it inside them
+            if ((i >> 3) == (j >> 3) && i != j) {
+                const uint32_t up = fa::tile_off<CH>(j, i >> 3) + (i & 7) * 2;
+                *reinterpret_cast<__nv_bfloat16*>(out + L::A + up) = __float2bfloat16_rn(0.f);
+                *reinterpret_cast<__nv_bfloat16*>(out + L::A + L::ATILE + up) = __float2bfloat16_rn(0.f);
+            }
         }
         if (lane == 0) unit = atomicAdd(next_unit, 1);
         unit = __shfl_sync(0xffffffffu, unit, 0);
     }
     __syncthreads();
-    for (int e = threadIdx.x; e < CH * CH / 8; e += THREADS) {
-        const int r = e / 8, c = (e % 8) * 8;
-        store_split8<CH>(out + L::A, out + L::A + L::ATILE, r, c, aq + r * S::PA + c);
-    }
-    __syncthreads();
-    // ---- (1 + B)^-1 over aq: the diagonal blocks by substitution (a lane owns a column), then block row after block row
-    if (warp < 4 && lane < 16) {
+    load_rows(P, W.vec, row0, cnt, P.v_col + h * Dv, Dv, W.Dvp, v_s, PV);      // over q
+    fa::cp_async_commit();
+    // ---- (1 + B)^-1 in place: the diagonal blocks by substitution (a lane owns a column), then block row after block row
+    if (warp < 4) {
         float x[16];
-        const float* b = ak + warp * 16 * S::PA + warp * 16;
+        float* b = ak + warp * 16 * S::PA + warp * 16;
+        if (lane < 16) {
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-            float v = i == lane ? 1.f : 0.f;
+            for (int i = 0; i < 16; ++i) {
+                float v = i == lane ? 1.f : 0.f;
 #pragma unroll
-            for (int m = 0; m < i; ++m) v = fmaf(-b[i * S::PA + m], x[m], v);
-            x[i] = v;
+                for (int m = 0; m < i; ++m) v = fmaf(-b[i * S::PA + m], x[m], v);
+                x[i] = v;
+            }
         }
+        __syncwarp();
+        if (lane < 16)
 #pragma unroll
-        for (int i = 0; i < 16; ++i) aq[(warp * 16 + i) * S::PA + warp * 16 + lane] = x[i];
+            for (int i = 0; i < 16; ++i) b[i * S::PA + lane] = x[i];
     }
     __syncthreads();
     for (int s = 1; s < 4; ++s) {
         const int i = threadIdx.x >> 4, c = threadIdx.x & 15;
+        const float* row = ak + (s * 16 + i) * S::PA;
         for (int r = 0; r < s; ++r) {
             float v = 0.f;
-            for (int m = r * 16; m < s * 16; ++m) v = fmaf(ak[(s * 16 + i) * S::PA + m], aq[m * S::PA + r * 16 + c], v);
+            for (int m = r * 16; m < s * 16; m += 4) {
+                const float4 f = *reinterpret_cast<const float4*>(row + m);
+                const float* y = ak + m * S::PA + r * 16 + c;
+                v = fmaf(f.x, y[0], fmaf(f.y, y[S::PA], fmaf(f.z, y[2 * S::PA], fmaf(f.w, y[3 * S::PA], v))));
+            }
             tmp[i * 52 + r * 16 + c] = v;
         }
         __syncthreads();
         for (int r = 0; r < s; ++r) {
             float v = 0.f;
 #pragma unroll
-            for (int m = 0; m < 16; ++m) v = fmaf(aq[(s * 16 + i) * S::PA + s * 16 + m], tmp[m * 52 + r * 16 + c], v);
-            aq[(s * 16 + i) * S::PA + r * 16 + c] = -v;
+            for (int m = 0; m < 16; ++m) v = fmaf(row[s * 16 + m], tmp[m * 52 + r * 16 + c], v);
+            ak[(s * 16 + i) * S::PA + r * 16 + c] = -v;
         }
         __syncthreads();
     }
@@ -285,9 +340,10 @@ __global__ void __launch_bounds__(THREADS) delta_chunk_kernel(const __grid_const
         const int r = e / 8, c = (e % 8) * 8;
         float f[8];
 #pragma unroll
-        for (int k = 0; k < 8; ++k) f[k] = c + k <= r ? aq[r * S::PA + c + k] * bt[c + k] : 0.f;
+        for (int k = 0; k < 8; ++k) f[k] = c + k <= r ? ak[r * S::PA + c + k] * bt[c + k] : 0.f;
         store_split8<CH>(smem + S::TH, smem + S::TL, r, c, f);
     }
+    fa::cp_async_wait<0>();
     __syncthreads();
     // ---- W and U: units of 16 columns
     const uint32_t th = smem_u32(smem + S::TH), tl = smem_u32(smem + S::TL);
@@ -341,21 +397,6 @@ __global__ void __launch_bounds__(THREADS) delta_chunk_kernel(const __grid_const
                 }
         }
     }
-    // ---- q G, k G_end / G and G_end
-    const float* Ge = G_s + (CH - 1) * S::PG;
-    for (int e = threadIdx.x; e < CH * DT / 8; e += THREADS) {
-        const int r = e / (DT / 8), d = (e % (DT / 8)) * 8;
-        float fq[8], fk[8];
-#pragma unroll
-        for (int k = 0; k < 8; ++k) {
-            const float G = G_s[r * S::PG + d + k];
-            fq[k] = __bfloat162float(q_s[r * S::PB + d + k]) * qn[r] * exp2f(G);
-            fk[k] = __bfloat162float(k_s[r * S::PB + d + k]) * kn[r] * exp2f(Ge[d + k] - G);
-        }
-        store_split8<DT>(out + L::Q, out + L::Q + L::TILE, r, d, fq);
-        store_split8<DT>(out + L::K, out + L::K + L::TILE, r, d, fk);
-    }
-    for (int d = threadIdx.x; d < DT; d += THREADS) reinterpret_cast<float*>(out + L::G)[d] = exp2f(Ge[d]);
 }
 
 // ---------------------------------------------------------------------------------------------- fixed decay, one chunk
@@ -454,25 +495,26 @@ __global__ void __launch_bounds__(THREADS) decay_chunk_kernel(const __grid_const
 template <int DT, int VS>
 struct StateSmem {
     using L = Work<DT>;
-    static constexpr int WQ = 0, KA = 4 * L::TILE, SH = KA + 2 * L::TILE + 2 * L::ATILE, SL = SH + VS * DT * 2, UH = SL + VS * DT * 2, UL = UH + VS * CH * 2;
+    static constexpr int WQ = 0, KA = 8 * L::TILE, SH = KA + 2 * L::TILE + 2 * L::ATILE, SL = SH + VS * DT * 2, UH = SL + VS * DT * 2, UL = UH + VS * CH * 2;
     static constexpr int BAR = UL + VS * CH * 2, TOTAL = BAR + 64;
 };
 
 // One CTA per (VS value columns, head, sequence), eight warps.  Of a chunk, warps 0-3 form u (64 rows) and then the new state, warps 4-7
 // the read-out; the state lives transposed, [value][key channel], in the accumulators of warps 0-3 and as two bf16 tiles in shared
-// memory for the products that read it.  Tiles arrive by bulk copies: those of a chunk's first half while the chunk before finishes.
+// memory for the products that read it.  Tiles arrive by bulk copies: W and q a chunk ahead, k and A while a chunk's first half runs.
 template <int DT, int VS, bool DELTA>
 __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_constant__ Params W) {
     using L = Work<DT>;
     using S = StateSmem<DT, VS>;
     constexpr int NT = DT / 32, MT = VS / 16, NB = VS / 8;         // state tiles of a warp: MT x NT of 16 x 8
     extern __shared__ __align__(128) unsigned char smem[];
-    uint64_t* bar = reinterpret_cast<uint64_t*>(smem + S::BAR);    // 0: W and q tiles, 1: k and A tiles
+    uint64_t* bar = reinterpret_cast<uint64_t*>(smem + S::BAR);    // 0, 1: W and q tiles of even and odd chunks, 2: k and A tiles
     const PtbRecurrence& P = W.P;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     if (threadIdx.x == 0) {
         mbar_init(&bar[0], 1);
         mbar_init(&bar[1], 1);
+        mbar_init(&bar[2], 1);
         mbar_fence_init();
     }
     __syncthreads();
@@ -489,16 +531,20 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
     auto tiles = [&](int c) { return W.work + ((size_t)(first + c) * P.H + h) * W.stride; };
     auto load_wq = [&](int c) {
         constexpr uint32_t bytes = (DELTA ? 4 : 2) * L::TILE;
-        mbar_expect_tx(&bar[0], bytes);
-        bulk_g2s(smem + S::WQ + (DELTA ? 0 : 2 * L::TILE), tiles(c) + (DELTA ? L::W : L::Q), bytes, &bar[0]);
+        mbar_expect_tx(&bar[c & 1], bytes);
+        bulk_g2s(smem + S::WQ + (c & 1) * 4 * L::TILE + (DELTA ? 0 : 2 * L::TILE), tiles(c) + (DELTA ? L::W : L::Q), bytes, &bar[c & 1]);
     };
     auto load_ka = [&](int c) {
         constexpr uint32_t bytes = 2 * L::TILE + 2 * L::ATILE;
-        mbar_expect_tx(&bar[1], bytes);
-        bulk_g2s(smem + S::KA, tiles(c) + L::K, bytes, &bar[1]);
+        mbar_expect_tx(&bar[2], bytes);
+        bulk_g2s(smem + S::KA, tiles(c) + L::K, bytes, &bar[2]);
     };
-    if (threadIdx.x == 0) { load_wq(0); load_ka(0); }
-    const uint32_t wh = smem_u32(smem + S::WQ), qh = wh + 2 * L::TILE, kh = smem_u32(smem + S::KA), ah = kh + 2 * L::TILE;
+    if (threadIdx.x == 0) {
+        load_wq(0);
+        load_ka(0);
+        if (chunks > 1) load_wq(1);
+    }
+    const uint32_t kh = smem_u32(smem + S::KA), ah = kh + 2 * L::TILE;
     const uint32_t sh = smem_u32(smem + S::SH), sl = smem_u32(smem + S::SL), uh = smem_u32(smem + S::UH), ul = smem_u32(smem + S::UL);
     const bool owner = warp < 4;                       // of the state channels d0 .. d0 + DT / 4
     const int wr = (warp & 3) * 16, d0 = (warp & 3) * (DT / 4);
@@ -527,43 +573,47 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
     }
     __syncthreads();
     bool ok = true;
-    for (int c = 0; c < chunks; ++c) {
+    float2 base[NB][2];                                // U (delta) or v (a pair of bf16 in x) of rows wr + g, wr + g + 8 of the chunk ahead
+    const bool pairs = (Dv & 1) == 0 && (P.ld & 1) == 0 && (P.v_col & 1) == 0 && ((uintptr_t)P.x & 3) == 0;
+    auto fetch = [&](int c) {
         const int row0 = sp.row0 + c * CH, cnt = min(CH, sp.count - c * CH);
-        const unsigned char* tile = tiles(c);
-        float acc[NB][4], ge[NT][2];
 #pragma unroll
         for (int n = 0; n < NB; ++n)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
-        float2 base[NB][2];                            // U (delta) or v of rows wr + g, wr + g + 8
+            for (int e = 0; e < 2; ++e) {
+                const int r = wr + g + 8 * e, v = v0 + n * 8 + 2 * t;
+                if constexpr (DELTA) base[n][e] = *reinterpret_cast<const float2*>(tiles(c) + L::U + ((size_t)r * W.Dvp + v) * 4);
+                else {
+                    uint32_t f = 0;
+                    if (r < cnt && v < Dv) {
+                        const __nv_bfloat16* x = (const __nv_bfloat16*)P.x + (size_t)(row0 + r) * P.ld + P.v_col + (size_t)h * Dv + v;
+                        if (pairs) f = *reinterpret_cast<const uint32_t*>(x);
+                        else f = *reinterpret_cast<const uint16_t*>(x) | (v + 1 < Dv ? (uint32_t)*reinterpret_cast<const uint16_t*>(x + 1) << 16 : 0u);
+                    }
+                    base[n][e].x = __uint_as_float(f);
+                }
+            }
+    };
+    if (owner) fetch(0);
+    for (int c = 0; c < chunks; ++c) {
+        const int row0 = sp.row0 + c * CH, cnt = min(CH, sp.count - c * CH);
+        const uint32_t wh = smem_u32(smem + S::WQ + (c & 1) * 4 * L::TILE), qh = wh + 2 * L::TILE;
+        float acc[NB][4], low[NB][4], ge[NT][2];       // products of the high parts; those with a low part
+#pragma unroll
+        for (int n = 0; n < NB; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[n][e] = low[n][e] = 0.f;
         if (owner) {
 #pragma unroll
             for (int n = 0; n < NT; ++n) {
-                const float2 f = *reinterpret_cast<const float2*>(tile + L::G + (d0 + n * 8 + 2 * t) * 4);
+                const float2 f = *reinterpret_cast<const float2*>(tiles(c) + L::G + (d0 + n * 8 + 2 * t) * 4);
                 ge[n][0] = f.x; ge[n][1] = f.y;
             }
-#pragma unroll
-            for (int n = 0; n < NB; ++n)
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const int r = wr + g + 8 * e, v = v0 + n * 8 + 2 * t;
-                    if constexpr (DELTA) base[n][e] = *reinterpret_cast<const float2*>(tile + L::U + ((size_t)r * W.Dvp + v) * 4);
-                    else {
-                        float2 f = make_float2(0.f, 0.f);
-                        if (r < cnt) {
-                            const __nv_bfloat16* x = (const __nv_bfloat16*)P.x + (size_t)(row0 + r) * P.ld + P.v_col + (size_t)h * Dv + v;
-                            if (v < Dv) f.x = __bfloat162float(x[0]);
-                            if (v + 1 < Dv) f.y = __bfloat162float(x[1]);
-                            if (P.silu) { f.x = silu(f.x); f.y = silu(f.y); }
-                        }
-                        base[n][e] = f;
-                    }
-                }
         }
-        if (ok) ok = mbar_wait(&bar[0], (uint32_t)(c & 1), P.status);
+        if (ok) ok = mbar_wait(&bar[c & 1], (uint32_t)((c >> 1) & 1), P.status);
         if (DELTA || !owner) {                         // W S (warps 0-3) or (q G) S (warps 4-7): 16 rows each
             const uint32_t th = owner ? wh : qh, tl = th + L::TILE;
-#pragma unroll 2
+#pragma unroll 4
             for (int ks = 0; ks < DT / 16; ++ks) {
                 uint32_t a[4], b[4];
                 fa::load_a<DT>(th, wr, ks, a);
@@ -573,28 +623,39 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                     uint32_t bh[4], bl[4];
                     fa::load_b<DT>(sh, n * 16, ks, bh);
                     fa::load_b<DT>(sl, n * 16, ks, bl);
-                    mma3(acc[2 * n], a, b, bh[0], bh[1], bl[0], bl[1]);
-                    mma3(acc[2 * n + 1], a, b, bh[2], bh[3], bl[2], bl[3]);
+                    fa::mma16816(acc[2 * n], a, bh[0], bh[1]);
+                    fa::mma16816(acc[2 * n + 1], a, bh[2], bh[3]);
+                    fa::mma16816(low[2 * n], b, bh[0], bh[1]);
+                    fa::mma16816(low[2 * n + 1], b, bh[2], bh[3]);
+                    fa::mma16816(low[2 * n], a, bl[0], bl[1]);
+                    fa::mma16816(low[2 * n + 1], a, bl[2], bl[3]);
                 }
             }
+#pragma unroll
+            for (int n = 0; n < NB; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) acc[n][e] += low[n][e];
         }
         if (owner) {                                   // u^T, split
 #pragma unroll
             for (int n = 0; n < NB; ++n)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const float2 f = base[n][e >> 1];
-                    const float u = ((e & 1) ? f.y : f.x) - acc[n][e];
+                    const float2 f = DELTA ? base[n][e >> 1] : unpack(__float_as_uint(base[n][e >> 1].x));
+                    float u = (e & 1) ? f.y : f.x;
+                    if constexpr (DELTA) u -= acc[n][e];
+                    else if (P.silu) u = silu(u);
                     const int v = n * 8 + 2 * t + (e & 1), r = wr + g + 8 * (e >> 1);
                     const __nv_bfloat16 hi = __float2bfloat16_rn(u);
                     const uint32_t off = fa::tile_off<CH>(v, r >> 3) + (r & 7) * 2;
                     *reinterpret_cast<__nv_bfloat16*>(smem + S::UH + off) = hi;
                     *reinterpret_cast<__nv_bfloat16*>(smem + S::UL + off) = __float2bfloat16_rn(u - __bfloat162float(hi));
                 }
+            if (c + 1 < chunks) fetch(c + 1);
         }
         __syncthreads();                               // u is there; W, q and the state tiles have been read
-        if (threadIdx.x == 0 && c + 1 < chunks && ok) load_wq(c + 1);
-        if (ok) ok = mbar_wait(&bar[1], (uint32_t)(c & 1), P.status);
+        if (threadIdx.x == 0 && c + 2 < chunks && ok) load_wq(c + 2);
+        if (ok) ok = mbar_wait(&bar[2], (uint32_t)(c & 1), P.status);
         if (owner) {
 #pragma unroll
             for (int m = 0; m < MT; ++m)
@@ -723,5 +784,6 @@ PTB_API int ptb_recurrence_chunked(const PtbRecurrence* args, void* work, long l
     p.Dvp = (args->Dv + 31) / 32 * 32;
     p.vec = args->D % 8 == 0 && args->Dv % 8 == 0 && args->ld % 8 == 0 && args->q_col % 8 == 0 && args->k_col % 8 == 0 && args->v_col % 8 == 0 &&
             ((uintptr_t)args->x & 15) == 0;
+    p.vec_a = args->D % 4 == 0 && args->ld_a % 4 == 0 && ((uintptr_t)args->a & 15) == 0;
     return args->D <= 64 ? rc::launch<64>(p, st) : rc::launch<128>(p, st);
 }

@@ -246,6 +246,123 @@ __global__ void __launch_bounds__(RS_THREADS) residual_norm_kernel(const Branch 
     }
 }
 
+// The same for the many rows of a prompt (bf16 branches of one part each): persistent CTAs, the inputs of the rows ahead arrive by bulk
+// copies in two stages of shared memory, the weights stay in registers.  W is a multiple of eight and at most 4 NK RS_THREADS.
+template <int NB> __host__ __device__ constexpr int stream_row_bytes(int W) { return W * (4 + 2 * NB); }
+template <int NK, int NB>
+__global__ void __launch_bounds__(RS_THREADS) residual_norm_stream_kernel(const Branch A, const Branch B, float eps, float* __restrict__ x,
+                                                                          const float* __restrict__ w, __nv_bfloat16* __restrict__ out, int n, int W,
+                                                                          int* status) {
+    extern __shared__ __align__(128) unsigned char smem[];
+    __shared__ float red[4][32];
+    __shared__ uint64_t bar[2];
+    const int nc = W / 4, stage = (stream_row_bytes<NB>(W) + 127) & ~127;
+    if (threadIdx.x == 0) {
+        mbar_init(&bar[0], 1);
+        mbar_init(&bar[1], 1);
+        mbar_fence_init();
+    }
+    __syncthreads();
+    pdl_wait();
+    pdl_launch_dependents();
+    auto load = [&](int row, int s) {
+        unsigned char* d = smem + s * stage;
+        mbar_expect_tx(&bar[s], (uint32_t)stream_row_bytes<NB>(W));
+        bulk_g2s(d, x + (size_t)row * W, W * 4, &bar[s]);
+        bulk_g2s(d + W * 4, (const __nv_bfloat16*)A.y + (size_t)row * A.ld, W * 2, &bar[s]);
+        if constexpr (NB == 2) bulk_g2s(d + W * 6, (const __nv_bfloat16*)B.y + (size_t)row * B.ld, W * 2, &bar[s]);
+    };
+    if (threadIdx.x == 0) {
+        load(blockIdx.x, 0);
+        if ((int)(blockIdx.x + gridDim.x) < n) load(blockIdx.x + gridDim.x, 1);
+    }
+    const float4 one = make_float4(1.f, 1.f, 1.f, 1.f);
+    float4 wa[NK], wb[NB == 2 ? NK : 1], wn[NK];
+#pragma unroll
+    for (int k = 0; k < NK; ++k) {
+        const int c = k * RS_THREADS + threadIdx.x;
+        wa[k] = c < nc && A.w ? load4<float>(A.w + c * 4) : one;
+        if constexpr (NB == 2) wb[k] = c < nc && B.w ? load4<float>(B.w + c * 4) : one;
+        wn[k] = c < nc ? load4<float>(w + c * 4) : one;
+    }
+    bool ok = true;
+    int it = 0;
+    for (int row = blockIdx.x; row < n; row += gridDim.x, ++it) {
+        const int s = it & 1;
+        if (ok) ok = mbar_wait(&bar[s], (uint32_t)((it >> 1) & 1), status);
+        const float* xs_s = reinterpret_cast<const float*>(smem + s * stage);
+        const __nv_bfloat16* a_s = reinterpret_cast<const __nv_bfloat16*>(smem + s * stage + W * 4);
+        const __nv_bfloat16* b_s = reinterpret_cast<const __nv_bfloat16*>(smem + s * stage + W * 6);
+        float4 a[NK], b[NB == 2 ? NK : 1];
+        float ra = A.g, rb = B.g, sa = 0.f, sb = 0.f;
+#pragma unroll
+        for (int k = 0; k < NK; ++k) {
+            const int c = k * RS_THREADS + threadIdx.x;
+            if (c < nc) {
+                a[k] = load4<__nv_bfloat16>(a_s + c * 4);
+                sa += a[k].x * a[k].x + a[k].y * a[k].y + a[k].z * a[k].z + a[k].w * a[k].w;
+                if constexpr (NB == 2) {
+                    b[k] = load4<__nv_bfloat16>(b_s + c * 4);
+                    sb += b[k].x * b[k].x + b[k].y * b[k].y + b[k].z * b[k].z + b[k].w * b[k].w;
+                }
+            }
+        }
+        if (A.w || (NB == 2 && B.w)) {
+            sa = warp_sum(sa);
+            if constexpr (NB == 2) sb = warp_sum(sb);
+            if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sa; red[1][threadIdx.x >> 5] = sb; }
+            __syncthreads();
+            sa = sb = 0.f;
+#pragma unroll
+            for (int i = 0; i < RS_THREADS / 32; ++i) { sa += red[0][i]; sb += red[1][i]; }
+            if (A.w) ra *= rsqrtf(sa / (float)W + eps);
+            if (NB == 2 && B.w) rb *= rsqrtf(sb / (float)W + eps);
+        }
+        float ss = 0.f;
+        float4 v[NK];
+#pragma unroll
+        for (int k = 0; k < NK; ++k) {
+            const int c = k * RS_THREADS + threadIdx.x;
+            if (c < nc) {
+                float4 r = load4<float>(xs_s + c * 4);
+                r.x += a[k].x * ra * wa[k].x; r.y += a[k].y * ra * wa[k].y; r.z += a[k].z * ra * wa[k].z; r.w += a[k].w * ra * wa[k].w;
+                if constexpr (NB == 2) { r.x += b[k].x * rb * wb[k].x; r.y += b[k].y * rb * wb[k].y; r.z += b[k].z * rb * wb[k].z; r.w += b[k].w * rb * wb[k].w; }
+                ss += r.x * r.x + r.y * r.y + r.z * r.z + r.w * r.w;
+                store4(x + (size_t)row * W + c * 4, r);
+                v[k] = r;
+            }
+        }
+        ss = warp_sum(ss);
+        if ((threadIdx.x & 31) == 0) red[2 + s][threadIdx.x >> 5] = ss;
+        __syncthreads();                               // and the stage has been read
+        if (threadIdx.x == 0 && ok && row + 2 * (int)gridDim.x < n) load(row + 2 * gridDim.x, s);
+        ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < RS_THREADS / 32; ++i) ss += red[2 + s][i];
+        const float rs = rsqrtf(ss / (float)W + eps);
+#pragma unroll
+        for (int k = 0; k < NK; ++k) {
+            const int c = k * RS_THREADS + threadIdx.x;
+            if (c < nc) store4(out + (size_t)row * W + c * 4, make_float4(v[k].x * rs * wn[k].x, v[k].y * rs * wn[k].y, v[k].z * rs * wn[k].z, v[k].w * rs * wn[k].w));
+        }
+    }
+}
+
+template <int NK, int NB>
+static cudaError_t residual_norm_stream(const Branch& A, const Branch& B, float eps, float* x, const float* w, void* out, int n, int W, int* status,
+                                        cudaStream_t st) {
+    const int smem = 2 * ((stream_row_bytes<NB>(W) + 127) & ~127);
+    auto k = residual_norm_stream_kernel<NK, NB>;
+    cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return e;
+    int dev = 0, sms = 0, per = 0;
+    if ((e = cudaGetDevice(&dev)) != cudaSuccess) return e;
+    if ((e = cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev)) != cudaSuccess) return e;
+    if ((e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per, k, RS_THREADS, smem)) != cudaSuccess) return e;
+    return ptb_launch(k, dim3(std::min(n, sms * std::max(1, per))), dim3(RS_THREADS), (size_t)smem, st, ptb_pdl_enabled(), A, B, eps, x, w,
+                      (__nv_bfloat16*)out, n, W, status);
+}
+
 template <typename T, int NB>
 static cudaError_t residual_norm_launch(const Branch& A, const Branch& B, float eps, float* x, const float* w, void* out, int n, int W, bool vec,
                                         cudaStream_t st) {
@@ -263,15 +380,22 @@ using namespace ptb;
 
 // x [n, W] fp32 += branch a (+ branch b, absent with yb null); h [n, W] (bf16 or fp32) = x / rms(x) * w unless w is null.  A branch: y in
 // bf16 (f32 = 0) or as the sum of `splits` fp32 matrices `stride` apart, row pitch ld; times g; RMS-normed with the fp32 weight w[W]
-// when that is given.  eps sits inside every root.
+// when that is given.  eps sits inside every root.  status: device int, set
+// non-zero if a copy never arrived.
 PTB_API int ptb_residual_norm(float* x, const void* ya, int f32a, int splits_a, long long stride_a, long long ld_a, const float* wa, float ga,
                               const void* yb, int f32b, int splits_b, long long stride_b, long long ld_b, const float* wb, float gb, float eps,
-                              const float* w, void* h, int n, int W, int bf16, cudaStream_t st) {
+                              const float* w, void* h, int n, int W, int bf16, int* status, cudaStream_t st) {
     if (n <= 0) return 0;
     const Branch A{ya, f32a, splits_a, stride_a, ld_a, wa, ga}, B{yb, f32b, splits_b, stride_b, ld_b, wb, gb};
     const uintptr_t bases = (uintptr_t)x | (uintptr_t)ya | (uintptr_t)yb | (uintptr_t)wa | (uintptr_t)wb | (uintptr_t)w | (uintptr_t)h;
     const bool vec = W % 4 == 0 && (bases & 15) == 0 && ld_a % 4 == 0 && ld_b % 4 == 0 && stride_a % 4 == 0 && stride_b % 4 == 0;
     if (!ya || (splits_a > 1 && !f32a) || (splits_b > 1 && !f32b)) { ptb_set_error("residual_norm: partials are fp32, and the first branch is there"); return -1; }
+    const bool stream = vec && bf16 && w && !f32a && !(yb && f32b) && n >= 1024 && W % 8 == 0 && ld_a % 8 == 0 && ld_b % 8 == 0 && W <= 16 * RS_THREADS;
+    if (stream) {
+        const bool small = W <= 8 * RS_THREADS;
+        PTB_CUDA_OK((yb ? (small ? residual_norm_stream<2, 2> : residual_norm_stream<4, 2>) : (small ? residual_norm_stream<2, 1> : residual_norm_stream<4, 1>))(A, B, eps, x, w, h, n, W, status, st));
+        return 0;
+    }
     if (bf16) PTB_CUDA_OK((yb ? residual_norm_launch<__nv_bfloat16, 2> : residual_norm_launch<__nv_bfloat16, 1>)(A, B, eps, x, w, h, n, W, vec, st));
     else PTB_CUDA_OK((yb ? residual_norm_launch<float, 2> : residual_norm_launch<float, 1>)(A, B, eps, x, w, h, n, W, vec, st));
     PTB_CUDA_OK(cudaGetLastError());

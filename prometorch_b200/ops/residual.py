@@ -28,7 +28,7 @@ def _decls(L):
     L.ptb_row_norm.argtypes = [vp, vp, ci, vp, cf, cf, vp, ci, ci, vp, ci, vp]
     L.ptb_gemm_bf16_splitk_f32.argtypes = [vp, ll, vp, ll, vp, ll, ci, ci, ci, ci, vp, vp, ci, vp]
     L.ptb_gemm_bf16_splitk_post_norm.argtypes = [vp, ll, vp, ll, ci, ci, ci, ci, vp, vp, cf, cf, vp, vp, vp, ci, vp]
-    L.ptb_residual_norm.argtypes = [vp, vp, ci, ci, ll, ll, vp, cf, vp, ci, ci, ll, ll, vp, cf, cf, vp, vp, ci, ci, ci, vp]
+    L.ptb_residual_norm.argtypes = [vp, vp, ci, ci, ll, ll, vp, cf, vp, ci, ci, ll, ll, vp, cf, cf, vp, vp, ci, ci, ci, vp, vp]
     for n in ("ptb_residual_norm", "ptb_embed_residual", "ptb_post_norm_add", "ptb_row_norm", "ptb_gemm_bf16_splitk_f32", "ptb_gemm_bf16_splitk_post_norm"):
         getattr(L, n).restype = ci
 
@@ -150,7 +150,7 @@ def residual_norm(x: torch.Tensor, branches: Sequence[Branch], eps: float, w: Op
     out = torch.empty(n, W, dtype=dtype or x.dtype, device=x.device) if w is not None else None
     assert len(branches) <= 2 and x.is_contiguous() and x.dtype == torch.float32 and all(b.y.stride(-1) == 1 for b in branches)
     N.check(N.lib().ptb_residual_norm(x.data_ptr(), *p[0], *p[1], float(eps), N.ptr(w), N.ptr(out), n, W,
-                                      _bf16(out) if out is not None else 0, _st(x)), "residual_norm")
+                                      _bf16(out) if out is not None else 0, _status(x.device).data_ptr(), _st(x)), "residual_norm")
     return out
 
 

@@ -284,14 +284,13 @@ def test_group_norm_gate_kernel(gs, groups, dtype):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("W", [64, 2048, 4096, 9000, 50])
-def test_residual_norm_kernel(dtype, W):
+@pytest.mark.parametrize("W,n", [(64, 19), (2048, 19), (4096, 19), (9000, 19), (50, 19), (264, 1500), (2048, 1100), (4096, 2500), (4104, 1030)])
+def test_residual_norm_kernel(dtype, W, n):
     from prometorch_b200.ops import residual as S
-    n = 19
     x, y, z = torch.randn(n, W), torch.randn(n, W).to(dtype), torch.randn(3, n, W)
     w = [torch.randn(W) for _ in range(3)]
     c = lambda t: t.cuda()
-    for make in (lambda f: [S.Branch(f(y), 0.5, f(w[0])), S.Branch(f(z), 0.25, f(w[1]))], lambda f: [S.Branch(f(z))], lambda f: [S.Branch(f(y), 1.0), S.Branch(f(y), 2.0, f(w[0]))]):
+    for make in (lambda f: [S.Branch(f(y))], lambda f: [S.Branch(f(y), 0.5, f(w[0])), S.Branch(f(y), 0.25, f(w[1]))], lambda f: [S.Branch(f(y), 0.5, f(w[0])), S.Branch(f(z), 0.25, f(w[1]))], lambda f: [S.Branch(f(z))], lambda f: [S.Branch(f(y), 1.0), S.Branch(f(y), 2.0, f(w[0]))]):
         xc, xg = x.clone(), x.cuda()
         want = S.residual_norm(xc, make(lambda t: t), 1e-3, w[2], torch.float32)
         got = S.residual_norm(xg, make(c), 1e-3, c(w[2]), dtype)
