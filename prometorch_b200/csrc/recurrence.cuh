@@ -15,7 +15,14 @@ template <typename T> __device__ __forceinline__ T rc_t(float v);
 template <> __device__ __forceinline__ float rc_t<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 rc_t<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
-__device__ __forceinline__ float softplus(float x) { return x > 15.f ? x + __expf(-x) : log1pf(__expf(x)); }
+// max(x, 0) + log(1 + z) with z = exp(-|x|) <= 1, by log(1 + z) = 2 artanh(s), s = z / (2 + z) <= 1/3, and the series of artanh through
+// s^13 (the next term is below 1e-8 of the sum).
+__device__ __forceinline__ float softplus(float x) {
+    const float z = __expf(-fabsf(x)), s = __fdividef(z, 2.f + z), q = s * s;
+    float p = fmaf(q, 1.f / 13.f, 1.f / 11.f);
+    p = fmaf(q, p, 1.f / 9.f); p = fmaf(q, p, 1.f / 7.f); p = fmaf(q, p, 1.f / 5.f); p = fmaf(q, p, 1.f / 3.f);
+    return fmaxf(x, 0.f) + 2.f * s * fmaf(q, p, 1.f);
+}
 // log of the decay of one head's key channel
 __device__ __forceinline__ float delta_log_decay(float a, float dt, float rate) { return -rate * softplus(a + dt); }
 

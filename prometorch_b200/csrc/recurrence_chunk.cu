@@ -20,6 +20,7 @@ namespace rc {
 
 constexpr int CH = 64, THREADS = 256, WARPS = 8;
 constexpr float LOG2E = 1.4426950408889634f;
+constexpr float MILD = -60.f;          // log2 of what a block of 16 tokens may keep of a channel: both factors of every pair stay finite
 
 // Workspace of one (chunk, head): bf16 tiles in the swizzled order of fa::tile_off, high parts then low parts.
 template <int DT>
@@ -97,7 +98,7 @@ struct DeltaSmem {
     static constexpr int PG = DT + 8;                  // pitch of the decays (floats)
     static constexpr int PA = CH + 4;                  // pitch of the 64 x 64 matrices (floats)
     static constexpr int K = 0, G = K + CH * PB * 2, E = G + CH * PG * 4, A = E + 4 * DT * 4, TH = A + CH * PA * 4, TL = TH + CH * CH * 2;
-    static constexpr int TMP = TL + CH * CH * 2, ROW = TMP + 16 * 52 * 4, Q = ROW + 3 * CH * 4 + 16;      // q, and v once q is done with
+    static constexpr int TMP = TL + CH * CH * 2, ROW = TMP + 16 * 52 * 4, Q = ROW + 3 * CH * 4 + 32;      // q, and v once q is done with
     static __host__ __device__ int total(int Dvp) { return Q + CH * (Dvp > DT ? Dvp + 8 : PB) * 2; }
 };
 
@@ -112,11 +113,13 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
     float* G_s = reinterpret_cast<float*>(smem + S::G);            // log2 of the product of decays up to and with a token
     float* E_s = reinterpret_cast<float*>(smem + S::E);            // ... of a whole block of 16
     float* ak = reinterpret_cast<float*>(smem + S::A);             // B, then (1 + B)^-1 in its place
-    float* tmp = reinterpret_cast<float*>(smem + S::TMP);
+    float* tmp = reinterpret_cast<float*>(smem + S::TMP);          // zeros until the inverse uses it
+    const float* zeros = tmp;
     float* qn = reinterpret_cast<float*>(smem + S::ROW);
     float* kn = qn + CH;
     float* bt = kn + CH;
     int* next_unit = reinterpret_cast<int*>(bt + CH);
+    int* mild = next_unit + 4;
     const PtbRecurrence& P = W.P;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     pdl_wait();
@@ -148,6 +151,7 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
         bt[threadIdx.x] = threadIdx.x < cnt ? sigmoid(__bfloat162float(((const __nv_bfloat16*)P.beta)[(size_t)(row0 + threadIdx.x) * P.ld_beta + h])) : 0.f;
     if (threadIdx.x == 0) *next_unit = WARPS;
     for (int e = threadIdx.x; e < CH * S::PA; e += THREADS) ak[e] = 0.f;
+    if (threadIdx.x < DT) tmp[threadIdx.x] = 0.f;
     {                                                  // the half of the q . k tiles that stays zero
         constexpr int above = 8 * 7 / 2;               // 8 x 8 blocks above the diagonal
         for (int e = threadIdx.x; e < above * 8; e += THREADS) {
@@ -190,6 +194,12 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
 #pragma unroll
         for (int i = 0; i < 16; ++i) G_s[(s * 16 + i) * S::PG + d] += base;
     }
+    if (warp >= 4) {                                   // whether a block's decays allow one reference for all its pairs
+        float least = 0.f;
+        for (int d = lane; d < DT; d += 32) least = fminf(least, E_s[(warp - 4) * DT + d]);
+        least = -warp_max(-least);
+        if (lane == 0) mild[warp - 4] = least > MILD;
+    }
     __syncthreads();
     // ---- q G, k G_end / G and G_end
     const float* Ge = G_s + (CH - 1) * S::PG;
@@ -210,12 +220,12 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
         store_split8<DT>(out + L::K, out + L::K + L::TILE, r, d, fk);
     }
     for (int d = threadIdx.x; d < DT; d += THREADS) reinterpret_cast<float*>(out + L::G)[d] = exp2f(Ge[d]);
-    // ---- q . k and k . k under the decays: units 0-5 are blocks of 16 x 16 below the diagonal on the tensor cores, the rest 32 pairs each
-    // of the diagonal blocks
-    for (int unit = warp; unit < 6 + 17;) {
-        if (unit < 6) {
-            const int s = unit < 1 ? 1 : unit < 3 ? 2 : 3, r = unit - (s == 1 ? 0 : s == 2 ? 1 : 3);
-            const float* base = G_s + (s * 16 - 1) * S::PG;        // both factors refer to the end of the block before s
+    // ---- q . k and k . k under the decays: units 0-9 are blocks of 16 x 16 on the tensor cores, six below the diagonal and those on it
+    // whose decays are mild; the others 32 pairs each of the remaining blocks on the diagonal
+    for (int unit = warp; unit < 10 + 17;) {
+        if (unit < 6 || (unit < 10 && mild[unit - 6])) {
+            const int s = unit >= 6 ? unit - 6 : unit < 1 ? 1 : unit < 3 ? 2 : 3, r = unit >= 6 ? s : unit - (s == 1 ? 0 : s == 2 ? 1 : 3);
+            const float* base = s ? G_s + (s * 16 - 1) * S::PG : zeros;       // both factors refer to the end of the block before s
             float cq[2][4], ck[2][4];
 #pragma unroll
             for (int n = 0; n < 2; ++n)
@@ -256,11 +266,11 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
                 for (int e = 0; e < 2; ++e) {
                     const int i = s * 16 + g + 8 * e, j = r * 16 + n * 8 + 2 * t;
                     const float a = qn[i], b = kn[i] * bt[i], k0 = kn[j], k1 = kn[j + 1];
-                    store_split<CH>(out + L::A, out + L::A + L::ATILE, i, j, cq[n][2 * e] * a * k0, cq[n][2 * e + 1] * a * k1);
-                    *reinterpret_cast<float2*>(ak + i * S::PA + j) = make_float2(ck[n][2 * e] * b * k0, ck[n][2 * e + 1] * b * k1);
+                    store_split<CH>(out + L::A, out + L::A + L::ATILE, i, j, j <= i ? cq[n][2 * e] * a * k0 : 0.f, j < i ? cq[n][2 * e + 1] * a * k1 : 0.f);
+                    *reinterpret_cast<float2*>(ak + i * S::PA + j) = make_float2(j < i ? ck[n][2 * e] * b * k0 : 0.f, j + 1 < i ? ck[n][2 * e + 1] * b * k1 : 0.f);
                 }
-        } else {
-            const int p = (unit - 6) * 32 + lane, s = p / 136, m = p % 136;
+        } else if (unit >= 10 && !mild[(unit - 10) * 32 / 136] + !mild[((unit - 10) * 32 + 31) / 136]) {
+            const int p = (unit - 10) * 32 + lane, s = p / 136, m = p % 136;
             int a = (int)((sqrtf(8.f * m + 1.f) - 1.f) * 0.5f);
             while (a * (a + 1) / 2 > m) --a;
             while ((a + 1) * (a + 2) / 2 <= m) ++a;
@@ -495,20 +505,22 @@ __global__ void __launch_bounds__(THREADS) decay_chunk_kernel(const __grid_const
 template <int DT, int VS>
 struct StateSmem {
     using L = Work<DT>;
-    static constexpr int WQ = 0, KA = 8 * L::TILE, SH = KA + 2 * L::TILE + 2 * L::ATILE, SL = SH + VS * DT * 2, UH = SL + VS * DT * 2, UL = UH + VS * CH * 2;
+    static constexpr int SLOT = 4 * L::TILE > 2 * L::TILE + 2 * L::ATILE ? 4 * L::TILE : 2 * L::TILE + 2 * L::ATILE, SH = 3 * SLOT, SL = SH + VS * DT * 2, UH = SL + VS * DT * 2, UL = UH + VS * CH * 2;
     static constexpr int BAR = UL + VS * CH * 2, TOTAL = BAR + 64;
 };
 
 // One CTA per (VS value columns, head, sequence), eight warps.  Of a chunk, warps 0-3 form u (64 rows) and then the new state, warps 4-7
 // the read-out; the state lives transposed, [value][key channel], in the accumulators of warps 0-3 and as two bf16 tiles in shared
-// memory for the products that read it.  Tiles arrive by bulk copies: W and q a chunk ahead, k and A while a chunk's first half runs.
+// memory for the products that read it.  Tiles arrive by bulk copies through three slots, in the order of their use: W and q of a chunk,
+// its k and A, W and q of the next, ...  Products of high parts and those with a low part have accumulators of their own, and every
+// accumulator waits for its turn among at least four, so that the tensor pipe is not held up by dependent products.
 template <int DT, int VS, bool DELTA>
 __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_constant__ Params W) {
     using L = Work<DT>;
     using S = StateSmem<DT, VS>;
     constexpr int NT = DT / 32, MT = VS / 16, NB = VS / 8;         // state tiles of a warp: MT x NT of 16 x 8
     extern __shared__ __align__(128) unsigned char smem[];
-    uint64_t* bar = reinterpret_cast<uint64_t*>(smem + S::BAR);    // 0, 1: W and q tiles of even and odd chunks, 2: k and A tiles
+    uint64_t* bar = reinterpret_cast<uint64_t*>(smem + S::BAR);    // one per slot
     const PtbRecurrence& P = W.P;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     if (threadIdx.x == 0) {
@@ -529,22 +541,21 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
         return;
     }
     auto tiles = [&](int c) { return W.work + ((size_t)(first + c) * P.H + h) * W.stride; };
-    auto load_wq = [&](int c) {
-        constexpr uint32_t bytes = (DELTA ? 4 : 2) * L::TILE;
-        mbar_expect_tx(&bar[c & 1], bytes);
-        bulk_g2s(smem + S::WQ + (c & 1) * 4 * L::TILE + (DELTA ? 0 : 2 * L::TILE), tiles(c) + (DELTA ? L::W : L::Q), bytes, &bar[c & 1]);
+    // load 2c: W and q of chunk c, load 2c + 1: its k and A; load i goes to slot i % 3 once load i - 3 has been read
+    auto load = [&](int i) {
+        const int s = i % 3;
+        if (i & 1) {
+            constexpr uint32_t bytes = 2 * L::TILE + 2 * L::ATILE;
+            mbar_expect_tx(&bar[s], bytes);
+            bulk_g2s(smem + s * S::SLOT, tiles(i >> 1) + L::K, bytes, &bar[s]);
+        } else {
+            constexpr uint32_t bytes = (DELTA ? 4 : 2) * L::TILE;
+            mbar_expect_tx(&bar[s], bytes);
+            bulk_g2s(smem + s * S::SLOT + (DELTA ? 0 : 2 * L::TILE), tiles(i >> 1) + (DELTA ? L::W : L::Q), bytes, &bar[s]);
+        }
     };
-    auto load_ka = [&](int c) {
-        constexpr uint32_t bytes = 2 * L::TILE + 2 * L::ATILE;
-        mbar_expect_tx(&bar[2], bytes);
-        bulk_g2s(smem + S::KA, tiles(c) + L::K, bytes, &bar[2]);
-    };
-    if (threadIdx.x == 0) {
-        load_wq(0);
-        load_ka(0);
-        if (chunks > 1) load_wq(1);
-    }
-    const uint32_t kh = smem_u32(smem + S::KA), ah = kh + 2 * L::TILE;
+    if (threadIdx.x == 0)
+        for (int i = 0; i < min(3, 2 * chunks); ++i) load(i);
     const uint32_t sh = smem_u32(smem + S::SH), sl = smem_u32(smem + S::SL), uh = smem_u32(smem + S::UH), ul = smem_u32(smem + S::UL);
     const bool owner = warp < 4;                       // of the state channels d0 .. d0 + DT / 4
     const int wr = (warp & 3) * 16, d0 = (warp & 3) * (DT / 4);
@@ -597,7 +608,8 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
     if (owner) fetch(0);
     for (int c = 0; c < chunks; ++c) {
         const int row0 = sp.row0 + c * CH, cnt = min(CH, sp.count - c * CH);
-        const uint32_t wh = smem_u32(smem + S::WQ + (c & 1) * 4 * L::TILE), qh = wh + 2 * L::TILE;
+        const uint32_t wh = smem_u32(smem + (2 * c % 3) * S::SLOT), qh = wh + 2 * L::TILE;
+        const uint32_t kh = smem_u32(smem + ((2 * c + 1) % 3) * S::SLOT), ah = kh + 2 * L::TILE;
         float acc[NB][4], low[NB][4], ge[NT][2];       // products of the high parts; those with a low part
 #pragma unroll
         for (int n = 0; n < NB; ++n)
@@ -610,7 +622,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                 ge[n][0] = f.x; ge[n][1] = f.y;
             }
         }
-        if (ok) ok = mbar_wait(&bar[c & 1], (uint32_t)((c >> 1) & 1), P.status);
+        if (ok) ok = mbar_wait(&bar[2 * c % 3], (uint32_t)((2 * c / 3) & 1), P.status);
         if (DELTA || !owner) {                         // W S (warps 0-3) or (q G) S (warps 4-7): 16 rows each
             const uint32_t th = owner ? wh : qh, tl = th + L::TILE;
 #pragma unroll 4
@@ -618,23 +630,16 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                 uint32_t a[4], b[4];
                 fa::load_a<DT>(th, wr, ks, a);
                 fa::load_a<DT>(tl, wr, ks, b);
+                uint32_t bh[MT][4], bl[MT][4];
 #pragma unroll
-                for (int n = 0; n < MT; ++n) {
-                    uint32_t bh[4], bl[4];
-                    fa::load_b<DT>(sh, n * 16, ks, bh);
-                    fa::load_b<DT>(sl, n * 16, ks, bl);
-                    fa::mma16816(acc[2 * n], a, bh[0], bh[1]);
-                    fa::mma16816(acc[2 * n + 1], a, bh[2], bh[3]);
-                    fa::mma16816(low[2 * n], b, bh[0], bh[1]);
-                    fa::mma16816(low[2 * n + 1], b, bh[2], bh[3]);
-                    fa::mma16816(low[2 * n], a, bl[0], bl[1]);
-                    fa::mma16816(low[2 * n + 1], a, bl[2], bl[3]);
-                }
+                for (int n = 0; n < MT; ++n) { fa::load_b<DT>(sh, n * 16, ks, bh[n]); fa::load_b<DT>(sl, n * 16, ks, bl[n]); }
+#pragma unroll
+                for (int n = 0; n < NB; ++n) fa::mma16816(acc[n], a, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+#pragma unroll
+                for (int n = 0; n < NB; ++n) fa::mma16816(low[n], b, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+#pragma unroll
+                for (int n = 0; n < NB; ++n) fa::mma16816(low[n], a, bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
             }
-#pragma unroll
-            for (int n = 0; n < NB; ++n)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) acc[n][e] += low[n][e];
         }
         if (owner) {                                   // u^T, split
 #pragma unroll
@@ -643,7 +648,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                 for (int e = 0; e < 4; ++e) {
                     const float2 f = DELTA ? base[n][e >> 1] : unpack(__float_as_uint(base[n][e >> 1].x));
                     float u = (e & 1) ? f.y : f.x;
-                    if constexpr (DELTA) u -= acc[n][e];
+                    if constexpr (DELTA) u -= acc[n][e] + low[n][e];
                     else if (P.silu) u = silu(u);
                     const int v = n * 8 + 2 * t + (e & 1), r = wr + g + 8 * (e >> 1);
                     const __nv_bfloat16 hi = __float2bfloat16_rn(u);
@@ -654,8 +659,8 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
             if (c + 1 < chunks) fetch(c + 1);
         }
         __syncthreads();                               // u is there; W, q and the state tiles have been read
-        if (threadIdx.x == 0 && c + 2 < chunks && ok) load_wq(c + 2);
-        if (ok) ok = mbar_wait(&bar[2], (uint32_t)(c & 1), P.status);
+        if (threadIdx.x == 0 && c + 1 < chunks && ok) load(2 * c + 3);
+        if (ok) ok = mbar_wait(&bar[(2 * c + 1) % 3], (uint32_t)(((2 * c + 1) / 3) & 1), P.status);
         if (owner) {
 #pragma unroll
             for (int m = 0; m < MT; ++m)
@@ -663,41 +668,59 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                 for (int n = 0; n < NT; ++n)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) X[m][n][e] *= ge[n][e & 1];
+            float Y[MT][NT][4];                        // products with a low part
 #pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int n = 0; n < NT; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) Y[m][n][e] = 0.f;
+#pragma unroll 2
             for (int ks = 0; ks < CH / 16; ++ks) {
-                uint32_t bh[NT / 2][4], bl[NT / 2][4];
+                uint32_t bh[NT / 2][4], bl[NT / 2][4], a[MT][4], b[MT][4];
 #pragma unroll
                 for (int n = 0; n < NT / 2; ++n) {
                     fa::load_b_t<DT>(kh, ks * 16, d0 / 8 + 2 * n, bh[n]);
                     fa::load_b_t<DT>(kh + L::TILE, ks * 16, d0 / 8 + 2 * n, bl[n]);
                 }
 #pragma unroll
-                for (int m = 0; m < MT; ++m) {
-                    uint32_t a[4], b[4];
-                    fa::load_a<CH>(uh, m * 16, ks, a);
-                    fa::load_a<CH>(ul, m * 16, ks, b);
+                for (int m = 0; m < MT; ++m) { fa::load_a<CH>(uh, m * 16, ks, a[m]); fa::load_a<CH>(ul, m * 16, ks, b[m]); }
 #pragma unroll
-                    for (int n = 0; n < NT / 2; ++n) {
-                        mma3(X[m][2 * n], a, b, bh[n][0], bh[n][1], bl[n][0], bl[n][1]);
-                        mma3(X[m][2 * n + 1], a, b, bh[n][2], bh[n][3], bl[n][2], bl[n][3]);
-                    }
-                }
+                for (int k = 0; k < 3; ++k)
+#pragma unroll
+                    for (int m = 0; m < MT; ++m)
+#pragma unroll
+                        for (int n = 0; n < NT; ++n) {
+                            const uint32_t* w = k == 2 ? bl[n / 2] : bh[n / 2];
+                            fa::mma16816(k == 0 ? X[m][n] : Y[m][n], k == 1 ? b[m] : a[m], w[2 * (n & 1)], w[2 * (n & 1) + 1]);
+                        }
             }
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int n = 0; n < NT; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) X[m][n][e] += Y[m][n][e];
             publish();
         } else {
             for (int ks = 0; ks <= wr / 16; ++ks) {
                 uint32_t a[4], b[4];
                 fa::load_a<CH>(ah, wr, ks, a);
                 fa::load_a<CH>(ah + L::ATILE, wr, ks, b);
+                uint32_t bh[MT][4], bl[MT][4];
 #pragma unroll
-                for (int n = 0; n < MT; ++n) {
-                    uint32_t bh[4], bl[4];
-                    fa::load_b<CH>(uh, n * 16, ks, bh);
-                    fa::load_b<CH>(ul, n * 16, ks, bl);
-                    mma3(acc[2 * n], a, b, bh[0], bh[1], bl[0], bl[1]);
-                    mma3(acc[2 * n + 1], a, b, bh[2], bh[3], bl[2], bl[3]);
-                }
+                for (int n = 0; n < MT; ++n) { fa::load_b<CH>(uh, n * 16, ks, bh[n]); fa::load_b<CH>(ul, n * 16, ks, bl[n]); }
+#pragma unroll
+                for (int n = 0; n < NB; ++n) fa::mma16816(acc[n], a, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+#pragma unroll
+                for (int n = 0; n < NB; ++n) fa::mma16816(low[n], b, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+#pragma unroll
+                for (int n = 0; n < NB; ++n) fa::mma16816(low[n], a, bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
             }
+#pragma unroll
+            for (int n = 0; n < NB; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) acc[n][e] += low[n][e];
 #pragma unroll
             for (int n = 0; n < NB; ++n)
 #pragma unroll
@@ -713,7 +736,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                 }
         }
         __syncthreads();                               // the new state is there; k, A and u have been read
-        if (threadIdx.x == 0 && c + 1 < chunks && ok) load_ka(c + 1);
+        if (threadIdx.x == 0 && c + 2 < chunks && ok) load(2 * c + 4);
     }
     if (owner) each_state([&](float& x, int v, int d) { if (ok && v < Dv && d < D) st[(size_t)d * Dv + v] = x; });
 }
@@ -743,7 +766,7 @@ static int launch(Params p, cudaStream_t st) {
     }
     // few CTAs: narrow slices, so that more of them share the walk
     const long long wide = (long long)((p.P.Dv + 31) / 32) * p.P.H * p.P.n_seqs;
-    if (wide < 56 ? launch_state<DT, 16>(p, st) : launch_state<DT, 32>(p, st)) return -1;
+    if (wide <= 74 ? launch_state<DT, 16>(p, st) : launch_state<DT, 32>(p, st)) return -1;
     PTB_CUDA_OK(cudaGetLastError());
     return 0;
 }
