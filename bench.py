@@ -327,8 +327,8 @@ def main():
     ap.add_argument("--warmup", type=int, default=16)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--prompt-len", type=int, default=128)
-    ap.add_argument("--model", default="qwen3-4b", choices=["qwen3-4b", "tiny", "kifusun"],
-                    help="kifusun: Kifusun beside Llama of equal size in the batching engine (benchmarks/kifusun_bench.py), 1 GPU")
+    ap.add_argument("--model", default="qwen3-4b", choices=["qwen3-4b", "tiny", "kifusun", "gelutar"],
+                    help="kifusun, gelutar: that model beside Llama of equal size in the batching engine (benchmarks/*_bench.py), 1 GPU")
     ap.add_argument("--max-seq", type=int, default=4096)
     ap.add_argument("--repeats", type=int, default=5, help="timed regions of --steps steps each (median is reported)")
     ap.add_argument("--train-steps", type=int, default=5, help="timed steps of the Llama-1.1B FSDP half (0 = skip)")
@@ -342,6 +342,10 @@ def main():
         sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
         import kifusun_bench
         return kifusun_bench.main([])
+    if args.model == "gelutar":
+        sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
+        import gelutar_bench
+        return gelutar_bench.main([])
     args.warmup = max(args.warmup, 3)
 
     import torch

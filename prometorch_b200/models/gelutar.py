@@ -132,6 +132,7 @@ class GelutarConfig:
                 "norm": {"eps": self.eps}, "logit_scale": self.logit_scale, "layers": layers}
 
 
+MERGE_GATES = 128                      # rows up to which the two low-rank gates are one product
 _LEFT = ("left.q", "left.k", "left.v")
 _CONV = ("right.q", "right.k", "right.v")
 
@@ -246,13 +247,15 @@ class PagedGelutar(PagedModel):
                 d["w_in"] = d["pack"].pack({**{n: L["mix." + n] for n in _LEFT + ("left.g", "right.b")}, "low": low,
                                             "conv": torch.cat([L["mix." + n] for n in _CONV])})
                 d["conv"] = torch.cat([L[f"mix.{n}.conv"] for n in _CONV]).t().contiguous()          # [taps, channels]
-                # both low-rank gates as one product: block-diagonal second matrices over the packed first ones
+                # few rows: both low-rank gates as one product, block-diagonal second matrices over the packed first ones; many rows: one
+                # product each, the decays' in fp32
                 ra, rg = RowPack.up(L["mix.right.a1"].shape[0]), L["mix.right.g1"].shape[0]
                 a2, g2 = L["mix.right.a2"], L["mix.right.g2"]
                 gates = a2.new_zeros(RowPack.up(a2.shape[0]) + g2.shape[0], RowPack.up(ra + rg))
                 gates[:a2.shape[0], :a2.shape[1]] = a2
                 gates[RowPack.up(a2.shape[0]):, ra:ra + rg] = g2
                 d["gates"], d["gate_cols"] = RowPack.pad(gates), RowPack.up(a2.shape[0])
+                d["a2"], d["g2"], d["rank_a"] = gates[:d["gate_cols"], :ra].contiguous(), RowPack.pad(gates[d["gate_cols"]:, ra:]), ra
                 d["attn"] = A.WindowAttention(a.heads, a.kv_heads, a.dim, a.vdim, min(a.window, A.UNBOUNDED), min(a.keep_first, A.UNBOUNDED), a.scale, L["mix.left.sink"])
                 d["delta"] = R.DeltaRule(b.heads, b.kv_heads, b.dim, b.vdim, L["mix.right.A_log"].exp(), L["mix.right.dt_bias"])
                 for n in ("left.q.norm", "left.k.norm", "right.norm", "left.out", "right.out"):
@@ -306,10 +309,14 @@ class PagedGelutar(PagedModel):
         p = linear(h, d["w_in"])
         q = A.proj_norm_write(p, tuple(pk.at[n] for n in _LEFT), a, d["left.q.norm"], d["left.k.norm"], eps, pos, req, page_table, kv.k[l], kv.v[l])
         c = R.short_conv(pk.cols(p, "conv"), d["conv"], kv.state[l]["conv"], pos, req, seqs)
-        gates = S.linear_f32(pk.cols(p, "low", padded=True), d["gates"])
-        r, at = d["delta"], d["gate_cols"]
-        o = R.delta_rule(c, r, pk.cols(p, "right.b"), gates[:, :r.heads * r.dim], kv.state[l]["S"], pos, req, seqs)
-        o = R.group_norm_gate(o, d["right.norm"], gates[:, at:at + r.heads * r.vdim], eps, self.dtype)
+        r, at, low = d["delta"], d["gate_cols"], pk.cols(p, "low", padded=True)
+        if p.shape[0] > MERGE_GATES:
+            decay, gate = S.linear_f32(low[:, :d["rank_a"]], d["a2"]), linear(low[:, d["rank_a"]:], d["g2"])
+        else:
+            gates = S.linear_f32(low, d["gates"])
+            decay, gate = gates[:, :at], gates[:, at:]
+        o = R.delta_rule(c, r, pk.cols(p, "right.b"), decay[:, :r.heads * r.dim], kv.state[l]["S"], pos, req, seqs)
+        o = R.group_norm_gate(o, d["right.norm"], gate[:, :r.heads * r.vdim], eps, self.dtype)
         y = attend(l, a, q, pk.cols(p, "left.g"))
         return [S.linear_branch(y, d["left.o"], 0.5, d["left.out"]), S.linear_branch(o, d["right.o"], 0.5, d["right.out"])]
 
