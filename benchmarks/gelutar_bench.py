@@ -89,9 +89,9 @@ def kernel_rows(z, window, prompt=4096, ctx=4096):
         seqs = R.Sequences.of([i * T for i in range(B + 1)], [0] * B, list(range(B)), "cuda")
         pos, req = torch.arange(T, dtype=torch.int32, device="cuda").repeat(B), torch.arange(B, dtype=torch.int32, device="cuda").repeat_interleave(T)
         S0 = torch.zeros(B, H, D, D, device="cuda")
-        x, xl, beta, aa = [rand(n, 3 * H * D) for _ in range(2)], [rand(n, 4 * H * D) for _ in range(2)], rand(n, H), torch.randn(n, H * D, device="cuda")
+        x, xl, beta, aa = [rand(n, 3 * H * D) for _ in range(2)], [rand(n, 4 * H * D) for _ in range(2)], rand(n, H), (rand(n, RANK), rand(H * D, RANK, scale=RANK ** -0.5))
         add(f"delta rule, {B} x {T} tokens", per_launch_us([lambda i=i: R.delta_rule(x[i], dr, beta, aa, S0, pos, req, seqs) for i in range(2)], 4),
-            n * H * D * (6 + 4 + 4), 2.0 * n * H * D * (3 * D + 4 * 64))
+            n * H * D * (6 + 4) + 2 * n * RANK, 2.0 * n * H * D * (3 * D + 4 * 64 + RANK))
         add(f"decay attention, {B} x {T} tokens", per_launch_us([lambda i=i: R.decay_attention(xl[i], dl, at, S0, pos, req, seqs) for i in range(2)], 4),
             n * H * D * (6 + 4), 2.0 * n * H * D * (2 * D + 64))
         del x, xl, aa
@@ -149,10 +149,10 @@ def kernel_rows(z, window, prompt=4096, ctx=4096):
             add(f"up projection + squared ReLU, {n} rows", per_launch_us([lambda i=i: gemm.linear_relu2(h, wu[i]) for i in range(sets)]), 2 * W * ff)
             add(f"gate / up projection + SiLU gate, {n} rows (llama)", per_launch_us([lambda i=i: gemm.linear_swiglu(h, wg[i]) for i in range(4)]), 4 * W * z["ff"])
         low, w2 = rand(n, 2 * RANK), [rand(2 * H * D, 2 * RANK) for _ in range(sets)]
+        wg2 = [rand(H * D, RANK) for _ in range(sets)]
         if big:
-            wa, wg2 = [rand(H * D, RANK) for _ in range(2)], [rand(H * D, RANK) for _ in range(2)]
-            us = per_launch_us([lambda i=i: (S.linear_f32(low[:, :RANK], wa[i]), gemm.linear(low[:, RANK:], wg2[i])) for i in range(2)])
-            add(f"two low-rank gates, {n} rows", us, 4 * n * RANK + 6 * n * H * D + 4 * H * D * RANK, 4.0 * n * RANK * H * D)
+            add(f"output gate of rank {RANK}, {n} rows", per_launch_us([lambda i=i: gemm.linear(low[:, RANK:], wg2[i]) for i in range(sets)]),
+                2 * n * RANK + 2 * n * H * D + 2 * H * D * RANK, 2.0 * n * RANK * H * D)
         else:
             add(f"two low-rank gates as one product, {n} rows", per_launch_us([lambda i=i: S.linear_f32(low, w2[i]) for i in range(sets)]),
                 4 * n * RANK + 8 * n * H * D + 4 * H * D * RANK, 4.0 * n * RANK * H * D)

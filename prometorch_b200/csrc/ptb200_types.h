@@ -88,5 +88,8 @@ typedef struct PtbRecurrence {
     int* status;
     const void* chunks;     // the matrix form: [n_chunks] int4 (first row, rows <= 64, sequence, 0), sequence by sequence
     const int* first_chunk; // [n_seqs]
-    int n_chunks, pad2;
+    int n_chunks, rank;
+    const void* low;        // the matrix form may take a as low low_w^T instead: [n][rank] of pitch ld_low, bf16
+    long long ld_low;
+    const void* low_w;      // [H D][rank], bf16
 } PtbRecurrence;

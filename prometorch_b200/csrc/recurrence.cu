@@ -378,7 +378,7 @@ int recurrence_check(const PtbRecurrence& p) {
         ptb_set_error("recurrence: bad sizes (H %d, G %d, D %d, Dv %d; D at most 512)", p.H, p.G, p.D, p.Dv);
         return -1;
     }
-    if (!p.x || !p.state || !p.out || !p.decay || (p.delta && (!p.a || !p.beta || !p.dt_bias))) { ptb_set_error("recurrence: missing operand"); return -1; }
+    if (!p.x || !p.state || !p.out || !p.decay || (p.delta && ((!p.a && !p.low) || !p.beta || !p.dt_bias))) { ptb_set_error("recurrence: missing operand"); return -1; }
     if ((p.seqs ? p.n_seqs : p.n) > 65535) { ptb_set_error("recurrence: more than 65535 sequences in one launch"); return -1; }
     return 0;
 }
@@ -420,6 +420,7 @@ PTB_API int ptb_recurrence(const PtbRecurrence* args, cudaStream_t st) {
     const PtbRecurrence& p = *args;
     if (p.n <= 0 || (p.seqs && p.n_seqs <= 0)) return 0;
     if (recurrence_check(p)) return -1;
+    if (p.delta && !p.a) { ptb_set_error("recurrence: token by token takes a, not its low-rank factors"); return -1; }
     if (p.bf16) PTB_CUDA_OK((p.delta ? recurrence_launch<__nv_bfloat16, true> : recurrence_launch<__nv_bfloat16, false>)(p, st));
     else PTB_CUDA_OK((p.delta ? recurrence_launch<float, true> : recurrence_launch<float, false>)(p, st));
     PTB_CUDA_OK(cudaGetLastError());

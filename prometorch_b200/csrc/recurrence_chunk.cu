@@ -8,6 +8,8 @@
 // W = (1 + B)^-1 beta (k G).  Two kernels:
 //   delta_chunk_kernel / decay_chunk_kernel   everything that does not depend on S, all chunks at once, into a workspace;
 //   chunk_state_kernel                        walks a sequence's chunks for a slice of value columns; S stays in registers.
+// What passes between them lies in the order of the mma fragments that will read it: a lane's 16 bytes are its four registers of a 16 x 16
+// block, so the walk loads its operands from L2 into registers, whole lines at a time, without shared memory.
 // Quotients of decays are never formed from products that could overflow: across blocks of 16 tokens both factors refer to the block
 // border between the two tokens and are at most 1, inside a block the exponent of every pair is taken directly.
 // Products run on the tensor cores with every fp32 operand split into two bf16 numbers (three products: 16 bits of both operands).
@@ -22,7 +24,11 @@ constexpr int CH = 64, THREADS = 256, WARPS = 8;
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float MILD = -60.f;          // log2 of what a block of 16 tokens may keep of a channel: both factors of every pair stay finite
 
-// Workspace of one (chunk, head): bf16 tiles in the swizzled order of fa::tile_off, high parts then low parts.
+// Workspace of one (chunk, head), in fragments of 512 bytes; the high parts of a matrix, then the low parts.
+//   W, Q  left operands   [4 row blocks][DT / 16 column blocks]
+//   K     right operand   [DT / 16 blocks of key channels][4 blocks of tokens]
+//   A     left operand    [4 row blocks][4 column blocks], those above the diagonal unused
+//   U     fp32            [Dvp / 16 column blocks][4 row blocks][2 halves of 8 columns][lane] the four accumulator registers
 template <int DT>
 struct Work {
     static constexpr int TILE = CH * DT * 2, ATILE = CH * CH * 2;
@@ -35,7 +41,7 @@ struct Params {
     unsigned char* work;
     size_t stride;                     // bytes per (chunk, head)
     int Dvp;                           // value columns rounded up to 32
-    int vec, vec_a;                    // 16-byte loads of x rows, of a
+    int vec, vec_a;                    // 16-byte loads of x rows, of a (or of low)
 };
 
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
@@ -52,7 +58,15 @@ __device__ __forceinline__ void mma3(float* d, const uint32_t* ah, const uint32_
     fa::mma16816(d, ah, bl0, bl1);
     fa::mma16816(d, ah, bh0, bh1);
 }
-// Store columns col, col + 1 (col even) of row r of a high and a low tile.
+// A lane's four registers of a fragment, given as pairs, to the high and the low part.
+__device__ __forceinline__ void store_frag(unsigned char* hi, int part, int frag, int lane, const float2* f) {
+    uint4 h, l;
+    split2(f[0].x, f[0].y, h.x, l.x); split2(f[1].x, f[1].y, h.y, l.y); split2(f[2].x, f[2].y, h.z, l.z); split2(f[3].x, f[3].y, h.w, l.w);
+    unsigned char* p = hi + ((size_t)frag * 32 + lane) * 16;
+    *reinterpret_cast<uint4*>(p) = h;
+    *reinterpret_cast<uint4*>(p + part) = l;
+}
+// Columns col, col + 1 (col even) of row r of a high and a low tile in shared memory.
 template <int DT>
 __device__ __forceinline__ void store_split(unsigned char* hi, unsigned char* lo, int r, int col, float a, float b) {
     uint32_t h, l;
@@ -134,7 +148,15 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
     unsigned char* out = W.work + ((size_t)blockIdx.x * P.H + h) * W.stride;
     load_rows(P, W.vec, row0, cnt, P.q_col + hk * D, D, DT, q_s, S::PB);
     load_rows(P, W.vec, row0, cnt, P.k_col + hk * D, D, DT, k_s, S::PB);
-    if (W.vec_a) {
+    __nv_bfloat16* low_s = reinterpret_cast<__nv_bfloat16*>(ak);   // over what the scores use later
+    const int rank = P.rank, RP = (rank + 15) / 16 * 16 + 8;
+    if (P.low) {
+        for (int e = threadIdx.x; e < CH * (RP / 8 - 1); e += THREADS) {
+            const int r = e / (RP / 8 - 1), c = (e % (RP / 8 - 1)) * 8;
+            const bool live = r < cnt && c < rank;
+            fa::cp_async16(smem_u32(low_s + r * RP + c), (const __nv_bfloat16*)P.low + (live ? (size_t)(row0 + r) * P.ld_low + c : 0), live);
+        }
+    } else if (W.vec_a) {
         for (int e = threadIdx.x; e < CH * DT / 4; e += THREADS) {
             const int r = e / (DT / 4), d = e % (DT / 4) * 4;
             const bool live = r < cnt && d < D;
@@ -150,20 +172,52 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
     if (threadIdx.x < CH)
         bt[threadIdx.x] = threadIdx.x < cnt ? sigmoid(__bfloat162float(((const __nv_bfloat16*)P.beta)[(size_t)(row0 + threadIdx.x) * P.ld_beta + h])) : 0.f;
     if (threadIdx.x == 0) *next_unit = WARPS;
-    for (int e = threadIdx.x; e < CH * S::PA; e += THREADS) ak[e] = 0.f;
     if (threadIdx.x < DT) tmp[threadIdx.x] = 0.f;
-    {                                                  // the half of the q . k tiles that stays zero
-        constexpr int above = 8 * 7 / 2;               // 8 x 8 blocks above the diagonal
-        for (int e = threadIdx.x; e < above * 8; e += THREADS) {
-            int b = e / 8, r = 0;
-            while (b >= 7 - r) { b -= 7 - r; ++r; }
-            const uint32_t off = fa::tile_off<CH>(r * 8 + e % 8, r + 1 + b);
-            *reinterpret_cast<uint4*>(out + L::A + off) = make_uint4(0, 0, 0, 0);
-            *reinterpret_cast<uint4*>(out + L::A + L::ATILE + off) = make_uint4(0, 0, 0, 0);
-        }
-    }
     fa::cp_async_wait<0>();
     __syncthreads();
+    if (P.low) {                                       // a = low low_w^T: a warp takes 16 channels (and half the rows when there are 4 blocks)
+        constexpr int UNITS = DT / 16, SHARE = WARPS / UNITS, RT = 4 / SHARE;
+        const int d0 = (warp % UNITS) * 16, rt0 = (warp / UNITS) * RT;
+        float c[RT][2][4];
+#pragma unroll
+        for (int r = 0; r < RT; ++r)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) c[r][e >> 2][e & 3] = 0.f;
+        const __nv_bfloat16* w[2];
+        bool live[2];
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            live[n] = d0 + n * 8 + g < D;
+            w[n] = (const __nv_bfloat16*)P.low_w + (size_t)(h * D + (live[n] ? d0 + n * 8 + g : 0)) * rank;
+        }
+#pragma unroll 4
+        for (int ks = 0; ks < (rank + 15) / 16; ++ks) {
+            uint32_t b[2][2];
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int u = 0; u < 2; ++u) {
+                    const int k = ks * 16 + 2 * t + 8 * u;         // rank is a multiple of eight
+                    b[n][u] = live[n] && k < rank ? *reinterpret_cast<const uint32_t*>(w[n] + k) : 0u;
+                }
+#pragma unroll
+            for (int r = 0; r < RT; ++r) {
+                uint32_t a[4];
+                fa::ldsm4(smem_u32(low_s + ((rt0 + r) * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * RP + ks * 16 + (lane >> 4) * 8), a[0], a[1], a[2], a[3]);
+                fa::mma16816(c[r][0], a, b[0][0], b[0][1]);
+                fa::mma16816(c[r][1], a, b[1][0], b[1][1]);
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < RT; ++r)
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+                    *reinterpret_cast<float2*>(G_s + ((rt0 + r) * 16 + g + 8 * e) * S::PG + d0 + n * 8 + 2 * t) = make_float2(c[r][n][2 * e], c[r][n][2 * e + 1]);
+        __syncthreads();
+    }
+    for (int e = threadIdx.x; e < CH * S::PA; e += THREADS) ak[e] = 0.f;
     for (int r = warp; r < CH; r += WARPS) {
         float a = 0.f, b = 0.f;
         for (int d = lane * 2; d < DT; d += 64) {
@@ -203,21 +257,26 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
     __syncthreads();
     // ---- q G, k G_end / G and G_end
     const float* Ge = G_s + (CH - 1) * S::PG;
-    for (int e = threadIdx.x; e < CH * DT / 8; e += THREADS) {
-        const int r = e / (DT / 8), d = (e % (DT / 8)) * 8;
-        const uint4 qr = *reinterpret_cast<const uint4*>(q_s + r * S::PB + d), kr = *reinterpret_cast<const uint4*>(k_s + r * S::PB + d);
-        const uint32_t *qp = reinterpret_cast<const uint32_t*>(&qr), *kp = reinterpret_cast<const uint32_t*>(&kr);
-        const float a = qn[r], b = kn[r];
-        float fq[8], fk[8];
+    for (int f = warp; f < DT / 4; f += WARPS) {
+        const int rb = f / (DT / 16), ks = f % (DT / 16), dp = f >> 2, kt = f & 3;
+        float2 x[4];
 #pragma unroll
-        for (int k = 0; k < 8; k += 4) {
-            const float4 G = *reinterpret_cast<const float4*>(G_s + r * S::PG + d + k), E = *reinterpret_cast<const float4*>(Ge + d + k);
-            const float2 q0 = unpack(qp[k / 2]), q1 = unpack(qp[k / 2 + 1]), k0 = unpack(kp[k / 2]), k1 = unpack(kp[k / 2 + 1]);
-            fq[k] = q0.x * a * exp2f(G.x); fq[k + 1] = q0.y * a * exp2f(G.y); fq[k + 2] = q1.x * a * exp2f(G.z); fq[k + 3] = q1.y * a * exp2f(G.w);
-            fk[k] = k0.x * b * exp2f(E.x - G.x); fk[k + 1] = k0.y * b * exp2f(E.y - G.y); fk[k + 2] = k1.x * b * exp2f(E.z - G.z); fk[k + 3] = k1.y * b * exp2f(E.w - G.w);
+        for (int u = 0; u < 4; ++u) {                  // row g + 8 (u & 1), columns 2t + 8 (u >> 1)
+            const int r = rb * 16 + g + 8 * (u & 1), d = ks * 16 + 2 * t + 8 * (u >> 1);
+            const float2 q = unpack(*reinterpret_cast<const uint32_t*>(q_s + r * S::PB + d)), G = *reinterpret_cast<const float2*>(G_s + r * S::PG + d);
+            x[u] = make_float2(q.x * qn[r] * exp2f(G.x), q.y * qn[r] * exp2f(G.y));
         }
-        store_split8<DT>(out + L::Q, out + L::Q + L::TILE, r, d, fq);
-        store_split8<DT>(out + L::K, out + L::K + L::TILE, r, d, fk);
+        store_frag(out + L::Q, L::TILE, f, lane, x);
+        uint32_t k[4];
+        fa::ldsm4_t(smem_u32(k_s + (kt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * S::PB + dp * 16 + (lane >> 4) * 8), k[0], k[1], k[2], k[3]);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {                  // tokens 2t + 8 (u & 1) and the next, channel g + 8 (u >> 1)
+            const int r = kt * 16 + 2 * t + 8 * (u & 1), d = dp * 16 + g + 8 * (u >> 1);
+            const float2 v = unpack(k[u]);
+            const float E = Ge[d];
+            x[u] = make_float2(v.x * kn[r] * exp2f(E - G_s[r * S::PG + d]), v.y * kn[r + 1] * exp2f(E - G_s[(r + 1) * S::PG + d]));
+        }
+        store_frag(out + L::K, L::TILE, f, lane, x);
     }
     for (int d = threadIdx.x; d < DT; d += THREADS) reinterpret_cast<float*>(out + L::G)[d] = exp2f(Ge[d]);
     // ---- q . k and k . k under the decays: units 0-9 are blocks of 16 x 16 on the tensor cores, six below the diagonal and those on it
@@ -260,15 +319,17 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
                     mma3(ck[n], kh, kl, bh[0], bh[1], bl[0], bl[1]);
                 }
             }
+            float2 x[4];
 #pragma unroll
             for (int n = 0; n < 2; ++n)
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int i = s * 16 + g + 8 * e, j = r * 16 + n * 8 + 2 * t;
                     const float a = qn[i], b = kn[i] * bt[i], k0 = kn[j], k1 = kn[j + 1];
-                    store_split<CH>(out + L::A, out + L::A + L::ATILE, i, j, j <= i ? cq[n][2 * e] * a * k0 : 0.f, j < i ? cq[n][2 * e + 1] * a * k1 : 0.f);
+                    x[n * 2 + e] = make_float2(j <= i ? cq[n][2 * e] * a * k0 : 0.f, j < i ? cq[n][2 * e + 1] * a * k1 : 0.f);
                     *reinterpret_cast<float2*>(ak + i * S::PA + j) = make_float2(j < i ? ck[n][2 * e] * b * k0 : 0.f, j + 1 < i ? ck[n][2 * e + 1] * b * k1 : 0.f);
                 }
+            store_frag(out + L::A, L::ATILE, s * 4 + r, lane, x);
         } else if (unit >= 10 && !mild[(unit - 10) * 32 / 136] + !mild[((unit - 10) * 32 + 31) / 136]) {
             const int p = (unit - 10) * 32 + lane, s = p / 136, m = p % 136;
             int a = (int)((sqrtf(8.f * m + 1.f) - 1.f) * 0.5f);
@@ -289,15 +350,17 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
             }
             const float f = sq * qn[i] * kn[j];
             const __nv_bfloat16 hi = __float2bfloat16_rn(f);
-            const uint32_t off = fa::tile_off<CH>(i, j >> 3) + (j & 7) * 2;
-            *reinterpret_cast<__nv_bfloat16*>(out + L::A + off) = hi;
-            *reinterpret_cast<__nv_bfloat16*>(out + L::A + L::ATILE + off) = __float2bfloat16_rn(f - __bfloat162float(hi));
-            if (i != j) ak[i * S::PA + j] = sk * kn[i] * kn[j] * bt[i];
-            // the tiles' 8 x 8 blocks on the diagonal: what lies above it inside them
-            if ((i >> 3) == (j >> 3) && i != j) {
-                const uint32_t up = fa::tile_off<CH>(j, i >> 3) + (i & 7) * 2;
-                *reinterpret_cast<__nv_bfloat16*>(out + L::A + up) = __float2bfloat16_rn(0.f);
-                *reinterpret_cast<__nv_bfloat16*>(out + L::A + L::ATILE + up) = __float2bfloat16_rn(0.f);
+            auto put = [&](int a, int b, __nv_bfloat16 x, __nv_bfloat16 y) {       // element (a, b) of the block, high and low part
+                unsigned char* p = out + L::A + (s * 5 * 32 + (a & 7) * 4 + ((b & 7) >> 1)) * 16 + ((a >> 3) + 2 * (b >> 3)) * 4 + (b & 1) * 2;
+                *reinterpret_cast<__nv_bfloat16*>(p) = x;
+                *reinterpret_cast<__nv_bfloat16*>(p + L::ATILE) = y;
+            };
+            if (!mild[s]) {
+                put(i & 15, j & 15, hi, __float2bfloat16_rn(f - __bfloat162float(hi)));
+                if (i != j) {
+                    ak[i * S::PA + j] = sk * kn[i] * kn[j] * bt[i];
+                    put(j & 15, i & 15, __float2bfloat16_rn(0.f), __float2bfloat16_rn(0.f));
+                }
             }
         }
         if (lane == 0) unit = atomicAdd(next_unit, 1);
@@ -361,21 +424,21 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
         const bool is_w = unit < DT / 16;
         const int n0 = (is_w ? unit : unit - DT / 16) * 16;
         uint32_t bh[4][4], bl[4][4];
-        if (is_w) {
 #pragma unroll
-            for (int ks = 0; ks < 4; ++ks)
-#pragma unroll
-                for (int u = 0; u < 4; ++u) {                      // n-block u >> 1, rows 2t, 2t + 1 (+ 8 for odd u)
-                    const int j = ks * 16 + 2 * t + 8 * (u & 1), d = n0 + g + 8 * (u >> 1);
-                    const float a = __bfloat162float(k_s[j * S::PB + d]) * kn[j] * exp2f(G_s[j * S::PG + d]);
-                    const float b = __bfloat162float(k_s[(j + 1) * S::PB + d]) * kn[j + 1] * exp2f(G_s[(j + 1) * S::PG + d]);
-                    split2(a, b, bh[ks][u], bl[ks][u]);
-                }
-        } else {
-#pragma unroll
-            for (int ks = 0; ks < 4; ++ks)
-                fa::ldsm4_t(smem_u32(v_s + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PV + n0 + (lane >> 4) * 8), bh[ks][0], bh[ks][1], bh[ks][2], bh[ks][3]);
+        for (int ks = 0; ks < 4; ++ks) {
+            const __nv_bfloat16* p = is_w ? k_s + n0 : v_s + n0;
+            const int pitch = is_w ? S::PB : PV;
+            fa::ldsm4_t(smem_u32(p + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + (lane >> 4) * 8), bh[ks][0], bh[ks][1], bh[ks][2], bh[ks][3]);
         }
+        if (is_w)
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks)
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {          // n-block u >> 1, rows 2t, 2t + 1 (+ 8 for odd u)
+                    const int j = ks * 16 + 2 * t + 8 * (u & 1), d = n0 + g + 8 * (u >> 1);
+                    const float2 k = unpack(bh[ks][u]);
+                    split2(k.x * kn[j] * exp2f(G_s[j * S::PG + d]), k.y * kn[j + 1] * exp2f(G_s[(j + 1) * S::PG + d]), bh[ks][u], bl[ks][u]);
+                }
 #pragma unroll
         for (int rb = 0; rb < 4; ++rb) {
             float c[2][4];
@@ -397,14 +460,14 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
                     }
                 }
             }
-#pragma unroll
-            for (int n = 0; n < 2; ++n)
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const int r = rb * 16 + g + 8 * e, col = n0 + n * 8 + 2 * t;
-                    if (is_w) store_split<DT>(out + L::W, out + L::W + L::TILE, r, col, c[n][2 * e], c[n][2 * e + 1]);
-                    else *reinterpret_cast<float2*>(out + L::U + ((size_t)r * W.Dvp + col) * 4) = make_float2(c[n][2 * e], c[n][2 * e + 1]);
-                }
+            if (is_w) {
+                const float2 x[4] = {make_float2(c[0][0], c[0][1]), make_float2(c[0][2], c[0][3]), make_float2(c[1][0], c[1][1]), make_float2(c[1][2], c[1][3])};
+                store_frag(out + L::W, L::TILE, rb * (DT / 16) + n0 / 16, lane, x);
+            } else {
+                float4* u = reinterpret_cast<float4*>(out + L::U) + ((n0 / 16) * 4 + rb) * 64 + lane;
+                u[0] = make_float4(c[0][0], c[0][1], c[0][2], c[0][3]);
+                u[32] = make_float4(c[1][0], c[1][1], c[1][2], c[1][3]);
+            }
         }
     }
 }
@@ -464,72 +527,86 @@ __global__ void __launch_bounds__(THREADS) decay_chunk_kernel(const __grid_const
         }
         store_split8<DT>(qh, ql, r, d, fq);
         store_split8<DT>(kh, kl, r, d, fk);
-        const float a = pw[r + 1], b = r < cnt ? pw[cnt - 1 - r] : 0.f;
-#pragma unroll
-        for (int k = 0; k < 8; ++k) { fq[k] *= a; fk[k] *= b; }
-        store_split8<DT>(out + L::Q, out + L::Q + L::TILE, r, d, fq);
-        store_split8<DT>(out + L::K, out + L::K + L::TILE, r, d, fk);
     }
     __syncthreads();
     const uint32_t a_h = smem_u32(qh), a_l = smem_u32(ql), b_h = smem_u32(kh), b_l = smem_u32(kl);
-    for (int unit = warp; unit < 16; unit += WARPS) {              // 16 x 16 blocks; those above the diagonal are zeros
+    for (int f = warp; f < DT / 4; f += WARPS) {       // q and k times their powers
+        const int rb = f / (DT / 16), ks = f % (DT / 16), dp = f >> 2, kt = f & 3;
+        uint32_t hi[4], lo[4];
+        float2 x[4];
+        fa::load_a<DT>(a_h, rb * 16, ks, hi);
+        fa::load_a<DT>(a_l, rb * 16, ks, lo);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const float2 a = unpack(hi[u]), b = unpack(lo[u]);
+            const float p = pw[rb * 16 + g + 8 * (u & 1) + 1];
+            x[u] = make_float2((a.x + b.x) * p, (a.y + b.y) * p);
+        }
+        store_frag(out + L::Q, L::TILE, f, lane, x);
+        fa::load_b_t<DT>(b_h, kt * 16, dp * 2, hi);
+        fa::load_b_t<DT>(b_l, kt * 16, dp * 2, lo);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const float2 a = unpack(hi[u]), b = unpack(lo[u]);
+            const int r = cnt - 1 - (kt * 16 + 2 * t + 8 * (u & 1));
+            x[u] = make_float2(r >= 0 ? (a.x + b.x) * pw[r] : 0.f, r >= 1 ? (a.y + b.y) * pw[r - 1] : 0.f);
+        }
+        store_frag(out + L::K, L::TILE, f, lane, x);
+    }
+    for (int unit = warp; unit < 16; unit += WARPS) {              // 16 x 16 blocks up to the diagonal
         const int s = unit >> 2, r = unit & 3;
+        if (r > s) continue;
         float c[2][4];
 #pragma unroll
         for (int n = 0; n < 2; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) c[n][e] = 0.f;
-        if (r <= s)
 #pragma unroll 2
-            for (int ks = 0; ks < DT / 16; ++ks) {
-                uint32_t ah[4], al[4], bh[4], bl[4];
-                fa::load_a<DT>(a_h, s * 16, ks, ah);
-                fa::load_a<DT>(a_l, s * 16, ks, al);
-                fa::load_b<DT>(b_h, r * 16, ks, bh);
-                fa::load_b<DT>(b_l, r * 16, ks, bl);
-                mma3(c[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
-                mma3(c[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
-            }
+        for (int ks = 0; ks < DT / 16; ++ks) {
+            uint32_t ah[4], al[4], bh[4], bl[4];
+            fa::load_a<DT>(a_h, s * 16, ks, ah);
+            fa::load_a<DT>(a_l, s * 16, ks, al);
+            fa::load_b<DT>(b_h, r * 16, ks, bh);
+            fa::load_b<DT>(b_l, r * 16, ks, bl);
+            mma3(c[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
+            mma3(c[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+        }
+        float2 x[4];
 #pragma unroll
         for (int n = 0; n < 2; ++n)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int i = s * 16 + g + 8 * e, j = r * 16 + n * 8 + 2 * t;
-                store_split<CH>(out + L::A, out + L::A + L::ATILE, i, j, j <= i ? c[n][2 * e] * pw[i - j] : 0.f, j + 1 <= i ? c[n][2 * e + 1] * pw[i - j - 1] : 0.f);
+                x[n * 2 + e] = make_float2(j <= i ? c[n][2 * e] * pw[i - j] : 0.f, j + 1 <= i ? c[n][2 * e + 1] * pw[i - j - 1] : 0.f);
             }
+        store_frag(out + L::A, L::ATILE, s * 4 + r, lane, x);
     }
     for (int d = threadIdx.x; d < DT; d += THREADS) reinterpret_cast<float*>(out + L::G)[d] = pw[cnt];
 }
 
 // ---------------------------------------------------------------------------------------------- the walk over a sequence's chunks
-template <int DT, int VS>
-struct StateSmem {
-    using L = Work<DT>;
-    static constexpr int SLOT = 4 * L::TILE > 2 * L::TILE + 2 * L::ATILE ? 4 * L::TILE : 2 * L::TILE + 2 * L::ATILE, SH = 3 * SLOT, SL = SH + VS * DT * 2, UH = SL + VS * DT * 2, UL = UH + VS * CH * 2;
-    static constexpr int BAR = UL + VS * CH * 2, TOTAL = BAR + 64;
-};
+__device__ __forceinline__ uint4 ld_once(const unsigned char* p) {
+    uint4 v;
+    asm volatile("ld.global.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+__device__ __forceinline__ void mma_u4(float* d, const uint4& a, uint32_t b0, uint32_t b1) {
+    const uint32_t f[4] = {a.x, a.y, a.z, a.w};
+    fa::mma16816(d, f, b0, b1);
+}
 
 // One CTA per (VS value columns, head, sequence), eight warps.  Of a chunk, warps 0-3 form u (64 rows) and then the new state, warps 4-7
 // the read-out; the state lives transposed, [value][key channel], in the accumulators of warps 0-3 and as two bf16 tiles in shared
-// memory for the products that read it.  Tiles arrive by bulk copies through three slots, in the order of their use: W and q of a chunk,
-// its k and A, W and q of the next, ...  Products of high parts and those with a low part have accumulators of their own, and every
-// accumulator waits for its turn among at least four, so that the tensor pipe is not held up by dependent products.
+// memory for the products that read it.  Every other operand is read by exactly one warp and comes from the workspace into registers:
+// the fragments of a chunk's second half are on their way during its first half, those of the next chunk's first half during the second.
 template <int DT, int VS, bool DELTA>
 __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_constant__ Params W) {
     using L = Work<DT>;
-    using S = StateSmem<DT, VS>;
-    constexpr int NT = DT / 32, MT = VS / 16, NB = VS / 8;         // state tiles of a warp: MT x NT of 16 x 8
-    extern __shared__ __align__(128) unsigned char smem[];
-    uint64_t* bar = reinterpret_cast<uint64_t*>(smem + S::BAR);    // one per slot
+    constexpr int KS = DT / 16, NT = DT / 32, MT = VS / 16, NB = VS / 8;       // state tiles of a warp: MT x NT of 16 x 8
+    constexpr int F3 = NT / 2 * 4;                     // fragments of the second half (the read-out uses up to four)
+    __shared__ __align__(128) unsigned char s_hi[VS * DT * 2], s_lo[VS * DT * 2], u_hi[VS * CH * 2], u_lo[VS * CH * 2];
     const PtbRecurrence& P = W.P;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-    if (threadIdx.x == 0) {
-        mbar_init(&bar[0], 1);
-        mbar_init(&bar[1], 1);
-        mbar_init(&bar[2], 1);
-        mbar_fence_init();
-    }
-    __syncthreads();
     pdl_wait();
     pdl_launch_dependents();
     const int h = blockIdx.y, v0 = blockIdx.x * VS, D = P.D, Dv = P.Dv;
@@ -540,26 +617,11 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
         if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
         return;
     }
-    auto tiles = [&](int c) { return W.work + ((size_t)(first + c) * P.H + h) * W.stride; };
-    // load 2c: W and q of chunk c, load 2c + 1: its k and A; load i goes to slot i % 3 once load i - 3 has been read
-    auto load = [&](int i) {
-        const int s = i % 3;
-        if (i & 1) {
-            constexpr uint32_t bytes = 2 * L::TILE + 2 * L::ATILE;
-            mbar_expect_tx(&bar[s], bytes);
-            bulk_g2s(smem + s * S::SLOT, tiles(i >> 1) + L::K, bytes, &bar[s]);
-        } else {
-            constexpr uint32_t bytes = (DELTA ? 4 : 2) * L::TILE;
-            mbar_expect_tx(&bar[s], bytes);
-            bulk_g2s(smem + s * S::SLOT + (DELTA ? 0 : 2 * L::TILE), tiles(i >> 1) + (DELTA ? L::W : L::Q), bytes, &bar[s]);
-        }
-    };
-    if (threadIdx.x == 0)
-        for (int i = 0; i < min(3, 2 * chunks); ++i) load(i);
-    const uint32_t sh = smem_u32(smem + S::SH), sl = smem_u32(smem + S::SL), uh = smem_u32(smem + S::UH), ul = smem_u32(smem + S::UL);
     const bool owner = warp < 4;                       // of the state channels d0 .. d0 + DT / 4
-    const int wr = (warp & 3) * 16, d0 = (warp & 3) * (DT / 4);
+    const int rb = warp & 3, wr = rb * 16, d0 = rb * (DT / 4);
+    const uint32_t sh = smem_u32(s_hi), sl = smem_u32(s_lo), uh = smem_u32(u_hi), ul = smem_u32(u_lo);
     float* st = P.state + (((size_t)sp.slot * P.H + h) * D) * Dv;
+    auto tiles = [&](int c) { return W.work + ((size_t)(first + c) * P.H + h) * W.stride; };
     float X[MT][NT][4];                                // S^T: row v0 + 16 m + g (+ 8), column d0 + 8 n + 2t (+ 1)
     auto each_state = [&](auto f) {
 #pragma unroll
@@ -575,46 +637,63 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
 #pragma unroll
             for (int n = 0; n < NT; ++n)
 #pragma unroll
-                for (int e = 0; e < 2; ++e)
-                    store_split<DT>(smem + S::SH, smem + S::SL, m * 16 + g + 8 * e, d0 + n * 8 + 2 * t, X[m][n][2 * e], X[m][n][2 * e + 1]);
+                for (int e = 0; e < 2; ++e) store_split<DT>(s_hi, s_lo, m * 16 + g + 8 * e, d0 + n * 8 + 2 * t, X[m][n][2 * e], X[m][n][2 * e + 1]);
     };
-    if (owner) {
-        each_state([&](float& x, int v, int d) { x = sp.pos0 > 0 && v < Dv && d < D ? st[(size_t)d * Dv + v] : 0.f; });
-        publish();
-    }
-    __syncthreads();
-    bool ok = true;
-    float2 base[NB][2];                                // U (delta) or v (a pair of bf16 in x) of rows wr + g, wr + g + 8 of the chunk ahead
+    uint4 ah[KS], al[KS], kh[F3 > 4 ? F3 : 4], kl[F3 > 4 ? F3 : 4], base[NB];
+    auto fetch_first = [&](int c) {                    // W or q of this warp's rows
+        if (!DELTA && owner) return;
+        const unsigned char* p = tiles(c) + (owner ? L::W : L::Q) + (rb * KS * 32 + lane) * 16;
+#pragma unroll
+        for (int k = 0; k < KS; ++k) { ah[k] = ld_once(p + k * 512); al[k] = ld_once(p + L::TILE + k * 512); }
+    };
+    auto fetch_second = [&](int c) {                   // k of this warp's channels, or A of its rows
+        if (owner) {
+            const unsigned char* p = tiles(c) + L::K + (d0 / 16 * 4 * 32 + lane) * 16;
+#pragma unroll
+            for (int k = 0; k < F3; ++k) { kh[k] = ld_once(p + k * 512); kl[k] = ld_once(p + L::TILE + k * 512); }
+        } else {
+            const unsigned char* p = tiles(c) + L::A + (rb * 4 * 32 + lane) * 16;
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+                if (k <= rb) { kh[k] = ld_once(p + k * 512); kl[k] = ld_once(p + L::ATILE + k * 512); }
+        }
+    };
     const bool pairs = (Dv & 1) == 0 && (P.ld & 1) == 0 && (P.v_col & 1) == 0 && ((uintptr_t)P.x & 3) == 0;
-    auto fetch = [&](int c) {
+    auto fetch_base = [&](int c) {                     // U in accumulator order, or v (two pairs of bf16 in x)
         const int row0 = sp.row0 + c * CH, cnt = min(CH, sp.count - c * CH);
 #pragma unroll
-        for (int n = 0; n < NB; ++n)
+        for (int n = 0; n < NB; ++n) {
+            if constexpr (DELTA) base[n] = ld_once(tiles(c) + L::U + (((v0 / 16 + (n >> 1)) * 4 + rb) * 64 + (n & 1) * 32 + lane) * 16);
+            else {
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int r = wr + g + 8 * e, v = v0 + n * 8 + 2 * t;
-                if constexpr (DELTA) base[n][e] = *reinterpret_cast<const float2*>(tiles(c) + L::U + ((size_t)r * W.Dvp + v) * 4);
-                else {
+                for (int e = 0; e < 2; ++e) {
+                    const int r = wr + g + 8 * e, v = v0 + n * 8 + 2 * t;
                     uint32_t f = 0;
                     if (r < cnt && v < Dv) {
                         const __nv_bfloat16* x = (const __nv_bfloat16*)P.x + (size_t)(row0 + r) * P.ld + P.v_col + (size_t)h * Dv + v;
                         if (pairs) f = *reinterpret_cast<const uint32_t*>(x);
                         else f = *reinterpret_cast<const uint16_t*>(x) | (v + 1 < Dv ? (uint32_t)*reinterpret_cast<const uint16_t*>(x + 1) << 16 : 0u);
                     }
-                    base[n][e].x = __uint_as_float(f);
+                    (e ? base[n].y : base[n].x) = f;
                 }
             }
+        }
     };
-    if (owner) fetch(0);
+    fetch_first(0);
+    if (owner) {
+        fetch_base(0);
+        each_state([&](float& x, int v, int d) { x = sp.pos0 > 0 && v < Dv && d < D ? st[(size_t)d * Dv + v] : 0.f; });
+        publish();
+    }
+    __syncthreads();
     for (int c = 0; c < chunks; ++c) {
         const int row0 = sp.row0 + c * CH, cnt = min(CH, sp.count - c * CH);
-        const uint32_t wh = smem_u32(smem + (2 * c % 3) * S::SLOT), qh = wh + 2 * L::TILE;
-        const uint32_t kh = smem_u32(smem + ((2 * c + 1) % 3) * S::SLOT), ah = kh + 2 * L::TILE;
         float acc[NB][4], low[NB][4], ge[NT][2];       // products of the high parts; those with a low part
 #pragma unroll
         for (int n = 0; n < NB; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) acc[n][e] = low[n][e] = 0.f;
+        fetch_second(c);
         if (owner) {
 #pragma unroll
             for (int n = 0; n < NT; ++n) {
@@ -622,45 +701,48 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                 ge[n][0] = f.x; ge[n][1] = f.y;
             }
         }
-        if (ok) ok = mbar_wait(&bar[2 * c % 3], (uint32_t)((2 * c / 3) & 1), P.status);
         if (DELTA || !owner) {                         // W S (warps 0-3) or (q G) S (warps 4-7): 16 rows each
-            const uint32_t th = owner ? wh : qh, tl = th + L::TILE;
-#pragma unroll 4
-            for (int ks = 0; ks < DT / 16; ++ks) {
-                uint32_t a[4], b[4];
-                fa::load_a<DT>(th, wr, ks, a);
-                fa::load_a<DT>(tl, wr, ks, b);
+#pragma unroll
+            for (int ks = 0; ks < KS; ++ks) {
                 uint32_t bh[MT][4], bl[MT][4];
 #pragma unroll
                 for (int n = 0; n < MT; ++n) { fa::load_b<DT>(sh, n * 16, ks, bh[n]); fa::load_b<DT>(sl, n * 16, ks, bl[n]); }
 #pragma unroll
-                for (int n = 0; n < NB; ++n) fa::mma16816(acc[n], a, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+                for (int n = 0; n < NB; ++n) mma_u4(acc[n], ah[ks], bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
 #pragma unroll
-                for (int n = 0; n < NB; ++n) fa::mma16816(low[n], b, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+                for (int n = 0; n < NB; ++n) mma_u4(low[n], al[ks], bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
 #pragma unroll
-                for (int n = 0; n < NB; ++n) fa::mma16816(low[n], a, bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
+                for (int n = 0; n < NB; ++n) mma_u4(low[n], ah[ks], bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
             }
         }
+        if (c + 1 < chunks) fetch_first(c + 1);
         if (owner) {                                   // u^T, split
 #pragma unroll
-            for (int n = 0; n < NB; ++n)
+            for (int n = 0; n < NB; ++n) {
+                float u[4];
+                if constexpr (DELTA) {
+                    u[0] = __uint_as_float(base[n].x); u[1] = __uint_as_float(base[n].y); u[2] = __uint_as_float(base[n].z); u[3] = __uint_as_float(base[n].w);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) u[e] -= acc[n][e] + low[n][e];
+                } else {
+                    const float2 a = unpack(base[n].x), b = unpack(base[n].y);
+                    u[0] = a.x; u[1] = a.y; u[2] = b.x; u[3] = b.y;
+                    if (P.silu)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) u[e] = silu(u[e]);
+                }
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const float2 f = DELTA ? base[n][e >> 1] : unpack(__float_as_uint(base[n][e >> 1].x));
-                    float u = (e & 1) ? f.y : f.x;
-                    if constexpr (DELTA) u -= acc[n][e] + low[n][e];
-                    else if (P.silu) u = silu(u);
                     const int v = n * 8 + 2 * t + (e & 1), r = wr + g + 8 * (e >> 1);
-                    const __nv_bfloat16 hi = __float2bfloat16_rn(u);
+                    const __nv_bfloat16 hi = __float2bfloat16_rn(u[e]);
                     const uint32_t off = fa::tile_off<CH>(v, r >> 3) + (r & 7) * 2;
-                    *reinterpret_cast<__nv_bfloat16*>(smem + S::UH + off) = hi;
-                    *reinterpret_cast<__nv_bfloat16*>(smem + S::UL + off) = __float2bfloat16_rn(u - __bfloat162float(hi));
+                    *reinterpret_cast<__nv_bfloat16*>(u_hi + off) = hi;
+                    *reinterpret_cast<__nv_bfloat16*>(u_lo + off) = __float2bfloat16_rn(u[e] - __bfloat162float(hi));
                 }
-            if (c + 1 < chunks) fetch(c + 1);
+            }
+            if (c + 1 < chunks) fetch_base(c + 1);
         }
-        __syncthreads();                               // u is there; W, q and the state tiles have been read
-        if (threadIdx.x == 0 && c + 1 < chunks && ok) load(2 * c + 3);
-        if (ok) ok = mbar_wait(&bar[(2 * c + 1) % 3], (uint32_t)(((2 * c + 1) / 3) & 1), P.status);
+        __syncthreads();                               // u is there; the state tiles have been read
         if (owner) {
 #pragma unroll
             for (int m = 0; m < MT; ++m)
@@ -668,21 +750,9 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                 for (int n = 0; n < NT; ++n)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) X[m][n][e] *= ge[n][e & 1];
-            float Y[MT][NT][4];                        // products with a low part
 #pragma unroll
-            for (int m = 0; m < MT; ++m)
-#pragma unroll
-                for (int n = 0; n < NT; ++n)
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) Y[m][n][e] = 0.f;
-#pragma unroll 2
             for (int ks = 0; ks < CH / 16; ++ks) {
-                uint32_t bh[NT / 2][4], bl[NT / 2][4], a[MT][4], b[MT][4];
-#pragma unroll
-                for (int n = 0; n < NT / 2; ++n) {
-                    fa::load_b_t<DT>(kh, ks * 16, d0 / 8 + 2 * n, bh[n]);
-                    fa::load_b_t<DT>(kh + L::TILE, ks * 16, d0 / 8 + 2 * n, bl[n]);
-                }
+                uint32_t a[MT][4], b[MT][4];
 #pragma unroll
                 for (int m = 0; m < MT; ++m) { fa::load_a<CH>(uh, m * 16, ks, a[m]); fa::load_a<CH>(ul, m * 16, ks, b[m]); }
 #pragma unroll
@@ -691,63 +761,50 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                     for (int m = 0; m < MT; ++m)
 #pragma unroll
                         for (int n = 0; n < NT; ++n) {
-                            const uint32_t* w = k == 2 ? bl[n / 2] : bh[n / 2];
-                            fa::mma16816(k == 0 ? X[m][n] : Y[m][n], k == 1 ? b[m] : a[m], w[2 * (n & 1)], w[2 * (n & 1) + 1]);
+                            const uint4& w = k == 2 ? kl[n / 2 * 4 + ks] : kh[n / 2 * 4 + ks];
+                            fa::mma16816(X[m][n], k == 1 ? b[m] : a[m], (n & 1) ? w.z : w.x, (n & 1) ? w.w : w.y);
                         }
             }
-#pragma unroll
-            for (int m = 0; m < MT; ++m)
-#pragma unroll
-                for (int n = 0; n < NT; ++n)
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) X[m][n][e] += Y[m][n][e];
             publish();
         } else {
-            for (int ks = 0; ks <= wr / 16; ++ks) {
-                uint32_t a[4], b[4];
-                fa::load_a<CH>(ah, wr, ks, a);
-                fa::load_a<CH>(ah + L::ATILE, wr, ks, b);
-                uint32_t bh[MT][4], bl[MT][4];
 #pragma unroll
-                for (int n = 0; n < MT; ++n) { fa::load_b<CH>(uh, n * 16, ks, bh[n]); fa::load_b<CH>(ul, n * 16, ks, bl[n]); }
+            for (int ks = 0; ks < CH / 16; ++ks)
+                if (ks <= rb) {
+                    uint32_t bh[MT][4], bl[MT][4];
 #pragma unroll
-                for (int n = 0; n < NB; ++n) fa::mma16816(acc[n], a, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+                    for (int n = 0; n < MT; ++n) { fa::load_b<CH>(uh, n * 16, ks, bh[n]); fa::load_b<CH>(ul, n * 16, ks, bl[n]); }
 #pragma unroll
-                for (int n = 0; n < NB; ++n) fa::mma16816(low[n], b, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+                    for (int n = 0; n < NB; ++n) mma_u4(acc[n], kh[ks], bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
 #pragma unroll
-                for (int n = 0; n < NB; ++n) fa::mma16816(low[n], a, bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
-            }
+                    for (int n = 0; n < NB; ++n) mma_u4(low[n], kl[ks], bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
 #pragma unroll
-            for (int n = 0; n < NB; ++n)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) acc[n][e] += low[n][e];
+                    for (int n = 0; n < NB; ++n) mma_u4(low[n], kh[ks], bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
+                }
 #pragma unroll
             for (int n = 0; n < NB; ++n)
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int r = wr + g + 8 * e, v = v0 + n * 8 + 2 * t;
                     float* o = P.out + (size_t)(row0 + r) * P.H * Dv + (size_t)h * Dv + v;
+                    const float x = acc[n][2 * e] + low[n][2 * e], y = acc[n][2 * e + 1] + low[n][2 * e + 1];
                     if (r >= cnt) continue;
-                    if (v + 1 < Dv && (Dv & 1) == 0) *reinterpret_cast<float2*>(o) = make_float2(acc[n][2 * e], acc[n][2 * e + 1]);
+                    if (v + 1 < Dv && (Dv & 1) == 0) *reinterpret_cast<float2*>(o) = make_float2(x, y);
                     else {
-                        if (v < Dv) o[0] = acc[n][2 * e];
-                        if (v + 1 < Dv) o[1] = acc[n][2 * e + 1];
+                        if (v < Dv) o[0] = x;
+                        if (v + 1 < Dv) o[1] = y;
                     }
                 }
         }
-        __syncthreads();                               // the new state is there; k, A and u have been read
-        if (threadIdx.x == 0 && c + 2 < chunks && ok) load(2 * c + 4);
+        __syncthreads();                               // the new state is there; u has been read
     }
-    if (owner) each_state([&](float& x, int v, int d) { if (ok && v < Dv && d < D) st[(size_t)d * Dv + v] = x; });
+    if (owner) each_state([&](float& x, int v, int d) { if (v < Dv && d < D) st[(size_t)d * Dv + v] = x; });
 }
 
 template <int DT, int VS>
 static int launch_state(const Params& p, cudaStream_t st) {
     const dim3 grid((p.P.Dv + VS - 1) / VS, p.P.H, p.P.n_seqs);
     auto kern = p.P.delta ? chunk_state_kernel<DT, VS, true> : chunk_state_kernel<DT, VS, false>;
-    constexpr int smem = StateSmem<DT, VS>::TOTAL;
-    PTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    PTB_CUDA_OK(ptb_launch(kern, grid, dim3(THREADS), (size_t)smem, st, ptb_pdl_enabled(), p));
+    PTB_CUDA_OK(ptb_launch(kern, grid, dim3(THREADS), 0, st, ptb_pdl_enabled(), p));
     return 0;
 }
 
@@ -807,6 +864,11 @@ PTB_API int ptb_recurrence_chunked(const PtbRecurrence* args, void* work, long l
     p.Dvp = (args->Dv + 31) / 32 * 32;
     p.vec = args->D % 8 == 0 && args->Dv % 8 == 0 && args->ld % 8 == 0 && args->q_col % 8 == 0 && args->k_col % 8 == 0 && args->v_col % 8 == 0 &&
             ((uintptr_t)args->x & 15) == 0;
+    if (args->delta && args->low &&
+        (!args->low_w || args->rank < 8 || args->rank > 256 || args->rank % 8 || args->ld_low % 8 || (((uintptr_t)args->low | (uintptr_t)args->low_w) & 15))) {
+        ptb_set_error("recurrence_chunked: a low-rank product of rank %d (a multiple of eight up to 256, 16-byte aligned rows)", args->rank);
+        return -1;
+    }
     p.vec_a = args->D % 4 == 0 && args->ld_a % 4 == 0 && ((uintptr_t)args->a & 15) == 0;
     return args->D <= 64 ? rc::launch<64>(p, st) : rc::launch<128>(p, st);
 }

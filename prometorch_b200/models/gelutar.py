@@ -132,7 +132,7 @@ class GelutarConfig:
                 "norm": {"eps": self.eps}, "logit_scale": self.logit_scale, "layers": layers}
 
 
-MERGE_GATES = 128                      # rows up to which the two low-rank gates are one product
+MERGE_GATES = 128                      # rows up to which the two low-rank gates are one product of their own
 _LEFT = ("left.q", "left.k", "left.v")
 _CONV = ("right.q", "right.k", "right.v")
 
@@ -247,8 +247,8 @@ class PagedGelutar(PagedModel):
                 d["w_in"] = d["pack"].pack({**{n: L["mix." + n] for n in _LEFT + ("left.g", "right.b")}, "low": low,
                                             "conv": torch.cat([L["mix." + n] for n in _CONV])})
                 d["conv"] = torch.cat([L[f"mix.{n}.conv"] for n in _CONV]).t().contiguous()          # [taps, channels]
-                # few rows: both low-rank gates as one product, block-diagonal second matrices over the packed first ones; many rows: one
-                # product each, the decays' in fp32
+                # few rows: both low-rank gates as one product, block-diagonal second matrices over the packed first ones; many rows: the
+                # output gate's alone, the decays' is formed where it is used
                 ra, rg = RowPack.up(L["mix.right.a1"].shape[0]), L["mix.right.g1"].shape[0]
                 a2, g2 = L["mix.right.a2"], L["mix.right.g2"]
                 gates = a2.new_zeros(RowPack.up(a2.shape[0]) + g2.shape[0], RowPack.up(ra + rg))
@@ -311,11 +311,11 @@ class PagedGelutar(PagedModel):
         c = R.short_conv(pk.cols(p, "conv"), d["conv"], kv.state[l]["conv"], pos, req, seqs)
         r, at, low = d["delta"], d["gate_cols"], pk.cols(p, "low", padded=True)
         if p.shape[0] > MERGE_GATES:
-            decay, gate = S.linear_f32(low[:, :d["rank_a"]], d["a2"]), linear(low[:, d["rank_a"]:], d["g2"])
+            decay, gate = (low[:, :d["rank_a"]], d["a2"]), linear(low[:, d["rank_a"]:], d["g2"])
         else:
             gates = S.linear_f32(low, d["gates"])
-            decay, gate = gates[:, :at], gates[:, at:]
-        o = R.delta_rule(c, r, pk.cols(p, "right.b"), decay[:, :r.heads * r.dim], kv.state[l]["S"], pos, req, seqs)
+            decay, gate = gates[:, :r.heads * r.dim], gates[:, at:]
+        o = R.delta_rule(c, r, pk.cols(p, "right.b"), decay, kv.state[l]["S"], pos, req, seqs)
         o = R.group_norm_gate(o, d["right.norm"], gate[:, :r.heads * r.vdim], eps, self.dtype)
         y = attend(l, a, q, pk.cols(p, "left.g"))
         return [S.linear_branch(y, d["left.o"], 0.5, d["left.out"]), S.linear_branch(o, d["right.o"], 0.5, d["right.out"])]

@@ -8,7 +8,7 @@ from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass
-from typing import List, Optional, Tuple
+from typing import List, Optional, Tuple, Union
 
 import torch
 
@@ -25,7 +25,8 @@ class RecurrenceArgs(C.Structure):
                 ("state", C.c_void_p), ("slots", C.c_int), ("n", C.c_int), ("H", C.c_int), ("G", C.c_int), ("D", C.c_int), ("Dv", C.c_int),
                 ("seqs", C.c_void_p), ("n_seqs", C.c_int), ("pos_stride", C.c_int), ("req_stride", C.c_int), ("pad", C.c_int),
                 ("pos", C.c_void_p), ("req", C.c_void_p), ("out", C.c_void_p), ("status", C.c_void_p),
-                ("chunks", C.c_void_p), ("first_chunk", C.c_void_p), ("n_chunks", C.c_int), ("pad2", C.c_int)]
+                ("chunks", C.c_void_p), ("first_chunk", C.c_void_p), ("n_chunks", C.c_int), ("rank", C.c_int),
+                ("low", C.c_void_p), ("ld_low", C.c_longlong), ("low_w", C.c_void_p)]
 
 
 @N.register_decls
@@ -135,36 +136,56 @@ def _unit(x):
     return x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6)
 
 
-def _run(args: RecurrenceArgs, x: torch.Tensor, seqs: Optional[Sequences], pos, req, state: torch.Tensor, out: torch.Tensor, chunked: Optional[bool]):
+def _runs_chunked(x: torch.Tensor, D: int, Dv: int, seqs: Optional[Sequences], chunked: Optional[bool]) -> bool:
+    """Whether the kernels of csrc/recurrence_chunk.cu take this pass: bf16 prompts of some length, head sizes up to 128."""
+    if seqs is None or x.dtype != torch.bfloat16 or max(D, Dv) > 128 or chunked is False:
+        return False
+    return bool(chunked) or max(c for _, c, _, _ in seqs.host) >= CHUNKED_FROM
+
+
+def _run(args: RecurrenceArgs, x: torch.Tensor, seqs: Optional[Sequences], pos, req, state: torch.Tensor, out: torch.Tensor, chunked: bool):
     args.x, args.ld, args.bf16 = x.data_ptr(), x.stride(0), int(x.dtype == torch.bfloat16)
     args.state, args.slots, args.n, args.out, args.status = state.data_ptr(), state.shape[0], x.shape[0], out.data_ptr(), _status(x.device).data_ptr()
     args.pos, args.pos_stride, args.req, args.req_stride = pos.data_ptr(), pos.stride(0), req.data_ptr(), req.stride(0)
     if seqs is not None:
         args.seqs, args.n_seqs = seqs.device.data_ptr(), len(seqs.host)
         args.chunks, args.n_chunks, args.first_chunk = seqs.chunks.data_ptr(), seqs.chunks.shape[0], seqs.first_chunk.data_ptr()
-        if chunked is None:
-            chunked = x.dtype == torch.bfloat16 and max(c for _, c, _, _ in seqs.host) >= CHUNKED_FROM
-        size = int(N.lib().ptb_recurrence_chunked_bytes(C.byref(args))) if chunked else -1
-        if size > 0:                                           # -1: sizes the chunk kernels do not take
-            work = torch.empty(size, dtype=torch.uint8, device=x.device)
-            N.check(N.lib().ptb_recurrence_chunked(C.byref(args), work.data_ptr(), size, _st(x)), "recurrence_chunked")
-            return
-    N.check(N.lib().ptb_recurrence(C.byref(args), _st(x)), "recurrence")
+    if chunked:
+        work = torch.empty(int(N.lib().ptb_recurrence_chunked_bytes(C.byref(args))), dtype=torch.uint8, device=x.device)
+        N.check(N.lib().ptb_recurrence_chunked(C.byref(args), work.data_ptr(), work.numel(), _st(x)), "recurrence_chunked")
+    else:
+        N.check(N.lib().ptb_recurrence(C.byref(args), _st(x)), "recurrence")
 
 
-def delta_rule(x: torch.Tensor, r: DeltaRule, beta: torch.Tensor, a: torch.Tensor, state: torch.Tensor, pos: torch.Tensor, req: torch.Tensor,
-               seqs: Optional[Sequences] = None, chunked: Optional[bool] = None) -> torch.Tensor:
-    """``x [n, 2 G dim + H vdim]``: q, k and v after their convolutions; ``beta [n, H]`` before its sigmoid (type of x), ``a [n, H
-    dim]`` fp32.  Advances ``state [slots, H, dim, vdim]``; returns o ``[n, H vdim]`` fp32."""
+def delta_rule(x: torch.Tensor, r: DeltaRule, beta: torch.Tensor, a: Union[torch.Tensor, Tuple[torch.Tensor, torch.Tensor]], state: torch.Tensor,
+               pos: torch.Tensor, req: torch.Tensor, seqs: Optional[Sequences] = None, chunked: Optional[bool] = None) -> torch.Tensor:
+    """``x [n, 2 G dim + H vdim]``: q, k and v after their convolutions; ``beta [n, H]`` before its sigmoid (type of x); ``a [n, H
+    dim]`` fp32, or its factors ``(low [n, rank], w [>= H dim, rank])`` in the type of x, whose product the chunk kernel forms itself.
+    Advances ``state [slots, H, dim, vdim]``; returns o ``[n, H vdim]`` fp32."""
     n, H, G, D, Dv = x.shape[0], r.heads, r.kv_heads, r.dim, r.vdim
     out = torch.empty(n, H * Dv, dtype=torch.float32, device=x.device)
     if x.is_cuda:
         _check(x)
-        assert a.dtype == torch.float32 and a.stride(1) == 1 and beta.dtype == x.dtype and state.is_contiguous()
-        args = RecurrenceArgs(q_col=0, k_col=G * D, v_col=2 * G * D, delta=1, beta=beta.data_ptr(), ld_beta=beta.stride(0), a=a.data_ptr(), ld_a=a.stride(0),
-                              decay=r.rate.data_ptr(), dt_bias=r.dt_bias.data_ptr(), H=H, G=G, D=D, Dv=Dv)
+        assert beta.dtype == x.dtype and state.is_contiguous()
+        chunked = _runs_chunked(x, D, Dv, seqs, chunked)
+        args = RecurrenceArgs(q_col=0, k_col=G * D, v_col=2 * G * D, delta=1, beta=beta.data_ptr(), ld_beta=beta.stride(0), decay=r.rate.data_ptr(),
+                              dt_bias=r.dt_bias.data_ptr(), H=H, G=G, D=D, Dv=Dv)
+        if isinstance(a, tuple):
+            low, w = a
+            rank = w.shape[1]
+            if chunked and rank % 8 == 0 and rank <= 256 and low.stride(0) % 8 == 0 and low.data_ptr() % 16 == 0 and w.is_contiguous():
+                assert low.dtype == w.dtype == x.dtype and low.shape[1] == rank and w.shape[0] >= H * D and low.stride(1) == 1
+                args.low, args.ld_low, args.low_w, args.rank = low.data_ptr(), low.stride(0), w.data_ptr(), rank
+            else:
+                from .residual import linear_f32
+                a = linear_f32(low, w)
+        if not isinstance(a, tuple):
+            assert a.dtype == torch.float32 and a.stride(1) == 1
+            args.a, args.ld_a = a.data_ptr(), a.stride(0)
         _run(args, x, seqs, pos, req, state, out, chunked)
         return out
+    if isinstance(a, tuple):
+        a = (a[0].float() @ a[1].float().t())[:, :H * D]
     f = x.float()
     q = (_unit(f[:, :G * D].reshape(n, G, D)) * D ** -0.5).repeat_interleave(H // G, 1)
     k = _unit(f[:, G * D:2 * G * D].reshape(n, G, D)).repeat_interleave(H // G, 1)
@@ -193,7 +214,7 @@ def decay_attention(x: torch.Tensor, r: DecayAttention, cols: Tuple[int, int, in
         _check(x)
         assert state.is_contiguous()
         args = RecurrenceArgs(q_col=cols[0], k_col=cols[1], v_col=cols[2], silu=int(r.silu), delta=0, decay=r.decay.data_ptr(), H=H, G=H, D=D, Dv=Dv)
-        _run(args, x, seqs, pos, req, state, out, chunked)
+        _run(args, x, seqs, pos, req, state, out, _runs_chunked(x, D, Dv, seqs, chunked))
         return out
     act = torch.nn.functional.silu if r.silu else (lambda t: t)
     q, k, v = (act(x[:, c:c + H * d].float()).reshape(n, H, d) for c, d in zip(cols, (D, D, Dv)))

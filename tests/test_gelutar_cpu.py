@@ -175,6 +175,15 @@ def test_delta_rule_in_portions():
         assert close(torch.cat(out), want) and close(state[1], S) and float(state[0].min()) == 5.0
 
 
+def test_delta_rule_takes_factors_of_its_decays():
+    r, x, beta, _ = delta_case()
+    low, w = torch.randn(40, 6), torch.randn(48, 6)
+    s, pos, req = seqs_of([40], [0], [0])
+    want, S = delta_oracle(r, x, beta, low @ w.t())
+    state = torch.zeros(1, 4, 12, 20)
+    assert close(R.delta_rule(x, r, beta, (low, w), state, pos, req, s), want) and close(state[0], S)
+
+
 def test_delta_rule_overwrites_a_key():
     """Two tokens with one key: with beta near 1 and no decay the second value replaces the first."""
     r = R.DeltaRule(1, 1, 4, 3, torch.tensor([1e-6]), torch.zeros(4))

@@ -231,6 +231,23 @@ def test_delta_rule_decays(shift, spread):
         assert torch.isfinite(got).all() and rel(got, want) < 1e-4 and rel(S, want_S) < 1e-4
 
 
+@pytest.mark.parametrize("H,G,D,Dv,rank", [(4, 2, 64, 64, 24), (2, 2, 128, 128, 128), (3, 1, 20, 36, 8), (2, 1, 96, 48, 256), (2, 1, 96, 48, 264)])
+def test_delta_rule_low_rank_decays(H, G, D, Dv, rank):
+    """The decays' projection given as its two factors."""
+    from prometorch_b200.ops import recurrence as R
+    lens, starts = [150, 1, 65], [0, 9, 3]
+    cpu, gpu, pos, req = batch(lens, starts, [1, 0, 2])
+    r, x, beta, _ = delta_inputs(H, G, D, Dv, sum(lens), torch.bfloat16)
+    low, w = torch.randn(sum(lens), rank + 16).bfloat16()[:, 8:8 + rank], (torch.randn(-(-H * D // 8) * 8, rank) * rank ** -0.5).bfloat16()
+    start = torch.randn(3, H, D, Dv)
+    want_S = start.clone()
+    want = R.delta_rule(x, r, beta, (low, w), want_S, pos, req, cpu)
+    for chunked in (False, True):
+        S = start.cuda()
+        got = R.delta_rule(x.cuda(), on_gpu(r), beta.cuda(), (low.cuda(), w.cuda()), S, pos.cuda(), req.cuda(), gpu, chunked=chunked)
+        assert rel(got, want) < 1e-4 and rel(S, want_S) < 1e-4
+
+
 def test_delta_rule_repeated_keys():
     """The same key over and over with beta near 1: the triangular system of a chunk is far from the identity."""
     from prometorch_b200.ops import recurrence as R
