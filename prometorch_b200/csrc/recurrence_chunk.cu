@@ -9,7 +9,7 @@
 //   delta_chunk_kernel / decay_chunk_kernel   everything that does not depend on S, all chunks at once, into a workspace;
 //   chunk_state_kernel                        walks a sequence's chunks for a slice of value columns; S stays in registers.
 // What passes between them lies in the order of the mma fragments that will read it: a lane's 16 bytes are its four registers of a 16 x 16
-// block, so the walk loads its operands from L2 into registers, whole lines at a time, without shared memory.
+// block, so the walk takes an operand with one 16-byte load per lane.
 // Quotients of decays are never formed from products that could overflow: across blocks of 16 tokens both factors refer to the block
 // border between the two tokens and are at most 1, inside a block the exponent of every pair is taken directly.
 // Products run on the tensor cores with every fp32 operand split into two bf16 numbers (three products: 16 bits of both operands).
@@ -590,6 +590,7 @@ __device__ __forceinline__ uint4 ld_once(const unsigned char* p) {
     asm volatile("ld.global.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
     return v;
 }
+__device__ __forceinline__ uint4 lds_frag(const unsigned char* p, int frag, int lane) { return *reinterpret_cast<const uint4*>(p + (frag * 32 + lane) * 16); }
 __device__ __forceinline__ void mma_u4(float* d, const uint4& a, uint32_t b0, uint32_t b1) {
     const uint32_t f[4] = {a.x, a.y, a.z, a.w};
     fa::mma16816(d, f, b0, b1);
@@ -597,16 +598,29 @@ __device__ __forceinline__ void mma_u4(float* d, const uint4& a, uint32_t b0, ui
 
 // One CTA per (VS value columns, head, sequence), eight warps.  Of a chunk, warps 0-3 form u (64 rows) and then the new state, warps 4-7
 // the read-out; the state lives transposed, [value][key channel], in the accumulators of warps 0-3 and as two bf16 tiles in shared
-// memory for the products that read it.  Every other operand is read by exactly one warp and comes from the workspace into registers:
-// the fragments of a chunk's second half are on their way during its first half, those of the next chunk's first half during the second.
+// memory for the products that read it.  The other operands arrive by bulk copies through three slots, in the order of their use: W and q
+// of a chunk, its k and A, W and q of the next, ...
+template <int DT, int VS>
+struct StateSmem {
+    using L = Work<DT>;
+    static constexpr int SLOT = 4 * L::TILE > 2 * L::TILE + 2 * L::ATILE ? 4 * L::TILE : 2 * L::TILE + 2 * L::ATILE, SH = 3 * SLOT, SL = SH + VS * DT * 2;
+    static constexpr int UH = SL + VS * DT * 2, UL = UH + VS * CH * 2, BAR = UL + VS * CH * 2, TOTAL = BAR + 64;
+};
 template <int DT, int VS, bool DELTA>
 __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_constant__ Params W) {
     using L = Work<DT>;
+    using S = StateSmem<DT, VS>;
     constexpr int KS = DT / 16, NT = DT / 32, MT = VS / 16, NB = VS / 8;       // state tiles of a warp: MT x NT of 16 x 8
-    constexpr int F3 = NT / 2 * 4;                     // fragments of the second half (the read-out uses up to four)
-    __shared__ __align__(128) unsigned char s_hi[VS * DT * 2], s_lo[VS * DT * 2], u_hi[VS * CH * 2], u_lo[VS * CH * 2];
+    extern __shared__ __align__(128) unsigned char smem[];
+    unsigned char *s_hi = smem + S::SH, *s_lo = smem + S::SL, *u_hi = smem + S::UH, *u_lo = smem + S::UL;
+    uint64_t* bar = reinterpret_cast<uint64_t*>(smem + S::BAR);    // one per slot
     const PtbRecurrence& P = W.P;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < 3; ++i) mbar_init(&bar[i], 1);
+        mbar_fence_init();
+    }
+    __syncthreads();
     pdl_wait();
     pdl_launch_dependents();
     const int h = blockIdx.y, v0 = blockIdx.x * VS, D = P.D, Dv = P.Dv;
@@ -622,6 +636,22 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
     const uint32_t sh = smem_u32(s_hi), sl = smem_u32(s_lo), uh = smem_u32(u_hi), ul = smem_u32(u_lo);
     float* st = P.state + (((size_t)sp.slot * P.H + h) * D) * Dv;
     auto tiles = [&](int c) { return W.work + ((size_t)(first + c) * P.H + h) * W.stride; };
+    // load 2c: W and q of chunk c, load 2c + 1: its k and A; load i goes to slot i % 3 once load i - 3 has been read
+    auto load = [&](int i) {
+        const int s = i % 3;
+        const unsigned char* src = tiles(i >> 1);
+        if (i & 1) {
+            constexpr uint32_t bytes = 2 * L::TILE + 2 * L::ATILE;
+            mbar_expect_tx(&bar[s], bytes);
+            bulk_g2s(smem + s * S::SLOT, src + L::K, bytes, &bar[s]);
+        } else {
+            constexpr uint32_t bytes = (DELTA ? 4 : 2) * L::TILE;
+            mbar_expect_tx(&bar[s], bytes);
+            bulk_g2s(smem + s * S::SLOT + (DELTA ? 0 : 2 * L::TILE), src + (DELTA ? L::W : L::Q), bytes, &bar[s]);
+        }
+    };
+    if (threadIdx.x == 0)
+        for (int i = 0; i < min(3, 2 * chunks); ++i) load(i);
     float X[MT][NT][4];                                // S^T: row v0 + 16 m + g (+ 8), column d0 + 8 n + 2t (+ 1)
     auto each_state = [&](auto f) {
 #pragma unroll
@@ -639,27 +669,9 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
 #pragma unroll
                 for (int e = 0; e < 2; ++e) store_split<DT>(s_hi, s_lo, m * 16 + g + 8 * e, d0 + n * 8 + 2 * t, X[m][n][2 * e], X[m][n][2 * e + 1]);
     };
-    uint4 ah[KS], al[KS], kh[F3 > 4 ? F3 : 4], kl[F3 > 4 ? F3 : 4], base[NB];
-    auto fetch_first = [&](int c) {                    // W or q of this warp's rows
-        if (!DELTA && owner) return;
-        const unsigned char* p = tiles(c) + (owner ? L::W : L::Q) + (rb * KS * 32 + lane) * 16;
-#pragma unroll
-        for (int k = 0; k < KS; ++k) { ah[k] = ld_once(p + k * 512); al[k] = ld_once(p + L::TILE + k * 512); }
-    };
-    auto fetch_second = [&](int c) {                   // k of this warp's channels, or A of its rows
-        if (owner) {
-            const unsigned char* p = tiles(c) + L::K + (d0 / 16 * 4 * 32 + lane) * 16;
-#pragma unroll
-            for (int k = 0; k < F3; ++k) { kh[k] = ld_once(p + k * 512); kl[k] = ld_once(p + L::TILE + k * 512); }
-        } else {
-            const unsigned char* p = tiles(c) + L::A + (rb * 4 * 32 + lane) * 16;
-#pragma unroll
-            for (int k = 0; k < 4; ++k)
-                if (k <= rb) { kh[k] = ld_once(p + k * 512); kl[k] = ld_once(p + L::ATILE + k * 512); }
-        }
-    };
+    uint4 base[NB];
     const bool pairs = (Dv & 1) == 0 && (P.ld & 1) == 0 && (P.v_col & 1) == 0 && ((uintptr_t)P.x & 3) == 0;
-    auto fetch_base = [&](int c) {                     // U in accumulator order, or v (two pairs of bf16 in x)
+    auto fetch_base = [&](int c) {                     // U in accumulator order, or v (two pairs of bf16)
         const int row0 = sp.row0 + c * CH, cnt = min(CH, sp.count - c * CH);
 #pragma unroll
         for (int n = 0; n < NB; ++n) {
@@ -679,21 +691,21 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
             }
         }
     };
-    fetch_first(0);
     if (owner) {
         fetch_base(0);
         each_state([&](float& x, int v, int d) { x = sp.pos0 > 0 && v < Dv && d < D ? st[(size_t)d * Dv + v] : 0.f; });
         publish();
     }
     __syncthreads();
+    bool ok = true;
     for (int c = 0; c < chunks; ++c) {
+        const unsigned char *wq = smem + (2 * c % 3) * S::SLOT, *ka = smem + ((2 * c + 1) % 3) * S::SLOT;
         const int row0 = sp.row0 + c * CH, cnt = min(CH, sp.count - c * CH);
         float acc[NB][4], low[NB][4], ge[NT][2];       // products of the high parts; those with a low part
 #pragma unroll
         for (int n = 0; n < NB; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) acc[n][e] = low[n][e] = 0.f;
-        fetch_second(c);
         if (owner) {
 #pragma unroll
             for (int n = 0; n < NT; ++n) {
@@ -701,21 +713,23 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                 ge[n][0] = f.x; ge[n][1] = f.y;
             }
         }
+        if (ok) ok = mbar_wait(&bar[2 * c % 3], (uint32_t)((2 * c / 3) & 1), P.status);
         if (DELTA || !owner) {                         // W S (warps 0-3) or (q G) S (warps 4-7): 16 rows each
+            const unsigned char* p = wq + (owner ? 0 : 2 * L::TILE);
 #pragma unroll
             for (int ks = 0; ks < KS; ++ks) {
+                const uint4 ah = lds_frag(p, rb * KS + ks, lane), al = lds_frag(p + L::TILE, rb * KS + ks, lane);
                 uint32_t bh[MT][4], bl[MT][4];
 #pragma unroll
                 for (int n = 0; n < MT; ++n) { fa::load_b<DT>(sh, n * 16, ks, bh[n]); fa::load_b<DT>(sl, n * 16, ks, bl[n]); }
 #pragma unroll
-                for (int n = 0; n < NB; ++n) mma_u4(acc[n], ah[ks], bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+                for (int n = 0; n < NB; ++n) mma_u4(acc[n], ah, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
 #pragma unroll
-                for (int n = 0; n < NB; ++n) mma_u4(low[n], al[ks], bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+                for (int n = 0; n < NB; ++n) mma_u4(low[n], al, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
 #pragma unroll
-                for (int n = 0; n < NB; ++n) mma_u4(low[n], ah[ks], bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
+                for (int n = 0; n < NB; ++n) mma_u4(low[n], ah, bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
             }
         }
-        if (c + 1 < chunks) fetch_first(c + 1);
         if (owner) {                                   // u^T, split
 #pragma unroll
             for (int n = 0; n < NB; ++n) {
@@ -742,7 +756,9 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
             }
             if (c + 1 < chunks) fetch_base(c + 1);
         }
-        __syncthreads();                               // u is there; the state tiles have been read
+        __syncthreads();                               // u is there; W, q and the state tiles have been read
+        if (threadIdx.x == 0 && c + 1 < chunks && ok) load(2 * c + 3);
+        if (ok) ok = mbar_wait(&bar[(2 * c + 1) % 3], (uint32_t)(((2 * c + 1) / 3) & 1), P.status);
         if (owner) {
 #pragma unroll
             for (int m = 0; m < MT; ++m)
@@ -753,6 +769,9 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
 #pragma unroll
             for (int ks = 0; ks < CH / 16; ++ks) {
                 uint32_t a[MT][4], b[MT][4];
+                uint4 kh[NT / 2], kl[NT / 2];
+#pragma unroll
+                for (int n = 0; n < NT / 2; ++n) { kh[n] = lds_frag(ka, (d0 / 16 + n) * 4 + ks, lane); kl[n] = lds_frag(ka + L::TILE, (d0 / 16 + n) * 4 + ks, lane); }
 #pragma unroll
                 for (int m = 0; m < MT; ++m) { fa::load_a<CH>(uh, m * 16, ks, a[m]); fa::load_a<CH>(ul, m * 16, ks, b[m]); }
 #pragma unroll
@@ -761,7 +780,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                     for (int m = 0; m < MT; ++m)
 #pragma unroll
                         for (int n = 0; n < NT; ++n) {
-                            const uint4& w = k == 2 ? kl[n / 2 * 4 + ks] : kh[n / 2 * 4 + ks];
+                            const uint4& w = k == 2 ? kl[n / 2] : kh[n / 2];
                             fa::mma16816(X[m][n], k == 1 ? b[m] : a[m], (n & 1) ? w.z : w.x, (n & 1) ? w.w : w.y);
                         }
             }
@@ -770,15 +789,16 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
 #pragma unroll
             for (int ks = 0; ks < CH / 16; ++ks)
                 if (ks <= rb) {
+                    const uint4 kh = lds_frag(ka + 2 * L::TILE, rb * 4 + ks, lane), kl = lds_frag(ka + 2 * L::TILE + L::ATILE, rb * 4 + ks, lane);
                     uint32_t bh[MT][4], bl[MT][4];
 #pragma unroll
                     for (int n = 0; n < MT; ++n) { fa::load_b<CH>(uh, n * 16, ks, bh[n]); fa::load_b<CH>(ul, n * 16, ks, bl[n]); }
 #pragma unroll
-                    for (int n = 0; n < NB; ++n) mma_u4(acc[n], kh[ks], bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+                    for (int n = 0; n < NB; ++n) mma_u4(acc[n], kh, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
 #pragma unroll
-                    for (int n = 0; n < NB; ++n) mma_u4(low[n], kl[ks], bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+                    for (int n = 0; n < NB; ++n) mma_u4(low[n], kl, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
 #pragma unroll
-                    for (int n = 0; n < NB; ++n) mma_u4(low[n], kh[ks], bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
+                    for (int n = 0; n < NB; ++n) mma_u4(low[n], kh, bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
                 }
 #pragma unroll
             for (int n = 0; n < NB; ++n)
@@ -795,16 +815,19 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                     }
                 }
         }
-        __syncthreads();                               // the new state is there; u has been read
+        __syncthreads();                               // the new state is there; k, A and u have been read
+        if (threadIdx.x == 0 && c + 2 < chunks && ok) load(2 * c + 4);
     }
-    if (owner) each_state([&](float& x, int v, int d) { if (v < Dv && d < D) st[(size_t)d * Dv + v] = x; });
+    if (owner) each_state([&](float& x, int v, int d) { if (ok && v < Dv && d < D) st[(size_t)d * Dv + v] = x; });
 }
 
 template <int DT, int VS>
 static int launch_state(const Params& p, cudaStream_t st) {
     const dim3 grid((p.P.Dv + VS - 1) / VS, p.P.H, p.P.n_seqs);
     auto kern = p.P.delta ? chunk_state_kernel<DT, VS, true> : chunk_state_kernel<DT, VS, false>;
-    PTB_CUDA_OK(ptb_launch(kern, grid, dim3(THREADS), 0, st, ptb_pdl_enabled(), p));
+    constexpr int smem = StateSmem<DT, VS>::TOTAL;
+    PTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    PTB_CUDA_OK(ptb_launch(kern, grid, dim3(THREADS), (size_t)smem, st, ptb_pdl_enabled(), p));
     return 0;
 }
 
