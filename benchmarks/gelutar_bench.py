@@ -5,8 +5,8 @@ kernel of Llama with the fraction of the roofline both reach.
 
 Random bf16 weights, random prompts.  A Gelutar model here alternates one parallel layer (window attention with the heads of the
 Llama model beside a delta rule with as many heads) with three lightning layers of the same heads; its two-matrix feed-forward is half
-as wide again, so the feed-forwards have the same parameters.  Engine: prompt passes and decode steps timed with CUDA events, the second
-of two identical repetitions.  Kernels: a CUDA graph of launches over rotating inputs that together exceed L2, time per launch from the
+as wide again, so the feed-forwards have the same parameters.  Engine: prompt passes and decode steps timed with CUDA events, the last
+of three identical repetitions (capturing the graphs of the first empties the allocator's cache, which the second refills).  Kernels: a CUDA graph of launches over rotating inputs that together exceed L2, time per launch from the
 median of its replays; `roof` is the slower of bytes over the measured copy bandwidth and FLOPs over the measured bf16 matrix
 throughput, and `frac` is roof / time.  One JSON object on the last line."""
 from __future__ import annotations
@@ -179,7 +179,7 @@ def main(argv=None):
                 weights = make(cfg, seed=0, dtype=torch.bfloat16, device="cuda")
                 for load in a.loads.split(","):
                     B, T, new = (int(x) for x in load.split("x"))
-                    pre, dec, ms = engine_rates(weights, B, T, new)
+                    pre, dec, ms = engine_rates(weights, B, T, new, reps=3)
                     res["engine"].append({"size": size, "model": name, "parameters": weights.num_parameters(), "batch": B, "prompt": T, "prefill_tok_s": pre,
                                           "decode_tok_s": dec, "decode_ms": ms})
                     print(res["engine"][-1], flush=True)

@@ -50,13 +50,13 @@ def llama_cfg(z):
                        num_attention_heads=z["heads"], num_key_value_heads=z["kv"], max_position_embeddings=8192, eos_token_id=-1)
 
 
-def engine_rates(weights, batch, prompt, new):
-    """(prompt tokens/s, decode tokens/s, ms per decode step)."""
+def engine_rates(weights, batch, prompt, new, reps=2):
+    """(prompt tokens/s, decode tokens/s, ms per decode step) of the last of ``reps`` identical repetitions."""
     eng = LLMEngine(device="cuda", max_pages=batch * ((prompt + new) // 64 + 2), max_active=batch)
     eng.set_weights(weights)
     g = torch.Generator().manual_seed(0)
     cfg = GenerationConfig(max_new_tokens=new, temperature=0.0, repetition_penalty=1.0, top_k=1)
-    for rep in range(2):
+    for rep in range(reps):
         for i in range(batch):
             eng.submit_request(Request(rep * batch + i, torch.randint(3, VOCAB, (prompt,), generator=g).tolist(), cfg))
         e = [torch.cuda.Event(enable_timing=True) for _ in range(3)]
