@@ -6,9 +6,9 @@ kernel of Llama with the fraction of the roofline both reach.
 Random bf16 weights, random prompts.  A Gelutar model here alternates one parallel layer (window attention with the heads of the
 Llama model beside a delta rule with as many heads) with three lightning layers of the same heads; its two-matrix feed-forward is half
 as wide again, so the feed-forwards have the same parameters.  Engine: prompt passes and decode steps timed with CUDA events, the last
-of three identical repetitions (capturing the graphs of the first empties the allocator's cache, which the second refills).  Kernels: a CUDA graph of launches over rotating inputs that together exceed L2, time per launch from the
-median of its replays; `roof` is the slower of bytes over the measured copy bandwidth and FLOPs over the measured bf16 matrix
-throughput, and `frac` is roof / time.  One JSON object on the last line."""
+of three identical repetitions (capturing the graphs of the first empties the allocator's cache, which the second refills).  Kernels: a
+CUDA graph of launches over rotating inputs that together exceed L2, time per launch from the median of its replays; `roof` is the slower
+of bytes over the measured copy bandwidth and FLOPs over the measured bf16 matrix throughput, and `frac` is roof / time.  One JSON object on the last line."""
 from __future__ import annotations
 
 import argparse
