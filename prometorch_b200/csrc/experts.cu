@@ -1,0 +1,280 @@
+// A mixture of experts for inference, the parts that take any size:
+//   route_kernel        a warp per token: sigmoid scores, the `top` experts with the largest corrected scores, their weights, and the
+//                       token's rank among an expert's rows (counted in shared memory, then once per CTA and expert in global memory);
+//   place_kernel        prefix sums of the counts: the place of every (token, expert) pair in the order by expert, and back;
+//   route_small_kernel  both for few tokens in one CTA;
+//   expert_simt_kernel  a grouped product over the sorted rows with FMAs in fp32 (fp32 models, sizes the tensor-core kernel cannot address).
+// Where a row lies inside its expert depends on the order of atomics; what is computed for it does not.
+#include "common.cuh"
+#include <algorithm>
+
+namespace ptb {
+namespace moe {
+
+constexpr int RT_WARPS = 8, RS_WARPS = 32, SMALL_TOKENS = 64;
+
+struct Route {
+    const float* z;                    // [splits][n] rows of pitch ld
+    int splits;
+    long long stride, ld;
+    const float* correction;           // [E]
+    int n, E, top;
+    float scale;
+    int* index;                        // [n][top] out: place in the order by expert
+    float* weight;                     // [n][top] out
+    int* token;                        // [n top] out
+    int* offsets;                      // [E + 1] out
+    int* expert;                       // [n][top] between the kernels
+    int* rank;                         // [n][top]
+    int* counts;                       // [E], zero at the start
+    int* status;
+};
+
+// One warp: choice scores of token i into c_s, its `top` experts in order to (e, w) by lane 0 of the callback.
+template <typename F>
+__device__ __forceinline__ void choose(const Route& R, int i, float* c_s, F chosen) {
+    const int lane = threadIdx.x & 31;
+    for (int e = lane; e < R.E; e += 32) {
+        float z = 0.f;
+        for (int s = 0; s < R.splits; ++s) z += R.z[s * R.stride + (size_t)i * R.ld + e];
+        c_s[e] = sigmoid(z) + R.correction[e];
+    }
+    __syncwarp();
+    float sum = 0.f, mine = 0.f;                       // lane k keeps the score of the k-th expert (and of k + 32, ... in turn)
+    for (int k = 0; k < R.top; ++k) {
+        float best = -INFINITY;
+        int at = R.E;
+        for (int e = lane; e < R.E; e += 32)
+            if (c_s[e] > best) { best = c_s[e]; at = e; }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float b = __shfl_xor_sync(0xffffffffu, best, o);
+            const int a = __shfl_xor_sync(0xffffffffu, at, o);
+            if (b > best || (b == best && a < at)) { best = b; at = a; }
+        }
+        if (at >= R.E) at = k;                         // scores that are not numbers: any expert will do
+        float z = 0.f;
+        for (int s = 0; s < R.splits; ++s) z += R.z[s * R.stride + (size_t)i * R.ld + at];
+        const float score = sigmoid(z);
+        sum += score;
+        if (lane == (k & 31)) mine = score;
+        __syncwarp();
+        if (lane == 0) {
+            c_s[at] = -INFINITY;
+            chosen(k, at);
+        }
+        __syncwarp();
+        if ((k & 31) == 31 || k + 1 == R.top) {        // unscaled for now: the sum is not known before the last
+            const int k0 = k & ~31;
+            if (k0 + lane <= k) R.weight[(size_t)i * R.top + k0 + lane] = mine;
+        }
+    }
+    const float f = R.scale / (sum + 1e-20f);
+    __syncwarp();
+    for (int k = lane; k < R.top; k += 32) R.weight[(size_t)i * R.top + k] *= f;
+}
+
+__global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const __grid_constant__ Route R) {
+    extern __shared__ float smem[];
+    const int warp = threadIdx.x >> 5;
+    float* c_s = smem + warp * R.E;
+    int* count = reinterpret_cast<int*>(smem + RT_WARPS * R.E);
+    int* base = count + R.E;
+    for (int e = threadIdx.x; e < R.E; e += blockDim.x) count[e] = 0;
+    pdl_wait();
+    pdl_launch_dependents();
+    __syncthreads();
+    const int i = blockIdx.x * RT_WARPS + warp;
+    if (i < R.n)
+        choose(R, i, c_s, [&](int k, int e) {
+            R.expert[(size_t)i * R.top + k] = e;
+            R.rank[(size_t)i * R.top + k] = atomicAdd(&count[e], 1);
+        });
+    __syncthreads();
+    for (int e = threadIdx.x; e < R.E; e += blockDim.x) base[e] = count[e] ? atomicAdd(&R.counts[e], count[e]) : 0;
+    __syncthreads();
+    if (i < R.n)
+        for (int k = threadIdx.x & 31; k < R.top; k += 32) {
+            const size_t p = (size_t)i * R.top + k;
+            R.rank[p] += base[R.expert[p]];
+        }
+}
+
+// Exclusive sums of count[0 .. E) to off[0 .. E], by the first warp.
+__device__ __forceinline__ void prefix(const int* count, int* off, int E) {
+    if (threadIdx.x < 32) {
+        int run = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int e = e0 + threadIdx.x, v = e < E ? count[e] : 0;
+            int s = v;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int t = __shfl_up_sync(0xffffffffu, s, o);
+                if ((int)threadIdx.x >= o) s += t;
+            }
+            if (e < E) off[e] = run + s - v;
+            run += __shfl_sync(0xffffffffu, s, 31);
+        }
+        if (threadIdx.x == 0) off[E] = run;
+    }
+}
+
+__global__ void __launch_bounds__(256) place_kernel(const __grid_constant__ Route R) {
+    extern __shared__ int off[];
+    pdl_wait();
+    pdl_launch_dependents();
+    prefix(R.counts, off, R.E);
+    __syncthreads();
+    if (blockIdx.x == 0)
+        for (int e = threadIdx.x; e <= R.E; e += blockDim.x) R.offsets[e] = off[e];
+    const long long total = (long long)R.n * R.top;
+    for (long long p = (long long)blockIdx.x * blockDim.x + threadIdx.x; p < total; p += (long long)gridDim.x * blockDim.x) {
+        const int at = off[R.expert[p]] + R.rank[p];
+        R.index[p] = at;
+        R.token[at] = (int)(p / R.top);
+    }
+}
+
+__global__ void __launch_bounds__(RS_WARPS * 32) route_small_kernel(const __grid_constant__ Route R) {
+    extern __shared__ float smem[];
+    const int warp = threadIdx.x >> 5;
+    float* c_s = smem + warp * R.E;
+    int* count = reinterpret_cast<int*>(smem + RS_WARPS * R.E);
+    int* off = count + R.E;
+    for (int e = threadIdx.x; e < R.E; e += blockDim.x) count[e] = 0;
+    pdl_wait();
+    pdl_launch_dependents();
+    __syncthreads();
+    for (int i = warp; i < R.n; i += RS_WARPS)
+        choose(R, i, c_s, [&](int k, int e) {
+            R.expert[(size_t)i * R.top + k] = e;
+            R.rank[(size_t)i * R.top + k] = atomicAdd(&count[e], 1);
+        });
+    __syncthreads();
+    prefix(count, off, R.E);
+    __syncthreads();
+    for (int e = threadIdx.x; e <= R.E; e += blockDim.x) R.offsets[e] = off[e];
+    for (int p = threadIdx.x; p < R.n * R.top; p += blockDim.x) {
+        const int at = off[R.expert[p]] + R.rank[p];
+        R.index[p] = at;
+        R.token[at] = p / R.top;
+    }
+}
+
+// ---------------------------------------------------------------------------------------------- grouped product, any size
+constexpr int ST_M = 32, ST_N = 64, ST_K = 32;
+
+template <typename T> __device__ __forceinline__ float f32_of(T v) { return (float)v; }
+
+// 32 sorted rows of one expert x 64 output columns per CTA; GATED: B has gate rows [0, N) and up rows [N, 2 N).
+template <typename T, bool GATED>
+__global__ void __launch_bounds__(256) expert_simt_kernel(const T* __restrict__ a, const int* __restrict__ token, long long lda, const T* __restrict__ b,
+                                                          T* __restrict__ out, const int* __restrict__ offsets, int rows, int E, int N, int K) {
+    __shared__ float as[ST_K][ST_M + 1], gs[ST_K][ST_N + 1], us[GATED ? ST_K : 1][ST_N + 1];
+    __shared__ int where[3];
+    pdl_wait();
+    pdl_launch_dependents();
+    if (threadIdx.x == 0) {                            // the expert and the rows of tile blockIdx.y
+        int t = blockIdx.y;
+        where[0] = -1;
+        for (int e = 0; e < E; ++e) {
+            const int lo = offsets[e], hi = offsets[e + 1], tiles = (hi - lo + ST_M - 1) / ST_M;
+            if (t < tiles) { where[0] = e; where[1] = lo + t * ST_M; where[2] = min(hi, lo + (t + 1) * ST_M); break; }
+            t -= tiles;
+        }
+    }
+    __syncthreads();
+    const int e = where[0], r0 = where[1], r1 = min(where[2], rows), n0 = blockIdx.x * ST_N;
+    if (e < 0) return;
+    const T* be = b + (size_t)e * (GATED ? 2 : 1) * N * K;
+    const int tx = threadIdx.x & 31, ty = threadIdx.x >> 5;            // columns tx, tx + 32; rows ty + 8 i
+    float g[4][2], u[4][2];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) g[i][j] = u[i][j] = 0.f;
+    for (int k0 = 0; k0 < K; k0 += ST_K) {
+        for (int i = threadIdx.x; i < ST_M * ST_K; i += 256) {
+            const int r = i / ST_K, k = k0 + i % ST_K;
+            float v = 0.f;
+            if (r0 + r < r1 && k < K) v = f32_of<T>(a[(size_t)(token ? token[r0 + r] : r0 + r) * lda + k]);
+            as[i % ST_K][r] = v;
+        }
+        for (int i = threadIdx.x; i < ST_N * ST_K; i += 256) {
+            const int n = n0 + i / ST_K, k = k0 + i % ST_K;
+            const bool in = n < N && k < K;
+            gs[i % ST_K][i / ST_K] = in ? f32_of<T>(be[(size_t)n * K + k]) : 0.f;
+            if constexpr (GATED) us[i % ST_K][i / ST_K] = in ? f32_of<T>(be[(size_t)(N + n) * K + k]) : 0.f;
+        }
+        __syncthreads();
+#pragma unroll 8
+        for (int k = 0; k < ST_K; ++k)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float x = as[k][ty + 8 * i];
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+                    g[i][j] = fmaf(x, gs[k][tx + 32 * j], g[i][j]);
+                    if constexpr (GATED) u[i][j] = fmaf(x, us[k][tx + 32 * j], u[i][j]);
+                }
+            }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const int r = r0 + ty + 8 * i, n = n0 + tx + 32 * j;
+            if (r < r1 && n < N) out[(size_t)r * N + n] = (T)(GATED ? silu(g[i][j]) * u[i][j] : g[i][j]);
+        }
+}
+
+}  // namespace moe
+}  // namespace ptb
+
+using namespace ptb;
+
+// Routing of n tokens: z [splits][n] fp32 logits (rows of pitch ld, splits `stride` apart), correction [E].  index [n, top]: the place of a
+// token's i-th expert in the order by expert; weight [n, top]: its score over the sum of the chosen ones, times scale; token [n top]: the
+// token of every place; offsets [E + 1].  work: 2 n top + E ints.
+PTB_API int ptb_expert_route(const float* z, int splits, long long stride, long long ld, const float* correction, int n, int E, int top, float scale, int* index,
+                             float* weight, int* token, int* offsets, int* work, int* status, cudaStream_t st) {
+    using namespace ptb::moe;
+    if (n <= 0) return 0;
+    if (E < 1 || top < 1 || top > E || E > 1024) { ptb_set_error("experts: %d of %d experts (at most 1024)", top, E); return -1; }
+    const size_t pairs = (size_t)n * top;
+    Route r{z, splits, stride, ld, correction, n, E, top, scale, index, weight, token, offsets, work, work + pairs, work + 2 * pairs, status};
+    const bool pdl = ptb_pdl_enabled();
+    if (n <= SMALL_TOKENS && E <= 256) {
+        const size_t smem = ((size_t)RS_WARPS * E + 2 * E + 1) * 4;
+        if (smem > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(route_small_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024));
+        PTB_CUDA_OK(ptb_launch(route_small_kernel, dim3(1), dim3(RS_WARPS * 32), smem, st, pdl, r));
+    } else {
+        PTB_CUDA_OK(cudaMemsetAsync(r.counts, 0, (size_t)E * 4, st));
+        PTB_CUDA_OK(ptb_launch(route_kernel, dim3((n + RT_WARPS - 1) / RT_WARPS), dim3(RT_WARPS * 32), ((size_t)RT_WARPS * E + 2 * E) * 4, st, false, r));
+        PTB_CUDA_OK(ptb_launch(place_kernel, dim3((unsigned)std::min<size_t>(1024, (pairs + 255) / 256)), dim3(256), (size_t)(E + 1) * 4, st, pdl, r));
+    }
+    PTB_CUDA_OK(cudaGetLastError());
+    return 0;
+}
+
+// out [rows, N] = A_e B_e^T for the rows of every expert e (offsets [E + 1]), in fp32 arithmetic; `gated`: B_e has 2 N rows and the result is
+// silu(gate) * up.  Row r of A is a[token[r]] (token null: a[r]), pitch lda.  bf16 or fp32 operands and result.
+PTB_API int ptb_expert_gemm_simt(const void* a, const int* token, long long lda, const void* b, int gated, void* out, const int* offsets, int rows, int E, int N,
+                                 int K, int bf16, int* status, cudaStream_t st) {
+    using namespace ptb::moe;
+    (void)status;
+    if (rows <= 0 || N <= 0 || K <= 0) return 0;
+    const long long tiles = std::min<long long>((long long)rows, rows / ST_M + E);
+    if (tiles > 65535) { ptb_set_error("experts: %d rows in one launch", rows); return -1; }
+    const dim3 grid((N + ST_N - 1) / ST_N, (unsigned)tiles);
+    const bool pdl = ptb_pdl_enabled();
+    auto go = [&](auto k, auto t) {
+        using T = decltype(t);
+        return ptb_launch(k, grid, dim3(256), 0, st, pdl, (const T*)a, token, lda, (const T*)b, (T*)out, offsets, rows, E, N, K);
+    };
+    if (bf16) PTB_CUDA_OK(gated ? go(expert_simt_kernel<__nv_bfloat16, true>, __nv_bfloat16()) : go(expert_simt_kernel<__nv_bfloat16, false>, __nv_bfloat16()));
+    else PTB_CUDA_OK(gated ? go(expert_simt_kernel<float, true>, 0.f) : go(expert_simt_kernel<float, false>, 0.f));
+    PTB_CUDA_OK(cudaGetLastError());
+    return 0;
+}

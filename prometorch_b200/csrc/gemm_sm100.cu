@@ -57,6 +57,24 @@ int ptb_make_tmap_bf16_3d(CUtensorMap* map, const void* base, long long n0, long
     return 0;
 }
 
+// 4-D bf16 tensor map: extents n[0] (contiguous) .. n[3], pitches of the outer three in elements, box sizes.
+int ptb_make_tmap_bf16_4d(CUtensorMap* map, const void* base, const long long* n, const long long* strides, const int* box) {
+    EncodeTiledFn enc = get_encode();
+    if (!enc) { ptb_set_error("cuTensorMapEncodeTiled is not available (no CUDA driver?)"); return -1; }
+    cuuint64_t dims[4], st[3];
+    cuuint32_t b[4], estr[4] = {1, 1, 1, 1};
+    for (int i = 0; i < 4; ++i) { dims[i] = (cuuint64_t)n[i]; b[i] = (cuuint32_t)box[i]; }
+    for (int i = 0; i < 3; ++i) {
+        st[i] = (cuuint64_t)strides[i] * 2;
+        if (st[i] & 15) { ptb_set_error("TMA operand needs 16-byte aligned pitches (%lld elements)", strides[i]); return -1; }
+    }
+    if ((uintptr_t)base & 15) { ptb_set_error("TMA operand needs a 16-byte aligned base"); return -1; }
+    CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, st, b, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) { ptb_set_error("cuTensorMapEncodeTiled failed with code %d", (int)r); return -1; }
+    return 0;
+}
+
 template <int BN, int STAGES, bool A_MN, bool B_MN>
 static int launch(const Operand& ta, const Operand& tb, const Params& p, int n_sm, cudaStream_t st) {
     auto kern = gemm_bf16_kernel<BN, STAGES, A_MN, B_MN>;

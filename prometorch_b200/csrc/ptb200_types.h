@@ -70,14 +70,14 @@ typedef struct PtbRecurrence {
     long long ld;
     int q_col, k_col, v_col;
     int silu;               // decay attention: q, k and v pass SiLU first
-    int delta;              // 1: gated delta rule; 0: decay attention (G == H)
+    int delta;              // 1: gated delta rule, decays per key channel; 2: one decay per head; 0: decay attention (G == H)
     int bf16;
     const void* beta;       // delta: [n][H] of pitch ld_beta in the type of x, before the sigmoid
     long long ld_beta;
-    const float* a;         // delta: [n][H D] of pitch ld_a
+    const void* a;          // delta 1: fp32 [n][H D] of pitch ld_a; delta 2: [n][H] of pitch ld_a in the type of x
     long long ld_a;
     const float* decay;     // [H]: the decay, or exp(A_log)
-    const float* dt_bias;   // delta: [H D]
+    const float* dt_bias;   // delta 1: [H D]; delta 2: [H]
     float* state;           // [slots][H][D][Dv]
     int slots, n, H, G, D, Dv;
     const void* seqs;       // [n_seqs] int4 (first row, rows, position of the first, slot); null: one token per row
@@ -93,3 +93,50 @@ typedef struct PtbRecurrence {
     long long ld_low;
     const void* low_w;      // [H D][rank], bf16
 } PtbRecurrence;
+
+// Softmax attention over the paged cache (window_attn.cuh has the meaning of the mask and of the two maps).
+typedef struct PtbWindowAttn {
+    const void* q;          // [n][H maps][Dp]
+    void* out;              // [n][H Dv]
+    const void* k_pages;    // [pages][G][64][maps Dp]
+    const void* v_pages;    // [pages][G][64] rows of v_ld, of which Dvp are read (the latent cache: the same rows as the keys)
+    const int* page_table;
+    const int* pos;         // rows: [n] of pos_stride
+    const int* req;         // rows: [n] of req_stride, rows of the page table
+    const float* sink;      // [H] or null
+    const void* gate;       // [n][H] of pitch gate_ld, in the type of q, or null
+    long long gate_ld;
+    float* work;            // rows: ptb_window_rows_work_floats(n, H maps, Dvp, nsplit) floats where nsplit or maps is above one
+    int* status;
+    const void* tiles;      // tiles: [n_tiles] int4 (first row, its position, rows <= 128, row of the page table or first row of the flat context)
+    const void* k_rot;      // flat: the rotated key part that all heads share, rows of rot_ld
+    long long k_ld, v_row, rot_ld;      // flat: pitches of the context's rows in k_pages ([rows][H][Dp]), v_pages ([rows][H][Dvp]) and k_rot
+    int n, H, G, D, Dp, Dv, Dvp, v_ld, maps;
+    int pos_stride, req_stride, pt_stride, n_pages;
+    int window, keep, chunked;
+    int max_keys, nsplit, bf16;
+    int n_tiles, flat_rows, rot_dim;    // flat_rows > 0: keys and values lie flat, flat_rows of them; q is [n][H][Dq], see ptb_window_attn_tiles
+    float scale, mix, mix_gain, mix_eps;
+} PtbWindowAttn;
+
+// What stands between two sublayers of a decoder with elementwise tanh norms: x += post(y); x += table[ids]; out = pre(x).
+typedef struct PtbTanhResidual {
+    float* x;               // [n][W]
+    const void* y;          // bf16 (f32 = 0) or the sum of `splits` fp32 matrices `stride` apart; rows of pitch ld
+    int f32, splits;
+    long long stride, ld;
+    const int* index;       // [n][top] rows of y, summed with `weight` [n][top]; null: row i is y's row i
+    const float* weight;
+    int top, y_rows;
+    float post_alpha, pre_alpha;
+    const float* post_w;
+    const float* post_b;
+    const float* pre_w;     // null: no out
+    const float* pre_b;
+    const int* ids;         // [n] of id_stride, or null
+    int id_stride, V;
+    const void* table;      // [V][W] in the type of out
+    void* out;              // [n][W] bf16 or fp32
+    int n, W, bf16, pad;
+    int* status;
+} PtbTanhResidual;

@@ -3,7 +3,7 @@
 //   recurrence_kernel                      one CTA per (32 value columns, head, sequence); the state stays in registers from the first
 //                                          token to the last.  One token per sequence in a decode pass, every token of a prompt in
 //                                          true fp32 arithmetic (recurrence_chunk.cu has the matrix form for bf16 prompts);
-//   group_norm_gate_kernel                 RMS norm of groups of columns, weight, sigmoid gate.
+//   group_norm_gate_kernel                 RMS norm of groups of columns, weight, sigmoid or SiLU gate.
 // A slot outside its extent sets PTB_ERR_BOUNDS and its sequence is skipped.
 #include "recurrence.cuh"
 #include <algorithm>
@@ -190,9 +190,11 @@ constexpr int RC_THREADS = 256, RC_WARPS = 8, RC_COLS = 32;
 
 // Thread (tx, ty): value columns v0 + 4 tx .. + 3, state rows ty, ty + 32, ...  One barrier per token: the next token's vectors are
 // staged, and this token's partial sums left, in buffers that alternate.
-template <typename T, bool DELTA, int RM>
+// MODE: `delta` of PtbRecurrence.
+template <typename T, int MODE, int RM>
 __global__ void __launch_bounds__(RC_THREADS) recurrence_kernel(const __grid_constant__ PtbRecurrence P) {
-    __shared__ float q_s[3][RM * 32], k_s[3][RM * 32], g_s[3][RM * 32];      // three: a slow warp may still update with the token before
+    constexpr bool DELTA = MODE != 0;
+    __shared__ float q_s[3][RM * 32], k_s[3][RM * 32], g_s[3][MODE == 1 ? RM * 32 : 1];      // three: a slow warp may still update with the token before
     __shared__ float red_s[2][RC_WARPS][4];
     __shared__ float4 part_s[2][RC_WARPS][8][2];
     pdl_wait();
@@ -228,14 +230,16 @@ __global__ void __launch_bounds__(RC_THREADS) recurrence_kernel(const __grid_con
             if (d < D) {
                 q = rc_f<T>(row[P.q_col + hk * D + d]);
                 k = rc_f<T>(row[P.k_col + hk * D + d]);
-                if constexpr (DELTA) g = expf(delta_log_decay(P.a[(size_t)(s.row0 + i) * P.ld_a + h * D + d], P.dt_bias[h * D + d], rate));
-                else if (P.silu) { q = silu(q); k = silu(k); }
+                if constexpr (MODE == 1) g = expf(delta_log_decay(((const float*)P.a)[(size_t)(s.row0 + i) * P.ld_a + h * D + d], P.dt_bias[h * D + d], rate));
+                else if (MODE == 0 && P.silu) { q = silu(q); k = silu(k); }
             }
             q_s[b][d] = q; k_s[b][d] = k;
-            if constexpr (DELTA) g_s[b][d] = g;
+            if constexpr (MODE == 1) g_s[b][d] = g;
             qq += q * q; kk += k * k; qk += q * k;
         }
         qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
+        if constexpr (MODE == 2)
+            if (threadIdx.x == 0) g_s[b][0] = expf(delta_log_decay(rc_f<T>(((const T*)P.a)[(size_t)(s.row0 + i) * P.ld_a + h]), P.dt_bias[h], rate));
         if (lane == 0) { red_s[i & 1][warp][0] = qq; red_s[i & 1][warp][1] = kk; red_s[i & 1][warp][2] = qk; }
     };
     stage(0);
@@ -257,7 +261,7 @@ __global__ void __launch_bounds__(RC_THREADS) recurrence_kernel(const __grid_con
 #pragma unroll
         for (int j = 0; j < RM; ++j) {
             const int d = ty + 32 * j;
-            const float g = DELTA ? g_s[c][d] : rate, k = k_s[c][d], q = q_s[c][d];
+            const float g = MODE == 1 ? g_s[c][d] : MODE == 2 ? g_s[c][0] : rate, k = k_s[c][d], q = q_s[c][d];
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 S[j][e] *= g;
@@ -313,7 +317,7 @@ __global__ void __launch_bounds__(RC_THREADS) recurrence_kernel(const __grid_con
 // TPG threads per group of gs columns; with V = 4, gs and every pitch are multiples of four.
 template <typename T, typename TG, int TPG, int V>
 __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const TG* __restrict__ gate,
-                                                              long long ld_gate, T* __restrict__ out, long long groups, int per_row, int gs, float eps) {
+                                                              long long ld_gate, T* __restrict__ out, long long groups, int per_row, int gs, float eps, int act) {
     __shared__ float red[8];
     pdl_wait();
     pdl_launch_dependents();
@@ -345,32 +349,32 @@ __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __res
         const Elems<TG, V> g = ld_elems<TG, V>(gp + c);
         Elems<T, V> r;
 #pragma unroll
-        for (int e = 0; e < V; ++e) r.v[e] = f.v[e] * rs * m.v[e] * sigmoid(g.v[e]);
+        for (int e = 0; e < V; ++e) r.v[e] = f.v[e] * rs * m.v[e] * (act ? silu(g.v[e]) : sigmoid(g.v[e]));
         st_elems<T, V>(op + c, r);
     }
 }
 
 template <typename T, typename TG>
 static cudaError_t norm_gate_launch(const float* o, const float* w, const void* gate, long long ld_gate, void* out, long long n, int per_row, int gs,
-                                    float eps, bool vec, cudaStream_t st) {
+                                    float eps, int act, bool vec, cudaStream_t st) {
     const long long groups = n * per_row;
     auto go = [&](auto k, int tpg) {
         return ptb_launch(k, dim3((unsigned)((groups + 256 / tpg - 1) / (256 / tpg))), dim3(256), 0, st, ptb_pdl_enabled(), o, w, (const TG*)gate, ld_gate,
-                          (T*)out, groups, per_row, gs, eps);
+                          (T*)out, groups, per_row, gs, eps, act);
     };
     if (gs > 512) return vec ? go(group_norm_gate_kernel<T, TG, 256, 4>, 256) : go(group_norm_gate_kernel<T, TG, 256, 1>, 256);
     return vec ? go(group_norm_gate_kernel<T, TG, 32, 4>, 32) : go(group_norm_gate_kernel<T, TG, 32, 1>, 32);
 }
 
-template <typename T, bool DELTA>
+template <typename T, int MODE>
 static cudaError_t recurrence_launch(const PtbRecurrence& p, cudaStream_t st) {
     const dim3 grid((p.Dv + RC_COLS - 1) / RC_COLS, p.H, p.seqs ? p.n_seqs : p.n);
     auto go = [&](auto k) { return ptb_launch(k, grid, dim3(RC_THREADS), 0, st, ptb_pdl_enabled(), p); };
-    if (p.D <= 32) return go(recurrence_kernel<T, DELTA, 1>);
-    if (p.D <= 64) return go(recurrence_kernel<T, DELTA, 2>);
-    if (p.D <= 128) return go(recurrence_kernel<T, DELTA, 4>);
-    if (p.D <= 256) return go(recurrence_kernel<T, DELTA, 8>);
-    return go(recurrence_kernel<T, DELTA, 16>);
+    if (p.D <= 32) return go(recurrence_kernel<T, MODE, 1>);
+    if (p.D <= 64) return go(recurrence_kernel<T, MODE, 2>);
+    if (p.D <= 128) return go(recurrence_kernel<T, MODE, 4>);
+    if (p.D <= 256) return go(recurrence_kernel<T, MODE, 8>);
+    return go(recurrence_kernel<T, MODE, 16>);
 }
 
 int recurrence_check(const PtbRecurrence& p) {
@@ -421,23 +425,25 @@ PTB_API int ptb_recurrence(const PtbRecurrence* args, cudaStream_t st) {
     if (p.n <= 0 || (p.seqs && p.n_seqs <= 0)) return 0;
     if (recurrence_check(p)) return -1;
     if (p.delta && !p.a) { ptb_set_error("recurrence: token by token takes a, not its low-rank factors"); return -1; }
-    if (p.bf16) PTB_CUDA_OK((p.delta ? recurrence_launch<__nv_bfloat16, true> : recurrence_launch<__nv_bfloat16, false>)(p, st));
-    else PTB_CUDA_OK((p.delta ? recurrence_launch<float, true> : recurrence_launch<float, false>)(p, st));
+    if (p.delta < 0 || p.delta > 2) { ptb_set_error("recurrence: kind %d", p.delta); return -1; }
+    auto go = p.bf16 ? (p.delta == 2 ? recurrence_launch<__nv_bfloat16, 2> : p.delta ? recurrence_launch<__nv_bfloat16, 1> : recurrence_launch<__nv_bfloat16, 0>)
+                     : (p.delta == 2 ? recurrence_launch<float, 2> : p.delta ? recurrence_launch<float, 1> : recurrence_launch<float, 0>);
+    PTB_CUDA_OK(go(p, st));
     PTB_CUDA_OK(cudaGetLastError());
     return 0;
 }
 
-// out [n, per_row gs] (bf16 or fp32) = o / rms(o) * w * sigmoid(gate), o fp32 in groups of gs columns, w [gs] fp32, gate [n, per_row gs] with
+// out [n, per_row gs] (bf16 or fp32) = o / rms(o) * w * act(gate), act the sigmoid (0) or SiLU (1), o fp32 in groups of gs columns, w [gs] fp32, gate [n, per_row gs] with
 // row pitch ld_gate in bf16 (gate_bf16) or fp32.
 PTB_API int ptb_group_norm_gate(const float* o, const float* w, const void* gate, int gate_bf16, long long ld_gate, void* out, int n, int per_row,
-                                int gs, float eps, int bf16, cudaStream_t st) {
+                                int gs, float eps, int act, int bf16, cudaStream_t st) {
     if (n <= 0 || per_row <= 0 || gs <= 0) return 0;
     const bool vec = gs % 4 == 0 && ld_gate % 4 == 0 && (((uintptr_t)o | (uintptr_t)w | (uintptr_t)out | (uintptr_t)gate) & 15) == 0;
     cudaError_t e;
-    if (bf16) e = gate_bf16 ? norm_gate_launch<__nv_bfloat16, __nv_bfloat16>(o, w, gate, ld_gate, out, n, per_row, gs, eps, vec, st)
-                            : norm_gate_launch<__nv_bfloat16, float>(o, w, gate, ld_gate, out, n, per_row, gs, eps, vec, st);
-    else e = gate_bf16 ? norm_gate_launch<float, __nv_bfloat16>(o, w, gate, ld_gate, out, n, per_row, gs, eps, vec, st)
-                       : norm_gate_launch<float, float>(o, w, gate, ld_gate, out, n, per_row, gs, eps, vec, st);
+    if (bf16) e = gate_bf16 ? norm_gate_launch<__nv_bfloat16, __nv_bfloat16>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, vec, st)
+                            : norm_gate_launch<__nv_bfloat16, float>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, vec, st);
+    else e = gate_bf16 ? norm_gate_launch<float, __nv_bfloat16>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, vec, st)
+                       : norm_gate_launch<float, float>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, vec, st);
     PTB_CUDA_OK(e);
     PTB_CUDA_OK(cudaGetLastError());
     return 0;

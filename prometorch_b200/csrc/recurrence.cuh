@@ -1,6 +1,6 @@
 // Recurrent layers with a matrix state S [D, Dv] per head and sequence, fp32:
 //   decay attention   S <- decay_h S + k v^T;  o = S^T q
-//   gated delta rule  S <- g S (g per key channel);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+//   gated delta rule  S <- g S (g per key channel, or one number);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 // with g = exp(-rate_h softplus(a + dt_bias)), beta a sigmoid, q and k unit vectors (q also times D^-1/2).
 #pragma once
 #include "common.cuh"

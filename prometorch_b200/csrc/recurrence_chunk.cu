@@ -6,12 +6,15 @@
 // where u is v for decay attention.  For the delta rule (1 + B) u = beta (v - (k G)^T S) with B_ij = beta_i k_i . (k_j G_i / G_j) for
 // j < i (a unit lower triangular system, the UT transform of delta-rule attention), hence u = U - W S with U = (1 + B)^-1 beta v and
 // W = (1 + B)^-1 beta (k G).  Two kernels:
-//   delta_chunk_kernel / decay_chunk_kernel   everything that does not depend on S, all chunks at once, into a workspace;
+//   delta_chunk_kernel / delta_head_chunk_kernel / decay_chunk_kernel   everything that does not depend on S, all chunks at once, into a
+//                        workspace;
 //   chunk_state_kernel                        walks a sequence's chunks for a slice of value columns; S stays in registers.
 // What passes between them lies in the order of the mma fragments that will read it: a lane's 16 bytes are its four registers of a 16 x 16
 // block, so the walk takes an operand with one 16-byte load per lane.
 // Quotients of decays are never formed from products that could overflow: across blocks of 16 tokens both factors refer to the block
 // border between the two tokens and are at most 1, inside a block the exponent of every pair is taken directly.
+// One decay per head: the quotients are numbers per pair of tokens, so they scale products of the bf16 q and k as they are, and the walk
+// takes q and k unscaled, with a factor per row for the product with q and for u on its way into the state.
 // Products run on the tensor cores with every fp32 operand split into two bf16 numbers (three products: 16 bits of both operands).
 #include "recurrence.cuh"
 #include "flash_attn.cuh"
@@ -28,11 +31,13 @@ constexpr float MILD = -60.f;          // log2 of what a block of 16 tokens may 
 //   W, Q  left operands   [4 row blocks][DT / 16 column blocks]
 //   K     right operand   [DT / 16 blocks of key channels][4 blocks of tokens]
 //   A     left operand    [4 row blocks][4 column blocks], those above the diagonal unused
+//   G     fp32            the decay of the whole chunk per key channel
 //   U     fp32            [Dvp / 16 column blocks][4 row blocks][2 halves of 8 columns][lane] the four accumulator registers
-template <int DT>
+// HEAD (one decay per head): Q and K have no low part, G is [chunk's decay, 3 unused, factor of every row of q (64), of u (64)].
+template <int DT, bool HEAD = false>
 struct Work {
-    static constexpr int TILE = CH * DT * 2, ATILE = CH * CH * 2;
-    static constexpr int W = 0, Q = 2 * TILE, K = 4 * TILE, A = 6 * TILE, G = A + 2 * ATILE, U = G + DT * 4;      // byte offsets
+    static constexpr int TILE = CH * DT * 2, ATILE = CH * CH * 2, PARTS = HEAD ? 1 : 2;
+    static constexpr int W = 0, Q = 2 * TILE, K = Q + PARTS * TILE, A = K + PARTS * TILE, G = A + 2 * ATILE, U = G + (HEAD ? 1024 : DT * 4);      // byte offsets
     static __host__ __device__ size_t bytes(int Dvp) { return (size_t)U + (size_t)CH * Dvp * 4; }
 };
 
@@ -105,6 +110,52 @@ __device__ __forceinline__ void load_rows(const PtbRecurrence& P, bool vec, int 
     }
 }
 
+// (1 + B)^-1 in place of the strictly lower B [64][PA]: the diagonal blocks by substitution (a lane owns a column), then block row after
+// block row.  tmp: 16 x 52 floats.  Starts and ends with all threads together.
+template <int PA>
+__device__ __forceinline__ void unit_lower_inverse(float* ak, float* tmp) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (warp < 4) {
+        float x[16];
+        float* b = ak + warp * 16 * PA + warp * 16;
+        if (lane < 16) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+                float v = i == lane ? 1.f : 0.f;
+#pragma unroll
+                for (int m = 0; m < i; ++m) v = fmaf(-b[i * PA + m], x[m], v);
+                x[i] = v;
+            }
+        }
+        __syncwarp();
+        if (lane < 16)
+#pragma unroll
+            for (int i = 0; i < 16; ++i) b[i * PA + lane] = x[i];
+    }
+    __syncthreads();
+    for (int s = 1; s < 4; ++s) {
+        const int i = threadIdx.x >> 4, c = threadIdx.x & 15;
+        const float* row = ak + (s * 16 + i) * PA;
+        for (int r = 0; r < s; ++r) {
+            float v = 0.f;
+            for (int m = r * 16; m < s * 16; m += 4) {
+                const float4 f = *reinterpret_cast<const float4*>(row + m);
+                const float* y = ak + m * PA + r * 16 + c;
+                v = fmaf(f.x, y[0], fmaf(f.y, y[PA], fmaf(f.z, y[2 * PA], fmaf(f.w, y[3 * PA], v))));
+            }
+            tmp[i * 52 + r * 16 + c] = v;
+        }
+        __syncthreads();
+        for (int r = 0; r < s; ++r) {
+            float v = 0.f;
+#pragma unroll
+            for (int m = 0; m < 16; ++m) v = fmaf(row[s * 16 + m], tmp[m * 52 + r * 16 + c], v);
+            ak[(s * 16 + i) * PA + r * 16 + c] = -v;
+        }
+        __syncthreads();
+    }
+}
+
 // ---------------------------------------------------------------------------------------------- delta rule, one chunk
 template <int DT>
 struct DeltaSmem {
@@ -160,12 +211,12 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
         for (int e = threadIdx.x; e < CH * DT / 4; e += THREADS) {
             const int r = e / (DT / 4), d = e % (DT / 4) * 4;
             const bool live = r < cnt && d < D;
-            fa::cp_async16(smem_u32(G_s + r * S::PG + d), P.a + (live ? (size_t)(row0 + r) * P.ld_a + h * D + d : 0), live);
+            fa::cp_async16(smem_u32(G_s + r * S::PG + d), (const float*)P.a + (live ? (size_t)(row0 + r) * P.ld_a + h * D + d : 0), live);
         }
     } else
         for (int e = threadIdx.x; e < CH * DT; e += THREADS) {
             const int r = e / DT, d = e % DT;
-            G_s[r * S::PG + d] = r < cnt && d < D ? P.a[(size_t)(row0 + r) * P.ld_a + h * D + d] : 0.f;
+            G_s[r * S::PG + d] = r < cnt && d < D ? ((const float*)P.a)[(size_t)(row0 + r) * P.ld_a + h * D + d] : 0.f;
         }
     fa::cp_async_commit();
     const float rate = P.decay[h] * LOG2E;
@@ -369,46 +420,7 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
     __syncthreads();
     load_rows(P, W.vec, row0, cnt, P.v_col + h * Dv, Dv, W.Dvp, v_s, PV);      // over q
     fa::cp_async_commit();
-    // ---- (1 + B)^-1 in place: the diagonal blocks by substitution (a lane owns a column), then block row after block row
-    if (warp < 4) {
-        float x[16];
-        float* b = ak + warp * 16 * S::PA + warp * 16;
-        if (lane < 16) {
-#pragma unroll
-            for (int i = 0; i < 16; ++i) {
-                float v = i == lane ? 1.f : 0.f;
-#pragma unroll
-                for (int m = 0; m < i; ++m) v = fmaf(-b[i * S::PA + m], x[m], v);
-                x[i] = v;
-            }
-        }
-        __syncwarp();
-        if (lane < 16)
-#pragma unroll
-            for (int i = 0; i < 16; ++i) b[i * S::PA + lane] = x[i];
-    }
-    __syncthreads();
-    for (int s = 1; s < 4; ++s) {
-        const int i = threadIdx.x >> 4, c = threadIdx.x & 15;
-        const float* row = ak + (s * 16 + i) * S::PA;
-        for (int r = 0; r < s; ++r) {
-            float v = 0.f;
-            for (int m = r * 16; m < s * 16; m += 4) {
-                const float4 f = *reinterpret_cast<const float4*>(row + m);
-                const float* y = ak + m * S::PA + r * 16 + c;
-                v = fmaf(f.x, y[0], fmaf(f.y, y[S::PA], fmaf(f.z, y[2 * S::PA], fmaf(f.w, y[3 * S::PA], v))));
-            }
-            tmp[i * 52 + r * 16 + c] = v;
-        }
-        __syncthreads();
-        for (int r = 0; r < s; ++r) {
-            float v = 0.f;
-#pragma unroll
-            for (int m = 0; m < 16; ++m) v = fmaf(row[s * 16 + m], tmp[m * 52 + r * 16 + c], v);
-            ak[(s * 16 + i) * S::PA + r * 16 + c] = -v;
-        }
-        __syncthreads();
-    }
+    unit_lower_inverse<S::PA>(ak, tmp);
     for (int e = threadIdx.x; e < CH * CH / 8; e += THREADS) {     // times beta, split
         const int r = e / 8, c = (e % 8) * 8;
         float f[8];
@@ -458,6 +470,197 @@ __global__ void __launch_bounds__(THREADS, 2) delta_chunk_kernel(const __grid_co
                         fa::mma16816(c[n], al, bh[ks][2 * n], bh[ks][2 * n + 1]);
                         fa::mma16816(c[n], ah, bh[ks][2 * n], bh[ks][2 * n + 1]);
                     }
+                }
+            }
+            if (is_w) {
+                const float2 x[4] = {make_float2(c[0][0], c[0][1]), make_float2(c[0][2], c[0][3]), make_float2(c[1][0], c[1][1]), make_float2(c[1][2], c[1][3])};
+                store_frag(out + L::W, L::TILE, rb * (DT / 16) + n0 / 16, lane, x);
+            } else {
+                float4* u = reinterpret_cast<float4*>(out + L::U) + ((n0 / 16) * 4 + rb) * 64 + lane;
+                u[0] = make_float4(c[0][0], c[0][1], c[0][2], c[0][3]);
+                u[32] = make_float4(c[1][0], c[1][1], c[1][2], c[1][3]);
+            }
+        }
+    }
+}
+
+// ---------------------------------------------------------------------------------------------- delta rule with one decay per head
+template <int DT>
+struct HeadSmem {
+    static constexpr int PB = DT + 8, PA = CH + 4;     // pitches of the bf16 tiles and of B
+    static constexpr int QB = CH * PB * 2 > CH * CH * 4 ? CH * PB * 2 : CH * CH * 4;         // q, and later the operand of W
+    static constexpr int K = 0, Q = K + CH * PB * 2, A = Q + QB, TH = A + CH * PA * 4, TL = TH + CH * CH * 2, TMP = TL + CH * CH * 2, ROW = TMP + 16 * 52 * 4;
+    static constexpr int V = ROW + 8 * CH * 4;
+    static __host__ __device__ int total(int Dvp) { return V + CH * (Dvp + 8) * 2; }
+};
+
+template <int DT>
+__global__ void __launch_bounds__(THREADS, 2) delta_head_chunk_kernel(const __grid_constant__ Params W) {
+    using S = HeadSmem<DT>;
+    using L = Work<DT, true>;
+    extern __shared__ __align__(128) unsigned char smem[];
+    __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem + S::Q);
+    __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem + S::K);
+    __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(smem + S::V);
+    float* ak = reinterpret_cast<float*>(smem + S::A);
+    float* tmp = reinterpret_cast<float*>(smem + S::TMP);
+    float* qn = reinterpret_cast<float*>(smem + S::ROW);           // per row: factors that make unit vectors,
+    float* kn = qn + CH;
+    float* bt = kn + CH;                                           // beta,
+    float* up = bt + CH;                                           // log2 of the decays of its block of 16 up to and with it,
+    float* rest = up + CH;                                         // and behind it
+    float* E = rest + CH;                                          // [4] of whole blocks; sums of four and fewer terms keep all their bits
+    const PtbRecurrence& P = W.P;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int h = blockIdx.y, D = P.D, Dv = P.Dv, hk = h / (P.H / P.G), PV = W.Dvp + 8;
+    const int4 chunk = reinterpret_cast<const int4*>(P.chunks)[blockIdx.x];
+    const int row0 = chunk.x, cnt = chunk.y;
+    if (row0 < 0 || cnt < 1 || cnt > CH || row0 + cnt > P.n) {
+        if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+        return;
+    }
+    unsigned char* out = W.work + ((size_t)blockIdx.x * P.H + h) * W.stride;
+    load_rows(P, W.vec, row0, cnt, P.q_col + hk * D, D, DT, q_s, S::PB);
+    load_rows(P, W.vec, row0, cnt, P.k_col + hk * D, D, DT, k_s, S::PB);
+    fa::cp_async_commit();
+    load_rows(P, W.vec, row0, cnt, P.v_col + h * Dv, Dv, W.Dvp, v_s, PV);
+    fa::cp_async_commit();
+    if (threadIdx.x < CH) {                            // two warps: a block of 16 tokens is half a warp
+        const int i = threadIdx.x;
+        const size_t r = (size_t)(row0 + (i < cnt ? i : 0));
+        bt[i] = i < cnt ? sigmoid(__bfloat162float(((const __nv_bfloat16*)P.beta)[r * P.ld_beta + h])) : 0.f;
+        // 2^-150 is 0
+        const float d = i < cnt ? fmaxf(-150.f, delta_log_decay(__bfloat162float(((const __nv_bfloat16*)P.a)[r * P.ld_a + h]), P.dt_bias[h], P.decay[h] * LOG2E)) : 0.f;
+        float a = d, b = d;
+#pragma unroll
+        for (int o = 1; o < 16; o <<= 1) {
+            const float x = __shfl_up_sync(0xffffffffu, a, o, 16), y = __shfl_down_sync(0xffffffffu, b, o, 16);
+            if ((i & 15) >= o) a += x;
+            if ((i & 15) + o < 16) b += y;
+        }
+        const float behind = __shfl_down_sync(0xffffffffu, b, 1, 16);
+        up[i] = a;
+        rest[i] = (i & 15) == 15 ? 0.f : behind;
+        if ((i & 15) == 15) E[i >> 4] = a;
+    }
+    fa::cp_async_wait<1>();
+    __syncthreads();
+    for (int r = warp; r < CH; r += WARPS) {
+        float a = 0.f, b = 0.f;
+        for (int d = lane * 2; d < DT; d += 64) {
+            const float2 x = unpack(*reinterpret_cast<const uint32_t*>(q_s + r * S::PB + d)), y = unpack(*reinterpret_cast<const uint32_t*>(k_s + r * S::PB + d));
+            a += x.x * x.x + x.y * x.y;
+            b += y.x * y.x + y.y * y.y;
+        }
+        a = warp_sum(a); b = warp_sum(b);
+        if (lane == 0) { qn[r] = rsqrtf(a + UNIT_EPS) * rsqrtf((float)D); kn[r] = rsqrtf(b + UNIT_EPS); }
+    }
+    // ---- q and k as they are, in fragment order
+    for (int f = warp; f < DT / 4; f += WARPS) {
+        const int rb = f / (DT / 16), ks = f % (DT / 16), dp = f >> 2, kt = f & 3;
+        uint32_t x[4];
+        fa::ldsm4(smem_u32(q_s + (rb * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * S::PB + ks * 16 + (lane >> 4) * 8), x[0], x[1], x[2], x[3]);
+        *reinterpret_cast<uint4*>(out + L::Q + ((size_t)f * 32 + lane) * 16) = make_uint4(x[0], x[1], x[2], x[3]);
+        fa::ldsm4_t(smem_u32(k_s + (kt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * S::PB + dp * 16 + (lane >> 4) * 8), x[0], x[1], x[2], x[3]);
+        *reinterpret_cast<uint4*>(out + L::K + ((size_t)f * 32 + lane) * 16) = make_uint4(x[0], x[1], x[2], x[3]);
+    }
+    __syncthreads();
+    if (threadIdx.x < CH) {
+        const int i = threadIdx.x, b = i >> 4;
+        float before = 0.f, after = 0.f;
+#pragma unroll
+        for (int r = 0; r < 4; ++r) { before += r < b ? E[r] : 0.f; after += r > b ? E[r] : 0.f; }
+        float* G = reinterpret_cast<float*>(out + L::G);
+        G[4 + i] = qn[i] * exp2f(up[i] + before);
+        G[4 + CH + i] = kn[i] * exp2f(rest[i] + after);
+        if (i == 0) G[0] = exp2f(E[0] + E[1] + E[2] + E[3]);
+    }
+    // ---- q . k and k . k in blocks of 16 x 16 up to the diagonal, scaled pair by pair
+    for (int unit = warp; unit < 10; unit += WARPS) {
+        const int s = unit < 1 ? 0 : unit < 3 ? 1 : unit < 6 ? 2 : 3, r = unit - s * (s + 1) / 2;
+        float cq[2][4], ck[2][4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) cq[n][e] = ck[n][e] = 0.f;
+#pragma unroll
+        for (int ks = 0; ks < DT / 16; ++ks) {
+            uint32_t q[4], k[4], b[4];
+            const int a_off = (s * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * S::PB + ks * 16 + (lane >> 4) * 8;
+            fa::ldsm4(smem_u32(q_s + a_off), q[0], q[1], q[2], q[3]);
+            fa::ldsm4(smem_u32(k_s + a_off), k[0], k[1], k[2], k[3]);
+            fa::ldsm4(smem_u32(k_s + (r * 16 + (lane & 7) + (lane >> 4) * 8) * S::PB + ks * 16 + ((lane >> 3) & 1) * 8), b[0], b[1], b[2], b[3]);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                fa::mma16816(cq[n], q, b[2 * n], b[2 * n + 1]);
+                fa::mma16816(ck[n], k, b[2 * n], b[2 * n + 1]);
+            }
+        }
+        float mid = 0.f;                               // whole blocks between the two
+        for (int m = r + 1; m < s; ++m) mid += E[m];
+        float2 x[4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int i = s * 16 + g + 8 * e, j = r * 16 + n * 8 + 2 * t;
+                float w[2];
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    const float d = s == r ? up[i] - up[j + c] : up[i] + mid + rest[j + c];
+                    w[c] = j + c <= i ? exp2f(d) * kn[j + c] : 0.f;
+                }
+                const float a = qn[i], b = kn[i] * bt[i];
+                x[n * 2 + e] = make_float2(cq[n][2 * e] * a * w[0], cq[n][2 * e + 1] * a * w[1]);
+                *reinterpret_cast<float2*>(ak + i * S::PA + j) = make_float2(j < i ? ck[n][2 * e] * b * w[0] : 0.f, j + 1 < i ? ck[n][2 * e + 1] * b * w[1] : 0.f);
+            }
+        store_frag(out + L::A, L::ATILE, s * 4 + r, lane, x);
+    }
+    __syncthreads();
+    unit_lower_inverse<S::PA>(ak, tmp);
+    // ---- times beta for U; times the factor of k's row as well, over q, for W
+    for (int e = threadIdx.x; e < CH * CH / 8; e += THREADS) {
+        const int r = e / 8, c = (e % 8) * 8;
+        float f[8], w[8], before = 0.f;
+        for (int m = 0; m < c / 16; ++m) before += E[m];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+            f[k] = c + k <= r ? ak[r * S::PA + c + k] * bt[c + k] : 0.f;
+            w[k] = f[k] * kn[c + k] * exp2f(up[c + k] + before);
+        }
+        store_split8<CH>(smem + S::TH, smem + S::TL, r, c, f);
+        store_split8<CH>(smem + S::Q, smem + S::Q + CH * CH * 2, r, c, w);
+    }
+    fa::cp_async_wait<0>();
+    __syncthreads();
+    for (int unit = warp; unit < DT / 16 + W.Dvp / 16; unit += WARPS) {        // W and U: units of 16 columns
+        const bool is_w = unit < DT / 16;
+        const int n0 = (is_w ? unit : unit - DT / 16) * 16;
+        const uint32_t th = smem_u32(smem + (is_w ? S::Q : S::TH)), tl = th + CH * CH * 2;
+        uint32_t b[4][4];
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) {
+            const __nv_bfloat16* p = is_w ? k_s + n0 : v_s + n0;
+            fa::ldsm4_t(smem_u32(p + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * (is_w ? S::PB : PV) + (lane >> 4) * 8), b[ks][0], b[ks][1], b[ks][2], b[ks][3]);
+        }
+#pragma unroll
+        for (int rb = 0; rb < 4; ++rb) {
+            float c[2][4];
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) c[n][e] = 0.f;
+#pragma unroll
+            for (int ks = 0; ks <= rb; ++ks) {
+                uint32_t ah[4], al[4];
+                fa::load_a<CH>(th, rb * 16, ks, ah);
+                fa::load_a<CH>(tl, rb * 16, ks, al);
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+                    fa::mma16816(c[n], al, b[ks][2 * n], b[ks][2 * n + 1]);
+                    fa::mma16816(c[n], ah, b[ks][2 * n], b[ks][2 * n + 1]);
                 }
             }
             if (is_w) {
@@ -600,16 +803,20 @@ __device__ __forceinline__ void mma_u4(float* d, const uint4& a, uint32_t b0, ui
 // the read-out; the state lives transposed, [value][key channel], in the accumulators of warps 0-3 and as two bf16 tiles in shared
 // memory for the products that read it.  The other operands arrive by bulk copies through three slots, in the order of their use: W and q
 // of a chunk, its k and A, W and q of the next, ...
-template <int DT, int VS>
+// With one decay per head (MODE 2) u enters the state times its row's factor, from a second pair of tiles.
+template <int DT, int VS, bool HEAD>
 struct StateSmem {
-    using L = Work<DT>;
-    static constexpr int SLOT = 4 * L::TILE > 2 * L::TILE + 2 * L::ATILE ? 4 * L::TILE : 2 * L::TILE + 2 * L::ATILE, SH = 3 * SLOT, SL = SH + VS * DT * 2;
-    static constexpr int UH = SL + VS * DT * 2, UL = UH + VS * CH * 2, BAR = UL + VS * CH * 2, TOTAL = BAR + 64;
+    using L = Work<DT, HEAD>;
+    static constexpr int EVEN = (2 + L::PARTS) * L::TILE, ODD = L::PARTS * L::TILE + 2 * L::ATILE;
+    static constexpr int SLOT = EVEN > ODD ? EVEN : ODD, SH = 3 * SLOT, SL = SH + VS * DT * 2;
+    static constexpr int UH = SL + VS * DT * 2, UL = UH + VS * CH * 2, FH = HEAD ? UL + VS * CH * 2 : UH, FL = HEAD ? FH + VS * CH * 2 : UL;
+    static constexpr int BAR = FL + VS * CH * 2, TOTAL = BAR + 64;
 };
-template <int DT, int VS, bool DELTA>
+template <int DT, int VS, int MODE>
 __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_constant__ Params W) {
-    using L = Work<DT>;
-    using S = StateSmem<DT, VS>;
+    constexpr bool DELTA = MODE != 0, HEAD = MODE == 2;
+    using L = Work<DT, HEAD>;
+    using S = StateSmem<DT, VS, HEAD>;
     constexpr int KS = DT / 16, NT = DT / 32, MT = VS / 16, NB = VS / 8;       // state tiles of a warp: MT x NT of 16 x 8
     extern __shared__ __align__(128) unsigned char smem[];
     unsigned char *s_hi = smem + S::SH, *s_lo = smem + S::SL, *u_hi = smem + S::UH, *u_lo = smem + S::UL;
@@ -641,11 +848,11 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
         const int s = i % 3;
         const unsigned char* src = tiles(i >> 1);
         if (i & 1) {
-            constexpr uint32_t bytes = 2 * L::TILE + 2 * L::ATILE;
+            constexpr uint32_t bytes = S::ODD;
             mbar_expect_tx(&bar[s], bytes);
             bulk_g2s(smem + s * S::SLOT, src + L::K, bytes, &bar[s]);
         } else {
-            constexpr uint32_t bytes = (DELTA ? 4 : 2) * L::TILE;
+            constexpr uint32_t bytes = DELTA ? S::EVEN : 2 * L::TILE;
             mbar_expect_tx(&bar[s], bytes);
             bulk_g2s(smem + s * S::SLOT + (DELTA ? 0 : 2 * L::TILE), src + (DELTA ? L::W : L::Q), bytes, &bar[s]);
         }
@@ -670,9 +877,14 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                 for (int e = 0; e < 2; ++e) store_split<DT>(s_hi, s_lo, m * 16 + g + 8 * e, d0 + n * 8 + 2 * t, X[m][n][2 * e], X[m][n][2 * e + 1]);
     };
     uint4 base[NB];
+    float fac[2] = {1.f, 1.f};                         // HEAD: the factors of this thread's rows of u (warps 0-3)
     const bool pairs = (Dv & 1) == 0 && (P.ld & 1) == 0 && (P.v_col & 1) == 0 && ((uintptr_t)P.x & 3) == 0;
     auto fetch_base = [&](int c) {                     // U in accumulator order, or v (two pairs of bf16)
         const int row0 = sp.row0 + c * CH, cnt = min(CH, sp.count - c * CH);
+        if constexpr (HEAD) {
+            const float* G = reinterpret_cast<const float*>(tiles(c) + L::G) + 4 + CH + wr + g;
+            fac[0] = G[0]; fac[1] = G[8];
+        }
 #pragma unroll
         for (int n = 0; n < NB; ++n) {
             if constexpr (DELTA) base[n] = ld_once(tiles(c) + L::U + (((v0 / 16 + (n >> 1)) * 4 + rb) * 64 + (n & 1) * 32 + lane) * 16);
@@ -706,7 +918,12 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
         for (int n = 0; n < NB; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) acc[n][e] = low[n][e] = 0.f;
-        if (owner) {
+        float rq[2] = {1.f, 1.f};                      // HEAD: the factors of this thread's rows of q (warps 4-7)
+        if constexpr (HEAD) {
+            const float* G = reinterpret_cast<const float*>(tiles(c) + L::G);
+            ge[0][0] = G[0];
+            if (!owner) { rq[0] = G[4 + wr + g]; rq[1] = G[4 + wr + g + 8]; }
+        } else if (owner) {
 #pragma unroll
             for (int n = 0; n < NT; ++n) {
                 const float2 f = *reinterpret_cast<const float2*>(tiles(c) + L::G + (d0 + n * 8 + 2 * t) * 4);
@@ -718,17 +935,24 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
             const unsigned char* p = wq + (owner ? 0 : 2 * L::TILE);
 #pragma unroll
             for (int ks = 0; ks < KS; ++ks) {
-                const uint4 ah = lds_frag(p, rb * KS + ks, lane), al = lds_frag(p + L::TILE, rb * KS + ks, lane);
+                const bool low_part = !HEAD || owner;          // q comes as it is
+                const uint4 ah = lds_frag(p, rb * KS + ks, lane), al = low_part ? lds_frag(p + L::TILE, rb * KS + ks, lane) : make_uint4(0, 0, 0, 0);
                 uint32_t bh[MT][4], bl[MT][4];
 #pragma unroll
                 for (int n = 0; n < MT; ++n) { fa::load_b<DT>(sh, n * 16, ks, bh[n]); fa::load_b<DT>(sl, n * 16, ks, bl[n]); }
 #pragma unroll
                 for (int n = 0; n < NB; ++n) mma_u4(acc[n], ah, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+                if (low_part)
 #pragma unroll
-                for (int n = 0; n < NB; ++n) mma_u4(low[n], al, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+                    for (int n = 0; n < NB; ++n) mma_u4(low[n], al, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
 #pragma unroll
                 for (int n = 0; n < NB; ++n) mma_u4(low[n], ah, bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
             }
+            if (HEAD && !owner)
+#pragma unroll
+                for (int n = 0; n < NB; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) { acc[n][e] *= rq[e >> 1]; low[n][e] *= rq[e >> 1]; }
         }
         if (owner) {                                   // u^T, split
 #pragma unroll
@@ -752,6 +976,12 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                     const uint32_t off = fa::tile_off<CH>(v, r >> 3) + (r & 7) * 2;
                     *reinterpret_cast<__nv_bfloat16*>(u_hi + off) = hi;
                     *reinterpret_cast<__nv_bfloat16*>(u_lo + off) = __float2bfloat16_rn(u[e] - __bfloat162float(hi));
+                    if constexpr (HEAD) {
+                        const float f = u[e] * fac[e >> 1];
+                        const __nv_bfloat16 fh = __float2bfloat16_rn(f);
+                        *reinterpret_cast<__nv_bfloat16*>(smem + S::FH + off) = fh;
+                        *reinterpret_cast<__nv_bfloat16*>(smem + S::FL + off) = __float2bfloat16_rn(f - __bfloat162float(fh));
+                    }
                 }
             }
             if (c + 1 < chunks) fetch_base(c + 1);
@@ -765,17 +995,17 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
 #pragma unroll
                 for (int n = 0; n < NT; ++n)
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) X[m][n][e] *= ge[n][e & 1];
+                    for (int e = 0; e < 4; ++e) X[m][n][e] *= HEAD ? ge[0][0] : ge[n][e & 1];
 #pragma unroll
             for (int ks = 0; ks < CH / 16; ++ks) {
                 uint32_t a[MT][4], b[MT][4];
                 uint4 kh[NT / 2], kl[NT / 2];
 #pragma unroll
-                for (int n = 0; n < NT / 2; ++n) { kh[n] = lds_frag(ka, (d0 / 16 + n) * 4 + ks, lane); kl[n] = lds_frag(ka + L::TILE, (d0 / 16 + n) * 4 + ks, lane); }
+                for (int n = 0; n < NT / 2; ++n) { kh[n] = lds_frag(ka, (d0 / 16 + n) * 4 + ks, lane); if constexpr (!HEAD) kl[n] = lds_frag(ka + L::TILE, (d0 / 16 + n) * 4 + ks, lane); }
 #pragma unroll
-                for (int m = 0; m < MT; ++m) { fa::load_a<CH>(uh, m * 16, ks, a[m]); fa::load_a<CH>(ul, m * 16, ks, b[m]); }
+                for (int m = 0; m < MT; ++m) { fa::load_a<CH>(uh + (S::FH - S::UH), m * 16, ks, a[m]); fa::load_a<CH>(ul + (S::FL - S::UL), m * 16, ks, b[m]); }
 #pragma unroll
-                for (int k = 0; k < 3; ++k)
+                for (int k = 0; k < (HEAD ? 2 : 3); ++k)
 #pragma unroll
                     for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -789,7 +1019,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
 #pragma unroll
             for (int ks = 0; ks < CH / 16; ++ks)
                 if (ks <= rb) {
-                    const uint4 kh = lds_frag(ka + 2 * L::TILE, rb * 4 + ks, lane), kl = lds_frag(ka + 2 * L::TILE + L::ATILE, rb * 4 + ks, lane);
+                    const uint4 kh = lds_frag(ka + L::PARTS * L::TILE, rb * 4 + ks, lane), kl = lds_frag(ka + L::PARTS * L::TILE + L::ATILE, rb * 4 + ks, lane);
                     uint32_t bh[MT][4], bl[MT][4];
 #pragma unroll
                     for (int n = 0; n < MT; ++n) { fa::load_b<CH>(uh, n * 16, ks, bh[n]); fa::load_b<CH>(ul, n * 16, ks, bl[n]); }
@@ -821,29 +1051,30 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
     if (owner) each_state([&](float& x, int v, int d) { if (ok && v < Dv && d < D) st[(size_t)d * Dv + v] = x; });
 }
 
-template <int DT, int VS>
+template <int DT, int VS, int MODE>
 static int launch_state(const Params& p, cudaStream_t st) {
     const dim3 grid((p.P.Dv + VS - 1) / VS, p.P.H, p.P.n_seqs);
-    auto kern = p.P.delta ? chunk_state_kernel<DT, VS, true> : chunk_state_kernel<DT, VS, false>;
-    constexpr int smem = StateSmem<DT, VS>::TOTAL;
-    PTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    PTB_CUDA_OK(ptb_launch(kern, grid, dim3(THREADS), (size_t)smem, st, ptb_pdl_enabled(), p));
+    constexpr int smem = StateSmem<DT, VS, MODE == 2>::TOTAL;
+    PTB_CUDA_OK(cudaFuncSetAttribute(chunk_state_kernel<DT, VS, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    PTB_CUDA_OK(ptb_launch(chunk_state_kernel<DT, VS, MODE>, grid, dim3(THREADS), (size_t)smem, st, ptb_pdl_enabled(), p));
     return 0;
+}
+template <int DT, int VS>
+static int launch_state(const Params& p, cudaStream_t st) {
+    return p.P.delta == 2 ? launch_state<DT, VS, 2>(p, st) : p.P.delta ? launch_state<DT, VS, 1>(p, st) : launch_state<DT, VS, 0>(p, st);
 }
 
 template <int DT>
 static int launch(Params p, cudaStream_t st) {
     const dim3 grid(p.P.n_chunks, p.P.H);
     const bool pdl = ptb_pdl_enabled();
-    if (p.P.delta) {
-        const int smem = DeltaSmem<DT>::total(p.Dvp);
-        PTB_CUDA_OK(cudaFuncSetAttribute(delta_chunk_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-        PTB_CUDA_OK(ptb_launch(delta_chunk_kernel<DT>, grid, dim3(THREADS), (size_t)smem, st, pdl, p));
-    } else {
-        constexpr int smem = 4 * Work<DT>::TILE;
-        PTB_CUDA_OK(cudaFuncSetAttribute(decay_chunk_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-        PTB_CUDA_OK(ptb_launch(decay_chunk_kernel<DT>, grid, dim3(THREADS), (size_t)smem, st, pdl, p));
-    }
+    auto go = [&](auto kern, int smem) {
+        PTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+        PTB_CUDA_OK(ptb_launch(kern, grid, dim3(THREADS), (size_t)smem, st, pdl, p));
+        return 0;
+    };
+    if (p.P.delta == 2 ? go(delta_head_chunk_kernel<DT>, HeadSmem<DT>::total(p.Dvp))
+                       : p.P.delta ? go(delta_chunk_kernel<DT>, DeltaSmem<DT>::total(p.Dvp)) : go(decay_chunk_kernel<DT>, 4 * Work<DT>::TILE)) return -1;
     // few CTAs: narrow slices, so that more of them share the walk
     const long long wide = (long long)((p.P.Dv + 31) / 32) * p.P.H * p.P.n_seqs;
     if (wide <= 74 ? launch_state<DT, 16>(p, st) : launch_state<DT, 32>(p, st)) return -1;
@@ -857,6 +1088,7 @@ int recurrence_check(const PtbRecurrence& p);
 
 static size_t chunk_bytes(const PtbRecurrence& p) {
     const int Dvp = (p.Dv + 31) / 32 * 32;
+    if (p.delta == 2) return p.D <= 64 ? rc::Work<64, true>::bytes(Dvp) : rc::Work<128, true>::bytes(Dvp);
     return p.D <= 64 ? rc::Work<64>::bytes(Dvp) : rc::Work<128>::bytes(Dvp);
 }
 

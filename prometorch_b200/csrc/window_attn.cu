@@ -4,7 +4,8 @@
 //                            values on their way to shared memory meanwhile; a weight enters the value product as the sum of two
 //                            bf16 numbers in the two halves of the 16-row operand;
 //   window_rows_f32_kernel   the same in true fp32 arithmetic (FMA);
-//   window_merge_kernel      joins the splits, the sink and the gate.
+//   window_merge_kernel      joins the splits, the maps, the sink and the gate.
+// With two maps the first half of a CTA's row blocks are the heads' first maps, the second half the second ones.
 // Page ids, positions and page-table columns are checked against their extents; a bad one sets PTB_ERR_BOUNDS and its key counts
 // as invisible.
 #include "window_attn.cuh"
@@ -124,24 +125,31 @@ __global__ void __launch_bounds__(PN_THREADS) proj_norm_write_kernel(const __gri
 }
 
 // ---------------------------------------------------------------------------------------------- one query row
+struct WindowRows {
+    PtbWindowAttn A;
+    int kcap, hg, groups;              // keys of a CTA; query heads of a CTA, CTAs per kv head
+    float scale_log2;                  // scale times log2(e)
+};
+
 // The cache slots (page * 64 + place, or -1) of the keys of split `split` of row `i`; returns their number.
-__device__ __forceinline__ int row_keys(const WindowAttnParams& P, int i, int split, int* krow) {
-    const int pos = P.pos[(size_t)i * P.pos_stride];
-    const Seen s = seen_by(pos, P.window, P.keep);
-    int per = (s.count + P.nsplit - 1) / P.nsplit;
+__device__ __forceinline__ int row_keys(const WindowRows& P, int i, int split, int* krow) {
+    const PtbWindowAttn& A = P.A;
+    const int pos = A.pos[(size_t)i * A.pos_stride];
+    const Seen s = seen_by(pos, A.window, A.keep, A.chunked);
+    int per = (s.count + A.nsplit - 1) / A.nsplit;
     if (pos < 0 || per > P.kcap) {                     // the host sizes the splits for the row that sees most
-        if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+        if (threadIdx.x == 0 && A.status) atomicExch(A.status, PTB_ERR_BOUNDS);
         per = min(per, P.kcap);
     }
     const int e0 = split * per, nk = max(0, min(per, s.count - e0));
-    const int* table = P.page_table + (size_t)P.req[(size_t)i * P.req_stride] * P.pt_stride;
+    const int* table = A.page_table + (size_t)A.req[(size_t)i * A.req_stride] * A.pt_stride;
     for (int e = threadIdx.x; e < P.kcap; e += blockDim.x) {
         int v = -1;
         if (e < nk) {
             const int j = e0 + e < s.kept ? e0 + e : s.lo + e0 + e - s.kept, col = j / WA_PAGE;
-            const int page = col < P.pt_stride ? table[col] : -1;
-            if (page >= 0 && page < P.n_pages) v = page * WA_PAGE + j % WA_PAGE;
-            else if (P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+            const int page = col < A.pt_stride ? table[col] : -1;
+            if (page >= 0 && page < A.n_pages) v = page * WA_PAGE + j % WA_PAGE;
+            else if (A.status) atomicExch(A.status, PTB_ERR_BOUNDS);
         }
         krow[e] = v;
     }
@@ -151,76 +159,94 @@ __device__ __forceinline__ size_t cache_row(int krow, int G, int g) { return ((s
 
 // Factor of a head's sum given its largest (log2) score and total: the sink joins the denominator, the gate multiplies.
 template <typename T>
-__device__ __forceinline__ float finish_factor(const WindowAttnParams& P, size_t i, int h, float m, float l) {
+__device__ __forceinline__ float finish_factor(const PtbWindowAttn& A, size_t i, int h, float m, float l) {
     float M = m, f = 1.f;
-    if (P.sink) {
-        const float s = P.sink[h] * WA_LOG2E;
+    if (A.sink) {
+        const float s = A.sink[h] * WA_LOG2E;
         M = fmaxf(m, s);
         f = m == -INFINITY ? 0.f : exp2f(m - M);
         l = l * f + exp2f(s - M);
     }
     f = l > 0.f ? f / l : 0.f;
-    if (P.gate) f *= sigmoid(wa_f<T>(((const T*)P.gate)[i * P.gate_ld + h]));
+    if (A.gate) f *= sigmoid(wa_f<T>(((const T*)A.gate)[i * A.gate_ld + h]));
     return f;
 }
 
 constexpr int WR_THREADS = 128, WR_WARPS = 4;
 
+// The query heads of a CTA: `n` of them from h0, all of kv head c.
+struct HeadGroup { int c, h0, n; };
+__device__ __forceinline__ HeadGroup head_group(const WindowRows& P) {
+    const int R = P.A.H / P.A.G, grp = blockIdx.y % P.groups;
+    HeadGroup g;
+    g.c = blockIdx.y / P.groups;
+    g.h0 = g.c * R + grp * P.hg;
+    g.n = min(P.hg, R - grp * P.hg);
+    return g;
+}
+
 struct WindowSmem {
     int v, q, w, hi, lo, ml, krow, pitch, ldw, ldh, total;      // byte offsets; pitches in bytes (v) and elements
-    __host__ __device__ WindowSmem(int R8, int Dp, int Dvp, int kcap, bool mma) {
+    __host__ __device__ WindowSmem(int rows, int Dp, int Dvp, int kcap, bool mma) {      // rows: of all maps
         pitch = Dvp * 2 + 16; ldw = kcap + 1; ldh = kcap + 8;
         v = 0;
         q = mma ? kcap * pitch : 0;
-        w = q + R8 * Dp * (mma ? 2 : 4);
-        hi = (w + R8 * ldw * 4 + 15) & ~15;
-        lo = hi + (mma ? R8 * ldh * 2 : 0);
-        ml = lo + (mma ? R8 * ldh * 2 : 0);
-        krow = ml + R8 * 8;
+        w = q + rows * Dp * (mma ? 2 : 4);
+        hi = (w + rows * ldw * 4 + 15) & ~15;
+        lo = hi + (mma ? rows * ldh * 2 : 0);
+        ml = lo + (mma ? rows * ldh * 2 : 0);
+        krow = ml + rows * 8;
         total = krow + kcap * 4;
     }
 };
 
-__global__ void __launch_bounds__(WR_THREADS) window_rows_mma_kernel(const __grid_constant__ WindowAttnParams P) {
+__global__ void __launch_bounds__(WR_THREADS) window_rows_mma_kernel(const __grid_constant__ WindowRows P) {
     extern __shared__ __align__(16) unsigned char smem[];
-    const int R = P.H / P.G, RB = (R + 7) / 8, R8 = RB * 8;
-    const WindowSmem L(R8, P.Dp, P.Dvp, P.kcap, true);
+    const PtbWindowAttn& A = P.A;
+    const int RB1 = (P.hg + 7) / 8, RB = RB1 * A.maps, R8 = RB1 * 8, rows = RB * 8;
+    const WindowSmem L(rows, A.Dp, A.Dvp, P.kcap, true);
     __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem + L.q);
     float* w_s = reinterpret_cast<float*>(smem + L.w);
     __nv_bfloat16* hi_s = reinterpret_cast<__nv_bfloat16*>(smem + L.hi);
     __nv_bfloat16* lo_s = reinterpret_cast<__nv_bfloat16*>(smem + L.lo);
     float2* ml_s = reinterpret_cast<float2*>(smem + L.ml);
     int* krow = reinterpret_cast<int*>(smem + L.krow);
-    const int split = blockIdx.x, c = blockIdx.y, i = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const int split = blockIdx.x, i = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const HeadGroup hg = head_group(P);
+    const int c = hg.c;
     pdl_wait();
     pdl_launch_dependents();
     const int nk = row_keys(P, i, split, krow);
     {
-        const uint4* src = reinterpret_cast<const uint4*>((const __nv_bfloat16*)P.q + ((size_t)i * P.H + c * R) * P.Dp);
+        const int ch = A.Dp / 8;
+        const uint4* src = reinterpret_cast<const uint4*>((const __nv_bfloat16*)A.q + ((size_t)i * A.H + hg.h0) * A.maps * A.Dp);
         uint4* dst = reinterpret_cast<uint4*>(q_s);
-        for (int e = threadIdx.x; e < R8 * P.Dp / 8; e += WR_THREADS) dst[e] = e < R * P.Dp / 8 ? src[e] : make_uint4(0, 0, 0, 0);
+        for (int e = threadIdx.x; e < rows * ch; e += WR_THREADS) {
+            const int row = e / ch, m = row / R8, r = row % R8;
+            dst[e] = r < hg.n ? src[(r * A.maps + m) * ch + e % ch] : make_uint4(0, 0, 0, 0);
+        }
     }
     __syncthreads();
     const int kgroups = (nk + 15) / 16;
     {                                                  // the values, while the scores are formed
-        const int vch = P.Dvp / 8;
+        const int vch = A.Dvp / 8;
         const uint32_t v0 = smem_u32(smem + L.v);
         for (int e = threadIdx.x; e < kgroups * 16 * vch; e += WR_THREADS) {
             const int r = e / vch, ch = e % vch, kr = krow[r];
-            fa::cp_async16(v0 + (uint32_t)(r * L.pitch + ch * 16), (const __nv_bfloat16*)P.v_pages + (kr >= 0 ? cache_row(kr, P.G, c) * P.Dvp + ch * 8 : 0), kr >= 0);
+            fa::cp_async16(v0 + (uint32_t)(r * L.pitch + ch * 16), (const __nv_bfloat16*)A.v_pages + (kr >= 0 ? cache_row(kr, A.G, c) * A.v_ld + ch * 8 : 0), kr >= 0);
         }
         fa::cp_async_commit();
     }
     // a lane's 16 bytes serve as its elements of two k16 steps of both operands, so the order inside a 32-element group cancels
     const uint4 zero4 = make_uint4(0, 0, 0, 0);
-    const __nv_bfloat16* kp = (const __nv_bfloat16*)P.k_pages;
-    const int nch = P.Dp / 8;
+    const int nch = A.Dp / 8, kpitch = A.maps * A.Dp;
     for (int u = warp; u < RB * kgroups; u += WR_WARPS) {
         const int kg = u % kgroups, rb = u / kgroups;
+        const __nv_bfloat16* kp = (const __nv_bfloat16*)A.k_pages + (rb / RB1) * A.Dp;
         const int r0 = krow[kg * 16 + g], r1 = krow[kg * 16 + g + 8];
-        const uint4* k0 = reinterpret_cast<const uint4*>(kp + cache_row(max(r0, 0), P.G, c) * P.Dp);
-        const uint4* k1 = reinterpret_cast<const uint4*>(kp + cache_row(max(r1, 0), P.G, c) * P.Dp);
-        const uint4* qv = reinterpret_cast<const uint4*>(q_s + (size_t)(rb * 8 + g) * P.Dp);
+        const uint4* k0 = reinterpret_cast<const uint4*>(kp + cache_row(max(r0, 0), A.G, c) * kpitch);
+        const uint4* k1 = reinterpret_cast<const uint4*>(kp + cache_row(max(r1, 0), A.G, c) * kpitch);
+        const uint4* qv = reinterpret_cast<const uint4*>(q_s + (size_t)(rb * 8 + g) * A.Dp);
         float acc[4] = {0.f, 0.f, 0.f, 0.f};
         for (int b0 = 0; b0 < nch; b0 += 16) {
             uint4 a[4], b[4];
@@ -246,13 +272,13 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_mma_kernel(const __gri
             w_s[(rb * 8 + 2 * t + (e & 1)) * L.ldw + kg * 16 + g + (e >> 1) * 8] = ((e >> 1) ? r1 : r0) >= 0 ? acc[e] * P.scale_log2 : -INFINITY;
     }
     __syncthreads();
-    for (int h = warp; h < R8; h += WR_WARPS) {
+    for (int h = warp; h < rows; h += WR_WARPS) {
         float m = -INFINITY, l = 0.f;
         for (int j = lane; j < kgroups * 16; j += 32) m = fmaxf(m, w_s[h * L.ldw + j]);
         m = warp_max(m);
         const float base = m == -INFINITY ? 0.f : m;
         for (int j = lane; j < kgroups * 16; j += 32) {
-            const float p = h < R ? exp2f(w_s[h * L.ldw + j] - base) : 0.f;
+            const float p = h % R8 < hg.n ? exp2f(w_s[h * L.ldw + j] - base) : 0.f;
             const __nv_bfloat16 hi = __float2bfloat16_rn(p);
             hi_s[h * L.ldh + j] = hi;
             lo_s[h * L.ldh + j] = __float2bfloat16_rn(p - __bfloat162float(hi));
@@ -265,10 +291,11 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_mma_kernel(const __gri
     __syncthreads();
     // rows 0-7 of the left operand carry the high halves of eight heads' weights, rows 8-15 the low halves; columns are values
     const uint32_t v0 = smem_u32(smem + L.v);
-    const int DC = (P.Dvp + 31) / 32;
+    const int DC = (A.Dvp + 31) / 32;
+    const bool merged = A.nsplit > 1 || A.maps > 1;
     for (int u = warp; u < RB * DC; u += WR_WARPS) {
         const int dc = u % DC, rb = u / DC;
-        const bool two = dc * 32 + 16 < P.Dvp;         // Dvp is a multiple of 16
+        const bool two = dc * 32 + 16 < A.Dvp;         // Dvp is a multiple of 16
         const __nv_bfloat16* hi_r = hi_s + (rb * 8 + g) * L.ldh + 2 * t;
         const __nv_bfloat16* lo_r = lo_s + (rb * 8 + g) * L.ldh + 2 * t;
         float acc[4][4];
@@ -293,49 +320,55 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_mma_kernel(const __gri
                 fa::mma16816(acc[3], a, b[2], b[3]);
             }
         }
-        const int hl = rb * 8 + g, h = c * R + hl;
-        if (hl >= R) continue;
-        const float2 ml = ml_s[hl];
-        const float f = P.nsplit > 1 ? 1.f : finish_factor<__nv_bfloat16>(P, i, h, ml.x, ml.y);
-        float* wk = P.work + (((size_t)i * P.nsplit + split) * P.H + h) * (P.Dvp + 2);
-        __nv_bfloat16* o = (__nv_bfloat16*)P.out + ((size_t)i * P.H + h) * P.Dv;
+        const int row = rb * 8 + g, hl = row % R8, h = hg.h0 + hl;
+        if (hl >= hg.n) continue;
+        const float2 ml = ml_s[row];
+        const float f = merged ? 1.f : finish_factor<__nv_bfloat16>(A, i, h, ml.x, ml.y);
+        float* wk = A.work + ((((size_t)i * A.nsplit + split) * A.H + h) * A.maps + row / R8) * (A.Dvp + 2);
+        __nv_bfloat16* o = (__nv_bfloat16*)A.out + ((size_t)i * A.H + h) * A.Dv;
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int d = dc * 32 + e * 8 + 2 * t;
             const float x = acc[e][0] + acc[e][2], y = acc[e][1] + acc[e][3];
-            if (P.nsplit > 1) {
-                if (d < P.Dvp) *reinterpret_cast<float2*>(wk + d) = make_float2(x, y);
+            if (merged) {
+                if (d < A.Dvp) *reinterpret_cast<float2*>(wk + d) = make_float2(x, y);
             } else {
-                if (d < P.Dv) o[d] = __float2bfloat16_rn(x * f);
-                if (d + 1 < P.Dv) o[d + 1] = __float2bfloat16_rn(y * f);
+                if (d < A.Dv) o[d] = __float2bfloat16_rn(x * f);
+                if (d + 1 < A.Dv) o[d + 1] = __float2bfloat16_rn(y * f);
             }
         }
-        if (P.nsplit > 1 && dc == 0 && t == 0) *reinterpret_cast<float2*>(wk + P.Dvp) = ml;
+        if (merged && dc == 0 && t == 0) *reinterpret_cast<float2*>(wk + A.Dvp) = ml;
     }
 }
 
-__global__ void __launch_bounds__(WR_THREADS) window_rows_f32_kernel(const __grid_constant__ WindowAttnParams P) {
+__global__ void __launch_bounds__(WR_THREADS) window_rows_f32_kernel(const __grid_constant__ WindowRows P) {
     extern __shared__ __align__(16) unsigned char smem[];
-    const int R = P.H / P.G, R8 = (R + 7) / 8 * 8;
-    const WindowSmem L(R8, P.Dp, P.Dvp, P.kcap, false);
-    float* q_s = reinterpret_cast<float*>(smem + L.q);
+    const PtbWindowAttn& A = P.A;
+    const int R8 = (P.hg + 7) / 8 * 8;
+    const WindowSmem L(R8 * A.maps, A.Dp, A.Dvp, P.kcap, false);
+    float* q_s = reinterpret_cast<float*>(smem + L.q);                 // [maps][n][Dp], the other arrays likewise
     float* w_s = reinterpret_cast<float*>(smem + L.w);
     float2* ml_s = reinterpret_cast<float2*>(smem + L.ml);
     int* krow = reinterpret_cast<int*>(smem + L.krow);
-    const int split = blockIdx.x, c = blockIdx.y, i = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int split = blockIdx.x, i = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const HeadGroup hg = head_group(P);
+    const int c = hg.c, rows = hg.n * A.maps, kpitch = A.maps * A.Dp;
     pdl_wait();
     pdl_launch_dependents();
     const int nk = row_keys(P, i, split, krow);
-    for (int e = threadIdx.x; e < R * P.Dp; e += WR_THREADS) q_s[e] = ((const float*)P.q)[((size_t)i * P.H + c * R) * P.Dp + e];
+    for (int e = threadIdx.x; e < rows * A.Dp; e += WR_THREADS) {
+        const int row = e / A.Dp, m = row / hg.n, r = row % hg.n;
+        q_s[e] = ((const float*)A.q)[(((size_t)i * A.H + hg.h0 + r) * A.maps + m) * A.Dp + e % A.Dp];
+    }
     __syncthreads();
-    for (int e = threadIdx.x; e < R * nk; e += WR_THREADS) {
+    for (int e = threadIdx.x; e < rows * nk; e += WR_THREADS) {
         const int h = e / nk, j = e % nk, r = krow[j];
         float s = -INFINITY;
         if (r >= 0) {
-            const float4* k4 = reinterpret_cast<const float4*>((const float*)P.k_pages + cache_row(r, P.G, c) * P.Dp);
-            const float4* q4 = reinterpret_cast<const float4*>(q_s + (size_t)h * P.Dp);
+            const float4* k4 = reinterpret_cast<const float4*>((const float*)A.k_pages + cache_row(r, A.G, c) * kpitch + (h / hg.n) * A.Dp);
+            const float4* q4 = reinterpret_cast<const float4*>(q_s + (size_t)h * A.Dp);
             float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-            for (int d = 0; d < P.Dp / 4; ++d) {
+            for (int d = 0; d < A.Dp / 4; ++d) {
                 const float4 x = k4[d], y = q4[d];
                 a.x = fmaf(x.x, y.x, a.x); a.y = fmaf(x.y, y.y, a.y); a.z = fmaf(x.z, y.z, a.z); a.w = fmaf(x.w, y.w, a.w);
             }
@@ -344,7 +377,7 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_f32_kernel(const __gri
         w_s[h * L.ldw + j] = s;
     }
     __syncthreads();
-    for (int h = warp; h < R; h += WR_WARPS) {
+    for (int h = warp; h < rows; h += WR_WARPS) {
         float m = -INFINITY, l = 0.f;
         for (int j = lane; j < nk; j += 32) m = fmaxf(m, w_s[h * L.ldw + j]);
         m = warp_max(m);
@@ -357,38 +390,75 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_f32_kernel(const __gri
         if (lane == 0) ml_s[h] = make_float2(m, l);
     }
     __syncthreads();
-    for (int e = threadIdx.x; e < R * P.Dvp; e += WR_THREADS) {
-        const int hl = e / P.Dvp, d = e % P.Dvp, h = c * R + hl;
+    const bool merged = A.nsplit > 1 || A.maps > 1;
+    for (int e = threadIdx.x; e < rows * A.Dvp; e += WR_THREADS) {
+        const int row = e / A.Dvp, d = e % A.Dvp, h = hg.h0 + row % hg.n;
         float a = 0.f;
         for (int j = 0; j < nk; ++j)
-            if (krow[j] >= 0) a = fmaf(w_s[hl * L.ldw + j], ((const float*)P.v_pages)[cache_row(krow[j], P.G, c) * P.Dvp + d], a);
-        const float2 ml = ml_s[hl];
-        float* wk = P.work + (((size_t)i * P.nsplit + split) * P.H + h) * (P.Dvp + 2);
-        if (P.nsplit > 1) {
+            if (krow[j] >= 0) a = fmaf(w_s[row * L.ldw + j], ((const float*)A.v_pages)[cache_row(krow[j], A.G, c) * A.v_ld + d], a);
+        const float2 ml = ml_s[row];
+        float* wk = A.work + ((((size_t)i * A.nsplit + split) * A.H + h) * A.maps + row / hg.n) * (A.Dvp + 2);
+        if (merged) {
             wk[d] = a;
-            if (d == 0) *reinterpret_cast<float2*>(wk + P.Dvp) = ml;
-        } else if (d < P.Dv) ((float*)P.out)[((size_t)i * P.H + h) * P.Dv + d] = a * finish_factor<float>(P, i, h, ml.x, ml.y);
+            if (d == 0) *reinterpret_cast<float2*>(wk + A.Dvp) = ml;
+        } else if (d < A.Dv) ((float*)A.out)[((size_t)i * A.H + h) * A.Dv + d] = a * finish_factor<float>(A, i, h, ml.x, ml.y);
     }
 }
 
 // One CTA per (head, row).
-template <typename T>
-__global__ void __launch_bounds__(128) window_merge_kernel(const __grid_constant__ WindowAttnParams P) {
+template <typename T, int MAPS>
+__global__ void __launch_bounds__(128) window_merge_kernel(const __grid_constant__ PtbWindowAttn P) {
+    __shared__ float red[4];
     pdl_wait();
     pdl_launch_dependents();
     const int h = blockIdx.x;
-    const size_t i = blockIdx.y, pitch = (size_t)P.H * (P.Dvp + 2);
-    const float* wk = P.work + i * P.nsplit * pitch + (size_t)h * (P.Dvp + 2);
-    float M = -INFINITY, l = 0.f;
-    for (int s = 0; s < P.nsplit; ++s) M = fmaxf(M, wk[s * pitch + P.Dvp]);
-    const float base = M == -INFINITY ? 0.f : M;
-    for (int s = 0; s < P.nsplit; ++s) l += wk[s * pitch + P.Dvp + 1] * exp2f(wk[s * pitch + P.Dvp] - base);
-    const float f = finish_factor<T>(P, i, h, M, l);
-    for (int d = threadIdx.x; d < P.Dv; d += blockDim.x) {
-        float a = 0.f;
+    const size_t i = blockIdx.y, pitch = (size_t)P.H * MAPS * (P.Dvp + 2);
+    const float* wk[MAPS];
+    float base[MAPS], f[MAPS];
+#pragma unroll
+    for (int m = 0; m < MAPS; ++m) {
+        wk[m] = P.work + i * P.nsplit * pitch + (size_t)(h * MAPS + m) * (P.Dvp + 2);
+        float M = -INFINITY, l = 0.f;
+        for (int s = 0; s < P.nsplit; ++s) M = fmaxf(M, wk[m][s * pitch + P.Dvp]);
+        base[m] = M == -INFINITY ? 0.f : M;
+        for (int s = 0; s < P.nsplit; ++s) l += wk[m][s * pitch + P.Dvp + 1] * exp2f(wk[m][s * pitch + P.Dvp] - base[m]);
+        f[m] = MAPS == 1 ? finish_factor<T>(P, i, h, M, l) : l > 0.f ? (m ? -P.mix : 1.f) / l : 0.f;
+    }
+    auto value = [&](int d) {
+        float r = 0.f;
+#pragma unroll
+        for (int m = 0; m < MAPS; ++m) {
+            float a = 0.f;
 #pragma unroll 4
-        for (int s = 0; s < P.nsplit; ++s) a += wk[s * pitch + d] * exp2f(wk[s * pitch + P.Dvp] - base);
-        ((T*)P.out)[(i * P.H + h) * P.Dv + d] = wa_t<T>(a * f);
+            for (int s = 0; s < P.nsplit; ++s) a += wk[m][s * pitch + d] * exp2f(wk[m][s * pitch + P.Dvp] - base[m]);
+            r = fmaf(a, f[m], r);
+        }
+        return r;
+    };
+    T* out = (T*)P.out + (i * P.H + h) * P.Dv;
+    if constexpr (MAPS == 1) {
+        for (int d = threadIdx.x; d < P.Dv; d += blockDim.x) out[d] = wa_t<T>(value(d));
+    } else {
+        constexpr int KEEP = 4;                        // values a thread keeps; wider heads form them again
+        float v[KEEP], ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) {
+            const int d = threadIdx.x + k * 128;
+            v[k] = d < P.Dv ? value(d) : 0.f;
+            ss += v[k] * v[k];
+        }
+        for (int d = threadIdx.x + KEEP * 128; d < P.Dv; d += 128) { const float a = value(d); ss += a * a; }
+        ss = warp_sum(ss);
+        if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+        __syncthreads();
+        float g = rsqrtf((red[0] + red[1] + red[2] + red[3]) / (float)P.Dv + P.mix_eps) * P.mix_gain;
+        if (P.gate) g *= sigmoid(wa_f<T>(((const T*)P.gate)[i * P.gate_ld + h]));
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) {
+            const int d = threadIdx.x + k * 128;
+            if (d < P.Dv) out[d] = wa_t<T>(v[k] * g);
+        }
+        for (int d = threadIdx.x + KEEP * 128; d < P.Dv; d += 128) out[d] = wa_t<T>(value(d) * g);
     }
 }
 
@@ -418,41 +488,42 @@ PTB_API int ptb_proj_norm_write(const void* x, long long ld, int q_col, int k_co
     return 0;
 }
 
-// Floats of workspace the row kernels need for `nsplit` > 1.
-PTB_API long long ptb_window_rows_work_floats(int n, int H, int Dvp, int nsplit) { return nsplit > 1 ? (long long)n * nsplit * H * (Dvp + 2) : 0; }
+// Floats of workspace the row kernels need (heads: H times the number of maps) where nsplit or the number of maps is above one.
+PTB_API long long ptb_window_rows_work_floats(int n, int heads, int Dvp, int nsplit) { return (long long)n * nsplit * heads * (Dvp + 2); }
 
-// Query rows q [n, H, Dp], each at its own position of its own sequence, against the cached keys it sees.  max_keys: the most keys any
-// row sees; nsplit CTAs share a row's keys (at most WA_KEYS each).  out [n, H Dv] in the type of q.
-PTB_API int ptb_window_attn_rows(const void* q, void* out, int n, int H, int G, int Dp, int Dv, int Dvp, const int* pos, int pos_stride,
-                                 const int* req, int req_stride, const int* page_table, int pt_stride, int n_pages, const void* k_pages,
-                                 const void* v_pages, const float* sink, const void* gate, long long gate_ld, int window, int keep, float scale,
-                                 int max_keys, float* work, int nsplit, int* status, int bf16, cudaStream_t st) {
-    if (n <= 0) return 0;
-    if (G <= 0 || H % G || Dp % 16 || Dvp % 16 || window < 1 || keep < 0 || G > 65535) {
-        ptb_set_error("window attention: bad sizes (H %d, G %d, Dp %d, Dvp %d, window %d, keep %d)", H, G, Dp, Dvp, window, keep);
+// Query rows, each at its own position of its own sequence, against the cached keys it sees; see PtbWindowAttn.  max_keys: the most keys
+// any row sees; nsplit CTAs share a row's keys (at most WA_KEYS each).
+PTB_API int ptb_window_attn_rows(const PtbWindowAttn* args, cudaStream_t st) {
+    const PtbWindowAttn& a = *args;
+    if (a.n <= 0) return 0;
+    if (a.G <= 0 || a.H % a.G || a.Dp % 16 || a.Dvp % 16 || a.v_ld % 8 || a.window < 1 || a.keep < 0 || a.maps < 1 || a.maps > 2 || (a.maps > 1 && a.sink)) {
+        ptb_set_error("window attention: bad sizes (H %d, G %d, Dp %d, Dvp %d, window %d, keep %d, maps %d)", a.H, a.G, a.Dp, a.Dvp, a.window, a.keep, a.maps);
         return -1;
     }
-    const int per = (std::max(1, max_keys) + nsplit - 1) / std::max(1, nsplit);
-    if (nsplit < 1 || per > WA_KEYS || (nsplit > 1 && !work)) {
-        ptb_set_error("window attention: %d splits for %d keys (at most %d keys per split, workspace needed above one)", nsplit, max_keys, WA_KEYS);
+    const int per = (std::max(1, a.max_keys) + a.nsplit - 1) / std::max(1, a.nsplit);
+    const bool merged = a.nsplit > 1 || a.maps > 1;
+    if (a.nsplit < 1 || per > WA_KEYS || (merged && !a.work)) {
+        ptb_set_error("window attention: %d splits for %d keys (at most %d keys per split, workspace needed above one)", a.nsplit, a.max_keys, WA_KEYS);
         return -1;
     }
-    if (n > 65535) { ptb_set_error("window attention: %d rows in one launch", n); return -1; }
-    WindowAttnParams p;
-    p.q = q; p.out = out; p.work = work; p.pos = pos; p.req = req; p.page_table = page_table; p.k_pages = k_pages; p.v_pages = v_pages;
-    p.sink = sink; p.gate = gate; p.gate_ld = gate_ld; p.pos_stride = pos_stride; p.req_stride = req_stride; p.pt_stride = pt_stride;
-    p.n_pages = n_pages; p.n = n; p.H = H; p.G = G; p.Dp = Dp; p.Dv = Dv; p.Dvp = Dvp; p.window = window; p.keep = keep; p.nsplit = nsplit;
-    p.kcap = (per + 15) & ~15; p.scale_log2 = scale * WA_LOG2E; p.status = status;
-    const int R8 = (H / G + 7) / 8 * 8;
-    const WindowSmem L(R8, Dp, Dvp, p.kcap, bf16 != 0);
-    if (L.total > 227 * 1024) { ptb_set_error("window attention: %d heads of %d need %d bytes of shared memory", H / G, Dp, L.total); return -1; }
-    auto kern = bf16 ? window_rows_mma_kernel : window_rows_f32_kernel;
+    WindowRows p;
+    p.A = a;
+    p.kcap = (per + 15) & ~15;
+    p.scale_log2 = a.scale * WA_LOG2E;
+    const int R = a.H / a.G;
+    p.hg = std::min(R, WA_HEADS);
+    p.groups = (R + p.hg - 1) / p.hg;
+    if (a.n > 65535 || a.G * p.groups > 65535) { ptb_set_error("window attention: %d rows of %d groups of heads in one launch", a.n, a.G * p.groups); return -1; }
+    const WindowSmem L((p.hg + 7) / 8 * 8 * a.maps, a.Dp, a.Dvp, p.kcap, a.bf16 != 0);
+    if (L.total > 227 * 1024) { ptb_set_error("window attention: %d heads of %d / %d need %d bytes of shared memory", p.hg, a.Dp, a.Dvp, L.total); return -1; }
+    auto kern = a.bf16 ? window_rows_mma_kernel : window_rows_f32_kernel;
     if (L.total > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     const bool pdl = ptb_pdl_enabled();
-    PTB_CUDA_OK(ptb_launch(kern, dim3(nsplit, G, n), dim3(WR_THREADS), (size_t)L.total, st, pdl, p));
-    if (nsplit > 1) {
-        if (bf16) PTB_CUDA_OK(ptb_launch(window_merge_kernel<__nv_bfloat16>, dim3(H, n), dim3(128), 0, st, pdl, p));
-        else PTB_CUDA_OK(ptb_launch(window_merge_kernel<float>, dim3(H, n), dim3(128), 0, st, pdl, p));
+    PTB_CUDA_OK(ptb_launch(kern, dim3(a.nsplit, a.G * p.groups, a.n), dim3(WR_THREADS), (size_t)L.total, st, pdl, p));
+    if (merged) {
+        auto merge = a.bf16 ? (a.maps > 1 ? window_merge_kernel<__nv_bfloat16, 2> : window_merge_kernel<__nv_bfloat16, 1>)
+                            : (a.maps > 1 ? window_merge_kernel<float, 2> : window_merge_kernel<float, 1>);
+        PTB_CUDA_OK(ptb_launch(merge, dim3(a.H, a.n), dim3(128), 0, st, pdl, a));
     }
     PTB_CUDA_OK(cudaGetLastError());
     return 0;

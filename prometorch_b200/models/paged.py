@@ -120,7 +120,7 @@ def register_model(config: type, weights: type, model: type, *names: str) -> Non
 
 
 def _ensure_builtin():
-    from . import gelutar, kifusun, llama_paged  # noqa: F401  (they register themselves)
+    from . import budorax, gelutar, kifusun, llama_paged  # noqa: F401  (they register themselves)
 
 
 def known_models() -> List[str]:

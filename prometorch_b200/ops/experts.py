@@ -1,0 +1,114 @@
+"""A mixture of experts for inference (csrc/experts.cu, csrc/experts_sm100.cu): a sigmoid router with a correction that has a say in the
+choice only, and gated experts ``down (silu(gate h) * (up h))``, each token using ``top`` of them.
+
+:func:`run` sorts the (token, expert) pairs by expert on the device, runs every expert over its rows (one grouped product for gate
+and up, one for down) and returns :class:`ExpertRows`: the rows where they lie, their places and weights.  What sums them up is the kernel
+that adds them to the stream (``ops/tanh_norm.py``).  Nothing depends on the counts on the host, so a decode pass can be a CUDA graph.
+CUDA tensors run the kernels, CPU tensors the plain math."""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass
+from typing import List
+
+import torch
+
+from .. import _native as N
+from .paged import _status
+from .residual import _st, linear_f32
+
+
+@N.register_decls
+def _decls(L):
+    vp, ci, cf, ll = C.c_void_p, C.c_int, C.c_float, C.c_longlong
+    L.ptb_expert_route.argtypes = [vp, ci, ll, ll, vp, ci, ci, ci, cf, vp, vp, vp, vp, vp, vp, vp]
+    L.ptb_expert_gemm_simt.argtypes = [vp, vp, ll, vp, ci, vp, vp, ci, ci, ci, ci, ci, vp, vp]
+    for n in ("ptb_expert_route", "ptb_expert_gemm_simt"):
+        getattr(L, n).restype = ci
+
+
+@dataclass
+class Experts:
+    """One layer's experts in the layout the kernels read; ``ff`` is rounded up to a multiple of eight with zeros."""
+    gate_up: torch.Tensor              # [E, 2 ff, W]: gate rows, then up rows
+    down: torch.Tensor                 # [E, W, ff]
+    router: torch.Tensor               # [E rounded up to eight, W]
+    correction: torch.Tensor           # [E] fp32
+    top: int
+    scale: float
+
+    @property
+    def count(self) -> int:
+        return self.gate_up.shape[0]
+
+    @classmethod
+    def of(cls, gate: List[torch.Tensor], up: List[torch.Tensor], down: List[torch.Tensor], router: torch.Tensor, correction: torch.Tensor, top: int,
+           scale: float) -> "Experts":
+        pad = lambda t, d: torch.nn.functional.pad(t, (0, 0, 0, -t.shape[0] % 8) if d == 0 else (0, -t.shape[1] % 8))
+        return cls(torch.stack([torch.cat([pad(g, 0), pad(u, 0)]) for g, u in zip(gate, up)]), torch.stack([pad(t, 1) for t in down]), pad(router, 0).contiguous(),
+                   correction.float(), top, scale)
+
+
+@dataclass
+class ExpertRows:
+    """Outputs of the chosen experts: row ``index[t, i]`` of ``y`` belongs to token t with the weight ``weight[t, i]``."""
+    y: torch.Tensor                    # [n top, W], sorted by expert
+    index: torch.Tensor                # [n, top] int32
+    weight: torch.Tensor               # [n, top] fp32
+
+    def combine(self) -> torch.Tensor:
+        return (self.y.float()[self.index.long()] * self.weight[..., None]).sum(1)
+
+
+@dataclass
+class Routing:
+    index: torch.Tensor                # [n, top] int32: place of every pair in the order by expert
+    weight: torch.Tensor               # [n, top] fp32
+    token: torch.Tensor                # [n top] int32: the token of every place
+    offsets: torch.Tensor              # [E + 1] int32: first place of every expert
+
+
+def route(h: torch.Tensor, e: Experts) -> Routing:
+    n, E, k = h.shape[0], e.count, e.top
+    z = linear_f32(h, e.router)
+    if h.is_cuda:
+        i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=h.device)
+        r = Routing(i32(n, k), torch.empty(n, k, dtype=torch.float32, device=h.device), i32(n * k), i32(E + 1))
+        work = i32(2 * n * k + E)
+        N.check(N.lib().ptb_expert_route(z.data_ptr(), 1, 0, z.stride(0), e.correction.data_ptr(), n, E, k, float(e.scale), r.index.data_ptr(), r.weight.data_ptr(),
+                                         r.token.data_ptr(), r.offsets.data_ptr(), work.data_ptr(), _status(h.device).data_ptr(), _st(h)), "expert_route")
+        return r
+    s = torch.sigmoid(z[:, :E])
+    chosen = torch.topk(s + e.correction, k, -1).indices
+    w = s.gather(1, chosen)
+    w = w / (w.sum(-1, keepdim=True) + 1e-20) * e.scale
+    order = torch.sort(chosen.flatten(), stable=True).indices
+    index = torch.empty_like(order)
+    index[order] = torch.arange(n * k)
+    offsets = torch.cat([torch.zeros(1, dtype=torch.long), torch.bincount(chosen.flatten(), minlength=E).cumsum(0)])
+    return Routing(index.view(n, k).int(), w, (order // k).int(), offsets.int())
+
+
+def run(h: torch.Tensor, e: Experts) -> ExpertRows:
+    """``h [n, W]`` through its tokens' experts."""
+    r = route(h, e)
+    n, W = h.shape
+    rows, F, E = n * e.top, e.down.shape[2], e.count
+    if h.is_cuda:
+        act = torch.empty(rows, F, dtype=h.dtype, device=h.device)
+        y = torch.empty(rows, W, dtype=h.dtype, device=h.device)
+        bf16, st, status = int(h.dtype == torch.bfloat16), _st(h), _status(h.device).data_ptr()
+        assert h.stride(1) == 1 and e.gate_up.dtype == h.dtype
+        N.check(N.lib().ptb_expert_gemm_simt(h.data_ptr(), r.token.data_ptr(), h.stride(0), e.gate_up.data_ptr(), 1, act.data_ptr(), r.offsets.data_ptr(), rows, E, F, W,
+                                             bf16, status, st), "expert_gemm")
+        N.check(N.lib().ptb_expert_gemm_simt(act.data_ptr(), 0, F, e.down.data_ptr(), 0, y.data_ptr(), r.offsets.data_ptr(), rows, E, W, F, bf16, status, st),
+                "expert_gemm")
+        return ExpertRows(y, r.index, r.weight)
+    x, at = h.float()[r.token.long()], r.offsets.tolist()
+    y = torch.zeros(rows, W)
+    for i in range(E):
+        lo, hi = at[i], at[i + 1]
+        if lo < hi:
+            g, u = (x[lo:hi] @ e.gate_up[i].float().t()).split([F, F], -1)
+            y[lo:hi] = (torch.nn.functional.silu(g) * u) @ e.down[i].float().t()
+    return ExpertRows(y.to(h.dtype), r.index, r.weight)

@@ -1,5 +1,5 @@
 """Recurrent layers with a matrix state per head (csrc/recurrence.cu, csrc/recurrence_chunk.cu): linear attention with a fixed decay,
-the gated delta rule with a decay per key channel, and the short causal convolution and the gated norm that go with them.
+the gated delta rule with a decay per key channel or per head, and the short causal convolution and the gated norm that go with them.
 
 A sequence's state is one slot of ``[slots, H, dim, vdim]`` fp32 (and ``[slots, taps - 1, channels]`` of convolution inputs); a token
 at position 0 starts from zero whatever the slot holds.  A decode pass gives one token per row (``seqs`` None: slot ``req[i]``,
@@ -36,7 +36,7 @@ def _decls(L):
     L.ptb_short_conv.restype = ci
     L.ptb_recurrence.argtypes = [C.POINTER(RecurrenceArgs), vp]
     L.ptb_recurrence.restype = ci
-    L.ptb_group_norm_gate.argtypes = [vp, vp, vp, ci, ll, vp, ci, ci, ci, cf, ci, vp]
+    L.ptb_group_norm_gate.argtypes = [vp, vp, vp, ci, ll, vp, ci, ci, ci, cf, ci, ci, vp]
     L.ptb_group_norm_gate.restype = ci
     L.ptb_recurrence_chunked.argtypes = [C.POINTER(RecurrenceArgs), vp, ll, vp]
     L.ptb_recurrence_chunked.restype = ci
@@ -113,13 +113,15 @@ def short_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, pos: 
 @dataclass
 class DeltaRule:
     """The gated delta rule of one layer: per head ``S <- g S; S <- S + k (beta (v - S^T k))^T; o = S^T q`` with q and k made unit
-    vectors (q also times dim^-1/2), ``beta`` a sigmoid and ``g = exp(-rate softplus(a + dt_bias))`` per head and key channel."""
+    vectors (q also times dim^-1/2), ``beta`` a sigmoid and ``g = exp(-rate softplus(a + dt_bias))`` per head and key channel, or with
+    ``head_decay`` one number per head."""
     heads: int
     kv_heads: int
     dim: int
     vdim: int
     rate: torch.Tensor                 # [H] fp32: exp(A_log)
-    dt_bias: torch.Tensor              # [H dim] fp32
+    dt_bias: torch.Tensor              # [H dim] fp32 ([H] with head_decay)
+    head_decay: bool = False
 
 
 @dataclass
@@ -160,8 +162,8 @@ def _run(args: RecurrenceArgs, x: torch.Tensor, seqs: Optional[Sequences], pos, 
 def delta_rule(x: torch.Tensor, r: DeltaRule, beta: torch.Tensor, a: Union[torch.Tensor, Tuple[torch.Tensor, torch.Tensor]], state: torch.Tensor,
                pos: torch.Tensor, req: torch.Tensor, seqs: Optional[Sequences] = None, chunked: Optional[bool] = None) -> torch.Tensor:
     """``x [n, 2 G dim + H vdim]``: q, k and v after their convolutions; ``beta [n, H]`` before its sigmoid (type of x); ``a [n, H
-    dim]`` fp32, or its factors ``(low [n, rank], w [>= H dim, rank])`` in the type of x, whose product the chunk kernel forms itself.
-    Advances ``state [slots, H, dim, vdim]``; returns o ``[n, H vdim]`` fp32."""
+    dim]`` fp32, or its factors ``(low [n, rank], w [>= H dim, rank])`` in the type of x, whose product the chunk kernel forms itself; one
+    decay per head: ``a [n, H]`` in the type of x.  Advances ``state [slots, H, dim, vdim]``; returns o ``[n, H vdim]`` fp32."""
     n, H, G, D, Dv = x.shape[0], r.heads, r.kv_heads, r.dim, r.vdim
     out = torch.empty(n, H * Dv, dtype=torch.float32, device=x.device)
     if x.is_cuda:
@@ -170,7 +172,10 @@ def delta_rule(x: torch.Tensor, r: DeltaRule, beta: torch.Tensor, a: Union[torch
         chunked = _runs_chunked(x, D, Dv, seqs, chunked)
         args = RecurrenceArgs(q_col=0, k_col=G * D, v_col=2 * G * D, delta=1, beta=beta.data_ptr(), ld_beta=beta.stride(0), decay=r.rate.data_ptr(),
                               dt_bias=r.dt_bias.data_ptr(), H=H, G=G, D=D, Dv=Dv)
-        if isinstance(a, tuple):
+        if r.head_decay:
+            assert a.dtype == x.dtype and a.shape[1] == H and a.stride(1) == 1
+            args.delta, args.a, args.ld_a = 2, a.data_ptr(), a.stride(0)
+        elif isinstance(a, tuple):
             low, w = a
             rank = w.shape[1]
             if chunked and rank % 8 == 0 and rank <= 256 and low.stride(0) % 8 == 0 and low.data_ptr() % 16 == 0 and w.is_contiguous():
@@ -179,7 +184,7 @@ def delta_rule(x: torch.Tensor, r: DeltaRule, beta: torch.Tensor, a: Union[torch
             else:
                 from .residual import linear_f32
                 a = linear_f32(low, w)
-        if not isinstance(a, tuple):
+        if not isinstance(a, tuple) and not r.head_decay:
             assert a.dtype == torch.float32 and a.stride(1) == 1
             args.a, args.ld_a = a.data_ptr(), a.stride(0)
         _run(args, x, seqs, pos, req, state, out, chunked)
@@ -190,7 +195,7 @@ def delta_rule(x: torch.Tensor, r: DeltaRule, beta: torch.Tensor, a: Union[torch
     q = (_unit(f[:, :G * D].reshape(n, G, D)) * D ** -0.5).repeat_interleave(H // G, 1)
     k = _unit(f[:, G * D:2 * G * D].reshape(n, G, D)).repeat_interleave(H // G, 1)
     v = f[:, 2 * G * D:].reshape(n, H, Dv)
-    g = torch.exp(-r.rate[:, None] * torch.nn.functional.softplus(a.float() + r.dt_bias, threshold=50.0).view(n, H, D))
+    g = torch.exp(-r.rate[:, None] * torch.nn.functional.softplus(a.float() + r.dt_bias, threshold=50.0).view(n, H, -1))       # [n, H, D or 1]
     b = torch.sigmoid(beta.float())
     o = out.view(n, H, Dv)
     for lo, count, at, slot in (seqs or Sequences.of_rows(pos, req)).host:
@@ -229,17 +234,17 @@ def decay_attention(x: torch.Tensor, r: DecayAttention, cols: Tuple[int, int, in
 
 
 # ------------------------------------------------------------------------------------------ output norm and gate
-def group_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, dtype) -> torch.Tensor:
-    """``o [n, K]`` fp32 in groups of ``len(weight)`` columns: RMS norm of every group times the fp32 ``weight``, times the sigmoid
-    of ``gate [n, K]`` (any row pitch; bf16 or fp32).  Returns ``[n, K]`` in ``dtype``."""
+def group_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, dtype, act: str = "sigmoid") -> torch.Tensor:
+    """``o [n, K]`` fp32 in groups of ``len(weight)`` columns: RMS norm of every group times the fp32 ``weight``, times the sigmoid (or
+    ``act="silu"``) of ``gate [n, K]`` (any row pitch; bf16 or fp32).  Returns ``[n, K]`` in ``dtype``."""
     n, K = o.shape
     gs = weight.shape[0]
     if o.is_cuda:
         out = torch.empty(n, K, dtype=dtype, device=o.device)
         assert o.is_contiguous() and gate.stride(1) == 1
         N.check(N.lib().ptb_group_norm_gate(o.data_ptr(), weight.data_ptr(), gate.data_ptr(), int(gate.dtype == torch.bfloat16), gate.stride(0),
-                                            out.data_ptr(), n, K // gs, gs, float(eps), int(dtype == torch.bfloat16), _st(o)), "group_norm_gate")
+                                            out.data_ptr(), n, K // gs, gs, float(eps), int(act == "silu"), int(dtype == torch.bfloat16), _st(o)), "group_norm_gate")
         return out
     x = o.float().reshape(n, K // gs, gs)
     y = (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * weight).reshape(n, K)
-    return (y * torch.sigmoid(gate.float())).to(dtype)
+    return (y * (torch.nn.functional.silu if act == "silu" else torch.sigmoid)(gate.float())).to(dtype)
