@@ -488,6 +488,15 @@ PTB_API int ptb_proj_norm_write(const void* x, long long ld, int q_col, int k_co
     return 0;
 }
 
+// Joins the splits and maps that row kernels left in a.work.
+int ptb_window_merge(const PtbWindowAttn& a, cudaStream_t st) {
+    auto merge = a.bf16 ? (a.maps > 1 ? window_merge_kernel<__nv_bfloat16, 2> : window_merge_kernel<__nv_bfloat16, 1>)
+                        : (a.maps > 1 ? window_merge_kernel<float, 2> : window_merge_kernel<float, 1>);
+    PTB_CUDA_OK(ptb_launch(merge, dim3(a.H, a.n), dim3(128), 0, st, ptb_pdl_enabled(), a));
+    PTB_CUDA_OK(cudaGetLastError());
+    return 0;
+}
+
 // Floats of workspace the row kernels need (heads: H times the number of maps) where nsplit or the number of maps is above one.
 PTB_API long long ptb_window_rows_work_floats(int n, int heads, int Dvp, int nsplit) { return (long long)n * nsplit * heads * (Dvp + 2); }
 
@@ -520,11 +529,5 @@ PTB_API int ptb_window_attn_rows(const PtbWindowAttn* args, cudaStream_t st) {
     if (L.total > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     const bool pdl = ptb_pdl_enabled();
     PTB_CUDA_OK(ptb_launch(kern, dim3(a.nsplit, a.G * p.groups, a.n), dim3(WR_THREADS), (size_t)L.total, st, pdl, p));
-    if (merged) {
-        auto merge = a.bf16 ? (a.maps > 1 ? window_merge_kernel<__nv_bfloat16, 2> : window_merge_kernel<__nv_bfloat16, 1>)
-                            : (a.maps > 1 ? window_merge_kernel<float, 2> : window_merge_kernel<float, 1>);
-        PTB_CUDA_OK(ptb_launch(merge, dim3(a.H, a.n), dim3(128), 0, st, pdl, a));
-    }
-    PTB_CUDA_OK(cudaGetLastError());
-    return 0;
+    return merged ? ptb_window_merge(a, st) : 0;
 }

@@ -246,7 +246,7 @@ class BudoraxWeights:
         g = torch.Generator(device=device).manual_seed(seed)
 
         def r(*s, scale=1.0, at=0.0):
-            return (at + torch.randn(*s, generator=g, device=device) * scale).to(dtype)
+            return (at + torch.randn(s, generator=g, device=device) * scale).to(dtype)
 
         def one(name, s):
             if name.endswith(".alpha"):
@@ -416,7 +416,7 @@ class PagedBudorax(PagedModel):
             return A.window_attention(q, a, batch.pos, batch.req, page_table, k, v, ns, top)
 
         def attend_latent(a, q, pages, gate):
-            if M.tiles_pay(q, a, batch.offs[-1], top):
+            if M.tiles_pay(q, a, batch.offs[-1]):
                 if not context:
                     context.append(M.PromptContext.of(batch.offs, batch.starts, batch.rows, self.device))
                 return M.latent_attention_tiles(q, a, context[0], batch.pos, page_table, pages, gate)

@@ -23,7 +23,9 @@ def _decls(L):
     vp, ci, cf, ll = C.c_void_p, C.c_int, C.c_float, C.c_longlong
     L.ptb_expert_route.argtypes = [vp, ci, ll, ll, vp, ci, ci, ci, cf, vp, vp, vp, vp, vp, vp, vp]
     L.ptb_expert_gemm_simt.argtypes = [vp, vp, ll, vp, ci, vp, vp, ci, ci, ci, ci, ci, vp, vp]
-    for n in ("ptb_expert_route", "ptb_expert_gemm_simt"):
+    L.ptb_expert_gather.argtypes = [vp, ll, vp, vp, ci, ci, ci, vp, vp]
+    L.ptb_expert_gemm.argtypes = [vp, ll, vp, ci, vp, vp, ci, ci, ci, ci, ci, ci, vp, vp]
+    for n in ("ptb_expert_route", "ptb_expert_gemm_simt", "ptb_expert_gather", "ptb_expert_gemm"):
         getattr(L, n).restype = ci
 
 
@@ -89,21 +91,30 @@ def route(h: torch.Tensor, e: Experts) -> Routing:
     return Routing(index.view(n, k).int(), w, (order // k).int(), offsets.int())
 
 
-def run(h: torch.Tensor, e: Experts) -> ExpertRows:
-    """``h [n, W]`` through its tokens' experts."""
-    r = route(h, e)
+FEW_ROWS = 48                          # mean rows of an expert below which its weights are the 128-row operand
+
+
+def products(h: torch.Tensor, e: Experts, r: Routing, simt: bool = False) -> torch.Tensor:
+    """The experts over their rows: ``[n top, W]`` in the order by expert.  bf16 rows of a multiple of eight go to the tensor cores;
+    everything else, or all with ``simt``, to the kernel that takes any size."""
     n, W = h.shape
     rows, F, E = n * e.top, e.down.shape[2], e.count
     if h.is_cuda:
-        act = torch.empty(rows, F, dtype=h.dtype, device=h.device)
-        y = torch.empty(rows, W, dtype=h.dtype, device=h.device)
-        bf16, st, status = int(h.dtype == torch.bfloat16), _st(h), _status(h.device).data_ptr()
+        bf16, st, status = h.dtype == torch.bfloat16, _st(h), _status(h.device).data_ptr()
+        act, y = torch.empty(rows, F, dtype=h.dtype, device=h.device), torch.empty(rows, W, dtype=h.dtype, device=h.device)
         assert h.stride(1) == 1 and e.gate_up.dtype == h.dtype
+        if bf16 and W % 8 == 0 and h.stride(0) % 8 == 0 and not simt:
+            x = torch.empty(rows, W, dtype=h.dtype, device=h.device)
+            few = int(rows < FEW_ROWS * E)
+            N.check(N.lib().ptb_expert_gather(h.data_ptr(), h.stride(0), r.token.data_ptr(), x.data_ptr(), rows, W, n, status, st), "expert_gather")
+            N.check(N.lib().ptb_expert_gemm(x.data_ptr(), W, e.gate_up.data_ptr(), 1, act.data_ptr(), r.offsets.data_ptr(), rows, E, F, W, few, 0, status, st), "expert_gemm")
+            N.check(N.lib().ptb_expert_gemm(act.data_ptr(), F, e.down.data_ptr(), 0, y.data_ptr(), r.offsets.data_ptr(), rows, E, W, F, few, 0, status, st), "expert_gemm")
+            return y
         N.check(N.lib().ptb_expert_gemm_simt(h.data_ptr(), r.token.data_ptr(), h.stride(0), e.gate_up.data_ptr(), 1, act.data_ptr(), r.offsets.data_ptr(), rows, E, F, W,
-                                             bf16, status, st), "expert_gemm")
-        N.check(N.lib().ptb_expert_gemm_simt(act.data_ptr(), 0, F, e.down.data_ptr(), 0, y.data_ptr(), r.offsets.data_ptr(), rows, E, W, F, bf16, status, st),
-                "expert_gemm")
-        return ExpertRows(y, r.index, r.weight)
+                                             int(bf16), status, st), "expert_gemm_simt")
+        N.check(N.lib().ptb_expert_gemm_simt(act.data_ptr(), 0, F, e.down.data_ptr(), 0, y.data_ptr(), r.offsets.data_ptr(), rows, E, W, F, int(bf16), status, st),
+                "expert_gemm_simt")
+        return y
     x, at = h.float()[r.token.long()], r.offsets.tolist()
     y = torch.zeros(rows, W)
     for i in range(E):
@@ -111,4 +122,10 @@ def run(h: torch.Tensor, e: Experts) -> ExpertRows:
         if lo < hi:
             g, u = (x[lo:hi] @ e.gate_up[i].float().t()).split([F, F], -1)
             y[lo:hi] = (torch.nn.functional.silu(g) * u) @ e.down[i].float().t()
-    return ExpertRows(y.to(h.dtype), r.index, r.weight)
+    return y.to(h.dtype)
+
+
+def run(h: torch.Tensor, e: Experts) -> ExpertRows:
+    """``h [n, W]`` through its tokens' experts."""
+    r = route(h, e)
+    return ExpertRows(products(h, e, r), r.index, r.weight)

@@ -28,7 +28,10 @@ def _decls(L):
     vp, ci, cf, ll = C.c_void_p, C.c_int, C.c_float, C.c_longlong
     L.ptb_latent_write.argtypes = [vp, ll, ci, ci, ci, ci, ci, vp, vp, cf, vp, vp, ci, vp, vp, ci, ci, vp, ci, vp, ci, vp, ci, ci, ci, vp, ci, vp]
     L.ptb_head_linear.argtypes = [vp, ll, ci, vp, ci, ci, ci, vp, ll, ci, ci, vp, ll, ci, ci, vp, vp, ci, vp, ci, vp, ci, vp]
-    for n in ("ptb_latent_write", "ptb_head_linear"):
+    L.ptb_latent_gather.argtypes = [vp, ci, ci, vp, ci, ci, vp, ci, vp, ci, vp, vp]
+    L.ptb_latent_q.argtypes = [vp, ll, vp, ci, ci, ci, ci, ci, vp, vp, ci, ci, vp, ci, vp, vp]
+    L.ptb_latent_attn_rows.argtypes = [C.POINTER(A.WindowArgs), vp]
+    for n in ("ptb_latent_write", "ptb_head_linear", "ptb_latent_gather", "ptb_latent_q", "ptb_latent_attn_rows"):
         getattr(L, n).restype = ci
 
 
@@ -115,6 +118,16 @@ def unfold_values(o: torch.Tensor, a: LatentAttention, gate: Optional[torch.Tens
 HEADS_PER_CTA = 32                     # of the row kernels
 
 
+def _runs_mma(q: torch.Tensor, a: LatentAttention) -> bool:
+    """Whether the kernel of csrc/latent_attn.cu takes these rows: latents up to 512 and their shared part fit its registers and rings."""
+    return q.dtype == torch.bfloat16 and a.rank_stored <= 512 and a.row <= 640
+
+
+def pick_splits(rows: int, heads: int, keys: int, sms: int = 148) -> int:
+    """CTAs that share a row's keys in the tensor-core kernel, which walks any number of pages: as many as fill the machine once."""
+    return max(1, min(-(-keys // PAGE), sms // max(1, rows * -(-heads // HEADS_PER_CTA))))
+
+
 def latent_attention(q: torch.Tensor, a: LatentAttention, pos: torch.Tensor, req: torch.Tensor, page_table: torch.Tensor, pages: torch.Tensor,
                      max_len: int, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Rows ``q [n, >= H (dim + rot_dim)]`` (as projected) at ``pos`` against the cached rows of their sequences, their own included;
@@ -127,27 +140,70 @@ def latent_attention(q: torch.Tensor, a: LatentAttention, pos: torch.Tensor, req
     args = A.WindowArgs(k_pages=pages.data_ptr(), v_pages=pages.data_ptr(), page_table=page_table.data_ptr(), pt_stride=page_table.stride(0), n_pages=pages.shape[0],
                         H=H, G=1, D=a.row, Dp=a.row, Dv=a.rank_stored, Dvp=a.rank_stored, v_ld=a.row, maps=1, window=A.UNBOUNDED, keep=0, chunked=0,
                         scale=float(a.scale), bf16=int(q.dtype == torch.bfloat16), status=_status(q.device).data_ptr(), max_keys=max(1, max_len))
-    A.run_rows(args, qs, o, pos, req, A.pick_splits(n, -(-H // HEADS_PER_CTA), max_len))
+    if _runs_mma(q, a):
+        A.run_rows(args, qs, o, pos, req, pick_splits(n, H, max_len), kernel=N.lib().ptb_latent_attn_rows)
+    else:
+        splits = A.pick_splits(n, -(-H // HEADS_PER_CTA), max_len)
+        if q.dtype == torch.bfloat16 and a.rank_stored > 512:                # a CTA's values have to fit its shared memory
+            splits = max(splits, -(-max_len // 32))
+        A.run_rows(args, qs, o, pos, req, splits)
     return unfold_values(o, a, gate)
 
 
 @dataclass
 class PromptContext:
-    """Where the context of every sequence of a prompt pass lies in the flat keys and values of that pass."""
-    tiles: A.PromptTiles
+    """The context of the sequences of a prompt pass, cached tokens included, laid out one after the other: the pages it comes from
+    (``[pieces, 4]`` int32: first row, row of the page table, page of the sequence, rows) and the query tiles with the first row of their
+    sequence's context."""
     rows: int
+    pieces: torch.Tensor
+    tiles: torch.Tensor
 
     @classmethod
     def of(cls, offs: List[int], starts: List[int], rows: List[int], device) -> "PromptContext":
-        raise NotImplementedError
+        pieces, tiles, base = [], [], 0
+        for lo, hi, at, r in zip(offs, offs[1:], starts, rows):
+            total = at + hi - lo
+            pieces += [(base + j, r, j // PAGE, min(PAGE, total - j)) for j in range(0, total, PAGE)]
+            tiles += [(lo + i, at + i, min(A.QUERY_TILE, hi - lo - i), base) for i in range(0, hi - lo, A.QUERY_TILE)]
+            base += total
+        tiles.sort(key=lambda t: -t[1])
+        up = lambda t: torch.tensor(t, dtype=torch.int32).to(device)
+        return cls(base, up(pieces), up(tiles))
 
 
-def tiles_pay(q: torch.Tensor, a: LatentAttention, rows: int, max_len: int) -> bool:
-    return False
+TILES_FROM = 32                        # rows of a prompt pass from which keys and values are formed
 
 
-def latent_attention_tiles(q, a, context, pos, page_table, pages, gate):
-    raise NotImplementedError
+def tiles_supported(a: LatentAttention) -> bool:
+    return A.stored(a.dim) <= 128 and A.stored(a.rot_dim) <= 64 and A.stored(a.vdim) <= 128
+
+
+def tiles_pay(q: torch.Tensor, a: LatentAttention, rows: int) -> bool:
+    return q.is_cuda and q.dtype == torch.bfloat16 and rows >= TILES_FROM and tiles_supported(a)
+
+
+def latent_attention_tiles(q: torch.Tensor, a: LatentAttention, context: PromptContext, pos: torch.Tensor, page_table: torch.Tensor, pages: torch.Tensor,
+                           gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """A prompt pass's rows ``q [n, >= H (dim + rot_dim)]`` (as projected) against the whole context of their sequences, on tcgen05."""
+    from .gemm import linear
+    n, H, status = q.shape[0], a.heads, _status(q.device).data_ptr()
+    flat = torch.empty(context.rows, a.row, dtype=q.dtype, device=q.device)
+    N.check(N.lib().ptb_latent_gather(pages.data_ptr(), pages.shape[0], a.row, page_table.data_ptr(), page_table.stride(0), page_table.shape[0], context.pieces.data_ptr(),
+                                      context.pieces.shape[0], flat.data_ptr(), context.rows, status, _st(q)), "latent_gather")
+    kv = linear(flat[:, :a.rank_stored], a.prompt)
+    Dp, Dvp, Rp = A.stored(a.dim), A.stored(a.vdim), A.stored(a.rot_dim)
+    Do = -(-Dp // 64) * 64
+    qs = torch.empty(n, H, Do + Rp, dtype=q.dtype, device=q.device)
+    N.check(N.lib().ptb_latent_q(q.data_ptr(), q.stride(0), qs.data_ptr(), n, H, a.dim, Do, Rp, N.ptr(a.rotary.cos), N.ptr(a.rotary.sin), a.rot_dim, a.rotary.positions,
+                                 pos.data_ptr(), pos.stride(0), status, _st(q)), "latent_q")
+    out = torch.empty(n, H * a.vdim, dtype=q.dtype, device=q.device)
+    args = A.WindowArgs(q=qs.data_ptr(), out=out.data_ptr(), k_pages=kv.data_ptr(), v_pages=kv[:, H * Dp:].data_ptr(), k_rot=flat[:, a.rank_stored:].data_ptr(),
+                        k_ld=kv.stride(0), v_row=kv.stride(0), rot_ld=a.row, gate=N.ptr(gate), gate_ld=gate.stride(0) if gate is not None else 0,
+                        tiles=context.tiles.data_ptr(), n_tiles=context.tiles.shape[0], n=n, H=H, G=H, D=a.dim, Dp=Dp, Dv=a.vdim, Dvp=Dvp, v_ld=Dvp, maps=1,
+                        window=A.UNBOUNDED, scale=float(a.scale), bf16=1, flat_rows=context.rows, rot_dim=a.rot_dim, status=status)
+    N.check(N.lib().ptb_window_attn_tiles(C.byref(args), _st(q)), "window_attn_tiles")
+    return out
 
 
 def latent_attention_reference(q, a: LatentAttention, pos, req, page_table, pages, gate=None) -> torch.Tensor:

@@ -161,8 +161,9 @@ def _args(q: torch.Tensor, a: WindowAttention, page_table: torch.Tensor, k_pages
                       bf16=int(q.dtype == torch.bfloat16), status=_status(q.device).data_ptr())
 
 
-def run_rows(args: WindowArgs, q: torch.Tensor, out: torch.Tensor, pos: torch.Tensor, req: torch.Tensor, nsplit: int, gate=None) -> torch.Tensor:
-    """The row kernels over all rows of ``q``, in launches whose workspace stays bounded."""
+def run_rows(args: WindowArgs, q: torch.Tensor, out: torch.Tensor, pos: torch.Tensor, req: torch.Tensor, nsplit: int, gate=None,
+             kernel=None) -> torch.Tensor:
+    """The row kernels over all rows of ``q``, in launches whose workspace stays bounded; ``kernel``: another entry point than the usual."""
     n = q.shape[0]
     st = torch.cuda.current_stream(q.device).cuda_stream
     merged = nsplit > 1 or args.maps > 1
@@ -175,7 +176,7 @@ def run_rows(args: WindowArgs, q: torch.Tensor, out: torch.Tensor, pos: torch.Te
         args.q, args.out, args.pos, args.req = q[lo:].data_ptr(), out[lo:].data_ptr(), pos[lo:].data_ptr(), req[lo:].data_ptr()
         if gate is not None:
             args.gate = gate[lo:].data_ptr()
-        N.check(N.lib().ptb_window_attn_rows(C.byref(args), st), "window_attn_rows")
+        N.check((kernel or N.lib().ptb_window_attn_rows)(C.byref(args), st), "attention rows")
     return out
 
 
