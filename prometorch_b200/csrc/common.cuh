@@ -117,6 +117,12 @@ __device__ __forceinline__ void bulk_g2s(void* dst, const void* src, uint32_t by
 }
 __device__ __forceinline__ void fence_proxy_async() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
 
+// Two neighbouring 16-byte stores as one: a thread that owns a row fills whole 32-byte sectors.  p is 32-byte aligned.
+__device__ __forceinline__ void st_global_32(void* p, const uint4& a, const uint4& b) {
+    asm volatile("st.global.v8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(p), "r"(a.x), "r"(a.y), "r"(a.z), "r"(a.w), "r"(b.x), "r"(b.y), "r"(b.z), "r"(b.w)
+                 : "memory");
+}
+
 // ---- programmatic dependent launch ---------------------------------------
 // wait: block until the preceding kernel in the stream has completed and its
 // writes are visible.  launch_dependents: allow the next kernel to begin its

@@ -3,6 +3,7 @@
 //                       token's rank among an expert's rows (counted in shared memory, then once per CTA and expert in global memory);
 //   place_kernel        prefix sums of the counts: the place of every (token, expert) pair in the order by expert, and back;
 //   route_small_kernel  both for few tokens in one CTA;
+//   route_rows_kernel   the router's product as well, for few tokens;
 //   expert_simt_kernel  a grouped product over the sorted rows with FMAs in fp32 (fp32 models, sizes the tensor-core kernel cannot address).
 // Where a row lies inside its expert depends on the order of atomics; what is computed for it does not.
 #include "common.cuh"
@@ -30,15 +31,22 @@ struct Route {
     int* status;
 };
 
-// One warp: choice scores of token i into c_s, its `top` experts in order to (e, w) by lane 0 of the callback.
-template <typename F>
-__device__ __forceinline__ void choose(const Route& R, int i, float* c_s, F chosen) {
-    const int lane = threadIdx.x & 31;
-    for (int e = lane; e < R.E; e += 32) {
+// The logit of token i and expert e.
+struct Logits {
+    const Route& R;
+    int i;
+    __device__ __forceinline__ float operator()(int e) const {
         float z = 0.f;
         for (int s = 0; s < R.splits; ++s) z += R.z[s * R.stride + (size_t)i * R.ld + e];
-        c_s[e] = sigmoid(z) + R.correction[e];
+        return z;
     }
+};
+
+// One warp: choice scores of token i into c_s, its `top` experts in order to (e, w) by lane 0 of the callback.
+template <typename Z, typename F>
+__device__ __forceinline__ void choose(const Route& R, int i, float* c_s, Z logit, F chosen) {
+    const int lane = threadIdx.x & 31;
+    for (int e = lane; e < R.E; e += 32) c_s[e] = sigmoid(logit(e)) + R.correction[e];
     __syncwarp();
     float sum = 0.f, mine = 0.f;                       // lane k keeps the score of the k-th expert (and of k + 32, ... in turn)
     for (int k = 0; k < R.top; ++k) {
@@ -53,9 +61,7 @@ __device__ __forceinline__ void choose(const Route& R, int i, float* c_s, F chos
             if (b > best || (b == best && a < at)) { best = b; at = a; }
         }
         if (at >= R.E) at = k;                         // scores that are not numbers: any expert will do
-        float z = 0.f;
-        for (int s = 0; s < R.splits; ++s) z += R.z[s * R.stride + (size_t)i * R.ld + at];
-        const float score = sigmoid(z);
+        const float score = sigmoid(logit(at));
         sum += score;
         if (lane == (k & 31)) mine = score;
         __syncwarp();
@@ -64,14 +70,12 @@ __device__ __forceinline__ void choose(const Route& R, int i, float* c_s, F chos
             chosen(k, at);
         }
         __syncwarp();
-        if ((k & 31) == 31 || k + 1 == R.top) {        // unscaled for now: the sum is not known before the last
-            const int k0 = k & ~31;
-            if (k0 + lane <= k) R.weight[(size_t)i * R.top + k0 + lane] = mine;
-        }
+        if ((k & 31) == 31 && k + 1 < R.top) R.weight[(size_t)i * R.top + k - 31 + lane] = mine;      // unscaled: the sum is not known yet
     }
     const float f = R.scale / (sum + 1e-20f);
-    __syncwarp();
-    for (int k = lane; k < R.top; k += 32) R.weight[(size_t)i * R.top + k] *= f;
+    const int k0 = (R.top - 1) & ~31;                  // the last ones are still in registers
+    for (int k = lane; k < k0; k += 32) R.weight[(size_t)i * R.top + k] *= f;
+    if (k0 + lane < R.top) R.weight[(size_t)i * R.top + k0 + lane] = mine * f;
 }
 
 __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const __grid_constant__ Route R) {
@@ -86,7 +90,7 @@ __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const __grid_const
     __syncthreads();
     const int i = blockIdx.x * RT_WARPS + warp;
     if (i < R.n)
-        choose(R, i, c_s, [&](int k, int e) {
+        choose(R, i, c_s, Logits{R, i}, [&](int k, int e) {
             R.expert[(size_t)i * R.top + k] = e;
             R.rank[(size_t)i * R.top + k] = atomicAdd(&count[e], 1);
         });
@@ -146,7 +150,7 @@ __global__ void __launch_bounds__(RS_WARPS * 32) route_small_kernel(const __grid
     pdl_launch_dependents();
     __syncthreads();
     for (int i = warp; i < R.n; i += RS_WARPS)
-        choose(R, i, c_s, [&](int k, int e) {
+        choose(R, i, c_s, Logits{R, i}, [&](int k, int e) {
             R.expert[(size_t)i * R.top + k] = e;
             R.rank[(size_t)i * R.top + k] = atomicAdd(&count[e], 1);
         });
@@ -156,6 +160,69 @@ __global__ void __launch_bounds__(RS_WARPS * 32) route_small_kernel(const __grid
     for (int e = threadIdx.x; e <= R.E; e += blockDim.x) R.offsets[e] = off[e];
     for (int p = threadIdx.x; p < R.n * R.top; p += blockDim.x) {
         const int at = off[R.expert[p]] + R.rank[p];
+        R.index[p] = at;
+        R.token[at] = p / R.top;
+    }
+}
+
+constexpr int RR_THREADS = 128, RR_WARPS = RR_THREADS / 32;
+
+// CTA (x, token): every gridDim.x-th group of RR_WARPS experts, a warp per expert.  Of a token's CTAs the last one to finish chooses; of the
+// tokens the last one puts all pairs in order.  h [n][W] of pitch ldh, w [E][W], both bf16 or fp32; z [n][E].  done [n + 1]: zero before
+// and after.
+template <typename T>
+__global__ void __launch_bounds__(RR_THREADS) route_rows_kernel(const __grid_constant__ Route R, const T* __restrict__ h, long long ldh, const T* __restrict__ w, int W,
+                                                                float* z, unsigned* done) {
+    extern __shared__ float c_s[];                     // [E], later counts [E] and offsets [E + 1]
+    __shared__ int last;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, i = blockIdx.y;
+    constexpr int V = 16 / sizeof(T);                  // elements of a 16-byte load
+    const bool vec = W % V == 0 && ldh % V == 0 && (((uintptr_t)w | (uintptr_t)h) & 15) == 0;
+    pdl_wait();
+    pdl_launch_dependents();
+    const T* x = h + (size_t)i * ldh;
+    for (int e = blockIdx.x * RR_WARPS + warp; e < R.E; e += gridDim.x * RR_WARPS) {
+        const T* row = w + (size_t)e * W;
+        float a = 0.f;
+        if (vec) {
+#pragma unroll 8
+            for (int c = lane * V; c < W; c += 32 * V) {
+                const uint4 p = *reinterpret_cast<const uint4*>(row + c), q = *reinterpret_cast<const uint4*>(x + c);
+                const T* u = reinterpret_cast<const T*>(&p);
+                const T* v = reinterpret_cast<const T*>(&q);
+#pragma unroll
+                for (int k = 0; k < V; ++k) a = fmaf((float)u[k], (float)v[k], a);
+            }
+        } else
+            for (int c = lane; c < W; c += 32) a = fmaf((float)row[c], (float)x[c], a);
+        a = warp_sum(a);
+        if (lane == 0) z[(size_t)i * R.E + e] = a;
+    }
+    auto finished = [&](unsigned* counter, unsigned of) {          // whether this CTA is the last of `of` to come here
+        __threadfence();
+        __syncthreads();
+        if (threadIdx.x == 0) {
+            last = atomicAdd(counter, 1u) == of - 1;
+            if (last) *counter = 0;
+        }
+        __syncthreads();
+        if (last) __threadfence();
+        return last != 0;
+    };
+    if (!finished(done + i, gridDim.x)) return;
+    if (warp == 0) choose(R, i, c_s, [&](int e) { return __ldcg(z + (size_t)i * R.E + e); }, [&](int k, int e) { R.expert[(size_t)i * R.top + k] = e; });
+    if (!finished(done + R.n, gridDim.y)) return;
+    int *count = reinterpret_cast<int*>(c_s), *off = count + R.E;
+    for (int e = threadIdx.x; e < R.E; e += RR_THREADS) count[e] = 0;
+    __syncthreads();
+    const int pairs = R.n * R.top;
+    for (int p = threadIdx.x; p < pairs; p += RR_THREADS) R.rank[p] = atomicAdd(&count[__ldcg(R.expert + p)], 1);
+    __syncthreads();
+    prefix(count, off, R.E);
+    __syncthreads();
+    for (int e = threadIdx.x; e <= R.E; e += RR_THREADS) R.offsets[e] = off[e];
+    for (int p = threadIdx.x; p < pairs; p += RR_THREADS) {
+        const int at = off[__ldcg(R.expert + p)] + R.rank[p];
         R.index[p] = at;
         R.token[at] = p / R.top;
     }
@@ -254,6 +321,27 @@ PTB_API int ptb_expert_route(const float* z, int splits, long long stride, long 
         PTB_CUDA_OK(ptb_launch(route_kernel, dim3((n + RT_WARPS - 1) / RT_WARPS), dim3(RT_WARPS * 32), ((size_t)RT_WARPS * E + 2 * E) * 4, st, false, r));
         PTB_CUDA_OK(ptb_launch(place_kernel, dim3((unsigned)std::min<size_t>(1024, (pairs + 255) / 256)), dim3(256), (size_t)(E + 1) * 4, st, pdl, r));
     }
+    PTB_CUDA_OK(cudaGetLastError());
+    return 0;
+}
+
+// The same from the rows themselves, for few tokens: h [n, W] (pitch ldh) and the router w [E, W], both bf16 or fp32.  work: 2 n top ints and n E floats;
+// done: n + 1 unsigned that are zero between calls, used by one stream at a time.
+PTB_API int ptb_expert_route_rows(const void* h, long long ldh, const void* w, int W, const float* correction, int n, int E, int top, float scale, int* index,
+                                  float* weight, int* token, int* offsets, int* work, unsigned* done, int bf16, cudaStream_t st) {
+    using namespace ptb::moe;
+    if (n <= 0) return 0;
+    const size_t pairs = (size_t)n * top;
+    if (E < 1 || top < 1 || top > E || E > 1024 || n > 65535 || W < 1) { ptb_set_error("experts: %d of %d experts (at most 1024), %d columns", top, E, W); return -1; }
+    const Route r{nullptr, 0, 0, 0, correction, n, E, top, scale, index, weight, token, offsets, work, work + pairs, nullptr, nullptr};
+    const bool pdl = ptb_pdl_enabled();
+    auto go = [&](auto k, auto t) {
+        using T = decltype(t);
+        const int groups = std::max(1, std::min((E + RR_WARPS - 1) / RR_WARPS, 148 * 8 / n));
+        return ptb_launch(k, dim3(groups, n), dim3(RR_THREADS), (2 * (size_t)E + 1) * 4, st, pdl, r, (const T*)h, ldh, (const T*)w, W,
+                          reinterpret_cast<float*>(work + 2 * pairs), done);
+    };
+    PTB_CUDA_OK(bf16 ? go(route_rows_kernel<__nv_bfloat16>, __nv_bfloat16()) : go(route_rows_kernel<float>, 0.f));
     PTB_CUDA_OK(cudaGetLastError());
     return 0;
 }

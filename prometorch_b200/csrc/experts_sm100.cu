@@ -171,6 +171,7 @@ __global__ void __launch_bounds__(THREADS, 1) expert_gemm_kernel(const __grid_co
         }
     } else {
         const int q = warp & 3;                        // tensor-memory lanes of this warp
+        const bool wide = P.N % 16 == 0 && ((uintptr_t)P.out & 31) == 0;
         bool ok = true;
         int tl = 0;
         for (int t = blockIdx.x; t < tiles && ok; t += gridDim.x, ++tl) {
@@ -208,16 +209,22 @@ __global__ void __launch_bounds__(THREADS, 1) expert_gemm_kernel(const __grid_co
                     tmem_ld_wait();
                     if (row < T.end) {
 #pragma unroll
-                        for (int j = 0; j < 32; j += 8) {      // N is a multiple of eight
-                            uint4 v;
-                            __nv_bfloat162* vh = reinterpret_cast<__nv_bfloat162*>(&v);
+                        for (int j = 0; j < 32; j += 16) {     // N is a multiple of eight
+                            uint4 v[2];
+                            __nv_bfloat162* vh = reinterpret_cast<__nv_bfloat162*>(v);
 #pragma unroll
-                            for (int i = 0; i < 4; ++i) {
+                            for (int i = 0; i < 8; ++i) {
                                 float x = __uint_as_float(g[j + 2 * i]), y = __uint_as_float(g[j + 2 * i + 1]);
                                 if constexpr (GATED) { x = silu(x) * __uint_as_float(u[j + 2 * i]); y = silu(y) * __uint_as_float(u[j + 2 * i + 1]); }
                                 vh[i] = __floats2bfloat162_rn(x, y);
                             }
-                            if (T.col + c + j < P.N) *reinterpret_cast<uint4*>(o + T.col + c + j) = v;
+                            __nv_bfloat16* dst = o + T.col + c + j;
+                            const int left = P.N - (T.col + c + j);
+                            if (left >= 16 && wide) st_global_32(dst, v[0], v[1]);
+                            else {
+                                if (left > 0) *reinterpret_cast<uint4*>(dst) = v[0];
+                                if (left > 8) *reinterpret_cast<uint4*>(dst + 8) = v[1];
+                            }
                         }
                     }
                 }

@@ -363,6 +363,8 @@ gemm_bf16_kernel(const __grid_constant__ Operand opA, const __grid_constant__ Op
     } else {
         // ------------------------------------------------------------------ epilogue (warps 2..5)
         const int q = warp & 3;                     // TMEM lane quarter this warp may read
+        // bf16 rows whose 64-byte pieces start on 32-byte boundaries go out in whole sectors
+        const bool wide = !(P.flags & (EPI_ACCUM | EPI_OUT_F32 | EPI_SCATTER_ADD | EPI_SCATTER_STORE | EPI_TRANS)) && P.ldc % 16 == 0 && ((uintptr_t)P.C & 31) == 0;
         int tl = 0;
         bool ok = true;
         for (int t = cta; t < num_tiles && ok; t += n_gemm, ++tl) {
@@ -439,7 +441,17 @@ gemm_bf16_kernel(const __grid_constant__ Operand opA, const __grid_constant__ Op
                         __nv_bfloat16* cp = reinterpret_cast<__nv_bfloat16*>(P.C) + (size_t)row * P.ldc + col;
                         if (col + 32 <= P.N) {
 #pragma unroll
+                            for (int j = 0; j < 32; j += 16) {
+                                if (!wide) break;
+                                uint4 o[2];
+                                __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(o);
+#pragma unroll
+                                for (int e = 0; e < 8; ++e) oh[e] = __floats2bfloat162_rn(v[j + 2 * e], v[j + 2 * e + 1]);
+                                st_global_32(cp + j, o[0], o[1]);
+                            }
+#pragma unroll
                             for (int j = 0; j < 32; j += 8) {
+                                if (wide) break;
                                 if (P.flags & EPI_ACCUM) {
                                     const uint4 pv = *reinterpret_cast<uint4*>(cp + j);
                                     const __nv_bfloat162* ph = reinterpret_cast<const __nv_bfloat162*>(&pv);

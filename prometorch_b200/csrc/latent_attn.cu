@@ -41,21 +41,24 @@ constexpr int HL_THREADS = 128, HL_ROWS = 4, HL_COLS = 32;
 // The columns of a head from N on for rows r0 .. r0 + rows: zeros up to rot_at, the rotated part, zeros.
 template <typename T>
 __device__ __forceinline__ void rotated_columns(const HeadLinear& P, int h, int r0, int rows) {
-    for (int e = threadIdx.x; e < rows * (P.os - P.N); e += HL_THREADS) {
-        const int r = r0 + e / (P.os - P.N), c = P.N + e % (P.os - P.N), d = c - P.rot_at;
-        float v = 0.f;
-        if (d >= 0 && d < P.rot) {
-            int pos = P.pos[(size_t)r * P.pos_stride];
-            if (pos < 0 || pos >= P.positions) {
-                if (P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
-                pos = 0;
-            }
-            const T* x = (const T*)P.x + (size_t)r * P.ldx + (size_t)h * P.xs + P.K;
-            const size_t at = (size_t)pos * (P.rot / 2) + d / 2;
-            const float cs = P.cos[at], sn = P.sin[at], a = (float)x[d], b = (float)x[d ^ 1];
-            v = (d & 1) ? a * cs + b * sn : a * cs - b * sn;
+    const int pairs = P.rot / 2, zeros = P.os - P.N - P.rot;
+#pragma unroll 4
+    for (int e = threadIdx.x; e < rows * pairs; e += HL_THREADS) {
+        const int r = r0 + e / pairs, d = e % pairs;
+        int pos = P.pos[(size_t)r * P.pos_stride];
+        if (pos < 0 || pos >= P.positions) {
+            if (P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+            pos = 0;
         }
-        ((T*)P.out)[(size_t)r * P.ldo + (size_t)h * P.os + c] = (T)v;
+        const T* x = (const T*)P.x + (size_t)r * P.ldx + (size_t)h * P.xs + P.K + 2 * d;
+        T* out = (T*)P.out + (size_t)r * P.ldo + (size_t)h * P.os + P.rot_at + 2 * d;
+        const float c = P.cos[(size_t)pos * pairs + d], s = P.sin[(size_t)pos * pairs + d], u = (float)x[0], v = (float)x[1];
+        out[0] = (T)(u * c - v * s);
+        out[1] = (T)(v * c + u * s);
+    }
+    for (int e = threadIdx.x; e < rows * zeros; e += HL_THREADS) {
+        const int r = r0 + e / zeros, k = e % zeros, c = P.N + k < P.rot_at ? P.N + k : P.N + k + P.rot;
+        ((T*)P.out)[(size_t)r * P.ldo + (size_t)h * P.os + c] = (T)0.f;
     }
 }
 

@@ -405,60 +405,78 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_f32_kernel(const __gri
     }
 }
 
-// One CTA per (head, row).
+// One CTA per (head, row, and with one map 64 columns): the factor of every split first, its lanes over the splits; then the warps share the
+// splits of 64 columns at a time and their sums meet in shared memory.
+constexpr int WM_THREADS = 256, WM_WARPS = WM_THREADS / 32, WM_COLS = 64;
 template <typename T, int MAPS>
-__global__ void __launch_bounds__(128) window_merge_kernel(const __grid_constant__ PtbWindowAttn P) {
-    __shared__ float red[4];
+__global__ void __launch_bounds__(WM_THREADS) window_merge_kernel(const __grid_constant__ PtbWindowAttn P) {
+    extern __shared__ float part_s[];                    // [WM_WARPS][cols] partial sums, then [MAPS][nsplit] factors
+    __shared__ float red[WM_WARPS];
+    const int cols = MAPS == 1 ? WM_COLS : (P.Dv + WM_COLS - 1) / WM_COLS * WM_COLS, c0 = MAPS == 1 ? blockIdx.z * WM_COLS : 0;
+    float* fac = part_s + WM_WARPS * cols;
     pdl_wait();
     pdl_launch_dependents();
-    const int h = blockIdx.x;
+    const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const size_t i = blockIdx.y, pitch = (size_t)P.H * MAPS * (P.Dvp + 2);
-    const float* wk[MAPS];
-    float base[MAPS], f[MAPS];
-#pragma unroll
-    for (int m = 0; m < MAPS; ++m) {
-        wk[m] = P.work + i * P.nsplit * pitch + (size_t)(h * MAPS + m) * (P.Dvp + 2);
+    const float* wk = P.work + i * P.nsplit * pitch + (size_t)(h * MAPS) * (P.Dvp + 2);
+    if (warp < MAPS) {                                 // a warp per map
+        const float* ml = wk + (size_t)warp * (P.Dvp + 2) + P.Dvp;
         float M = -INFINITY, l = 0.f;
-        for (int s = 0; s < P.nsplit; ++s) M = fmaxf(M, wk[m][s * pitch + P.Dvp]);
-        base[m] = M == -INFINITY ? 0.f : M;
-        for (int s = 0; s < P.nsplit; ++s) l += wk[m][s * pitch + P.Dvp + 1] * exp2f(wk[m][s * pitch + P.Dvp] - base[m]);
-        f[m] = MAPS == 1 ? finish_factor<T>(P, i, h, M, l) : l > 0.f ? (m ? -P.mix : 1.f) / l : 0.f;
+        for (int s = lane; s < P.nsplit; s += 32) M = fmaxf(M, ml[s * pitch]);
+        M = warp_max(M);
+        const float base = M == -INFINITY ? 0.f : M;
+        for (int s = lane; s < P.nsplit; s += 32) {
+            const float e = exp2f(ml[s * pitch] - base);
+            fac[warp * P.nsplit + s] = e;
+            l += ml[s * pitch + 1] * e;
+        }
+        l = warp_sum(l);
+        const float f = MAPS == 1 ? finish_factor<T>(P, i, h, M, l) : l > 0.f ? (warp ? -P.mix : 1.f) / l : 0.f;
+        __syncwarp();
+        for (int s = lane; s < P.nsplit; s += 32) fac[warp * P.nsplit + s] *= f;
     }
-    auto value = [&](int d) {
-        float r = 0.f;
-#pragma unroll
-        for (int m = 0; m < MAPS; ++m) {
-            float a = 0.f;
-#pragma unroll 4
-            for (int s = 0; s < P.nsplit; ++s) a += wk[m][s * pitch + d] * exp2f(wk[m][s * pitch + P.Dvp] - base[m]);
-            r = fmaf(a, f[m], r);
+    __syncthreads();
+    const int m = warp % MAPS;
+    const float* f = fac + m * P.nsplit;
+    for (int c = 0; c < cols; c += WM_COLS) {
+        const int d = c0 + c + lane * 2;               // elements d and d + 1 (Dvp is even)
+        float2 r = make_float2(0.f, 0.f);
+        if (d < P.Dvp) {
+            const float* p = wk + (size_t)m * (P.Dvp + 2) + d;
+#pragma unroll 8
+            for (int s = warp / MAPS; s < P.nsplit; s += WM_WARPS / MAPS) {
+                const float2 v = *reinterpret_cast<const float2*>(p + s * pitch);
+                r.x = fmaf(v.x, f[s], r.x);
+                r.y = fmaf(v.y, f[s], r.y);
+            }
         }
-        return r;
-    };
+        *reinterpret_cast<float2*>(part_s + warp * cols + c + lane * 2) = r;
+    }
+    __syncthreads();
     T* out = (T*)P.out + (i * P.H + h) * P.Dv;
-    if constexpr (MAPS == 1) {
-        for (int d = threadIdx.x; d < P.Dv; d += blockDim.x) out[d] = wa_t<T>(value(d));
-    } else {
-        constexpr int KEEP = 4;                        // values a thread keeps; wider heads form them again
-        float v[KEEP], ss = 0.f;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < cols; c += WM_THREADS) {
+        float v = 0.f;
 #pragma unroll
-        for (int k = 0; k < KEEP; ++k) {
-            const int d = threadIdx.x + k * 128;
-            v[k] = d < P.Dv ? value(d) : 0.f;
-            ss += v[k] * v[k];
+        for (int w = 0; w < WM_WARPS; ++w) v += part_s[w * cols + c];
+        if (c0 + c >= P.Dv) v = 0.f;
+        if constexpr (MAPS == 1) {
+            if (c0 + c < P.Dv) out[c0 + c] = wa_t<T>(v);
+        } else {
+            part_s[c] = v;                               // the same thread reads it again
+            ss += v * v;
         }
-        for (int d = threadIdx.x + KEEP * 128; d < P.Dv; d += 128) { const float a = value(d); ss += a * a; }
+    }
+    if constexpr (MAPS == 2) {
         ss = warp_sum(ss);
-        if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+        if (lane == 0) red[warp] = ss;
         __syncthreads();
-        float g = rsqrtf((red[0] + red[1] + red[2] + red[3]) / (float)P.Dv + P.mix_eps) * P.mix_gain;
-        if (P.gate) g *= sigmoid(wa_f<T>(((const T*)P.gate)[i * P.gate_ld + h]));
+        ss = 0.f;
 #pragma unroll
-        for (int k = 0; k < KEEP; ++k) {
-            const int d = threadIdx.x + k * 128;
-            if (d < P.Dv) out[d] = wa_t<T>(v[k] * g);
-        }
-        for (int d = threadIdx.x + KEEP * 128; d < P.Dv; d += 128) out[d] = wa_t<T>(value(d) * g);
+        for (int w = 0; w < WM_WARPS; ++w) ss += red[w];
+        float g = rsqrtf(ss / (float)P.Dv + P.mix_eps) * P.mix_gain;
+        if (P.gate) g *= sigmoid(wa_f<T>(((const T*)P.gate)[i * P.gate_ld + h]));
+        for (int c = threadIdx.x; c < P.Dv; c += WM_THREADS) out[c] = wa_t<T>(part_s[c] * g);
     }
 }
 
@@ -492,7 +510,11 @@ PTB_API int ptb_proj_norm_write(const void* x, long long ld, int q_col, int k_co
 int ptb_window_merge(const PtbWindowAttn& a, cudaStream_t st) {
     auto merge = a.bf16 ? (a.maps > 1 ? window_merge_kernel<__nv_bfloat16, 2> : window_merge_kernel<__nv_bfloat16, 1>)
                         : (a.maps > 1 ? window_merge_kernel<float, 2> : window_merge_kernel<float, 1>);
-    PTB_CUDA_OK(ptb_launch(merge, dim3(a.H, a.n), dim3(128), 0, st, ptb_pdl_enabled(), a));
+    const int blocks = (a.Dv + WM_COLS - 1) / WM_COLS;
+    const size_t smem = ((size_t)WM_WARPS * (a.maps > 1 ? blocks : 1) * WM_COLS + (size_t)a.maps * a.nsplit) * 4;
+    if (smem > 200 * 1024) { ptb_set_error("window attention: %d splits, heads of %d", a.nsplit, a.Dv); return -1; }
+    if (smem > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(merge, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    PTB_CUDA_OK(ptb_launch(merge, dim3(a.H, a.n, a.maps > 1 ? 1 : blocks), dim3(WM_THREADS), smem, st, ptb_pdl_enabled(), a));
     PTB_CUDA_OK(cudaGetLastError());
     return 0;
 }

@@ -25,7 +25,8 @@ def _decls(L):
     L.ptb_expert_gemm_simt.argtypes = [vp, vp, ll, vp, ci, vp, vp, ci, ci, ci, ci, ci, vp, vp]
     L.ptb_expert_gather.argtypes = [vp, ll, vp, vp, ci, ci, ci, vp, vp]
     L.ptb_expert_gemm.argtypes = [vp, ll, vp, ci, vp, vp, ci, ci, ci, ci, ci, ci, vp, vp]
-    for n in ("ptb_expert_route", "ptb_expert_gemm_simt", "ptb_expert_gather", "ptb_expert_gemm"):
+    L.ptb_expert_route_rows.argtypes = [vp, ll, vp, ci, vp, ci, ci, ci, cf, vp, vp, vp, vp, vp, vp, ci, vp]
+    for n in ("ptb_expert_route", "ptb_expert_route_rows", "ptb_expert_gemm_simt", "ptb_expert_gather", "ptb_expert_gemm"):
         getattr(L, n).restype = ci
 
 
@@ -38,6 +39,9 @@ class Experts:
     correction: torch.Tensor           # [E] fp32
     top: int
     scale: float
+
+    def __post_init__(self):
+        self.done = torch.zeros(ROUTE_ROWS + 1, dtype=torch.int32, device=self.router.device)      # counters of the row router, zero between launches
 
     @property
     def count(self) -> int:
@@ -70,16 +74,27 @@ class Routing:
     offsets: torch.Tensor              # [E + 1] int32: first place of every expert
 
 
+ROUTE_ROWS = 64                        # tokens up to which the kernel that chooses forms the logits as well
+
+
 def route(h: torch.Tensor, e: Experts) -> Routing:
-    n, E, k = h.shape[0], e.count, e.top
-    z = linear_f32(h, e.router)
+    n, E, k, W = h.shape[0], e.count, e.top, h.shape[1]
     if h.is_cuda:
         i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=h.device)
         r = Routing(i32(n, k), torch.empty(n, k, dtype=torch.float32, device=h.device), i32(n * k), i32(E + 1))
-        work = i32(2 * n * k + E)
-        N.check(N.lib().ptb_expert_route(z.data_ptr(), 1, 0, z.stride(0), e.correction.data_ptr(), n, E, k, float(e.scale), r.index.data_ptr(), r.weight.data_ptr(),
-                                         r.token.data_ptr(), r.offsets.data_ptr(), work.data_ptr(), _status(h.device).data_ptr(), _st(h)), "expert_route")
+        few = n <= ROUTE_ROWS and E * W <= 1 << 21
+        work = i32(2 * n * k + (n * E if few else E))
+        out = (r.index.data_ptr(), r.weight.data_ptr(), r.token.data_ptr(), r.offsets.data_ptr(), work.data_ptr())
+        if few:
+            assert h.dtype == e.router.dtype and h.stride(1) == 1
+            N.check(N.lib().ptb_expert_route_rows(h.data_ptr(), h.stride(0), e.router.data_ptr(), W, e.correction.data_ptr(), n, E, k, float(e.scale), *out,
+                                                  e.done.data_ptr(), int(h.dtype == torch.bfloat16), _st(h)), "expert_route_rows")
+            return r
+        z = linear_f32(h, e.router)
+        N.check(N.lib().ptb_expert_route(z.data_ptr(), 1, 0, z.stride(0), e.correction.data_ptr(), n, E, k, float(e.scale), *out, _status(h.device).data_ptr(), _st(h)),
+                "expert_route")
         return r
+    z = linear_f32(h, e.router)
     s = torch.sigmoid(z[:, :E])
     chosen = torch.topk(s + e.correction, k, -1).indices
     w = s.gather(1, chosen)
