@@ -242,13 +242,14 @@ __device__ __forceinline__ float gelu_tanh(float x) {
     return x / (1.0f + __expf(-k2 * (x + 0.044715f * x * x * x)));
 }
 
-// tanh with its relative accuracy at both ends (the fast-math tanhf is a hardware approximation): near zero Lambert's continued fraction
-// x / (1 + x^2 / (3 + x^2 / (5 + x^2 / (7 + x^2 / 9)))) as one quotient, whose next term is below 1e-9 there; else 1 - 2 / (e^2x + 1).
+// tanh with its relative accuracy at both ends (the fast-math tanhf is a hardware approximation), one quotient either way: near zero
+// Lambert's continued fraction x / (1 + x^2 / (3 + x^2 / (5 + x^2 / (7 + x^2 / 9)))), whose next term is below 1e-9 there; else
+// (e^2x - 1) / (e^2x + 1), which no longer cancels.
 __device__ __forceinline__ float tanh_accurate(float x) {
-    const float a = fabsf(x), q = x * x;
-    const float small = x * fmaf(q, fmaf(q, 1.f, 105.f), 945.f) / fmaf(q, fmaf(q, 15.f, 420.f), 945.f);
-    const float big = copysignf(1.f - 2.f / (__expf(2.f * fminf(a, 30.f)) + 1.f), x);
-    return a < 0.55f ? small : big;
+    const float a = fabsf(x), q = x * x, e = __expf(2.f * fminf(a, 30.f));
+    const bool near = a < 0.55f;
+    const float num = near ? a * fmaf(q, fmaf(q, 1.f, 105.f), 945.f) : e - 1.f, den = near ? fmaf(q, fmaf(q, 15.f, 420.f), 945.f) : e + 1.f;
+    return copysignf(__fdividef(num, den), x);
 }
 
 }  // namespace ptb

@@ -42,11 +42,16 @@ struct Logits {
     }
 };
 
-// One warp: choice scores of token i into c_s, its `top` experts in order to (e, w) by lane 0 of the callback.
+// One warp: choice scores of token i into c_s [E] and plain ones behind them, its `top` experts one after the other to lane 0 of the callback.
 template <typename Z, typename F>
 __device__ __forceinline__ void choose(const Route& R, int i, float* c_s, Z logit, F chosen) {
     const int lane = threadIdx.x & 31;
-    for (int e = lane; e < R.E; e += 32) c_s[e] = sigmoid(logit(e)) + R.correction[e];
+    float* s_s = c_s + R.E;
+    for (int e = lane; e < R.E; e += 32) {
+        const float s = sigmoid(logit(e));
+        s_s[e] = s;
+        c_s[e] = s + R.correction[e];
+    }
     __syncwarp();
     float sum = 0.f, mine = 0.f;                       // lane k keeps the score of the k-th expert (and of k + 32, ... in turn)
     for (int k = 0; k < R.top; ++k) {
@@ -61,7 +66,7 @@ __device__ __forceinline__ void choose(const Route& R, int i, float* c_s, Z logi
             if (b > best || (b == best && a < at)) { best = b; at = a; }
         }
         if (at >= R.E) at = k;                         // scores that are not numbers: any expert will do
-        const float score = sigmoid(logit(at));
+        const float score = s_s[at];
         sum += score;
         if (lane == (k & 31)) mine = score;
         __syncwarp();
@@ -81,8 +86,8 @@ __device__ __forceinline__ void choose(const Route& R, int i, float* c_s, Z logi
 __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const __grid_constant__ Route R) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5;
-    float* c_s = smem + warp * R.E;
-    int* count = reinterpret_cast<int*>(smem + RT_WARPS * R.E);
+    float* c_s = smem + warp * 2 * R.E;
+    int* count = reinterpret_cast<int*>(smem + RT_WARPS * 2 * R.E);
     int* base = count + R.E;
     for (int e = threadIdx.x; e < R.E; e += blockDim.x) count[e] = 0;
     pdl_wait();
@@ -142,8 +147,8 @@ __global__ void __launch_bounds__(256) place_kernel(const __grid_constant__ Rout
 __global__ void __launch_bounds__(RS_WARPS * 32) route_small_kernel(const __grid_constant__ Route R) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5;
-    float* c_s = smem + warp * R.E;
-    int* count = reinterpret_cast<int*>(smem + RS_WARPS * R.E);
+    float* c_s = smem + warp * 2 * R.E;
+    int* count = reinterpret_cast<int*>(smem + RS_WARPS * 2 * R.E);
     int* off = count + R.E;
     for (int e = threadIdx.x; e < R.E; e += blockDim.x) count[e] = 0;
     pdl_wait();
@@ -173,7 +178,7 @@ constexpr int RR_THREADS = 128, RR_WARPS = RR_THREADS / 32;
 template <typename T>
 __global__ void __launch_bounds__(RR_THREADS) route_rows_kernel(const __grid_constant__ Route R, const T* __restrict__ h, long long ldh, const T* __restrict__ w, int W,
                                                                 float* z, unsigned* done) {
-    extern __shared__ float c_s[];                     // [E], later counts [E] and offsets [E + 1]
+    extern __shared__ float c_s[];                     // [2 E], later counts [E] and offsets [E + 1]
     __shared__ int last;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, i = blockIdx.y;
     constexpr int V = 16 / sizeof(T);                  // elements of a 16-byte load
@@ -313,12 +318,14 @@ PTB_API int ptb_expert_route(const float* z, int splits, long long stride, long 
     Route r{z, splits, stride, ld, correction, n, E, top, scale, index, weight, token, offsets, work, work + pairs, work + 2 * pairs, status};
     const bool pdl = ptb_pdl_enabled();
     if (n <= SMALL_TOKENS && E <= 256) {
-        const size_t smem = ((size_t)RS_WARPS * E + 2 * E + 1) * 4;
-        if (smem > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(route_small_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024));
+        const size_t smem = ((size_t)RS_WARPS * 2 * E + 2 * E + 1) * 4;
+        if (smem > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(route_small_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
         PTB_CUDA_OK(ptb_launch(route_small_kernel, dim3(1), dim3(RS_WARPS * 32), smem, st, pdl, r));
     } else {
         PTB_CUDA_OK(cudaMemsetAsync(r.counts, 0, (size_t)E * 4, st));
-        PTB_CUDA_OK(ptb_launch(route_kernel, dim3((n + RT_WARPS - 1) / RT_WARPS), dim3(RT_WARPS * 32), ((size_t)RT_WARPS * E + 2 * E) * 4, st, false, r));
+        const size_t smem = ((size_t)RT_WARPS * 2 * E + 2 * E) * 4;
+        if (smem > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
+        PTB_CUDA_OK(ptb_launch(route_kernel, dim3((n + RT_WARPS - 1) / RT_WARPS), dim3(RT_WARPS * 32), smem, st, false, r));
         PTB_CUDA_OK(ptb_launch(place_kernel, dim3((unsigned)std::min<size_t>(1024, (pairs + 255) / 256)), dim3(256), (size_t)(E + 1) * 4, st, pdl, r));
     }
     PTB_CUDA_OK(cudaGetLastError());

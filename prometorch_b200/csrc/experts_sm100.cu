@@ -1,8 +1,8 @@
 // Grouped products of a mixture of experts on the 5th-generation tensor cores, bf16.  Rows are sorted by expert; the row counts are read
 // from device memory, so nothing waits for the host.
 //   expert_gather_kernel   the rows of the tokens in the order by expert;
-//   expert_gemm_kernel     persistent CTAs walk the tiles of all experts.  192 threads: warp 0 TMA producer, warp 1 owns tensor memory and
-//                          issues the MMAs, warps 2-5 epilogue; two accumulators, so an epilogue overlaps the next tile's main loop.
+//   expert_gemm_kernel     persistent CTAs walk the tiles of all experts.  320 threads: warp 0 TMA producer, warp 1 owns tensor memory and
+//                          issues the MMAs, warps 2-9 epilogue; two accumulators, so an epilogue overlaps the next tile's main loop.
 //     many rows per expert: 128 rows x 256 weight rows; gated, these are 128 gate rows and the 128 up rows that go with them;
 //     few: the weight is the 128-row operand (gated: one tile of gate and one of up rows, two accumulators), 32 tokens are the columns.
 //   Gated products leave silu(gate) * up.
@@ -71,7 +71,7 @@ __global__ void __launch_bounds__(THREADS, 1) expert_gemm_kernel(const __grid_co
     const int kblocks = (P.K + BK - 1) / BK, col_tiles = (P.N + C::COLS - 1) / C::COLS;
     if (threadIdx.x == 0) {
         for (int s = 0; s < C::STAGES; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
-        for (int b = 0; b < 2; ++b) { mbar_init(&acc_full[b], 1); mbar_init(&acc_empty[b], 4); }
+        for (int b = 0; b < 2; ++b) { mbar_init(&acc_full[b], 1); mbar_init(&acc_empty[b], EPI_WARPS); }
         mbar_fence_init();
         prefetch_tmap(&tmT);
         prefetch_tmap(&tmW);
@@ -170,7 +170,7 @@ __global__ void __launch_bounds__(THREADS, 1) expert_gemm_kernel(const __grid_co
             }
         }
     } else {
-        const int q = warp & 3;                        // tensor-memory lanes of this warp
+        const int q = warp & 3, half = warp >= 6;      // tensor-memory lanes of this warp; the half of a tile it stores
         const bool wide = P.N % 16 == 0 && ((uintptr_t)P.out & 31) == 0;
         bool ok = true;
         int tl = 0;
@@ -187,11 +187,11 @@ __global__ void __launch_bounds__(THREADS, 1) expert_gemm_kernel(const __grid_co
                 tmem_ld32(acc, g);
                 if constexpr (GATED) tmem_ld32(acc + C::ROWS, u);
                 tmem_ld_wait();
-                if (f < P.N) {
+                if (f < P.N) {                         // four warps take the even tokens, four the odd ones
                     __nv_bfloat16* o = P.out + (size_t)T.row * P.N + f;
 #pragma unroll
                     for (int j = 0; j < 32; ++j)
-                        if (j < n) {
+                        if (j < n && (j & 1) == half) {
                             float v = __uint_as_float(g[j]);
                             if constexpr (GATED) v = silu(v) * __uint_as_float(u[j]);
                             o[(size_t)j * P.N] = __float2bfloat16_rn(v);
@@ -201,7 +201,7 @@ __global__ void __launch_bounds__(THREADS, 1) expert_gemm_kernel(const __grid_co
                 const int row = T.row + q * 32 + lane;
                 __nv_bfloat16* o = P.out + (size_t)row * P.N;
 #pragma unroll 1
-                for (int c = 0; c < C::COLS; c += 32) {
+                for (int c = half * (C::COLS / 2); c < (half + 1) * (C::COLS / 2); c += 32) {
                     if (T.col + c >= P.N) break;
                     uint32_t g[32], u[32];
                     tmem_ld32(acc + c, g);

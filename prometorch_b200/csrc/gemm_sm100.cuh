@@ -8,8 +8,9 @@
 //   C[M,N] (+)= op(A) * op(B)      A: M x K,  B: N x K  ("K-major": K contiguous)
 //                                  or stored transposed ("MN-major": M resp. N contiguous)
 //
-// Warp roles (192 threads): warp 0 = TMA producer, warp 1 = TMEM allocator + MMA
-// issuer, warps 2..5 = epilogue (warp w reads TMEM lanes 32*(w%4) .. +32).
+// Warp roles (320 threads): warp 0 = TMA producer, warp 1 = TMEM allocator + MMA
+// issuer, warps 2..9 = epilogue (warp w reads TMEM lanes 32*(w%4) .. +32; the first
+// four take the left half of a tile's columns, the others the right half).
 // The reference's GEMM is cublasSgemm in fp32 (aten/src/ATen/cuda/CUDABlas.cu:455-479).
 #pragma once
 #include "common.cuh"
@@ -21,7 +22,7 @@ namespace gemm {
 constexpr int BM = 128;
 constexpr int BK = 64;              // 64 bf16 = one 128-byte swizzle row
 constexpr int UMMA_K = 16;
-constexpr int THREADS = 192;
+constexpr int THREADS = 320, EPI_WARPS = 8;
 constexpr int TMEM_COLS = 512;
 
 constexpr int MAX_SHARDS = 8;
@@ -257,7 +258,7 @@ gemm_bf16_kernel(const __grid_constant__ Operand opA, const __grid_constant__ Op
 
     if (threadIdx.x == 0) {
         for (int s = 0; s < STAGES; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
-        for (int b = 0; b < 2; ++b) { mbar_init(&acc_full[b], 1); mbar_init(&acc_empty[b], 4); }
+        for (int b = 0; b < 2; ++b) { mbar_init(&acc_full[b], 1); mbar_init(&acc_empty[b], EPI_WARPS); }
         *abort_flag = 0;
         mbar_fence_init();
         prefetch_tmap(&opA.map[0]);
@@ -361,7 +362,7 @@ gemm_bf16_kernel(const __grid_constant__ Operand opA, const __grid_constant__ Op
             if (!ok) *abort_flag = 1;
         }
     } else {
-        // ------------------------------------------------------------------ epilogue (warps 2..5)
+        // ------------------------------------------------------------------ epilogue (warps 2..9)
         const int q = warp & 3;                     // TMEM lane quarter this warp may read
         // bf16 rows whose 64-byte pieces start on 32-byte boundaries go out in whole sectors
         const bool wide = !(P.flags & (EPI_ACCUM | EPI_OUT_F32 | EPI_SCATTER_ADD | EPI_SCATTER_STORE | EPI_TRANS)) && P.ldc % 16 == 0 && ((uintptr_t)P.C & 31) == 0;
@@ -376,8 +377,10 @@ gemm_bf16_kernel(const __grid_constant__ Operand opA, const __grid_constant__ Op
             tc_fence_after();
             const int row = m0 + q * 32 + lane;
             const uint32_t taddr = tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(b * BN);
+            constexpr int PIECES = BN / 32, LEFT = (PIECES + 1) / 2;           // of 32 columns; a tile of one piece leaves the right half idle
+            const int c_lo = warp < 6 ? 0 : LEFT * 32, c_hi = warp < 6 ? LEFT * 32 : BN;
 #pragma unroll 1
-            for (int c = 0; c < BN; c += 32) {
+            for (int c = c_lo; c < c_hi; c += 32) {
                 uint32_t r[32];
                 tmem_ld32(taddr + c, r);
                 tmem_ld_wait();

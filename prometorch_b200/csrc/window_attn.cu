@@ -405,15 +405,15 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_f32_kernel(const __gri
     }
 }
 
-// One CTA per (head, row, and with one map 64 columns): the factor of every split first, its lanes over the splits; then the warps share the
-// splits of 64 columns at a time and their sums meet in shared memory.
+// One CTA per (head, row, and with one map `cols` columns): the factor of every split first, its lanes over the splits; then `share` warps per
+// map take the splits of 64 columns together, the warps left over other columns, and their sums meet in shared memory.
 constexpr int WM_THREADS = 256, WM_WARPS = WM_THREADS / 32, WM_COLS = 64;
 template <typename T, int MAPS>
-__global__ void __launch_bounds__(WM_THREADS) window_merge_kernel(const __grid_constant__ PtbWindowAttn P) {
-    extern __shared__ float part_s[];                    // [WM_WARPS][cols] partial sums, then [MAPS][nsplit] factors
+__global__ void __launch_bounds__(WM_THREADS) window_merge_kernel(const __grid_constant__ PtbWindowAttn P, int cols, int share) {
+    extern __shared__ float part_s[];                  // [MAPS share][cols] partial sums, then [MAPS][nsplit] factors
     __shared__ float red[WM_WARPS];
-    const int cols = MAPS == 1 ? WM_COLS : (P.Dv + WM_COLS - 1) / WM_COLS * WM_COLS, c0 = MAPS == 1 ? blockIdx.z * WM_COLS : 0;
-    float* fac = part_s + WM_WARPS * cols;
+    const int c0 = blockIdx.z * cols, parts = MAPS * share;
+    float* fac = part_s + parts * cols;
     pdl_wait();
     pdl_launch_dependents();
     const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -436,29 +436,28 @@ __global__ void __launch_bounds__(WM_THREADS) window_merge_kernel(const __grid_c
         for (int s = lane; s < P.nsplit; s += 32) fac[warp * P.nsplit + s] *= f;
     }
     __syncthreads();
-    const int m = warp % MAPS;
+    const int m = warp % MAPS, mine = warp / MAPS % share;
     const float* f = fac + m * P.nsplit;
-    for (int c = 0; c < cols; c += WM_COLS) {
+    for (int c = warp / parts * WM_COLS; c < cols; c += WM_WARPS / parts * WM_COLS) {
         const int d = c0 + c + lane * 2;               // elements d and d + 1 (Dvp is even)
         float2 r = make_float2(0.f, 0.f);
         if (d < P.Dvp) {
             const float* p = wk + (size_t)m * (P.Dvp + 2) + d;
 #pragma unroll 8
-            for (int s = warp / MAPS; s < P.nsplit; s += WM_WARPS / MAPS) {
+            for (int s = mine; s < P.nsplit; s += share) {
                 const float2 v = *reinterpret_cast<const float2*>(p + s * pitch);
                 r.x = fmaf(v.x, f[s], r.x);
                 r.y = fmaf(v.y, f[s], r.y);
             }
         }
-        *reinterpret_cast<float2*>(part_s + warp * cols + c + lane * 2) = r;
+        *reinterpret_cast<float2*>(part_s + warp % parts * cols + c + lane * 2) = r;
     }
     __syncthreads();
     T* out = (T*)P.out + (i * P.H + h) * P.Dv;
     float ss = 0.f;
     for (int c = threadIdx.x; c < cols; c += WM_THREADS) {
         float v = 0.f;
-#pragma unroll
-        for (int w = 0; w < WM_WARPS; ++w) v += part_s[w * cols + c];
+        for (int w = 0; w < parts; ++w) v += part_s[w * cols + c];
         if (c0 + c >= P.Dv) v = 0.f;
         if constexpr (MAPS == 1) {
             if (c0 + c < P.Dv) out[c0 + c] = wa_t<T>(v);
@@ -510,11 +509,13 @@ PTB_API int ptb_proj_norm_write(const void* x, long long ld, int q_col, int k_co
 int ptb_window_merge(const PtbWindowAttn& a, cudaStream_t st) {
     auto merge = a.bf16 ? (a.maps > 1 ? window_merge_kernel<__nv_bfloat16, 2> : window_merge_kernel<__nv_bfloat16, 1>)
                         : (a.maps > 1 ? window_merge_kernel<float, 2> : window_merge_kernel<float, 1>);
-    const int blocks = (a.Dv + WM_COLS - 1) / WM_COLS;
-    const size_t smem = ((size_t)WM_WARPS * (a.maps > 1 ? blocks : 1) * WM_COLS + (size_t)a.maps * a.nsplit) * 4;
+    int share = 1;
+    while (share * 2 * a.maps <= WM_WARPS && share * 8 <= a.nsplit) share *= 2;
+    const int padded = (a.Dv + WM_COLS - 1) / WM_COLS * WM_COLS, cols = a.maps == 1 && share * a.maps == WM_WARPS ? WM_COLS : padded;
+    const size_t smem = ((size_t)a.maps * share * cols + (size_t)a.maps * a.nsplit) * 4;
     if (smem > 200 * 1024) { ptb_set_error("window attention: %d splits, heads of %d", a.nsplit, a.Dv); return -1; }
     if (smem > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(merge, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    PTB_CUDA_OK(ptb_launch(merge, dim3(a.H, a.n, a.maps > 1 ? 1 : blocks), dim3(WM_THREADS), smem, st, ptb_pdl_enabled(), a));
+    PTB_CUDA_OK(ptb_launch(merge, dim3(a.H, a.n, padded / cols), dim3(WM_THREADS), smem, st, ptb_pdl_enabled(), a, cols, share));
     PTB_CUDA_OK(cudaGetLastError());
     return 0;
 }
