@@ -194,6 +194,8 @@ static int gemm_core(void* const* a_ptrs, int a_shards, int a_shard_rows, long l
     p.pdl = sk.pdl;
     fill_staging(p.stA, stage_a);
     fill_staging(p.stB, stage_b);
+    // an ordinary product sets itself up under the end of the kernel before it (what it accumulates into, or shares with peers, it must not)
+    if (!p.stA.seq && !p.stB.seq && a_shards == 1 && b_shards == 1 && !(flags & (EPI_ACCUM | EPI_SCATTER_ADD | EPI_SCATTER_STORE))) p.pdl = ptb_pdl_enabled() ? 1 : 0;
     // stager CTAs are needed unless every staged operand is filled by an external copier
     p.stager_ctas = ((p.stA.seq && !(stage_a && stage_a->external)) || (p.stB.seq && !(stage_b && stage_b->external))) ? 1 : 0;
     if ((p.stA.seq && (p.stA.shard_rows % STAGE_ROWS)) || (p.stB.seq && (p.stB.shard_rows % STAGE_ROWS))) {

@@ -41,8 +41,8 @@ __device__ __forceinline__ void st(T* p, const Vals<V>& r) {
     }
 }
 
-// TY: type of y, T: of out and the table.  U rows at a time: their loads are in flight together.
-template <typename T, typename TY, int V, int U>
+// TY: type of y, T: of out and the table.
+template <typename T, typename TY, int V>
 __global__ void __launch_bounds__(TN_THREADS) tanh_residual_kernel(const __grid_constant__ PtbTanhResidual P) {
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
     const bool live = c < P.W;
@@ -55,74 +55,51 @@ __global__ void __launch_bounds__(TN_THREADS) tanh_residual_kernel(const __grid_
     pdl_wait();
     pdl_launch_dependents();
     if (!live) return;
-    for (int row0 = blockIdx.y * U; row0 < P.n; row0 += gridDim.y * U) {
-        Vals<V> x[U], y[U], again[U];
-        const int rows = min(U, P.n - row0);
-#pragma unroll
-        for (int u = 0; u < U; ++u)
-            if (u < rows) x[u] = ld<V>(P.x + (size_t)(row0 + u) * P.W + c);
+    for (int row = blockIdx.y; row < P.n; row += gridDim.y) {
+        Vals<V> x = ld<V>(P.x + (size_t)row * P.W + c), y;
         if (P.index) {
 #pragma unroll
-            for (int u = 0; u < U; ++u)
-#pragma unroll
-                for (int e = 0; e < V; ++e) y[u].v[e] = 0.f;
+            for (int e = 0; e < V; ++e) y.v[e] = 0.f;
 #pragma unroll 4
-            for (int k = 0; k < P.top; ++k)
-#pragma unroll
-                for (int u = 0; u < U; ++u)
-                    if (u < rows) {
-                        const size_t at = (size_t)(row0 + u) * P.top + k;
-                        int r = P.index[at];
-                        const float f = P.weight[at];
-                        if (r < 0 || r >= P.y_rows) {
-                            if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
-                            r = 0;
-                        }
-                        const Vals<V> t = ld<V>((const TY*)P.y + (size_t)r * P.ld + c);
-#pragma unroll
-                        for (int e = 0; e < V; ++e) y[u].v[e] = fmaf(f, t.v[e], y[u].v[e]);
-                    }
-        } else {
-#pragma unroll
-            for (int u = 0; u < U; ++u)
-                if (u < rows) y[u] = ld<V>((const TY*)P.y + (size_t)(row0 + u) * P.ld + c);
-#pragma unroll 4
-            for (int s = 1; s < P.splits; ++s)
-#pragma unroll
-                for (int u = 0; u < U; ++u)
-                    if (u < rows) {
-                        const Vals<V> t = ld<V>((const TY*)P.y + s * P.stride + (size_t)(row0 + u) * P.ld + c);
-#pragma unroll
-                        for (int e = 0; e < V; ++e) y[u].v[e] += t.v[e];
-                    }
-        }
-        if (P.ids) {
-#pragma unroll
-            for (int u = 0; u < U; ++u)
-                if (u < rows) {
-                    int id = P.ids[(size_t)(row0 + u) * P.id_stride];
-                    if (id < 0 || id >= P.V) {
-                        if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
-                        id = 0;
-                    }
-                    again[u] = ld<V>((const T*)P.table + (size_t)id * P.W + c);
+            for (int k = 0; k < P.top; ++k) {
+                int r = P.index[(size_t)row * P.top + k];
+                const float f = P.weight[(size_t)row * P.top + k];
+                if (r < 0 || r >= P.y_rows) {
+                    if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+                    r = 0;
                 }
-        }
+                const Vals<V> t = ld<V>((const TY*)P.y + (size_t)r * P.ld + c);
 #pragma unroll
-        for (int u = 0; u < U; ++u)
-            if (u < rows) {
-#pragma unroll
-                for (int e = 0; e < V; ++e) {
-                    x[u].v[e] += fmaf(tanh_accurate(P.post_alpha * y[u].v[e]), wo.v[e], bo.v[e]);
-                    if (P.ids) x[u].v[e] += again[u].v[e];
-                }
-                st<V>(P.x + (size_t)(row0 + u) * P.W + c, x[u]);
-                if (P.pre_w) {
-#pragma unroll
-                    for (int e = 0; e < V; ++e) x[u].v[e] = fmaf(tanh_accurate(P.pre_alpha * x[u].v[e]), wi.v[e], bi.v[e]);
-                    st<V>((T*)P.out + (size_t)(row0 + u) * P.W + c, x[u]);
-                }
+                for (int e = 0; e < V; ++e) y.v[e] = fmaf(f, t.v[e], y.v[e]);
             }
+        } else {
+            const TY* p = (const TY*)P.y + (size_t)row * P.ld + c;
+            y = ld<V>(p);
+#pragma unroll 4
+            for (int s = 1; s < P.splits; ++s) {
+                const Vals<V> t = ld<V>(p + s * P.stride);
+#pragma unroll
+                for (int e = 0; e < V; ++e) y.v[e] += t.v[e];
+            }
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) x.v[e] += fmaf(tanh_accurate(P.post_alpha * y.v[e]), wo.v[e], bo.v[e]);
+        if (P.ids) {
+            int id = P.ids[(size_t)row * P.id_stride];
+            if (id < 0 || id >= P.V) {
+                if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+                id = 0;
+            }
+            const Vals<V> t = ld<V>((const T*)P.table + (size_t)id * P.W + c);
+#pragma unroll
+            for (int e = 0; e < V; ++e) x.v[e] += t.v[e];
+        }
+        st<V>(P.x + (size_t)row * P.W + c, x);
+        if (P.pre_w) {
+#pragma unroll
+            for (int e = 0; e < V; ++e) x.v[e] = fmaf(tanh_accurate(P.pre_alpha * x.v[e]), wi.v[e], bi.v[e]);
+            st<V>((T*)P.out + (size_t)row * P.W + c, x);
+        }
     }
 }
 
@@ -149,13 +126,12 @@ __global__ void __launch_bounds__(TN_THREADS) softcap_kernel(const float* __rest
 
 template <typename T, typename TY>
 static cudaError_t tanh_residual_launch(const PtbTanhResidual& p, bool vec, cudaStream_t s) {
-    // few rows: small CTAs spread a row over more SMs; many: up to eight CTAs of 256 threads per SM walk them, two rows at a time
+    // few rows: small CTAs spread a row over more SMs; many: up to eight CTAs of 256 threads per SM walk them
     const bool many = p.n >= 1024;
     const int lanes = vec ? p.W / 4 : p.W, threads = std::min(many ? TN_THREADS : 64, (lanes + 31) / 32 * 32), cols = (lanes + threads - 1) / threads;
-    const int u = many ? 2 : 1, rows = std::max(1, std::min((p.n + u - 1) / u, 148 * 8 * (TN_THREADS / threads) / cols));
+    const int rows = std::max(1, std::min(p.n, 148 * 8 * (TN_THREADS / threads) / cols));
     auto go = [&](auto k) { return ptb_launch(k, dim3(cols, std::min(rows, 65535)), dim3(threads), 0, s, ptb_pdl_enabled(), p); };
-    if (many) return vec ? go(tanh_residual_kernel<T, TY, 4, 2>) : go(tanh_residual_kernel<T, TY, 1, 2>);
-    return vec ? go(tanh_residual_kernel<T, TY, 4, 1>) : go(tanh_residual_kernel<T, TY, 1, 1>);
+    return vec ? go(tanh_residual_kernel<T, TY, 4>) : go(tanh_residual_kernel<T, TY, 1>);
 }
 
 }  // namespace ptb
