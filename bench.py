@@ -327,8 +327,8 @@ def main():
     ap.add_argument("--warmup", type=int, default=16)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--prompt-len", type=int, default=128)
-    ap.add_argument("--model", default="qwen3-4b", choices=["qwen3-4b", "tiny", "kifusun", "gelutar"],
-                    help="kifusun, gelutar: that model beside Llama of equal size in the batching engine (benchmarks/*_bench.py), 1 GPU")
+    ap.add_argument("--model", default="qwen3-4b", choices=["qwen3-4b", "tiny", "kifusun", "gelutar", "budorax"],
+                    help="kifusun, gelutar, budorax: that model beside Llama of equal size in the batching engine (benchmarks/*_bench.py), 1 GPU")
     ap.add_argument("--max-seq", type=int, default=4096)
     ap.add_argument("--repeats", type=int, default=5, help="timed regions of --steps steps each (median is reported)")
     ap.add_argument("--train-steps", type=int, default=5, help="timed steps of the Llama-1.1B FSDP half (0 = skip)")
@@ -346,6 +346,10 @@ def main():
         sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
         import gelutar_bench
         return gelutar_bench.main([])
+    if args.model == "budorax":
+        sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
+        import budorax_bench
+        return budorax_bench.main([])
     args.warmup = max(args.warmup, 3)
 
     import torch
