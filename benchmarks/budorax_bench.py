@@ -101,9 +101,10 @@ def kernel_rows(z, chunk, prompt=4096, ctx=4096):
                                         Dp=la.row, Dv=KV_RANK, Dvp=KV_RANK, v_ld=la.row, maps=1, window=A.UNBOUNDED, scale=0.1, bf16=1, max_keys=n)
                     A.run_rows(args, qs[i], o, pos, req, ns, kernel=A.N.lib().ptb_latent_attn_rows)
                 add(f"decode latent attention, batch {B}, {n} keys", per_launch_us([lambda i=i: rows(i) for i in range(sets)]), 2 * B * n * la.row, 2.0 * B * n * H * (la.row + KV_RANK))
-                add(f"queries through W_uk, {B} rows", per_launch_us([lambda i=i: M.fold_queries(lq[i], la, pos) for i in range(sets)]), 2 * H * D * KV_RANK, 2.0 * B * H * D * KV_RANK)
-                add(f"latents through W_uv and gate, {B} rows", per_launch_us([lambda i=i: M.unfold_values(o, la, gate[:B]) for i in range(sets)]), 2 * H * D * KV_RANK,
-                    2.0 * B * H * D * KV_RANK)
+                add(f"queries through W_uk, {B} rows", per_launch_us([lambda i=i: M.fold_queries(lq[i], la, pos) for i in range(sets)]),
+                    2 * H * D * KV_RANK + 2 * B * H * (D + ROT + la.row), 2.0 * B * H * D * KV_RANK)
+                add(f"latents through W_uv and gate, {B} rows", per_launch_us([lambda i=i: M.unfold_values(o, la, gate[:B]) for i in range(sets)]),
+                    2 * H * D * KV_RANK + 2 * B * H * (KV_RANK + D), 2.0 * B * H * D * KV_RANK)
             q2, lens, nl = [rand(B, H * D) for _ in range(sets)], pos + 1, P.pick_splits(B, G, n)
             add(f"decode attention, batch {B}, {n} keys (llama)", per_launch_us([lambda i=i: P.paged_attention_decode(q2[i], H, G, D, lens, table, kp[i], vp[i], nsplit=nl) for i in range(sets)]),
                 4 * B * n * G * D, 4.0 * B * n * H * D)
