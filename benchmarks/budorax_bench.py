@@ -140,7 +140,7 @@ def kernel_rows(z, chunk, prompt=4096, ctx=4096):
         st = lambda: torch.cuda.current_stream().cuda_stream
         gu = lambda i: N.check(N.lib().ptb_expert_gemm(xs.data_ptr(), W, ex[i].gate_up.data_ptr(), 1, act.data_ptr(), rt[i].offsets.data_ptr(), rows_, EXPERTS, ff, W, few, 0, 0, st()))
         dn = lambda i: N.check(N.lib().ptb_expert_gemm(act.data_ptr(), ff, ex[i].down.data_ptr(), 0, y.data_ptr(), rt[i].offsets.data_ptr(), rows_, EXPERTS, W, ff, few, 0, 0, st()))
-        ga = lambda i: N.check(N.lib().ptb_expert_gather(h.data_ptr(), W, rt[i].token.data_ptr(), xs.data_ptr(), rows_, W, n, 0, st()))
+        ga = lambda i: N.check(N.lib().ptb_expert_gather(h.data_ptr(), W, rt[i].token.data_ptr(), rt[i].offsets[-1:].data_ptr(), xs.data_ptr(), rows_, W, n, 0, st()))
         ga(0)
         add(f"experts gate / up + SiLU gate, {n} rows", per_launch_us([lambda i=i: gu(i) for i in range(2)], 6), 2 * (rows_ * W + live * 2 * ff * W + rows_ * ff), 4.0 * rows_ * ff * W)
         add(f"experts down, {n} rows", per_launch_us([lambda i=i: dn(i) for i in range(2)], 6), 2 * (rows_ * W + live * ff * W + rows_ * ff), 2.0 * rows_ * ff * W)

@@ -1,10 +1,12 @@
 // A mixture of experts for inference, the parts that take any size:
-//   route_kernel        a warp per token: sigmoid scores, the `top` experts with the largest corrected scores, their weights, and the
-//                       token's rank among an expert's rows (counted in shared memory, then once per CTA and expert in global memory);
+//   route_kernel        a warp per token: scores (sigmoid, or softmax over all outputs), the `top` outputs with the largest corrected scores,
+//                       their weights, and the token's rank among an expert's rows (counted in shared memory, then once per CTA and expert
+//                       in global memory);
 //   place_kernel        prefix sums of the counts: the place of every (token, expert) pair in the order by expert, and back;
 //   route_small_kernel  both for few tokens in one CTA;
 //   route_rows_kernel   the router's product as well, for few tokens;
 //   expert_simt_kernel  a grouped product over the sorted rows with FMAs in fp32 (fp32 models, sizes the tensor-core kernel cannot address).
+// The router may have more outputs than there are experts: those behind them are identities, without rows; their place is -1.
 // Where a row lies inside its expert depends on the order of atomics; what is computed for it does not.
 #include "common.cuh"
 #include <algorithm>
@@ -18,9 +20,10 @@ struct Route {
     const float* z;                    // [splits][n] rows of pitch ld
     int splits;
     long long stride, ld;
-    const float* correction;           // [E]
+    const float* correction;           // [O]
     int n, E, top;
-    float scale;
+    int O, softmax;                    // router outputs: the experts and the identities behind them
+    float scale;                       // weights: scores over their sum times scale; softmax: the scores times scale
     int* index;                        // [n][top] out: place in the order by expert
     float* weight;                     // [n][top] out
     int* token;                        // [n top] out
@@ -42,22 +45,36 @@ struct Logits {
     }
 };
 
-// One warp: choice scores of token i into c_s [E] and plain ones behind them, its `top` experts one after the other to lane 0 of the callback.
+// One warp: choice scores of token i into c_s [O] and plain ones behind them, its `top` outputs one after the other to lane 0 of the callback.
 template <typename Z, typename F>
 __device__ __forceinline__ void choose(const Route& R, int i, float* c_s, Z logit, F chosen) {
     const int lane = threadIdx.x & 31;
-    float* s_s = c_s + R.E;
-    for (int e = lane; e < R.E; e += 32) {
-        const float s = sigmoid(logit(e));
-        s_s[e] = s;
-        c_s[e] = s + R.correction[e];
-    }
+    float* s_s = c_s + R.O;
+    if (R.softmax) {
+        float most = -INFINITY, all = 0.f;
+        for (int e = lane; e < R.O; e += 32) {
+            s_s[e] = logit(e);
+            most = fmaxf(most, s_s[e]);
+        }
+        most = warp_max(most);
+        for (int e = lane; e < R.O; e += 32) all += s_s[e] = expf(s_s[e] - most);
+        all = 1.f / warp_sum(all);
+        for (int e = lane; e < R.O; e += 32) {
+            s_s[e] *= all;
+            c_s[e] = s_s[e] + R.correction[e];
+        }
+    } else
+        for (int e = lane; e < R.O; e += 32) {
+            const float s = sigmoid(logit(e));
+            s_s[e] = s;
+            c_s[e] = s + R.correction[e];
+        }
     __syncwarp();
     float sum = 0.f, mine = 0.f;                       // lane k keeps the score of the k-th expert (and of k + 32, ... in turn)
     for (int k = 0; k < R.top; ++k) {
         float best = -INFINITY;
-        int at = R.E;
-        for (int e = lane; e < R.E; e += 32)
+        int at = R.O;
+        for (int e = lane; e < R.O; e += 32)
             if (c_s[e] > best) { best = c_s[e]; at = e; }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
@@ -65,7 +82,7 @@ __device__ __forceinline__ void choose(const Route& R, int i, float* c_s, Z logi
             const int a = __shfl_xor_sync(0xffffffffu, at, o);
             if (b > best || (b == best && a < at)) { best = b; at = a; }
         }
-        if (at >= R.E) at = k;                         // scores that are not numbers: any expert will do
+        if (at >= R.O) at = k;                         // scores that are not numbers: any expert will do
         const float score = s_s[at];
         sum += score;
         if (lane == (k & 31)) mine = score;
@@ -77,7 +94,7 @@ __device__ __forceinline__ void choose(const Route& R, int i, float* c_s, Z logi
         __syncwarp();
         if ((k & 31) == 31 && k + 1 < R.top) R.weight[(size_t)i * R.top + k - 31 + lane] = mine;      // unscaled: the sum is not known yet
     }
-    const float f = R.scale / (sum + 1e-20f);
+    const float f = R.softmax ? R.scale : R.scale / (sum + 1e-20f);
     const int k0 = (R.top - 1) & ~31;                  // the last ones are still in registers
     for (int k = lane; k < k0; k += 32) R.weight[(size_t)i * R.top + k] *= f;
     if (k0 + lane < R.top) R.weight[(size_t)i * R.top + k0 + lane] = mine * f;
@@ -86,8 +103,8 @@ __device__ __forceinline__ void choose(const Route& R, int i, float* c_s, Z logi
 __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const __grid_constant__ Route R) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5;
-    float* c_s = smem + warp * 2 * R.E;
-    int* count = reinterpret_cast<int*>(smem + RT_WARPS * 2 * R.E);
+    float* c_s = smem + warp * 2 * R.O;
+    int* count = reinterpret_cast<int*>(smem + RT_WARPS * 2 * R.O);
     int* base = count + R.E;
     for (int e = threadIdx.x; e < R.E; e += blockDim.x) count[e] = 0;
     pdl_wait();
@@ -97,7 +114,7 @@ __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const __grid_const
     if (i < R.n)
         choose(R, i, c_s, Logits{R, i}, [&](int k, int e) {
             R.expert[(size_t)i * R.top + k] = e;
-            R.rank[(size_t)i * R.top + k] = atomicAdd(&count[e], 1);
+            if (e < R.E) R.rank[(size_t)i * R.top + k] = atomicAdd(&count[e], 1);
         });
     __syncthreads();
     for (int e = threadIdx.x; e < R.E; e += blockDim.x) base[e] = count[e] ? atomicAdd(&R.counts[e], count[e]) : 0;
@@ -105,7 +122,7 @@ __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const __grid_const
     if (i < R.n)
         for (int k = threadIdx.x & 31; k < R.top; k += 32) {
             const size_t p = (size_t)i * R.top + k;
-            R.rank[p] += base[R.expert[p]];
+            if (R.expert[p] < R.E) R.rank[p] += base[R.expert[p]];
         }
 }
 
@@ -138,17 +155,17 @@ __global__ void __launch_bounds__(256) place_kernel(const __grid_constant__ Rout
         for (int e = threadIdx.x; e <= R.E; e += blockDim.x) R.offsets[e] = off[e];
     const long long total = (long long)R.n * R.top;
     for (long long p = (long long)blockIdx.x * blockDim.x + threadIdx.x; p < total; p += (long long)gridDim.x * blockDim.x) {
-        const int at = off[R.expert[p]] + R.rank[p];
+        const int e = R.expert[p], at = e < R.E ? off[e] + R.rank[p] : -1;
         R.index[p] = at;
-        R.token[at] = (int)(p / R.top);
+        if (at >= 0) R.token[at] = (int)(p / R.top);
     }
 }
 
 __global__ void __launch_bounds__(RS_WARPS * 32) route_small_kernel(const __grid_constant__ Route R) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5;
-    float* c_s = smem + warp * 2 * R.E;
-    int* count = reinterpret_cast<int*>(smem + RS_WARPS * 2 * R.E);
+    float* c_s = smem + warp * 2 * R.O;
+    int* count = reinterpret_cast<int*>(smem + RS_WARPS * 2 * R.O);
     int* off = count + R.E;
     for (int e = threadIdx.x; e < R.E; e += blockDim.x) count[e] = 0;
     pdl_wait();
@@ -157,28 +174,28 @@ __global__ void __launch_bounds__(RS_WARPS * 32) route_small_kernel(const __grid
     for (int i = warp; i < R.n; i += RS_WARPS)
         choose(R, i, c_s, Logits{R, i}, [&](int k, int e) {
             R.expert[(size_t)i * R.top + k] = e;
-            R.rank[(size_t)i * R.top + k] = atomicAdd(&count[e], 1);
+            if (e < R.E) R.rank[(size_t)i * R.top + k] = atomicAdd(&count[e], 1);
         });
     __syncthreads();
     prefix(count, off, R.E);
     __syncthreads();
     for (int e = threadIdx.x; e <= R.E; e += blockDim.x) R.offsets[e] = off[e];
     for (int p = threadIdx.x; p < R.n * R.top; p += blockDim.x) {
-        const int at = off[R.expert[p]] + R.rank[p];
+        const int e = R.expert[p], at = e < R.E ? off[e] + R.rank[p] : -1;
         R.index[p] = at;
-        R.token[at] = p / R.top;
+        if (at >= 0) R.token[at] = p / R.top;
     }
 }
 
 constexpr int RR_THREADS = 128, RR_WARPS = RR_THREADS / 32;
 
 // CTA (x, token): every gridDim.x-th group of RR_WARPS experts, a warp per expert.  Of a token's CTAs the last one to finish chooses; of the
-// tokens the last one puts all pairs in order.  h [n][W] of pitch ldh, w [E][W], both bf16 or fp32; z [n][E].  done [n + 1]: zero before
+// tokens the last one puts all pairs in order.  h [n][W] of pitch ldh, w [O][W], both bf16 or fp32; z [n][O].  done [n + 1]: zero before
 // and after.
 template <typename T>
 __global__ void __launch_bounds__(RR_THREADS) route_rows_kernel(const __grid_constant__ Route R, const T* __restrict__ h, long long ldh, const T* __restrict__ w, int W,
                                                                 float* z, unsigned* done) {
-    extern __shared__ float c_s[];                     // [2 E], later counts [E] and offsets [E + 1]
+    extern __shared__ float c_s[];                     // [2 O], later counts [E] and offsets [E + 1]
     __shared__ int last;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, i = blockIdx.y;
     constexpr int V = 16 / sizeof(T);                  // elements of a 16-byte load
@@ -186,7 +203,7 @@ __global__ void __launch_bounds__(RR_THREADS) route_rows_kernel(const __grid_con
     pdl_wait();
     pdl_launch_dependents();
     const T* x = h + (size_t)i * ldh;
-    for (int e = blockIdx.x * RR_WARPS + warp; e < R.E; e += gridDim.x * RR_WARPS) {
+    for (int e = blockIdx.x * RR_WARPS + warp; e < R.O; e += gridDim.x * RR_WARPS) {
         const T* row = w + (size_t)e * W;
         float a = 0.f;
         if (vec) {
@@ -201,7 +218,7 @@ __global__ void __launch_bounds__(RR_THREADS) route_rows_kernel(const __grid_con
         } else
             for (int c = lane; c < W; c += 32) a = fmaf((float)row[c], (float)x[c], a);
         a = warp_sum(a);
-        if (lane == 0) z[(size_t)i * R.E + e] = a;
+        if (lane == 0) z[(size_t)i * R.O + e] = a;
     }
     auto finished = [&](unsigned* counter, unsigned of) {          // whether this CTA is the last of `of` to come here
         __threadfence();
@@ -215,21 +232,24 @@ __global__ void __launch_bounds__(RR_THREADS) route_rows_kernel(const __grid_con
         return last != 0;
     };
     if (!finished(done + i, gridDim.x)) return;
-    if (warp == 0) choose(R, i, c_s, [&](int e) { return __ldcg(z + (size_t)i * R.E + e); }, [&](int k, int e) { R.expert[(size_t)i * R.top + k] = e; });
+    if (warp == 0) choose(R, i, c_s, [&](int e) { return __ldcg(z + (size_t)i * R.O + e); }, [&](int k, int e) { R.expert[(size_t)i * R.top + k] = e; });
     if (!finished(done + R.n, gridDim.y)) return;
     int *count = reinterpret_cast<int*>(c_s), *off = count + R.E;
     for (int e = threadIdx.x; e < R.E; e += RR_THREADS) count[e] = 0;
     __syncthreads();
     const int pairs = R.n * R.top;
-    for (int p = threadIdx.x; p < pairs; p += RR_THREADS) R.rank[p] = atomicAdd(&count[__ldcg(R.expert + p)], 1);
+    for (int p = threadIdx.x; p < pairs; p += RR_THREADS) {
+        const int e = __ldcg(R.expert + p);
+        if (e < R.E) R.rank[p] = atomicAdd(&count[e], 1);
+    }
     __syncthreads();
     prefix(count, off, R.E);
     __syncthreads();
     for (int e = threadIdx.x; e <= R.E; e += RR_THREADS) R.offsets[e] = off[e];
     for (int p = threadIdx.x; p < pairs; p += RR_THREADS) {
-        const int at = off[__ldcg(R.expert + p)] + R.rank[p];
+        const int e = __ldcg(R.expert + p), at = e < R.E ? off[e] + R.rank[p] : -1;
         R.index[p] = at;
-        R.token[at] = p / R.top;
+        if (at >= 0) R.token[at] = p / R.top;
     }
 }
 
@@ -306,24 +326,25 @@ __global__ void __launch_bounds__(256) expert_simt_kernel(const T* __restrict__ 
 
 using namespace ptb;
 
-// Routing of n tokens: z [splits][n] fp32 logits (rows of pitch ld, splits `stride` apart), correction [E].  index [n, top]: the place of a
-// token's i-th expert in the order by expert; weight [n, top]: its score over the sum of the chosen ones, times scale; token [n top]: the
-// token of every place; offsets [E + 1].  work: 2 n top + E ints.
-PTB_API int ptb_expert_route(const float* z, int splits, long long stride, long long ld, const float* correction, int n, int E, int top, float scale, int* index,
-                             float* weight, int* token, int* offsets, int* work, int* status, cudaStream_t st) {
+// Routing of n tokens over O >= E router outputs: z [splits][n] fp32 logits (rows of pitch ld, splits `stride` apart), correction [O].  index
+// [n, top]: the place of a token's i-th expert in the order by expert, -1 for an output behind the experts; weight [n, top]: its sigmoid score over
+// the sum of the chosen ones, times scale (softmax: its score times scale); token [n top]: the token of every place; offsets [E + 1].  work:
+// 2 n top + E ints.
+PTB_API int ptb_expert_route(const float* z, int splits, long long stride, long long ld, const float* correction, int n, int E, int O, int softmax, int top, float scale,
+                             int* index, float* weight, int* token, int* offsets, int* work, int* status, cudaStream_t st) {
     using namespace ptb::moe;
     if (n <= 0) return 0;
-    if (E < 1 || top < 1 || top > E || E > 1024) { ptb_set_error("experts: %d of %d experts (at most 1024)", top, E); return -1; }
+    if (E < 1 || O < E || top < 1 || top > O || O > 1024) { ptb_set_error("experts: %d of %d outputs (at most 1024), %d experts", top, O, E); return -1; }
     const size_t pairs = (size_t)n * top;
-    Route r{z, splits, stride, ld, correction, n, E, top, scale, index, weight, token, offsets, work, work + pairs, work + 2 * pairs, status};
+    Route r{z, splits, stride, ld, correction, n, E, top, O, softmax, scale, index, weight, token, offsets, work, work + pairs, work + 2 * pairs, status};
     const bool pdl = ptb_pdl_enabled();
-    if (n <= SMALL_TOKENS && E <= 256) {
-        const size_t smem = ((size_t)RS_WARPS * 2 * E + 2 * E + 1) * 4;
+    if (n <= SMALL_TOKENS && O <= 256) {
+        const size_t smem = ((size_t)RS_WARPS * 2 * O + 2 * E + 1) * 4;
         if (smem > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(route_small_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
         PTB_CUDA_OK(ptb_launch(route_small_kernel, dim3(1), dim3(RS_WARPS * 32), smem, st, pdl, r));
     } else {
         PTB_CUDA_OK(cudaMemsetAsync(r.counts, 0, (size_t)E * 4, st));
-        const size_t smem = ((size_t)RT_WARPS * 2 * E + 2 * E) * 4;
+        const size_t smem = ((size_t)RT_WARPS * 2 * O + 2 * E) * 4;
         if (smem > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
         PTB_CUDA_OK(ptb_launch(route_kernel, dim3((n + RT_WARPS - 1) / RT_WARPS), dim3(RT_WARPS * 32), smem, st, false, r));
         PTB_CUDA_OK(ptb_launch(place_kernel, dim3((unsigned)std::min<size_t>(1024, (pairs + 255) / 256)), dim3(256), (size_t)(E + 1) * 4, st, pdl, r));
@@ -332,20 +353,23 @@ PTB_API int ptb_expert_route(const float* z, int splits, long long stride, long 
     return 0;
 }
 
-// The same from the rows themselves, for few tokens: h [n, W] (pitch ldh) and the router w [E, W], both bf16 or fp32.  work: 2 n top ints and n E floats;
+// The same from the rows themselves, for few tokens: h [n, W] (pitch ldh) and the router w [O, W], both bf16 or fp32.  work: 2 n top ints and n O floats;
 // done: n + 1 unsigned that are zero between calls, used by one stream at a time.
-PTB_API int ptb_expert_route_rows(const void* h, long long ldh, const void* w, int W, const float* correction, int n, int E, int top, float scale, int* index,
-                                  float* weight, int* token, int* offsets, int* work, unsigned* done, int bf16, cudaStream_t st) {
+PTB_API int ptb_expert_route_rows(const void* h, long long ldh, const void* w, int W, const float* correction, int n, int E, int O, int softmax, int top,
+                                  float scale, int* index, float* weight, int* token, int* offsets, int* work, unsigned* done, int bf16, cudaStream_t st) {
     using namespace ptb::moe;
     if (n <= 0) return 0;
     const size_t pairs = (size_t)n * top;
-    if (E < 1 || top < 1 || top > E || E > 1024 || n > 65535 || W < 1) { ptb_set_error("experts: %d of %d experts (at most 1024), %d columns", top, E, W); return -1; }
-    const Route r{nullptr, 0, 0, 0, correction, n, E, top, scale, index, weight, token, offsets, work, work + pairs, nullptr, nullptr};
+    if (E < 1 || O < E || top < 1 || top > O || O > 1024 || n > 65535 || W < 1) {
+        ptb_set_error("experts: %d of %d outputs (at most 1024), %d experts, %d columns", top, O, E, W);
+        return -1;
+    }
+    const Route r{nullptr, 0, 0, 0, correction, n, E, top, O, softmax, scale, index, weight, token, offsets, work, work + pairs, nullptr, nullptr};
     const bool pdl = ptb_pdl_enabled();
     auto go = [&](auto k, auto t) {
         using T = decltype(t);
-        const int groups = std::max(1, std::min((E + RR_WARPS - 1) / RR_WARPS, 148 * 8 / n));
-        return ptb_launch(k, dim3(groups, n), dim3(RR_THREADS), (2 * (size_t)E + 1) * 4, st, pdl, r, (const T*)h, ldh, (const T*)w, W,
+        const int groups = std::max(1, std::min((O + RR_WARPS - 1) / RR_WARPS, 148 * 8 / n));
+        return ptb_launch(k, dim3(groups, n), dim3(RR_THREADS), (2 * (size_t)O + 1) * 4, st, pdl, r, (const T*)h, ldh, (const T*)w, W,
                           reinterpret_cast<float*>(work + 2 * pairs), done);
     };
     PTB_CUDA_OK(bf16 ? go(route_rows_kernel<__nv_bfloat16>, __nv_bfloat16()) : go(route_rows_kernel<float>, 0.f));

@@ -19,10 +19,11 @@ using namespace ptb::gemm;
 
 constexpr int MAX_EXPERTS = 1024, WT = 128;            // WT: weight rows of a box
 
-__global__ void __launch_bounds__(256) expert_gather_kernel(const uint4* __restrict__ h, long long ld, const int* __restrict__ token, uint4* __restrict__ out, int rows,
-                                                            int vec, int tokens, int* status) {
+__global__ void __launch_bounds__(256) expert_gather_kernel(const uint4* __restrict__ h, long long ld, const int* __restrict__ token, const int* __restrict__ count,
+                                                            uint4* __restrict__ out, int rows, int vec, int tokens, int* status) {
     pdl_wait();
     pdl_launch_dependents();
+    rows = min(rows, *count);
     for (int r = blockIdx.x; r < rows; r += gridDim.x) {
         int t = token[r];
         if (t < 0 || t >= tokens) {
@@ -263,12 +264,13 @@ static int launch(const void* a, long long lda, const void* w, const Params& p, 
 
 using namespace ptb;
 
-// out [rows, W] = h[token[r]] (rows of h [tokens] of pitch ld), bf16; W, ld multiples of eight, 16-byte aligned.
-PTB_API int ptb_expert_gather(const void* h, long long ld, const int* token, void* out, int rows, int W, int tokens, int* status, cudaStream_t st) {
+// out [rows, W] = h[token[r]] (rows of h [tokens] of pitch ld), bf16, for the first `count` (on the device) of at most `rows` rows; W, ld multiples
+// of eight, 16-byte aligned.
+PTB_API int ptb_expert_gather(const void* h, long long ld, const int* token, const int* count, void* out, int rows, int W, int tokens, int* status, cudaStream_t st) {
     if (rows <= 0) return 0;
     if (W % 8 || ld % 8 || (((uintptr_t)h | (uintptr_t)out) & 15)) { ptb_set_error("expert_gather: %d columns of pitch %lld", W, ld); return -1; }
     const int vec = W / 8, threads = std::min(256, (vec + 31) / 32 * 32);
-    PTB_CUDA_OK(ptb_launch(moe100::expert_gather_kernel, dim3(std::min(rows, 148 * 16)), dim3(threads), 0, st, ptb_pdl_enabled(), (const uint4*)h, ld / 8, token, (uint4*)out,
+    PTB_CUDA_OK(ptb_launch(moe100::expert_gather_kernel, dim3(std::min(rows, 148 * 16)), dim3(threads), 0, st, ptb_pdl_enabled(), (const uint4*)h, ld / 8, token, count, (uint4*)out,
                            rows, vec, tokens, status));
     PTB_CUDA_OK(cudaGetLastError());
     return 0;

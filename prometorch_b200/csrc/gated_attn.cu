@@ -17,13 +17,16 @@ constexpr int GA_WARPS = GA_THREADS / 32;
 
 // ---------------------------------------------------------------------------------------------- norm + page write
 struct HeadNormParams {
-    const void* qkv;                   // [n, H D + G D + G Dv]: q heads, k heads, v heads
+    const void* qkv;                   // [n] rows: q heads, k heads from k_col on, v heads from v_col on
     long long ld;
+    int k_col, v_col;
     void* q_out;                       // [n, H, Dp], the pad filled with zeros
     void* k_pages;
     void* v_pages;
-    const float* qw;                   // [D]
-    const float* kw;                   // [D]
+    const float* qw;                   // [D] or null
+    const float* kw;                   // [D] or null
+    const float* gain;                 // [positions]: q times the entry of its position; or null
+    int positions;
     const void* v_first;               // rows of another layer's values [n, G Dv] (pitch v_first_ld), or null
     long long v_first_ld;
     float lam;                         // v = (1 - lam) v + lam v_first
@@ -81,6 +84,11 @@ __global__ void __launch_bounds__(256) head_norm_write_kernel(const __grid_const
         if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
         page = -1;
     }
+    float factor = 1.f;
+    if (P.gain) {
+        if ((pos < 0 || pos >= P.positions) && threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+        factor = P.gain[min(max(pos, 0), P.positions - 1)];
+    }
     const T* row = (const T*)P.qkv + i * P.ld;
     const int sub = threadIdx.x % lph, group = threadIdx.x / lph, groups = blockDim.x / lph;
     const int heads = P.H + 2 * P.G;
@@ -89,7 +97,7 @@ __global__ void __launch_bounds__(256) head_norm_write_kernel(const __grid_const
     for (int h = group; h < heads; h += groups) {
         const bool is_q = h < P.H, is_v = h >= P.H + P.G;
         const int width = is_v ? P.Dv : P.D, padded = is_v ? P.Dvp : P.Dp;
-        const T* src = row + (is_v ? (size_t)(P.H + P.G) * P.D + (size_t)(h - P.H - P.G) * P.Dv : (size_t)h * P.D);
+        const T* src = row + (is_v ? P.v_col + (size_t)(h - P.H - P.G) * P.Dv : is_q ? (size_t)h * P.D : P.k_col + (size_t)(h - P.H) * P.D);
         T* dst;
         if (is_q) dst = (T*)P.q_out + (i * P.H + h) * P.Dp;
         else {
@@ -113,6 +121,7 @@ __global__ void __launch_bounds__(256) head_norm_write_kernel(const __grid_const
             }
             for (int o = lph / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
             rs = rsqrtf(ss / (float)width + P.eps);
+            if (is_q) rs *= factor;
         }
         const float* w = is_q ? P.qw : P.kw;
         const T* vf = is_v && P.v_first ? (const T*)P.v_first + i * P.v_first_ld + (size_t)(h - P.H - P.G) * P.Dv : nullptr;
@@ -123,7 +132,7 @@ __global__ void __launch_bounds__(256) head_norm_write_kernel(const __grid_const
                     Vec8T<T>::load(src + c, f);
                     if (!is_v) {
 #pragma unroll
-                        for (int e = 0; e < 8; ++e) f[e] = f[e] * rs * w[c + e];
+                        for (int e = 0; e < 8; ++e) f[e] = f[e] * rs * (w ? w[c + e] : 1.f);
                     } else if (vf) {
                         float g[8];
                         Vec8T<T>::load(vf + c, g);
@@ -139,7 +148,7 @@ __global__ void __launch_bounds__(256) head_norm_write_kernel(const __grid_const
                 float f = 0.f;
                 if (c < width) {
                     f = ga_f(src[c]);
-                    if (!is_v) f = f * rs * w[c];
+                    if (!is_v) f = f * rs * (w ? w[c] : 1.f);
                     else if (vf) f = (1.f - P.lam) * f + P.lam * ga_f(vf[c]);
                 }
                 dst[c] = ga_t<T>(f);
@@ -429,26 +438,28 @@ __global__ void __launch_bounds__(256) gated_merge_kernel(const float* __restric
 
 using namespace ptb;
 
-// After the packed projection qkv [n, H D + G D + G Dv] (pitch ld): q_out [n, H, Dp] = RMS norm of the q heads (weight qw [D]), the
-// k heads' norm (kw) and the values go to the page slot of (req, pos).  v_first (pitch v_first_ld, optional) mixes another layer's
+// After the packed projection qkv (pitch ld; q heads first, k and v heads at k_col and v_col): q_out [n, H, Dp] = RMS norm of the q heads (weight qw
+// [D]; null: none) times gain[pos] (fp32 [positions]; null: 1), the k heads' norm (kw) and the values go to the page slot of (req, pos).  v_first (pitch v_first_ld, optional) mixes another layer's
 // values in: v = (1 - lam) v + lam v_first.  Dp, Dvp: sizes as stored, multiples of 16; the pad is zero.
-PTB_API int ptb_head_norm_write(const void* qkv, long long ld, void* q_out, void* k_pages, void* v_pages, const float* qw, const float* kw,
+PTB_API int ptb_head_norm_write(const void* qkv, long long ld, int k_col, int v_col, void* q_out, void* k_pages, void* v_pages, const float* qw, const float* kw,
+                                const float* gain, int positions,
                                 const void* v_first, long long v_first_ld, float lam, const int* pos, int pos_stride, const int* req,
                                 int req_stride, const int* page_table, int pt_stride, int n_pages, int n, int H, int G, int D, int Dp,
                                 int Dv, int Dvp, float eps, int* status, int bf16, cudaStream_t st) {
     if (n <= 0) return 0;
-    if (H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || Dp % 16 || Dvp % 16 || Dp < D || Dvp < Dv) {
+    if (H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || Dp % 16 || Dvp % 16 || Dp < D || Dvp < Dv || (gain && positions < 1)) {
         ptb_set_error("head_norm_write: bad sizes (H %d, G %d, D %d/%d, Dv %d/%d)", H, G, D, Dp, Dv, Dvp);
         return -1;
     }
     HeadNormParams p;
+    p.k_col = k_col; p.v_col = v_col; p.gain = gain; p.positions = positions;
     p.qkv = qkv; p.ld = ld; p.q_out = q_out; p.k_pages = k_pages; p.v_pages = v_pages; p.qw = qw; p.kw = kw; p.v_first = v_first;
     p.v_first_ld = v_first_ld; p.lam = lam; p.pos = pos; p.req = req; p.page_table = page_table; p.pos_stride = pos_stride;
     p.req_stride = req_stride; p.pt_stride = pt_stride; p.n_pages = n_pages; p.H = H; p.G = G; p.D = D; p.Dp = Dp; p.Dv = Dv; p.Dvp = Dvp;
     p.eps = eps; p.status = status;
     const int elt = bf16 ? 2 : 4;
     const bool vec = D % 8 == 0 && Dv % 8 == 0 && ld % 8 == 0 && (!v_first || v_first_ld % 8 == 0) && ((uintptr_t)qkv & 15) == 0 &&
-                     ((uintptr_t)v_first & 15) == 0 && ((size_t)(H + G) * D * elt) % 16 == 0;
+                     ((uintptr_t)v_first & 15) == 0 && ((size_t)k_col * elt) % 16 == 0 && ((size_t)v_col * elt) % 16 == 0;
     const int steps = (std::max(Dp, Dvp) + (vec ? 7 : 0)) / (vec ? 8 : 1);
     int lph = 1;
     while (lph < steps && lph < 32) lph *= 2;

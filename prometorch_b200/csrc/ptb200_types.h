@@ -70,14 +70,14 @@ typedef struct PtbRecurrence {
     long long ld;
     int q_col, k_col, v_col;
     int silu;               // decay attention: q, k and v pass SiLU first
-    int delta;              // 1: gated delta rule, decays per key channel; 2: one decay per head; 0: decay attention (G == H)
+    int delta;              // 1: gated delta rule, decays per key channel; 2: one decay per head; 0: decay attention (G == H); 3: state-space step
     int bf16;
     const void* beta;       // delta: [n][H] of pitch ld_beta in the type of x, before the sigmoid
     long long ld_beta;
-    const void* a;          // delta 1: fp32 [n][H D] of pitch ld_a; delta 2: [n][H] of pitch ld_a in the type of x
+    const void* a;          // delta 1: fp32 [n][H D] of pitch ld_a; delta 2, 3: [n][H] of pitch ld_a in the type of x
     long long ld_a;
     const float* decay;     // [H]: the decay, or exp(A_log)
-    const float* dt_bias;   // delta 1: [H D]; delta 2: [H]
+    const float* dt_bias;   // delta 1: [H D]; delta 2, 3: [H]
     float* state;           // [slots][H][D][Dv]
     int slots, n, H, G, D, Dv;
     const void* seqs;       // [n_seqs] int4 (first row, rows, position of the first, slot); null: one token per row
@@ -92,6 +92,7 @@ typedef struct PtbRecurrence {
     const void* low;        // the matrix form may take a as low low_w^T instead: [n][rank] of pitch ld_low, bf16
     long long ld_low;
     const void* low_w;      // [H D][rank], bf16
+    const float* skip;      // delta 3: [H]
 } PtbRecurrence;
 
 // Softmax attention over the paged cache (window_attn.cuh has the meaning of the mask and of the two maps).
@@ -109,12 +110,14 @@ typedef struct PtbWindowAttn {
     float* work;            // rows: ptb_window_rows_work_floats(n, H maps, Dvp, nsplit) floats where nsplit or maps is above one
     int* status;
     const void* tiles;      // tiles: [n_tiles] int4 (first row, its position, rows <= 128, row of the page table or first row of the flat context)
+    const float* rel;       // [H][rel_n]: added to a score by the key's distance, the last entry for all beyond; or null
     const void* k_rot;      // flat: the rotated key part that all heads share, rows of rot_ld
     long long k_ld, v_row, rot_ld;      // flat: pitches of the context's rows in k_pages ([rows][H][Dp]), v_pages ([rows][H][Dvp]) and k_rot
     int n, H, G, D, Dp, Dv, Dvp, v_ld, maps;
     int pos_stride, req_stride, pt_stride, n_pages;
     int window, keep, chunked;
     int max_keys, nsplit, bf16;
+    int rel_n;
     int n_tiles, flat_rows, rot_dim;    // flat_rows > 0: keys and values lie flat, flat_rows of them; q is [n][H][Dq], see ptb_window_attn_tiles
     float scale, mix, mix_gain, mix_eps;
 } PtbWindowAttn;
@@ -140,3 +143,54 @@ typedef struct PtbTanhResidual {
     int n, W, bf16, pad;
     int* status;
 } PtbTanhResidual;
+
+// Token, pair and position tables into the residual streams of every token.
+typedef struct PtbPairEmbed {
+    const int* ids;         // [n] of id_stride
+    const int* pos;         // [n] of pos_stride
+    const int* req;         // [n] of req_stride: slots
+    int* last;              // [slots]: the id a sequence ended with; what it held counts for positions above zero
+    const void* seqs;       // [n_seqs] int4 (first row, rows, position of the first, slot): a prompt pass; null: one token per row
+    const void* table;      // [V][W]
+    const void* pairs;      // [rows + 1][W]: row (id before * mul_before + id * mul_id) mod rows, the last one for a first token
+    const void* at;         // [positions][W]
+    float* x;               // [n][streams][W]
+    int* status;
+    long long mul_before, mul_id;
+    int id_stride, pos_stride, req_stride, slots, n_seqs, n, V, rows, positions, W, streams, bf16;
+} PtbPairEmbed;
+
+// A matrix [n][W] in bf16 (f32 = 0), or the sum of `splits` fp32 matrices `stride` apart; rows of pitch ld.  y null: absent.
+typedef struct PtbDense {
+    const void* y;
+    int f32, splits;
+    long long stride, ld;
+} PtbDense;
+
+// Between two sublayers: with `mix`, stream t becomes sum_s mix[s][t] x_s + way_out[t] f sigmoid(gate + gate_bias), f the sum of y and of `top`
+// weighed rows; then u = sum_s way_in[s] x_s (null: their sum), h = (u - mean) / sqrt(variance + eps) norm, and with `conv` conv_out = h + the
+// causal convolution of h over the sequence's tokens, one token per sequence.
+typedef struct PtbStreamStep {
+    float* x;               // [n][streams][W]
+    const float* mix;       // [streams][streams] from, to; null: the streams stay as they are
+    const float* way_out;   // [streams]
+    const float* way_in;    // [streams]
+    PtbDense y, gate;
+    const float* gate_bias; // [W]
+    const int* index_of;    // [n][top] rows of `experts`, -1: the token's own row of `self`; null: none
+    const float* weight;    // [n][top]
+    const void* experts;    // [e_rows] of pitch e_ld, in the compute type
+    const void* self;       // [n][W]
+    long long e_ld;
+    const float* norm;      // [W]; null: no h
+    void* h;                // [m][W] bf16 or fp32
+    const float* conv;      // [taps][W], the current token's tap last, or null
+    void* conv_state;       // [slots][taps - 1][W] in the type of h
+    void* conv_out;         // [m][W]
+    const int* pos;
+    const int* req;
+    const long long* index; // [m] rows of x, or null (m = n)
+    int* status;
+    int top, e_rows, taps, slots, pos_stride, req_stride, n, m, W, streams, bf16;
+    float eps;
+} PtbStreamStep;

@@ -1,9 +1,10 @@
 // Recurrent layers token by token, and what surrounds them:
-//   short_conv_kernel / conv_tail_kernel   causal convolution over time per channel, SiLU; the last inputs stay in the sequence's slot;
+//   short_conv_kernel / conv_tail_kernel   causal convolution over time per channel, then SiLU, or the input added; the last inputs stay in the
+//                                          sequence's slot;
 //   recurrence_kernel                      one CTA per (32 value columns, head, sequence); the state stays in registers from the first
 //                                          token to the last.  One token per sequence in a decode pass, every token of a prompt in
 //                                          true fp32 arithmetic (recurrence_chunk.cu has the matrix form for bf16 prompts);
-//   group_norm_gate_kernel                 RMS norm of groups of columns, weight, sigmoid or SiLU gate.
+//   group_norm_gate_kernel                 RMS norm of groups of columns, weight, sigmoid or SiLU gate (behind the norm, or ahead of it).
 // A slot outside its extent sets PTB_ERR_BOUNDS and its sequence is skipped.
 #include "recurrence.cuh"
 #include <algorithm>
@@ -15,6 +16,8 @@ struct ConvParams {
     const void* x;
     long long ld;
     const float* w;                    // [taps][C]
+    const float* bias;                 // [C] or null
+    int add;                           // the result is the input plus the convolution, without SiLU
     void* state;                       // [slots][taps - 1][C]
     void* out;                         // [n][C]
     const int* pos;
@@ -81,6 +84,15 @@ __device__ __forceinline__ Elems<T, E> conv_input(const ConvParams& P, int i, in
     return ld_elems<T, E>((const T*)P.state + ((size_t)slot * (P.taps - 1) + (P.taps - 1 - (m - in_batch))) * P.C + c);
 }
 
+template <int E>
+__device__ __forceinline__ void conv_bias(const ConvParams& P, int c, Elems<float, E>& b) {
+    if (P.bias) b = ld_elems<float, E>(P.bias + c);
+    else {
+#pragma unroll
+        for (int e = 0; e < E; ++e) b.v[e] = 0.f;
+    }
+}
+
 // A prompt pass with a fixed number of taps: weights and the last inputs stay in registers while a thread walks its rows.
 template <typename T, int E, int TAPS>
 __global__ void __launch_bounds__(256) short_conv_taps_kernel(const __grid_constant__ ConvParams P) {
@@ -89,7 +101,8 @@ __global__ void __launch_bounds__(256) short_conv_taps_kernel(const __grid_const
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * E;
     if (c >= P.C) return;
     const int lo = blockIdx.y * CONV_TOKENS, hi = min(lo + CONV_TOKENS, P.n);
-    Elems<float, E> w[TAPS], x[TAPS];                  // x[m]: the input m tokens back
+    Elems<float, E> w[TAPS], x[TAPS], bias;            // x[m]: the input m tokens back
+    conv_bias(P, c, bias);
 #pragma unroll
     for (int m = 0; m < TAPS; ++m) w[m] = ld_elems<float, E>(P.w + (size_t)(TAPS - 1 - m) * P.C + c);
     int before = -1;                                   // slot of the row before
@@ -120,7 +133,8 @@ __global__ void __launch_bounds__(256) short_conv_taps_kernel(const __grid_const
             float a = x[TAPS - 1].v[e] * w[TAPS - 1].v[e];
 #pragma unroll
             for (int m = TAPS - 2; m >= 0; --m) a = fmaf(x[m].v[e], w[m].v[e], a);
-            acc.v[e] = silu(a);
+            a += bias.v[e];
+            acc.v[e] = P.add ? now.v[e] + a : silu(a);
 #pragma unroll
             for (int m = TAPS - 1; m > 0; --m) x[m].v[e] = x[m - 1].v[e];
         }
@@ -135,6 +149,8 @@ __global__ void __launch_bounds__(256) short_conv_kernel(const __grid_constant__
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * E;
     if (c >= P.C) return;
     const int per = P.seqs ? CONV_TOKENS : 1, lo = blockIdx.y * per, hi = min(lo + per, P.n);
+    Elems<float, E> bias;
+    conv_bias(P, c, bias);
     for (int i = lo; i < hi; ++i) {
         const int pos = P.pos[(size_t)i * P.pos_stride];
         int slot = P.req[(size_t)i * P.req_stride], in_batch = 0;
@@ -149,7 +165,7 @@ __global__ void __launch_bounds__(256) short_conv_kernel(const __grid_constant__
         {
             const Elems<float, E> w = ld_elems<float, E>(P.w + (size_t)(P.taps - 1) * P.C + c);
 #pragma unroll
-            for (int e = 0; e < E; ++e) acc.v[e] = now.v[e] * w.v[e];
+            for (int e = 0; e < E; ++e) acc.v[e] = fmaf(now.v[e], w.v[e], bias.v[e]);
         }
         T* st = (T*)P.state + (size_t)max(slot, 0) * (P.taps - 1) * P.C + c;
         for (int m = P.taps - 1; m >= 1; --m) {
@@ -162,7 +178,7 @@ __global__ void __launch_bounds__(256) short_conv_kernel(const __grid_constant__
         }
         if (!P.seqs && slot >= 0 && P.taps > 1) st_elems<T, E>(st + (size_t)(P.taps - 2) * P.C, now);
 #pragma unroll
-        for (int e = 0; e < E; ++e) acc.v[e] = silu(acc.v[e]);
+        for (int e = 0; e < E; ++e) acc.v[e] = P.add ? now.v[e] + acc.v[e] : silu(acc.v[e]);
         st_elems<T, E>((T*)P.out + (size_t)i * P.C + c, acc);
     }
 }
@@ -193,8 +209,8 @@ constexpr int RC_THREADS = 256, RC_WARPS = 8, RC_COLS = 32;
 // MODE: `delta` of PtbRecurrence.
 template <typename T, int MODE, int RM>
 __global__ void __launch_bounds__(RC_THREADS) recurrence_kernel(const __grid_constant__ PtbRecurrence P) {
-    constexpr bool DELTA = MODE != 0;
-    __shared__ float q_s[3][RM * 32], k_s[3][RM * 32], g_s[3][MODE == 1 ? RM * 32 : 1];      // three: a slow warp may still update with the token before
+    constexpr bool DELTA = MODE == 1 || MODE == 2;
+    __shared__ float q_s[3][RM * 32], k_s[3][RM * 32], g_s[3][MODE == 1 ? RM * 32 : 2];      // three: a slow warp may still update with the token before
     __shared__ float red_s[2][RC_WARPS][4];
     __shared__ float4 part_s[2][RC_WARPS][8][2];
     pdl_wait();
@@ -220,7 +236,7 @@ __global__ void __launch_bounds__(RC_THREADS) recurrence_kernel(const __grid_con
                 for (int e = 0; e < live; ++e) S[i][e] = st[(size_t)d * Dv + col + e];
         }
     }
-    const float rate = P.decay[h];
+    const float rate = P.decay[h], skip = MODE == 3 ? P.skip[h] : 0.f;
     auto stage = [&](int i) {
         const int b = i % 3;
         const T* row = (const T*)P.x + (size_t)(s.row0 + i) * P.ld;
@@ -238,6 +254,12 @@ __global__ void __launch_bounds__(RC_THREADS) recurrence_kernel(const __grid_con
             qq += q * q; kk += k * k; qk += q * k;
         }
         qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
+        if constexpr (MODE == 3)
+            if (threadIdx.x == 0) {                    // the decay and the step
+                const float dt = softplus(rc_f<T>(((const T*)P.a)[(size_t)(s.row0 + i) * P.ld_a + h]) + P.dt_bias[h]);
+                g_s[b][0] = expf(-rate * dt);
+                g_s[b][1] = dt;
+            }
         if constexpr (MODE == 2)
             if (threadIdx.x == 0) g_s[b][0] = expf(delta_log_decay(rc_f<T>(((const T*)P.a)[(size_t)(s.row0 + i) * P.ld_a + h]), P.dt_bias[h], rate));
         if (lane == 0) { red_s[i & 1][warp][0] = qq; red_s[i & 1][warp][1] = kk; red_s[i & 1][warp][2] = qk; }
@@ -250,7 +272,7 @@ __global__ void __launch_bounds__(RC_THREADS) recurrence_kernel(const __grid_con
         float v[4] = {0.f, 0.f, 0.f, 0.f}, beta = 1.f;
         for (int e = 0; e < live; ++e) {
             v[e] = rc_f<T>(((const T*)P.x)[r * P.ld + P.v_col + (size_t)h * Dv + col + e]);
-            if (!DELTA && P.silu) v[e] = silu(v[e]);
+            if (MODE == 0 && P.silu) v[e] = silu(v[e]);
         }
         if constexpr (DELTA) beta = sigmoid(rc_f<T>(((const T*)P.beta)[r * P.ld_beta + h]));
         float qq = 0.f, kk = 0.f, qk = 0.f;
@@ -261,7 +283,7 @@ __global__ void __launch_bounds__(RC_THREADS) recurrence_kernel(const __grid_con
 #pragma unroll
         for (int j = 0; j < RM; ++j) {
             const int d = ty + 32 * j;
-            const float g = MODE == 1 ? g_s[c][d] : MODE == 2 ? g_s[c][0] : rate, k = k_s[c][d], q = q_s[c][d];
+            const float g = MODE == 1 ? g_s[c][d] : MODE >= 2 ? g_s[c][0] : rate, k = k_s[c][d], q = q_s[c][d];
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 S[j][e] *= g;
@@ -292,9 +314,9 @@ __global__ void __launch_bounds__(RC_THREADS) recurrence_kernel(const __grid_con
         const float a4[4] = {ak.x, ak.y, ak.z, ak.w}, r4[4] = {aq.x, aq.y, aq.z, aq.w};
         float u[4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) u[e] = DELTA ? beta * (v[e] - a4[e] * kn) : v[e];
+        for (int e = 0; e < 4; ++e) u[e] = DELTA ? beta * (v[e] - a4[e] * kn) : MODE == 3 ? g_s[c][1] * v[e] : v[e];
         if (ty == 0)
-            for (int e = 0; e < live; ++e) P.out[r * P.H * Dv + (size_t)h * Dv + col + e] = qn * (r4[e] + qk * kn * u[e]);
+            for (int e = 0; e < live; ++e) P.out[r * P.H * Dv + (size_t)h * Dv + col + e] = qn * (r4[e] + qk * kn * u[e]) + (MODE == 3 ? skip * v[e] : 0.f);
 #pragma unroll
         for (int j = 0; j < RM; ++j) {
             const float k = k_s[c][ty + 32 * j] * kn;
@@ -317,7 +339,8 @@ __global__ void __launch_bounds__(RC_THREADS) recurrence_kernel(const __grid_con
 // TPG threads per group of gs columns; with V = 4, gs and every pitch are multiples of four.
 template <typename T, typename TG, int TPG, int V>
 __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const TG* __restrict__ gate,
-                                                              long long ld_gate, T* __restrict__ out, long long groups, int per_row, int gs, float eps, int act) {
+                                                              long long ld_gate, T* __restrict__ out, long long groups, int per_row, int gs, float eps, int act, int first,
+                                                              int w_row) {
     __shared__ float red[8];
     pdl_wait();
     pdl_launch_dependents();
@@ -327,9 +350,16 @@ __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __res
     const long long row = grp / per_row;
     const int at = (int)(grp % per_row) * gs;
     const float* src = o + row * per_row * gs + at;
+    const TG* gp = gate + row * ld_gate + at;
+    const float* wp = w + (w_row ? at : 0);
     float ss = 0.f;
     for (int c = t * V; c < gs; c += TPG * V) {
-        const Elems<float, V> f = ld_elems<float, V>(src + c);
+        Elems<float, V> f = ld_elems<float, V>(src + c);
+        if (first) {
+            const Elems<TG, V> g = ld_elems<TG, V>(gp + c);
+#pragma unroll
+            for (int e = 0; e < V; ++e) f.v[e] *= act ? silu(g.v[e]) : sigmoid(g.v[e]);
+        }
 #pragma unroll
         for (int e = 0; e < V; ++e) ss += f.v[e] * f.v[e];
     }
@@ -342,10 +372,9 @@ __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __res
         for (int i = 0; i < 8; ++i) ss += red[i];
     }
     const float rs = rsqrtf(ss / (float)gs + eps);
-    const TG* gp = gate + row * ld_gate + at;
     T* op = out + row * per_row * gs + at;
     for (int c = t * V; c < gs; c += TPG * V) {
-        const Elems<float, V> f = ld_elems<float, V>(src + c), m = ld_elems<float, V>(w + c);
+        const Elems<float, V> f = ld_elems<float, V>(src + c), m = ld_elems<float, V>(wp + c);
         const Elems<TG, V> g = ld_elems<TG, V>(gp + c);
         Elems<T, V> r;
 #pragma unroll
@@ -356,11 +385,11 @@ __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __res
 
 template <typename T, typename TG>
 static cudaError_t norm_gate_launch(const float* o, const float* w, const void* gate, long long ld_gate, void* out, long long n, int per_row, int gs,
-                                    float eps, int act, bool vec, cudaStream_t st) {
+                                    float eps, int act, int first, int w_row, bool vec, cudaStream_t st) {
     const long long groups = n * per_row;
     auto go = [&](auto k, int tpg) {
         return ptb_launch(k, dim3((unsigned)((groups + 256 / tpg - 1) / (256 / tpg))), dim3(256), 0, st, ptb_pdl_enabled(), o, w, (const TG*)gate, ld_gate,
-                          (T*)out, groups, per_row, gs, eps, act);
+                          (T*)out, groups, per_row, gs, eps, act, first, w_row);
     };
     if (gs > 512) return vec ? go(group_norm_gate_kernel<T, TG, 256, 4>, 256) : go(group_norm_gate_kernel<T, TG, 256, 1>, 256);
     return vec ? go(group_norm_gate_kernel<T, TG, 32, 4>, 32) : go(group_norm_gate_kernel<T, TG, 32, 1>, 32);
@@ -382,7 +411,7 @@ int recurrence_check(const PtbRecurrence& p) {
         ptb_set_error("recurrence: bad sizes (H %d, G %d, D %d, Dv %d; D at most 512)", p.H, p.G, p.D, p.Dv);
         return -1;
     }
-    if (!p.x || !p.state || !p.out || !p.decay || (p.delta && ((!p.a && !p.low) || !p.beta || !p.dt_bias))) { ptb_set_error("recurrence: missing operand"); return -1; }
+    if (!p.x || !p.state || !p.out || !p.decay || (p.delta && ((!p.a && !p.low) || (p.delta == 3 ? !p.skip : !p.beta) || !p.dt_bias))) { ptb_set_error("recurrence: missing operand"); return -1; }
     if ((p.seqs ? p.n_seqs : p.n) > 65535) { ptb_set_error("recurrence: more than 65535 sequences in one launch"); return -1; }
     return 0;
 }
@@ -391,17 +420,17 @@ int recurrence_check(const PtbRecurrence& p) {
 
 using namespace ptb;
 
-// out [n, C] = silu(causal convolution of x [n, C] (pitch ld)) with w [taps][C] fp32, the current token's tap last; state [slots][taps - 1][C]
-// in the type of x.  seqs [n_seqs] int4 (first row, rows, first position, slot): a prompt pass; null: one token per row.
-PTB_API int ptb_short_conv(const void* x, long long ld, const float* w, int C, int taps, void* state, void* out, int n, int slots, const int* pos,
+// out [n, C] = silu(causal convolution of x [n, C] (pitch ld) + bias) with w [taps][C] and bias [C] (or null) fp32, the current token's tap last; `add`:
+// out = x + the convolution + bias.  state [slots][taps - 1][C] in the type of x.  seqs [n_seqs] int4 (first row, rows, first position, slot): a prompt pass; null: one token per row.
+PTB_API int ptb_short_conv(const void* x, long long ld, const float* w, const float* bias, int add, int C, int taps, void* state, void* out, int n, int slots, const int* pos,
                            int pos_stride, const int* req, int req_stride, const void* seqs, int n_seqs, int* status, int bf16, cudaStream_t st) {
     if (n <= 0 || C <= 0) return 0;
     if (taps < 1 || slots < 1 || n_seqs > 65535) { ptb_set_error("short_conv: %d taps, %d slots, %d sequences", taps, slots, n_seqs); return -1; }
     const int per = seqs ? CONV_TOKENS : 1;
     const long long rows = ((long long)n + per - 1) / per;
     if (rows > 65535) { ptb_set_error("short_conv: %d rows in one launch", n); return -1; }
-    ConvParams p{x, ld, w, state, out, pos, req, (const int4*)seqs, C, taps, n, slots, pos_stride, req_stride, n_seqs, status};
-    const bool vec = C % 8 == 0 && ld % 8 == 0 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)state | (uintptr_t)out) & 15) == 0;
+    ConvParams p{x, ld, w, bias, add, state, out, pos, req, (const int4*)seqs, C, taps, n, slots, pos_stride, req_stride, n_seqs, status};
+    const bool vec = C % 8 == 0 && ld % 8 == 0 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)bias | (uintptr_t)state | (uintptr_t)out) & 15) == 0;
     const int lanes = vec ? C / 8 : C, threads = lanes >= 256 ? 256 : (lanes + 31) / 32 * 32;
     const dim3 grid((lanes + threads - 1) / threads, (unsigned)rows);
     const bool pdl = ptb_pdl_enabled();
@@ -425,25 +454,25 @@ PTB_API int ptb_recurrence(const PtbRecurrence* args, cudaStream_t st) {
     if (p.n <= 0 || (p.seqs && p.n_seqs <= 0)) return 0;
     if (recurrence_check(p)) return -1;
     if (p.delta && !p.a) { ptb_set_error("recurrence: token by token takes a, not its low-rank factors"); return -1; }
-    if (p.delta < 0 || p.delta > 2) { ptb_set_error("recurrence: kind %d", p.delta); return -1; }
-    auto go = p.bf16 ? (p.delta == 2 ? recurrence_launch<__nv_bfloat16, 2> : p.delta ? recurrence_launch<__nv_bfloat16, 1> : recurrence_launch<__nv_bfloat16, 0>)
-                     : (p.delta == 2 ? recurrence_launch<float, 2> : p.delta ? recurrence_launch<float, 1> : recurrence_launch<float, 0>);
+    if (p.delta < 0 || p.delta > 3) { ptb_set_error("recurrence: kind %d", p.delta); return -1; }
+    auto go = p.bf16 ? (p.delta == 3 ? recurrence_launch<__nv_bfloat16, 3> : p.delta == 2 ? recurrence_launch<__nv_bfloat16, 2> : p.delta ? recurrence_launch<__nv_bfloat16, 1> : recurrence_launch<__nv_bfloat16, 0>)
+                     : (p.delta == 3 ? recurrence_launch<float, 3> : p.delta == 2 ? recurrence_launch<float, 2> : p.delta ? recurrence_launch<float, 1> : recurrence_launch<float, 0>);
     PTB_CUDA_OK(go(p, st));
     PTB_CUDA_OK(cudaGetLastError());
     return 0;
 }
 
 // out [n, per_row gs] (bf16 or fp32) = o / rms(o) * w * act(gate), act the sigmoid (0) or SiLU (1), o fp32 in groups of gs columns, w [gs] fp32, gate [n, per_row gs] with
-// row pitch ld_gate in bf16 (gate_bf16) or fp32.
+// row pitch ld_gate in bf16 (gate_bf16) or fp32.  first: out = g / rms(g) * w with g = o act(gate) instead; w_row: w is [per_row gs].
 PTB_API int ptb_group_norm_gate(const float* o, const float* w, const void* gate, int gate_bf16, long long ld_gate, void* out, int n, int per_row,
-                                int gs, float eps, int act, int bf16, cudaStream_t st) {
+                                int gs, float eps, int act, int first, int w_row, int bf16, cudaStream_t st) {
     if (n <= 0 || per_row <= 0 || gs <= 0) return 0;
     const bool vec = gs % 4 == 0 && ld_gate % 4 == 0 && (((uintptr_t)o | (uintptr_t)w | (uintptr_t)out | (uintptr_t)gate) & 15) == 0;
     cudaError_t e;
-    if (bf16) e = gate_bf16 ? norm_gate_launch<__nv_bfloat16, __nv_bfloat16>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, vec, st)
-                            : norm_gate_launch<__nv_bfloat16, float>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, vec, st);
-    else e = gate_bf16 ? norm_gate_launch<float, __nv_bfloat16>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, vec, st)
-                       : norm_gate_launch<float, float>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, vec, st);
+    if (bf16) e = gate_bf16 ? norm_gate_launch<__nv_bfloat16, __nv_bfloat16>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, first, w_row, vec, st)
+                            : norm_gate_launch<__nv_bfloat16, float>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, first, w_row, vec, st);
+    else e = gate_bf16 ? norm_gate_launch<float, __nv_bfloat16>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, first, w_row, vec, st)
+                       : norm_gate_launch<float, float>(o, w, gate, ld_gate, out, n, per_row, gs, eps, act, first, w_row, vec, st);
     PTB_CUDA_OK(e);
     PTB_CUDA_OK(cudaGetLastError());
     return 0;

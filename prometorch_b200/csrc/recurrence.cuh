@@ -1,7 +1,8 @@
 // Recurrent layers with a matrix state S [D, Dv] per head and sequence, fp32:
 //   decay attention   S <- decay_h S + k v^T;  o = S^T q
 //   gated delta rule  S <- g S (g per key channel, or one number);  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
-// with g = exp(-rate_h softplus(a + dt_bias)), beta a sigmoid, q and k unit vectors (q also times D^-1/2).
+// with g = exp(-rate_h softplus(a + dt_bias)), beta a sigmoid, q and k unit vectors (q also times D^-1/2);
+//   state-space step  S <- exp(-rate_h dt) S + dt k v^T;  o = S^T q + skip_h v,  dt = softplus(a + dt_bias) per head, q and k per group of heads.
 #pragma once
 #include "common.cuh"
 #include "ptb200_types.h"

@@ -6,7 +6,7 @@
 // where u is v for decay attention.  For the delta rule (1 + B) u = beta (v - (k G)^T S) with B_ij = beta_i k_i . (k_j G_i / G_j) for
 // j < i (a unit lower triangular system, the UT transform of delta-rule attention), hence u = U - W S with U = (1 + B)^-1 beta v and
 // W = (1 + B)^-1 beta (k G).  Two kernels:
-//   delta_chunk_kernel / delta_head_chunk_kernel / decay_chunk_kernel   everything that does not depend on S, all chunks at once, into a
+//   delta_chunk_kernel / delta_head_chunk_kernel / ssd_chunk_kernel / decay_chunk_kernel   everything that does not depend on S, all chunks at once, into a
 //                        workspace;
 //   chunk_state_kernel                        walks a sequence's chunks for a slice of value columns; S stays in registers.
 // What passes between them lies in the order of the mma fragments that will read it: a lane's 16 bytes are its four registers of a 16 x 16
@@ -15,6 +15,9 @@
 // border between the two tokens and are at most 1, inside a block the exponent of every pair is taken directly.
 // One decay per head: the quotients are numbers per pair of tokens, so they scale products of the bf16 q and k as they are, and the walk
 // takes q and k unscaled, with a factor per row for the product with q and for u on its way into the state.
+// State-space steps (MODE 3): q and k belong to a group of heads, so a chunk's fragments of q, k and the products q . k are made once per group
+// (ssd_chunk_kernel) and only the pairs' factors per head; u is v, exact in bf16, and the step joins A and the factor of u on its way into
+// the state.
 // Products run on the tensor cores with every fp32 operand split into two bf16 numbers (three products: 16 bits of both operands).
 #include "recurrence.cuh"
 #include "flash_attn.cuh"
@@ -41,9 +44,16 @@ struct Work {
     static __host__ __device__ size_t bytes(int Dvp) { return (size_t)U + (size_t)CH * Dvp * 4; }
 };
 
+// State-space steps: q and k of every (chunk, group) first, as in Work without low parts, then of every (chunk, head) A and G.
+template <int DT>
+struct SsdWork {
+    static constexpr int Q = 0, K = Work<DT>::TILE, GROUP = 2 * Work<DT>::TILE, A = 0, G = 2 * Work<DT>::ATILE, HEAD = G + 1024;
+};
+
 struct Params {
     PtbRecurrence P;
     unsigned char* work;
+    unsigned char* shared;             // MODE 3: the part that the heads of a group share
     size_t stride;                     // bytes per (chunk, head)
     int Dvp;                           // value columns rounded up to 32
     int vec, vec_a;                    // 16-byte loads of x rows, of a (or of low)
@@ -675,6 +685,122 @@ __global__ void __launch_bounds__(THREADS, 2) delta_head_chunk_kernel(const __gr
     }
 }
 
+// ---------------------------------------------------------------------------------------------- state-space steps, one chunk
+// One CTA per (chunk, group, share of the group's heads).
+constexpr int SSD_HEADS = THREADS / CH;                // heads whose decays are formed at once
+template <int DT>
+__global__ void __launch_bounds__(THREADS) ssd_chunk_kernel(const __grid_constant__ Params W, int heads) {
+    using L = Work<DT>;
+    using M = SsdWork<DT>;
+    constexpr int PB = DT + 8, UNITS = 10;
+    extern __shared__ __align__(128) unsigned char smem[];
+    __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
+    __nv_bfloat16* k_s = q_s + CH * PB;
+    __shared__ __align__(16) float4 qk_s[UNITS][2][32];            // products of the blocks up to the diagonal, a lane's accumulators
+    __shared__ float up_s[SSD_HEADS][CH], rest_s[SSD_HEADS][CH], dt_s[SSD_HEADS][CH], E_s[SSD_HEADS][4];
+    const PtbRecurrence& P = W.P;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int grp = blockIdx.y, R = P.H / P.G, D = P.D;
+    const int4 chunk = reinterpret_cast<const int4*>(P.chunks)[blockIdx.x];
+    const int row0 = chunk.x, cnt = chunk.y;
+    if (row0 < 0 || cnt < 1 || cnt > CH || row0 + cnt > P.n) {
+        if (threadIdx.x == 0 && P.status) atomicExch(P.status, PTB_ERR_BOUNDS);
+        return;
+    }
+    load_rows(P, W.vec, row0, cnt, P.q_col + grp * D, D, DT, q_s, PB);
+    load_rows(P, W.vec, row0, cnt, P.k_col + grp * D, D, DT, k_s, PB);
+    fa::cp_async_commit();
+    fa::cp_async_wait<0>();
+    __syncthreads();
+    if (blockIdx.z == 0) {
+        unsigned char* out = W.shared + ((size_t)blockIdx.x * P.G + grp) * M::GROUP;
+        for (int f = warp; f < DT / 4; f += WARPS) {
+            const int rb = f / (DT / 16), ks = f % (DT / 16), dp = f >> 2, kt = f & 3;
+            uint32_t x[4];
+            fa::ldsm4(smem_u32(q_s + (rb * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PB + ks * 16 + (lane >> 4) * 8), x[0], x[1], x[2], x[3]);
+            *reinterpret_cast<uint4*>(out + M::Q + ((size_t)f * 32 + lane) * 16) = make_uint4(x[0], x[1], x[2], x[3]);
+            fa::ldsm4_t(smem_u32(k_s + (kt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PB + dp * 16 + (lane >> 4) * 8), x[0], x[1], x[2], x[3]);
+            *reinterpret_cast<uint4*>(out + M::K + ((size_t)f * 32 + lane) * 16) = make_uint4(x[0], x[1], x[2], x[3]);
+        }
+    }
+    for (int unit = warp; unit < UNITS; unit += WARPS) {
+        const int s = unit < 1 ? 0 : unit < 3 ? 1 : unit < 6 ? 2 : 3, r = unit - s * (s + 1) / 2;
+        float c[2][4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) c[n][e] = 0.f;
+#pragma unroll
+        for (int ks = 0; ks < DT / 16; ++ks) {
+            uint32_t q[4], b[4];
+            fa::ldsm4(smem_u32(q_s + (s * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PB + ks * 16 + (lane >> 4) * 8), q[0], q[1], q[2], q[3]);
+            fa::ldsm4(smem_u32(k_s + (r * 16 + (lane & 7) + (lane >> 4) * 8) * PB + ks * 16 + ((lane >> 3) & 1) * 8), b[0], b[1], b[2], b[3]);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) fa::mma16816(c[n], q, b[2 * n], b[2 * n + 1]);
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n) qk_s[unit][n][lane] = make_float4(c[n][0], c[n][1], c[n][2], c[n][3]);
+    }
+    const int h0 = blockIdx.z * heads, h1 = min(R, h0 + heads);
+    for (int hb = h0; hb < h1; hb += SSD_HEADS) {
+        __syncthreads();                               // the products are there; the heads before are done with
+        const int mine = threadIdx.x / CH, i = threadIdx.x % CH, live = min(SSD_HEADS, h1 - hb);
+        if (mine < live) {
+            const int h = grp * R + hb + mine;
+            float dt = 0.f;
+            if (i < cnt) dt = softplus(__bfloat162float(((const __nv_bfloat16*)P.a)[(size_t)(row0 + i) * P.ld_a + h]) + P.dt_bias[h]);
+            const float d = fmaxf(-150.f, -P.decay[h] * LOG2E * dt);           // 2^-150 is 0
+            float a = d, b = d;
+#pragma unroll
+            for (int o = 1; o < 16; o <<= 1) {
+                const float x = __shfl_up_sync(0xffffffffu, a, o, 16), y = __shfl_down_sync(0xffffffffu, b, o, 16);
+                if ((i & 15) >= o) a += x;
+                if ((i & 15) + o < 16) b += y;
+            }
+            const float behind = __shfl_down_sync(0xffffffffu, b, 1, 16);
+            dt_s[mine][i] = dt;
+            up_s[mine][i] = a;
+            rest_s[mine][i] = (i & 15) == 15 ? 0.f : behind;
+            if ((i & 15) == 15) E_s[mine][i >> 4] = a;
+        }
+        __syncthreads();
+        if (mine < live) {
+            const int b = i >> 4;
+            float before = 0.f, after = 0.f;
+#pragma unroll
+            for (int r = 0; r < 4; ++r) { before += r < b ? E_s[mine][r] : 0.f; after += r > b ? E_s[mine][r] : 0.f; }
+            float* G = reinterpret_cast<float*>(W.work + ((size_t)blockIdx.x * P.H + grp * R + hb + mine) * W.stride + M::G);
+            G[4 + i] = exp2f(up_s[mine][i] + before);
+            G[4 + CH + i] = dt_s[mine][i] * exp2f(rest_s[mine][i] + after);
+            if (i == 0) G[0] = exp2f(E_s[mine][0] + E_s[mine][1] + E_s[mine][2] + E_s[mine][3]);
+        }
+        for (int u = warp; u < live * UNITS; u += WARPS) {
+            const int hl = u / UNITS, unit = u % UNITS, s = unit < 1 ? 0 : unit < 3 ? 1 : unit < 6 ? 2 : 3, r = unit - s * (s + 1) / 2;
+            float mid = 0.f;                           // whole blocks between the two
+            for (int m = r + 1; m < s; ++m) mid += E_s[hl][m];
+            float2 x[4];
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                const float4 c = qk_s[unit][n][lane];
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int i2 = s * 16 + g + 8 * e, j = r * 16 + n * 8 + 2 * t;
+                    float w[2];
+#pragma unroll
+                    for (int k = 0; k < 2; ++k) {
+                        const float d = s == r ? up_s[hl][i2] - up_s[hl][j + k] : up_s[hl][i2] + mid + rest_s[hl][j + k];
+                        w[k] = j + k <= i2 ? exp2f(d) * dt_s[hl][j + k] : 0.f;
+                    }
+                    x[n * 2 + e] = make_float2((e ? c.z : c.x) * w[0], (e ? c.w : c.y) * w[1]);
+                }
+            }
+            store_frag(W.work + ((size_t)blockIdx.x * P.H + grp * R + hb + hl) * W.stride + M::A, L::ATILE, s * 4 + r, lane, x);
+        }
+    }
+}
+
 // ---------------------------------------------------------------------------------------------- fixed decay, one chunk
 template <int DT>
 __global__ void __launch_bounds__(THREADS) decay_chunk_kernel(const __grid_constant__ Params W) {
@@ -803,20 +929,23 @@ __device__ __forceinline__ void mma_u4(float* d, const uint4& a, uint32_t b0, ui
 // the read-out; the state lives transposed, [value][key channel], in the accumulators of warps 0-3 and as two bf16 tiles in shared
 // memory for the products that read it.  The other operands arrive by bulk copies through three slots, in the order of their use: W and q
 // of a chunk, its k and A, W and q of the next, ...
-// With one decay per head (MODE 2) u enters the state times its row's factor, from a second pair of tiles.
-template <int DT, int VS, bool HEAD>
+// With one decay per head (MODE 2, 3) u enters the state times its row's factor, from a second pair of tiles.
+template <int DT, int VS, int MODE>
 struct StateSmem {
+    static constexpr bool HEAD = MODE >= 2;
     using L = Work<DT, HEAD>;
-    static constexpr int EVEN = (2 + L::PARTS) * L::TILE, ODD = L::PARTS * L::TILE + 2 * L::ATILE;
+    static constexpr int Q_AT = MODE == 3 ? 0 : 2 * L::TILE;       // of q in its slot
+    static constexpr int EVEN = Q_AT + L::PARTS * L::TILE, ODD = L::PARTS * L::TILE + 2 * L::ATILE;
     static constexpr int SLOT = EVEN > ODD ? EVEN : ODD, SH = 3 * SLOT, SL = SH + VS * DT * 2;
     static constexpr int UH = SL + VS * DT * 2, UL = UH + VS * CH * 2, FH = HEAD ? UL + VS * CH * 2 : UH, FL = HEAD ? FH + VS * CH * 2 : UL;
     static constexpr int BAR = FL + VS * CH * 2, TOTAL = BAR + 64;
 };
 template <int DT, int VS, int MODE>
 __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_constant__ Params W) {
-    constexpr bool DELTA = MODE != 0, HEAD = MODE == 2;
+    constexpr bool DELTA = MODE == 1 || MODE == 2, HEAD = MODE >= 2, SSD = MODE == 3;
     using L = Work<DT, HEAD>;
-    using S = StateSmem<DT, VS, HEAD>;
+    using S = StateSmem<DT, VS, MODE>;
+    using M = SsdWork<DT>;
     constexpr int KS = DT / 16, NT = DT / 32, MT = VS / 16, NB = VS / 8;       // state tiles of a warp: MT x NT of 16 x 8
     extern __shared__ __align__(128) unsigned char smem[];
     unsigned char *s_hi = smem + S::SH, *s_lo = smem + S::SL, *u_hi = smem + S::UH, *u_lo = smem + S::UL;
@@ -843,11 +972,18 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
     const uint32_t sh = smem_u32(s_hi), sl = smem_u32(s_lo), uh = smem_u32(u_hi), ul = smem_u32(u_lo);
     float* st = P.state + (((size_t)sp.slot * P.H + h) * D) * Dv;
     auto tiles = [&](int c) { return W.work + ((size_t)(first + c) * P.H + h) * W.stride; };
+    auto factors = [&](int c) { return reinterpret_cast<const float*>(tiles(c) + (SSD ? M::G : L::G)); };
     // load 2c: W and q of chunk c, load 2c + 1: its k and A; load i goes to slot i % 3 once load i - 3 has been read
     auto load = [&](int i) {
         const int s = i % 3;
         const unsigned char* src = tiles(i >> 1);
-        if (i & 1) {
+        if constexpr (SSD) {
+            const unsigned char* both = W.shared + ((size_t)(first + (i >> 1)) * P.G + h / (P.H / P.G)) * M::GROUP;
+            unsigned char* dst = smem + s * S::SLOT;
+            mbar_expect_tx(&bar[s], (i & 1) ? S::ODD : S::EVEN);
+            bulk_g2s(dst, both + ((i & 1) ? M::K : M::Q), L::TILE, &bar[s]);
+            if (i & 1) bulk_g2s(dst + L::TILE, src + M::A, 2 * L::ATILE, &bar[s]);
+        } else if (i & 1) {
             constexpr uint32_t bytes = S::ODD;
             mbar_expect_tx(&bar[s], bytes);
             bulk_g2s(smem + s * S::SLOT, src + L::K, bytes, &bar[s]);
@@ -882,7 +1018,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
     auto fetch_base = [&](int c) {                     // U in accumulator order, or v (two pairs of bf16)
         const int row0 = sp.row0 + c * CH, cnt = min(CH, sp.count - c * CH);
         if constexpr (HEAD) {
-            const float* G = reinterpret_cast<const float*>(tiles(c) + L::G) + 4 + CH + wr + g;
+            const float* G = factors(c) + 4 + CH + wr + g;
             fac[0] = G[0]; fac[1] = G[8];
         }
 #pragma unroll
@@ -909,6 +1045,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
         publish();
     }
     __syncthreads();
+    const float skip = SSD ? P.skip[h] : 0.f;
     bool ok = true;
     for (int c = 0; c < chunks; ++c) {
         const unsigned char *wq = smem + (2 * c % 3) * S::SLOT, *ka = smem + ((2 * c + 1) % 3) * S::SLOT;
@@ -920,7 +1057,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
             for (int e = 0; e < 4; ++e) acc[n][e] = low[n][e] = 0.f;
         float rq[2] = {1.f, 1.f};                      // HEAD: the factors of this thread's rows of q (warps 4-7)
         if constexpr (HEAD) {
-            const float* G = reinterpret_cast<const float*>(tiles(c) + L::G);
+            const float* G = factors(c);
             ge[0][0] = G[0];
             if (!owner) { rq[0] = G[4 + wr + g]; rq[1] = G[4 + wr + g + 8]; }
         } else if (owner) {
@@ -932,7 +1069,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
         }
         if (ok) ok = mbar_wait(&bar[2 * c % 3], (uint32_t)((2 * c / 3) & 1), P.status);
         if (DELTA || !owner) {                         // W S (warps 0-3) or (q G) S (warps 4-7): 16 rows each
-            const unsigned char* p = wq + (owner ? 0 : 2 * L::TILE);
+            const unsigned char* p = wq + (owner ? 0 : S::Q_AT);
 #pragma unroll
             for (int ks = 0; ks < KS; ++ks) {
                 const bool low_part = !HEAD || owner;          // q comes as it is
@@ -965,7 +1102,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                 } else {
                     const float2 a = unpack(base[n].x), b = unpack(base[n].y);
                     u[0] = a.x; u[1] = a.y; u[2] = b.x; u[3] = b.y;
-                    if (P.silu)
+                    if (MODE == 0 && P.silu)
 #pragma unroll
                         for (int e = 0; e < 4; ++e) u[e] = silu(u[e]);
                 }
@@ -975,7 +1112,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                     const __nv_bfloat16 hi = __float2bfloat16_rn(u[e]);
                     const uint32_t off = fa::tile_off<CH>(v, r >> 3) + (r & 7) * 2;
                     *reinterpret_cast<__nv_bfloat16*>(u_hi + off) = hi;
-                    *reinterpret_cast<__nv_bfloat16*>(u_lo + off) = __float2bfloat16_rn(u[e] - __bfloat162float(hi));
+                    if constexpr (!SSD) *reinterpret_cast<__nv_bfloat16*>(u_lo + off) = __float2bfloat16_rn(u[e] - __bfloat162float(hi));
                     if constexpr (HEAD) {
                         const float f = u[e] * fac[e >> 1];
                         const __nv_bfloat16 fh = __float2bfloat16_rn(f);
@@ -1022,13 +1159,14 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                     const uint4 kh = lds_frag(ka + L::PARTS * L::TILE, rb * 4 + ks, lane), kl = lds_frag(ka + L::PARTS * L::TILE + L::ATILE, rb * 4 + ks, lane);
                     uint32_t bh[MT][4], bl[MT][4];
 #pragma unroll
-                    for (int n = 0; n < MT; ++n) { fa::load_b<CH>(uh, n * 16, ks, bh[n]); fa::load_b<CH>(ul, n * 16, ks, bl[n]); }
+                    for (int n = 0; n < MT; ++n) { fa::load_b<CH>(uh, n * 16, ks, bh[n]); if constexpr (!SSD) fa::load_b<CH>(ul, n * 16, ks, bl[n]); }
 #pragma unroll
                     for (int n = 0; n < NB; ++n) mma_u4(acc[n], kh, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
 #pragma unroll
                     for (int n = 0; n < NB; ++n) mma_u4(low[n], kl, bh[n / 2][2 * (n & 1)], bh[n / 2][2 * (n & 1) + 1]);
+                    if constexpr (!SSD)
 #pragma unroll
-                    for (int n = 0; n < NB; ++n) mma_u4(low[n], kh, bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
+                        for (int n = 0; n < NB; ++n) mma_u4(low[n], kh, bl[n / 2][2 * (n & 1)], bl[n / 2][2 * (n & 1) + 1]);
                 }
 #pragma unroll
             for (int n = 0; n < NB; ++n)
@@ -1036,7 +1174,12 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
                 for (int e = 0; e < 2; ++e) {
                     const int r = wr + g + 8 * e, v = v0 + n * 8 + 2 * t;
                     float* o = P.out + (size_t)(row0 + r) * P.H * Dv + (size_t)h * Dv + v;
-                    const float x = acc[n][2 * e] + low[n][2 * e], y = acc[n][2 * e + 1] + low[n][2 * e + 1];
+                    float x = acc[n][2 * e] + low[n][2 * e], y = acc[n][2 * e + 1] + low[n][2 * e + 1];
+                    if constexpr (SSD) {                 // v is still in its tile
+                        auto own = [&](int c) { return __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(u_hi + fa::tile_off<CH>(c, r >> 3) + (r & 7) * 2)); };
+                        x = fmaf(skip, own(n * 8 + 2 * t), x);
+                        y = fmaf(skip, own(n * 8 + 2 * t + 1), y);
+                    }
                     if (r >= cnt) continue;
                     if (v + 1 < Dv && (Dv & 1) == 0) *reinterpret_cast<float2*>(o) = make_float2(x, y);
                     else {
@@ -1054,14 +1197,14 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_state_kernel(const __grid_co
 template <int DT, int VS, int MODE>
 static int launch_state(const Params& p, cudaStream_t st) {
     const dim3 grid((p.P.Dv + VS - 1) / VS, p.P.H, p.P.n_seqs);
-    constexpr int smem = StateSmem<DT, VS, MODE == 2>::TOTAL;
+    constexpr int smem = StateSmem<DT, VS, MODE>::TOTAL;
     PTB_CUDA_OK(cudaFuncSetAttribute(chunk_state_kernel<DT, VS, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     PTB_CUDA_OK(ptb_launch(chunk_state_kernel<DT, VS, MODE>, grid, dim3(THREADS), (size_t)smem, st, ptb_pdl_enabled(), p));
     return 0;
 }
 template <int DT, int VS>
 static int launch_state(const Params& p, cudaStream_t st) {
-    return p.P.delta == 2 ? launch_state<DT, VS, 2>(p, st) : p.P.delta ? launch_state<DT, VS, 1>(p, st) : launch_state<DT, VS, 0>(p, st);
+    return p.P.delta == 3 ? launch_state<DT, VS, 3>(p, st) : p.P.delta == 2 ? launch_state<DT, VS, 2>(p, st) : p.P.delta ? launch_state<DT, VS, 1>(p, st) : launch_state<DT, VS, 0>(p, st);
 }
 
 template <int DT>
@@ -1073,7 +1216,16 @@ static int launch(Params p, cudaStream_t st) {
         PTB_CUDA_OK(ptb_launch(kern, grid, dim3(THREADS), (size_t)smem, st, pdl, p));
         return 0;
     };
-    if (p.P.delta == 2 ? go(delta_head_chunk_kernel<DT>, HeadSmem<DT>::total(p.Dvp))
+    if (p.P.delta == 3) {
+        p.shared = p.work;
+        p.work += (size_t)p.P.n_chunks * p.P.G * SsdWork<DT>::GROUP;
+        const int R = p.P.H / p.P.G;                   // shares of whole batches of heads, about three CTAs per SM
+        const long long most = std::max<long long>(1, 444LL / std::max<long long>(1, (long long)p.P.n_chunks * p.P.G));
+        const int heads = (int)((R + most - 1) / most + SSD_HEADS - 1) / SSD_HEADS * SSD_HEADS, smem = 2 * CH * (DT + 8) * 2;
+        auto kern = ssd_chunk_kernel<DT>;
+        PTB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+        PTB_CUDA_OK(ptb_launch(kern, dim3(p.P.n_chunks, p.P.G, (R + heads - 1) / heads), dim3(THREADS), (size_t)smem, st, pdl, p, heads));
+    } else if (p.P.delta == 2 ? go(delta_head_chunk_kernel<DT>, HeadSmem<DT>::total(p.Dvp))
                        : p.P.delta ? go(delta_chunk_kernel<DT>, DeltaSmem<DT>::total(p.Dvp)) : go(decay_chunk_kernel<DT>, 4 * Work<DT>::TILE)) return -1;
     // few CTAs: narrow slices, so that more of them share the walk
     const long long wide = (long long)((p.P.Dv + 31) / 32) * p.P.H * p.P.n_seqs;
@@ -1088,6 +1240,7 @@ int recurrence_check(const PtbRecurrence& p);
 
 static size_t chunk_bytes(const PtbRecurrence& p) {
     const int Dvp = (p.Dv + 31) / 32 * 32;
+    if (p.delta == 3) return rc::SsdWork<64>::HEAD;                // and what a group's heads share
     if (p.delta == 2) return p.D <= 64 ? rc::Work<64, true>::bytes(Dvp) : rc::Work<128, true>::bytes(Dvp);
     return p.D <= 64 ? rc::Work<64>::bytes(Dvp) : rc::Work<128>::bytes(Dvp);
 }
@@ -1100,7 +1253,8 @@ using namespace ptb;
 PTB_API long long ptb_recurrence_chunked_bytes(const PtbRecurrence* args) {
     const PtbRecurrence& p = *args;
     if (!p.bf16 || p.D > 128 || p.Dv > 128 || p.n_chunks < 1) return -1;
-    return (long long)chunk_bytes(p) * p.n_chunks * p.H;
+    const long long shared = p.delta == 3 ? (long long)p.G * (p.D <= 64 ? rc::SsdWork<64>::GROUP : rc::SsdWork<128>::GROUP) : 0;
+    return ((long long)chunk_bytes(p) * p.H + shared) * p.n_chunks;
 }
 
 // ptb_recurrence for a prompt pass, in chunks of 64 rows; see PtbRecurrence.
@@ -1115,6 +1269,7 @@ PTB_API int ptb_recurrence_chunked(const PtbRecurrence* args, void* work, long l
     rc::Params p;
     p.P = *args;
     p.work = (unsigned char*)work;
+    p.shared = nullptr;
     p.stride = chunk_bytes(*args);
     p.Dvp = (args->Dv + 31) / 32 * 32;
     p.vec = args->D % 8 == 0 && args->Dv % 8 == 0 && args->ld % 8 == 0 && args->q_col % 8 == 0 && args->k_col % 8 == 0 && args->v_col % 8 == 0 &&

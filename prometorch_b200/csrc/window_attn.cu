@@ -131,8 +131,13 @@ struct WindowRows {
     float scale_log2;                  // scale times log2(e)
 };
 
-// The cache slots (page * 64 + place, or -1) of the keys of split `split` of row `i`; returns their number.
-__device__ __forceinline__ int row_keys(const WindowRows& P, int i, int split, int* krow) {
+// The cache slots (page * 64 + place, or -1) of the keys of split `split` of row `i`; returns their number and (dist) how the distance of the key
+// at place e of the list follows from e.
+struct Distance {
+    int pos, e0, kept, lo;
+    __device__ __forceinline__ int operator()(int e) const { return pos - (e0 + e < kept ? e0 + e : lo + e0 + e - kept); }
+};
+__device__ __forceinline__ int row_keys(const WindowRows& P, int i, int split, int* krow, Distance& dist) {
     const PtbWindowAttn& A = P.A;
     const int pos = A.pos[(size_t)i * A.pos_stride];
     const Seen s = seen_by(pos, A.window, A.keep, A.chunked);
@@ -142,6 +147,7 @@ __device__ __forceinline__ int row_keys(const WindowRows& P, int i, int split, i
         per = min(per, P.kcap);
     }
     const int e0 = split * per, nk = max(0, min(per, s.count - e0));
+    dist = Distance{pos, e0, s.kept, s.lo};
     const int* table = A.page_table + (size_t)A.req[(size_t)i * A.req_stride] * A.pt_stride;
     for (int e = threadIdx.x; e < P.kcap; e += blockDim.x) {
         int v = -1;
@@ -156,6 +162,11 @@ __device__ __forceinline__ int row_keys(const WindowRows& P, int i, int split, i
     return nk;
 }
 __device__ __forceinline__ size_t cache_row(int krow, int G, int g) { return ((size_t)(krow / WA_PAGE) * G + g) * WA_PAGE + krow % WA_PAGE; }
+
+// What a key's distance adds to a score of head h, in units of log2.
+__device__ __forceinline__ float rel_log2(const PtbWindowAttn& A, int h, int distance) {
+    return __ldg(A.rel + (size_t)h * A.rel_n + min(max(distance, 0), A.rel_n - 1)) * WA_LOG2E;
+}
 
 // Factor of a head's sum given its largest (log2) score and total: the sink joins the denominator, the gate multiplies.
 template <typename T>
@@ -216,7 +227,8 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_mma_kernel(const __gri
     const int c = hg.c;
     pdl_wait();
     pdl_launch_dependents();
-    const int nk = row_keys(P, i, split, krow);
+    Distance dist;
+    const int nk = row_keys(P, i, split, krow, dist);
     {
         const int ch = A.Dp / 8;
         const uint4* src = reinterpret_cast<const uint4*>((const __nv_bfloat16*)A.q + ((size_t)i * A.H + hg.h0) * A.maps * A.Dp);
@@ -268,8 +280,12 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_mma_kernel(const __gri
             }
         }
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-            w_s[(rb * 8 + 2 * t + (e & 1)) * L.ldw + kg * 16 + g + (e >> 1) * 8] = ((e >> 1) ? r1 : r0) >= 0 ? acc[e] * P.scale_log2 : -INFINITY;
+        for (int e = 0; e < 4; ++e) {
+            const int row = rb * 8 + 2 * t + (e & 1), j = kg * 16 + g + (e >> 1) * 8;
+            float s = acc[e] * P.scale_log2;
+            if (A.rel && row % R8 < hg.n) s += rel_log2(A, hg.h0 + row % R8, dist(j));
+            w_s[row * L.ldw + j] = ((e >> 1) ? r1 : r0) >= 0 ? s : -INFINITY;
+        }
     }
     __syncthreads();
     for (int h = warp; h < rows; h += WR_WARPS) {
@@ -355,7 +371,8 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_f32_kernel(const __gri
     const int c = hg.c, rows = hg.n * A.maps, kpitch = A.maps * A.Dp;
     pdl_wait();
     pdl_launch_dependents();
-    const int nk = row_keys(P, i, split, krow);
+    Distance dist;
+    const int nk = row_keys(P, i, split, krow, dist);
     for (int e = threadIdx.x; e < rows * A.Dp; e += WR_THREADS) {
         const int row = e / A.Dp, m = row / hg.n, r = row % hg.n;
         q_s[e] = ((const float*)A.q)[(((size_t)i * A.H + hg.h0 + r) * A.maps + m) * A.Dp + e % A.Dp];
@@ -373,6 +390,7 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_f32_kernel(const __gri
                 a.x = fmaf(x.x, y.x, a.x); a.y = fmaf(x.y, y.y, a.y); a.z = fmaf(x.z, y.z, a.z); a.w = fmaf(x.w, y.w, a.w);
             }
             s = ((a.x + a.y) + (a.z + a.w)) * P.scale_log2;
+            if (A.rel) s += rel_log2(A, hg.h0 + h % hg.n, dist(j));
         }
         w_s[h * L.ldw + j] = s;
     }
@@ -528,7 +546,7 @@ PTB_API long long ptb_window_rows_work_floats(int n, int heads, int Dvp, int nsp
 PTB_API int ptb_window_attn_rows(const PtbWindowAttn* args, cudaStream_t st) {
     const PtbWindowAttn& a = *args;
     if (a.n <= 0) return 0;
-    if (a.G <= 0 || a.H % a.G || a.Dp % 16 || a.Dvp % 16 || a.v_ld % 8 || a.window < 1 || a.keep < 0 || a.maps < 1 || a.maps > 2 || (a.maps > 1 && a.sink)) {
+    if (a.G <= 0 || a.H % a.G || a.Dp % 16 || a.Dvp % 16 || a.v_ld % 8 || a.window < 1 || a.keep < 0 || a.maps < 1 || a.maps > 2 || (a.maps > 1 && a.sink) || (a.rel && a.rel_n < 1)) {
         ptb_set_error("window attention: bad sizes (H %d, G %d, Dp %d, Dvp %d, window %d, keep %d, maps %d)", a.H, a.G, a.Dp, a.Dvp, a.window, a.keep, a.maps);
         return -1;
     }

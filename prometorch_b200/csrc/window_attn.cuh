@@ -1,6 +1,7 @@
 // Softmax attention over the paged cache.  The query at position p sees the keys from `low(p)` to p and the first `keep` tokens of its
 // sequence; low is p - window + 1 (a sliding window) or, chunked, the first position of p's chunk of `window` positions.  A sink adds
 // exp(sink_h) to a head's denominator; a gate scales the head's output by its sigmoid.
+// A distance bias adds rel[h][min(p - j, rel_n - 1)] to the scaled score of key j.
 // Two maps: q and k of a head are [map 1, map 2], each an attention of its own over the same values, and the output is
 // d / sqrt(mean(d^2) + mix_eps) * mix_gain with d = a1 - mix a2.
 #pragma once

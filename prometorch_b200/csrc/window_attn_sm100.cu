@@ -24,6 +24,7 @@ namespace wa100 {
 
 using namespace ptb::gemm;
 
+constexpr int MAX_REL = 8192;          // entries of a head's distance bias (one map, keys from pages)
 constexpr int BQ = 128, BKV = 128, NTHREADS = 320, SUB = BKV * 128;      // SUB: bytes of 128 rows of 64 columns
 
 struct Params {
@@ -37,8 +38,9 @@ template <int KT, int DV, int MAPS>
 struct Sm {
     static constexpr int NK = KT == 3 ? 5 : 4, V_BYTES = BKV * DV * 2, P_BYTES = BQ * BKV * 2;
     static constexpr int OFF_K = MAPS * KT * SUB, OFF_V = OFF_K + NK * SUB, OFF_P = OFF_V + 2 * V_BYTES, OFF_RED = OFF_P + P_BYTES;
-    static constexpr int OFF_BAR = OFF_RED + 2 * BQ * 4, TOTAL = OFF_BAR + 256 + 1024;
-    static_assert(TOTAL <= 227 * 1024, "shared memory of a CTA");
+    static constexpr int OFF_BAR = OFF_RED + 2 * BQ * 4, OFF_REL = OFF_BAR + 256, TOTAL = OFF_REL + 1024;        // and the head's distance bias
+    static constexpr int MOST = TOTAL + (MAPS == 1 && KT < 3 ? MAX_REL * 4 : 0);
+    static_assert(MOST <= 227 * 1024, "shared memory of a CTA");
 };
 
 __device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
@@ -101,6 +103,7 @@ window_tiles_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     uint64_t* o_full = bars + 18;        // [1]
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 19);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+    float* rel = reinterpret_cast<float*>(smem + S::OFF_REL);
 
     const PtbWindowAttn& A = P.A;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -121,6 +124,8 @@ window_tiles_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         tmem_alloc(tmem_slot, 512);
         tmem_relinquish();
     }
+    if (A.rel)                                           // a weight of the model: no kernel before this one writes it
+        for (int e = threadIdx.x; e < A.rel_n; e += NTHREADS) rel[e] = A.rel[(size_t)h * A.rel_n + e] * WA_LOG2E;
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
@@ -263,6 +268,17 @@ window_tiles_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
                 for (int i = 0; i < 32; ++i) sc[32 + i] = __uint_as_float(r[i]) * P.scale_log2;
             }
             const int key0 = pg.at(e) * WA_PAGE;
+            if (A.rel) {
+                const int far = A.rel_n - 1, d0 = q_pos - key0;
+                if (T.y - (key0 + 63) >= far) {          // all keys of the page lie beyond the table for every row of the tile
+                    const float b = rel[far];
+#pragma unroll
+                    for (int i = 0; i < 64; ++i) sc[i] += b;
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 64; ++i) sc[i] += rel[min(max(d0 - i, 0), far)];
+                }
+            }
             // some row of the tile does not see all 64 keys: one lies ahead of it, or below its lowest and not among the kept
             if (!there || key0 + 63 > T.y || (last_low > key0 && key0 + 63 >= A.keep)) {
                 const int ahead = there ? q_pos - key0 : -1, behind = q_low - 1 - key0, kept = A.keep - key0;
@@ -418,10 +434,10 @@ static int launch(const Params& p, cudaStream_t st) {
     using S = Sm<KT, DV, MAPS>;
     static bool attr = false;
     if (!attr) {
-        PTB_CUDA_OK(cudaFuncSetAttribute(window_tiles_kernel<KT, DV, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, S::TOTAL));
+        PTB_CUDA_OK(cudaFuncSetAttribute(window_tiles_kernel<KT, DV, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, S::MOST));
         attr = true;
     }
-    PTB_CUDA_OK(ptb_launch(window_tiles_kernel<KT, DV, MAPS>, dim3(a.H, a.n_tiles), dim3(NTHREADS), (size_t)S::TOTAL, st, ptb_pdl_enabled(), mq, mk, mr, mv, p));
+    PTB_CUDA_OK(ptb_launch(window_tiles_kernel<KT, DV, MAPS>, dim3(a.H, a.n_tiles), dim3(NTHREADS), (size_t)S::TOTAL + (a.rel ? (size_t)a.rel_n * 4 : 0), st, ptb_pdl_enabled(), mq, mk, mr, mv, p));
     PTB_CUDA_OK(cudaGetLastError());
     return 0;
 }
@@ -442,7 +458,7 @@ PTB_API int ptb_window_attn_tiles(const PtbWindowAttn* args, cudaStream_t st) {
     const bool flat = a.flat_rows > 0;
     if (a.G <= 0 || a.H % a.G || a.Dp % 16 || a.Dvp % 16 || a.Dp > 128 || a.Dvp > 128 || a.Dv > a.Dvp || a.window < 1 || a.keep < 0 || a.n_tiles > 65535 ||
         a.maps < 1 || a.maps > 2 || (a.maps == 2 && (a.sink || flat)) || (flat && (a.G != a.H || a.rot_dim > 64 || a.k_ld % 8 || a.v_row % 8 || a.rot_ld % 8)) ||
-        (!flat && a.v_ld != a.Dvp)) {
+        (!flat && a.v_ld != a.Dvp) || (a.rel && (flat || a.maps > 1 || a.rel_n < 1 || a.rel_n > wa100::MAX_REL))) {
         ptb_set_error("window attention (tcgen05): bad sizes (H %d, G %d, Dp %d, Dvp %d, window %d, keep %d, maps %d, %d tiles)", a.H, a.G, a.Dp, a.Dvp, a.window, a.keep,
                       a.maps, a.n_tiles);
         return -1;

@@ -77,7 +77,7 @@ class PagedModel:
 
     def state_shapes(self) -> List[Dict[str, Tuple[tuple, torch.dtype]]]:
         """What each layer keeps per sequence besides pages: name -> (shape, dtype).  The engine holds one slot of it per page-table
-        row; a pass whose first token stands at position 0 takes the slot's content as zero."""
+        row; a pass whose first token stands at position 0 takes the slot's content as zero.  Entries past the layers' are the model's own."""
         return [{} for _ in self.kv_shapes()]
 
     def kept_tokens(self) -> int:
@@ -120,7 +120,7 @@ def register_model(config: type, weights: type, model: type, *names: str) -> Non
 
 
 def _ensure_builtin():
-    from . import budorax, gelutar, kifusun, llama_paged  # noqa: F401  (they register themselves)
+    from . import budorax, gelutar, kifusun, llama_paged, tifepel  # noqa: F401  (they register themselves)
 
 
 def known_models() -> List[str]:

@@ -1,31 +1,33 @@
-"""A mixture of experts for inference (csrc/experts.cu, csrc/experts_sm100.cu): a sigmoid router with a correction that has a say in the
-choice only, and gated experts ``down (silu(gate h) * (up h))``, each token using ``top`` of them.
+"""A mixture of experts for inference (csrc/experts.cu, csrc/experts_sm100.cu): a router (sigmoid, or softmax over all its outputs) with a
+correction that has a say in the choice only, and gated experts ``down (silu(gate h) * (up h))``, each token using ``top`` of them.  Router
+outputs behind the experts are identities: they return the token's row itself.
 
 :func:`run` sorts the (token, expert) pairs by expert on the device, runs every expert over its rows (one grouped product for gate
 and up, one for down) and returns :class:`ExpertRows`: the rows where they lie, their places and weights.  What sums them up is the kernel
-that adds them to the stream (``ops/tanh_norm.py``).  Nothing depends on the counts on the host, so a decode pass can be a CUDA graph.
+that adds them to the stream (``ops/tanh_norm.py``, ``ops/streams.py``).  Nothing depends on the counts on the host, so a decode pass can be a CUDA graph.
 CUDA tensors run the kernels, CPU tensors the plain math."""
 from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass
-from typing import List
+from typing import List, Optional
 
 import torch
 
 from .. import _native as N
 from .paged import _status
-from .residual import _st, linear_f32
+from .gemm import linear_swiglu
+from .residual import Branch, _st, linear_branch, linear_f32
 
 
 @N.register_decls
 def _decls(L):
     vp, ci, cf, ll = C.c_void_p, C.c_int, C.c_float, C.c_longlong
-    L.ptb_expert_route.argtypes = [vp, ci, ll, ll, vp, ci, ci, ci, cf, vp, vp, vp, vp, vp, vp, vp]
+    L.ptb_expert_route.argtypes = [vp, ci, ll, ll, vp, ci, ci, ci, ci, ci, cf, vp, vp, vp, vp, vp, vp, vp]
     L.ptb_expert_gemm_simt.argtypes = [vp, vp, ll, vp, ci, vp, vp, ci, ci, ci, ci, ci, vp, vp]
-    L.ptb_expert_gather.argtypes = [vp, ll, vp, vp, ci, ci, ci, vp, vp]
+    L.ptb_expert_gather.argtypes = [vp, ll, vp, vp, vp, ci, ci, ci, vp, vp]
     L.ptb_expert_gemm.argtypes = [vp, ll, vp, ci, vp, vp, ci, ci, ci, ci, ci, ci, vp, vp]
-    L.ptb_expert_route_rows.argtypes = [vp, ll, vp, ci, vp, ci, ci, ci, cf, vp, vp, vp, vp, vp, vp, ci, vp]
+    L.ptb_expert_route_rows.argtypes = [vp, ll, vp, ci, vp, ci, ci, ci, ci, ci, cf, vp, vp, vp, vp, vp, vp, ci, vp]
     for n in ("ptb_expert_route", "ptb_expert_route_rows", "ptb_expert_gemm_simt", "ptb_expert_gather", "ptb_expert_gemm"):
         getattr(L, n).restype = ci
 
@@ -35,10 +37,11 @@ class Experts:
     """One layer's experts in the layout the kernels read; ``ff`` is rounded up to a multiple of eight with zeros."""
     gate_up: torch.Tensor              # [E, 2 ff, W]: gate rows, then up rows
     down: torch.Tensor                 # [E, W, ff]
-    router: torch.Tensor               # [E rounded up to eight, W]
-    correction: torch.Tensor           # [E] fp32
+    router: torch.Tensor               # [outputs rounded up to eight, W]
+    correction: torch.Tensor           # [outputs] fp32: the experts, then the identities
     top: int
-    scale: float
+    scale: float                       # sigmoid scores: weights are scores over the sum of the chosen ones, times scale; softmax: the scores times scale
+    softmax: bool = False
 
     def __post_init__(self):
         self.done = torch.zeros(ROUTE_ROWS + 1, dtype=torch.int32, device=self.router.device)      # counters of the row router, zero between launches
@@ -47,23 +50,33 @@ class Experts:
     def count(self) -> int:
         return self.gate_up.shape[0]
 
+    @property
+    def outputs(self) -> int:
+        return self.correction.shape[0]
+
     @classmethod
     def of(cls, gate: List[torch.Tensor], up: List[torch.Tensor], down: List[torch.Tensor], router: torch.Tensor, correction: torch.Tensor, top: int,
-           scale: float) -> "Experts":
+           scale: float, softmax: bool = False) -> "Experts":
         pad = lambda t, d: torch.nn.functional.pad(t, (0, 0, 0, -t.shape[0] % 8) if d == 0 else (0, -t.shape[1] % 8))
         return cls(torch.stack([torch.cat([pad(g, 0), pad(u, 0)]) for g, u in zip(gate, up)]), torch.stack([pad(t, 1) for t in down]), pad(router, 0).contiguous(),
-                   correction.float(), top, scale)
+                   correction.float().contiguous(), top, scale, softmax)
 
 
 @dataclass
 class ExpertRows:
-    """Outputs of the chosen experts: row ``index[t, i]`` of ``y`` belongs to token t with the weight ``weight[t, i]``."""
+    """Outputs of the chosen experts: row ``index[t, i]`` of ``y`` belongs to token t with the weight ``weight[t, i]``; where the index is -1 it is the
+    token's own row of ``h``."""
     y: torch.Tensor                    # [n top, W], sorted by expert
     index: torch.Tensor                # [n, top] int32
     weight: torch.Tensor               # [n, top] fp32
+    h: Optional[torch.Tensor] = None   # [n, W] what the experts read
 
     def combine(self) -> torch.Tensor:
-        return (self.y.float()[self.index.long()] * self.weight[..., None]).sum(1)
+        i = self.index.long()
+        if self.h is None:
+            return (self.y.float()[i] * self.weight[..., None]).sum(1)
+        rows = torch.where((i < 0)[..., None], self.h.float()[:, None, :], self.y.float()[i.clamp_min(0)])
+        return (rows * self.weight[..., None]).sum(1)
 
 
 @dataclass
@@ -78,34 +91,36 @@ ROUTE_ROWS = 64                        # tokens up to which the kernel that choo
 
 
 def route(h: torch.Tensor, e: Experts) -> Routing:
-    n, E, k, W = h.shape[0], e.count, e.top, h.shape[1]
+    n, E, O, k, W = h.shape[0], e.count, e.outputs, e.top, h.shape[1]
     if h.is_cuda:
         i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=h.device)
         r = Routing(i32(n, k), torch.empty(n, k, dtype=torch.float32, device=h.device), i32(n * k), i32(E + 1))
-        few = n <= ROUTE_ROWS and E * W <= 1 << 21
-        work = i32(2 * n * k + (n * E if few else E))
+        few = n <= ROUTE_ROWS and O * W <= 1 << 21
+        work = i32(2 * n * k + (n * O if few else E))
         out = (r.index.data_ptr(), r.weight.data_ptr(), r.token.data_ptr(), r.offsets.data_ptr(), work.data_ptr())
         if few:
             assert h.dtype == e.router.dtype and h.stride(1) == 1
-            N.check(N.lib().ptb_expert_route_rows(h.data_ptr(), h.stride(0), e.router.data_ptr(), W, e.correction.data_ptr(), n, E, k, float(e.scale), *out,
+            N.check(N.lib().ptb_expert_route_rows(h.data_ptr(), h.stride(0), e.router.data_ptr(), W, e.correction.data_ptr(), n, E, O, int(e.softmax), k, float(e.scale), *out,
                                                   e.done.data_ptr(), int(h.dtype == torch.bfloat16), _st(h)), "expert_route_rows")
             return r
         z = linear_f32(h, e.router)
-        N.check(N.lib().ptb_expert_route(z.data_ptr(), 1, 0, z.stride(0), e.correction.data_ptr(), n, E, k, float(e.scale), *out, _status(h.device).data_ptr(), _st(h)),
+        N.check(N.lib().ptb_expert_route(z.data_ptr(), 1, 0, z.stride(0), e.correction.data_ptr(), n, E, O, int(e.softmax), k, float(e.scale), *out, _status(h.device).data_ptr(), _st(h)),
                 "expert_route")
         return r
     z = linear_f32(h, e.router)
-    s = torch.sigmoid(z[:, :E])
+    s = torch.softmax(z[:, :O], -1) if e.softmax else torch.sigmoid(z[:, :O])
     chosen = torch.topk(s + e.correction, k, -1).indices
     w = s.gather(1, chosen)
-    w = w / (w.sum(-1, keepdim=True) + 1e-20) * e.scale
+    w = w * e.scale if e.softmax else w / (w.sum(-1, keepdim=True) + 1e-20) * e.scale
     order = torch.sort(chosen.flatten(), stable=True).indices
     index = torch.empty_like(order)
     index[order] = torch.arange(n * k)
-    offsets = torch.cat([torch.zeros(1, dtype=torch.long), torch.bincount(chosen.flatten(), minlength=E).cumsum(0)])
+    index[chosen.flatten() >= E] = -1
+    offsets = torch.cat([torch.zeros(1, dtype=torch.long), torch.bincount(chosen.flatten(), minlength=O)[:E].cumsum(0)])
     return Routing(index.view(n, k).int(), w, (order // k).int(), offsets.int())
 
 
+GATED_FROM = 128                       # rows above which the shared expert runs as a grouped product of one expert
 FEW_ROWS = 48                          # mean rows of an expert below which its weights are the 128-row operand
 
 
@@ -121,7 +136,7 @@ def products(h: torch.Tensor, e: Experts, r: Routing, simt: bool = False) -> tor
         if bf16 and W % 8 == 0 and h.stride(0) % 8 == 0 and not simt:
             x = torch.empty(rows, W, dtype=h.dtype, device=h.device)
             few = int(rows < FEW_ROWS * E)
-            N.check(N.lib().ptb_expert_gather(h.data_ptr(), h.stride(0), r.token.data_ptr(), x.data_ptr(), rows, W, n, status, st), "expert_gather")
+            N.check(N.lib().ptb_expert_gather(h.data_ptr(), h.stride(0), r.token.data_ptr(), r.offsets[E:].data_ptr(), x.data_ptr(), rows, W, n, status, st), "expert_gather")
             N.check(N.lib().ptb_expert_gemm(x.data_ptr(), W, e.gate_up.data_ptr(), 1, act.data_ptr(), r.offsets.data_ptr(), rows, E, F, W, few, 0, status, st), "expert_gemm")
             N.check(N.lib().ptb_expert_gemm(act.data_ptr(), F, e.down.data_ptr(), 0, y.data_ptr(), r.offsets.data_ptr(), rows, E, W, F, few, 0, status, st), "expert_gemm")
             return y
@@ -143,4 +158,30 @@ def products(h: torch.Tensor, e: Experts, r: Routing, simt: bool = False) -> tor
 def run(h: torch.Tensor, e: Experts) -> ExpertRows:
     """``h [n, W]`` through its tokens' experts."""
     r = route(h, e)
-    return ExpertRows(products(h, e, r), r.index, r.weight)
+    return ExpertRows(products(h, e, r), r.index, r.weight, h)
+
+
+@dataclass
+class SharedExpert:
+    """A gated expert that every token uses; ``ff`` is rounded up to a multiple of eight with zeros."""
+    gate_up: torch.Tensor              # [2 ff, W]: gate rows, then up rows
+    down: torch.Tensor                 # [W rounded up to eight, ff]
+
+    @classmethod
+    def of(cls, gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor) -> "SharedExpert":
+        pad = lambda t: torch.nn.functional.pad(t, (0, 0, 0, -t.shape[0] % 8))
+        return cls(torch.cat([pad(gate), pad(up)]), pad(torch.nn.functional.pad(down, (0, -down.shape[1] % 8))))
+
+
+def run_shared(h: torch.Tensor, e: SharedExpert) -> Branch:
+    """``h [n, W]`` through the shared expert, as a branch for the kernel that adds it to the stream."""
+    n, W = h.shape
+    F = e.down.shape[1]
+    if h.is_cuda and h.dtype == torch.bfloat16 and n > GATED_FROM and W % 8 == 0 and h.stride(0) % 8 == 0:
+        act = torch.empty(n, F, dtype=h.dtype, device=h.device)
+        offsets = torch.tensor([0, n], dtype=torch.int32).to(h.device)
+        N.check(N.lib().ptb_expert_gemm(h.data_ptr(), h.stride(0), e.gate_up.data_ptr(), 1, act.data_ptr(), offsets.data_ptr(), n, 1, F, W, 0, 0,
+                                        _status(h.device).data_ptr(), _st(h)), "expert_gemm")
+    else:
+        act = linear_swiglu(h, e.gate_up)
+    return linear_branch(act, e.down)

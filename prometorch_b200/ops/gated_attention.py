@@ -21,7 +21,7 @@ KEYS_PER_CTA = 128                     # GA_KEYS of csrc/gated_attn.cuh
 @N.register_decls
 def _decls(L):
     vp, ci, cf, ll = C.c_void_p, C.c_int, C.c_float, C.c_longlong
-    L.ptb_head_norm_write.argtypes = [vp, ll, vp, vp, vp, vp, vp, vp, ll, cf, vp, ci, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, ci, cf, vp, ci, vp]
+    L.ptb_head_norm_write.argtypes = [vp, ll, ci, ci, vp, vp, vp, vp, vp, vp, ci, vp, ll, cf, vp, ci, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, ci, cf, vp, ci, vp]
     L.ptb_head_norm_write.restype = ci
     L.ptb_gated_rows_work_floats.argtypes = [ci, ci, ci, ci]
     L.ptb_gated_rows_work_floats.restype = ll
@@ -100,34 +100,38 @@ class GatedAttention:
         return stored(self.vdim)
 
 
-def head_norm_write(qkv: torch.Tensor, a: GatedAttention, q_weight: torch.Tensor, k_weight: torch.Tensor, eps: float, pos: torch.Tensor,
-                    req: torch.Tensor, page_table: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
-                    v_first: Optional[torch.Tensor] = None, lam: float = 0.0) -> torch.Tensor:
-    """``qkv [n, H dim + G dim + G vdim]`` -> q ``[n, H, stored dim]`` after the heads' norm; keys (normalised) and values
+def head_norm_write(qkv: torch.Tensor, a, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float, pos: torch.Tensor, req: torch.Tensor,
+                    page_table: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, v_first: Optional[torch.Tensor] = None, lam: float = 0.0,
+                    cols: Optional[Tuple[int, int]] = None, gain: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``a``: anything with the sizes of a :class:`GatedAttention`.  ``qkv [n, *]``: q heads, then k and v heads (at the columns ``cols``, by default one
+    after the other) -> q ``[n, H, stored dim]`` after the heads' norm (a weight may be None), times ``gain[pos]`` (fp32 ``[positions]``); keys (normalised) and values
     ``(1 - lam) v + lam v_first`` go to the page slot of ``(req[i], pos[i])``.  ``pos`` / ``req``: int32 vectors of any stride."""
     n, H, G, D, Dv, Dp, Dvp = qkv.shape[0], a.heads, a.kv_heads, a.dim, a.vdim, a.dim_stored, a.vdim_stored
+    kc, vc = cols or (H * D, (H + G) * D)
     q = torch.empty(n, H, Dp, dtype=qkv.dtype, device=qkv.device)
     if qkv.is_cuda:
         if qkv.dtype not in (torch.bfloat16, torch.float32):
             raise TypeError(f"head_norm_write takes bf16 or fp32, got {qkv.dtype}")
         assert qkv.stride(1) == 1 and (v_first is None or v_first.stride(1) == 1) and pos.dtype == req.dtype == page_table.dtype == torch.int32
         st = torch.cuda.current_stream(qkv.device).cuda_stream
-        N.check(N.lib().ptb_head_norm_write(qkv.data_ptr(), qkv.stride(0), q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), q_weight.data_ptr(),
-                                            k_weight.data_ptr(), N.ptr(v_first), v_first.stride(0) if v_first is not None else 0, float(lam),
+        N.check(N.lib().ptb_head_norm_write(qkv.data_ptr(), qkv.stride(0), kc, vc, q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), N.ptr(q_weight),
+                                            N.ptr(k_weight), N.ptr(gain), gain.shape[0] if gain is not None else 0, N.ptr(v_first), v_first.stride(0) if v_first is not None else 0, float(lam),
                                             pos.data_ptr(), pos.stride(0), req.data_ptr(), req.stride(0), page_table.data_ptr(),
                                             page_table.stride(0), k_pages.shape[0], n, H, G, D, Dp, Dv, Dvp, float(eps),
                                             _status(qkv.device).data_ptr(), int(qkv.dtype == torch.bfloat16), st), "head_norm_write")
         return q
     x = qkv.float()
-    qs, ks, v = x[:, :H * D].reshape(n, H, D), x[:, H * D:(H + G) * D].reshape(n, G, D), x[:, (H + G) * D:(H + G) * D + G * Dv].reshape(n, G, Dv)
+    qs, ks, v = x[:, :H * D].reshape(n, H, D), x[:, kc:kc + G * D].reshape(n, G, D), x[:, vc:vc + G * Dv].reshape(n, G, Dv)
 
     def norm(t, w):
-        return t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * w
+        t = t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps)
+        return t if w is None else t * w
     if v_first is not None:
         v = (1 - lam) * v + lam * v_first.float().reshape(n, G, Dv)
     q.zero_()
-    q[..., :D] = norm(qs, q_weight).to(q.dtype)
     p = pos.long()
+    qn = norm(qs, q_weight)
+    q[..., :D] = (qn if gain is None else qn * gain[p][:, None, None]).to(q.dtype)
     pages = page_table[req.long(), p // PAGE].long()
     k_pages[pages, :, p % PAGE] = torch.nn.functional.pad(norm(ks, k_weight), (0, Dp - D)).to(k_pages.dtype)
     v_pages[pages, :, p % PAGE] = torch.nn.functional.pad(v, (0, Dvp - Dv)).to(v_pages.dtype)

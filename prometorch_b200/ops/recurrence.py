@@ -1,5 +1,6 @@
 """Recurrent layers with a matrix state per head (csrc/recurrence.cu, csrc/recurrence_chunk.cu): linear attention with a fixed decay,
-the gated delta rule with a decay per key channel or per head, and the short causal convolution and the gated norm that go with them.
+the gated delta rule with a decay per key channel or per head, state-space steps, and the short causal convolution and the gated norm that go
+with them.
 
 A sequence's state is one slot of ``[slots, H, dim, vdim]`` fp32 (and ``[slots, taps - 1, channels]`` of convolution inputs); a token
 at position 0 starts from zero whatever the slot holds.  A decode pass gives one token per row (``seqs`` None: slot ``req[i]``,
@@ -26,17 +27,17 @@ class RecurrenceArgs(C.Structure):
                 ("seqs", C.c_void_p), ("n_seqs", C.c_int), ("pos_stride", C.c_int), ("req_stride", C.c_int), ("pad", C.c_int),
                 ("pos", C.c_void_p), ("req", C.c_void_p), ("out", C.c_void_p), ("status", C.c_void_p),
                 ("chunks", C.c_void_p), ("first_chunk", C.c_void_p), ("n_chunks", C.c_int), ("rank", C.c_int),
-                ("low", C.c_void_p), ("ld_low", C.c_longlong), ("low_w", C.c_void_p)]
+                ("low", C.c_void_p), ("ld_low", C.c_longlong), ("low_w", C.c_void_p), ("skip", C.c_void_p)]
 
 
 @N.register_decls
 def _decls(L):
     vp, ci, cf, ll = C.c_void_p, C.c_int, C.c_float, C.c_longlong
-    L.ptb_short_conv.argtypes = [vp, ll, vp, ci, ci, vp, vp, ci, ci, vp, ci, vp, ci, vp, ci, vp, ci, vp]
+    L.ptb_short_conv.argtypes = [vp, ll, vp, vp, ci, ci, ci, vp, vp, ci, ci, vp, ci, vp, ci, vp, ci, vp, ci, vp]
     L.ptb_short_conv.restype = ci
     L.ptb_recurrence.argtypes = [C.POINTER(RecurrenceArgs), vp]
     L.ptb_recurrence.restype = ci
-    L.ptb_group_norm_gate.argtypes = [vp, vp, vp, ci, ll, vp, ci, ci, ci, cf, ci, ci, vp]
+    L.ptb_group_norm_gate.argtypes = [vp, vp, vp, ci, ll, vp, ci, ci, ci, cf, ci, ci, ci, ci, vp]
     L.ptb_group_norm_gate.restype = ci
     L.ptb_recurrence_chunked.argtypes = [C.POINTER(RecurrenceArgs), vp, ll, vp]
     L.ptb_recurrence_chunked.restype = ci
@@ -85,17 +86,17 @@ def _check(t: torch.Tensor):
 
 # ------------------------------------------------------------------------------------------ short convolution
 def short_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, pos: torch.Tensor, req: torch.Tensor,
-               seqs: Optional[Sequences] = None) -> torch.Tensor:
+               seqs: Optional[Sequences] = None, bias: Optional[torch.Tensor] = None, add: bool = False) -> torch.Tensor:
     """``x [n, C]`` (any row pitch), ``weight [taps, C]`` fp32 with the current token's tap last: per channel the weighted sum of a
-    token and the taps - 1 before it, then SiLU; ``state [slots, taps - 1, C]`` in the type of x brings the inputs from before the
-    batch and takes the last ones along.  Returns ``[n, C]``."""
+    token and the taps - 1 before it, plus ``bias [C]`` fp32, then SiLU; with ``add`` the input plus that sum
+    instead; ``state [slots, taps - 1, C]`` in the type of x brings the inputs from before the batch and takes the last ones along.  Returns ``[n, C]``."""
     n, Ch = x.shape
     taps = weight.shape[0]
     out = torch.empty(n, Ch, dtype=x.dtype, device=x.device)
     if x.is_cuda:
         _check(x)
         assert state.dtype == x.dtype and state.is_contiguous() and weight.is_contiguous()
-        N.check(N.lib().ptb_short_conv(x.data_ptr(), x.stride(0), weight.data_ptr(), Ch, taps, state.data_ptr(), out.data_ptr(), n, state.shape[0],
+        N.check(N.lib().ptb_short_conv(x.data_ptr(), x.stride(0), weight.data_ptr(), N.ptr(bias), int(add), Ch, taps, state.data_ptr(), out.data_ptr(), n, state.shape[0],
                                        pos.data_ptr(), pos.stride(0), req.data_ptr(), req.stride(0), seqs.device.data_ptr() if seqs else 0,
                                        len(seqs.host) if seqs else 0, _status(x.device).data_ptr(), int(x.dtype == torch.bfloat16), _st(x)), "short_conv")
         return out
@@ -104,7 +105,8 @@ def short_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, pos: 
         before[:max(0, taps - 1 - at)] = 0                      # rows from before position 0
         full = torch.cat([before, x[lo:lo + count].float()])
         y = sum(full[i:i + count] * weight[i].float() for i in range(taps))
-        out[lo:lo + count] = torch.nn.functional.silu(y).to(out.dtype)
+        y = y if bias is None else y + bias
+        out[lo:lo + count] = (x[lo:lo + count].float() + y if add else torch.nn.functional.silu(y)).to(out.dtype)
         state[slot] = full[full.shape[0] - (taps - 1):].to(state.dtype)
     return out
 
@@ -132,6 +134,19 @@ class DecayAttention:
     vdim: int
     decay: torch.Tensor                # [H] fp32
     silu: bool = True
+
+
+@dataclass
+class StateSpace:
+    """The recurrence of a state-space layer: per head ``S <- exp(-rate dt) S + dt k v^T; o = S^T q + skip v`` with the step
+    ``dt = softplus(a + dt_bias)``; q and k are shared by the heads of a group."""
+    heads: int
+    groups: int
+    dim: int                           # rows of the state: size of q and k
+    vdim: int
+    rate: torch.Tensor                 # [H] fp32: exp(A_log)
+    dt_bias: torch.Tensor              # [H] fp32
+    skip: torch.Tensor                 # [H] fp32
 
 
 def _unit(x):
@@ -233,18 +248,49 @@ def decay_attention(x: torch.Tensor, r: DecayAttention, cols: Tuple[int, int, in
     return out
 
 
+def state_space(x: torch.Tensor, r: StateSpace, cols: Tuple[int, int, int], a: torch.Tensor, state: torch.Tensor, pos: torch.Tensor, req: torch.Tensor,
+                seqs: Optional[Sequences] = None, chunked: Optional[bool] = None) -> torch.Tensor:
+    """``x [n, *]``: q and k (group by group) and v (head by head) at the columns ``cols``; ``a [n, H]`` in the type of x.  Advances ``state
+    [slots, H, dim, vdim]``; returns o ``[n, H vdim]`` fp32."""
+    n, H, G, D, Dv = x.shape[0], r.heads, r.groups, r.dim, r.vdim
+    out = torch.empty(n, H * Dv, dtype=torch.float32, device=x.device)
+    if x.is_cuda:
+        _check(x)
+        assert a.dtype == x.dtype and a.shape[1] == H and a.stride(1) == 1 and state.is_contiguous()
+        args = RecurrenceArgs(q_col=cols[0], k_col=cols[1], v_col=cols[2], delta=3, a=a.data_ptr(), ld_a=a.stride(0), decay=r.rate.data_ptr(),
+                              dt_bias=r.dt_bias.data_ptr(), skip=r.skip.data_ptr(), H=H, G=G, D=D, Dv=Dv)
+        _run(args, x, seqs, pos, req, state, out, _runs_chunked(x, D, Dv, seqs, chunked))
+        return out
+    q, k, v = (x[:, c:c + h * d].float().reshape(n, h, d) for c, h, d in zip(cols, (G, G, H), (D, D, Dv)))
+    q, k = q.repeat_interleave(H // G, 1), k.repeat_interleave(H // G, 1)
+    dt = torch.nn.functional.softplus(a.float() + r.dt_bias, threshold=50.0)
+    g, o = torch.exp(-r.rate * dt), out.view(n, H, Dv)
+    for lo, count, at, slot in (seqs or Sequences.of_rows(pos, req)).host:
+        S = state[slot].clone() if at > 0 else torch.zeros_like(state[slot])
+        for i in range(lo, lo + count):
+            S = S * g[i][:, None, None] + k[i][:, :, None] * (dt[i][:, None] * v[i])[:, None, :]
+            o[i] = torch.einsum("hdv,hd->hv", S, q[i]) + r.skip[:, None] * v[i]
+        state[slot] = S
+    return out
+
+
 # ------------------------------------------------------------------------------------------ output norm and gate
-def group_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, dtype, act: str = "sigmoid") -> torch.Tensor:
+def group_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, dtype, act: str = "sigmoid",
+                    groups: Optional[int] = None, gate_first: bool = False) -> torch.Tensor:
     """``o [n, K]`` fp32 in groups of ``len(weight)`` columns: RMS norm of every group times the fp32 ``weight``, times the sigmoid (or
-    ``act="silu"``) of ``gate [n, K]`` (any row pitch; bf16 or fp32).  Returns ``[n, K]`` in ``dtype``."""
+    ``act="silu"``) of ``gate [n, K]`` (any row pitch; bf16 or fp32).  With ``groups`` the weight is ``[K]`` and that many equal groups are normed;
+    ``gate_first``: the gate multiplies ``o`` ahead of the norm.  Returns ``[n, K]`` in ``dtype``."""
     n, K = o.shape
-    gs = weight.shape[0]
+    gs = K // groups if groups else weight.shape[0]
+    assert K % gs == 0 and weight.shape[0] == (K if groups else gs)
     if o.is_cuda:
         out = torch.empty(n, K, dtype=dtype, device=o.device)
         assert o.is_contiguous() and gate.stride(1) == 1
         N.check(N.lib().ptb_group_norm_gate(o.data_ptr(), weight.data_ptr(), gate.data_ptr(), int(gate.dtype == torch.bfloat16), gate.stride(0),
-                                            out.data_ptr(), n, K // gs, gs, float(eps), int(act == "silu"), int(dtype == torch.bfloat16), _st(o)), "group_norm_gate")
+                                            out.data_ptr(), n, K // gs, gs, float(eps), int(act == "silu"), int(gate_first), int(bool(groups)),
+                                            int(dtype == torch.bfloat16), _st(o)), "group_norm_gate")
         return out
-    x = o.float().reshape(n, K // gs, gs)
-    y = (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * weight).reshape(n, K)
-    return (y * (torch.nn.functional.silu if act == "silu" else torch.sigmoid)(gate.float())).to(dtype)
+    g = (torch.nn.functional.silu if act == "silu" else torch.sigmoid)(gate.float())
+    x = (o.float() * g if gate_first else o.float()).reshape(n, K // gs, gs)
+    y = (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * (weight.view(-1, gs) if groups else weight)).reshape(n, K)
+    return (y if gate_first else y * g).to(dtype)

@@ -1,14 +1,17 @@
 """Softmax attention over the paged cache inside a sliding window or inside chunks of positions (csrc/window_attn.cu,
 csrc/window_attn_sm100.cu), with what designs add to it: the first tokens of a sequence stay visible, a learned sink joins every head's
-denominator, a gate scales every head's output, two maps weigh the same values and their difference is normed.
+denominator, a gate scales every head's output, two maps weigh the same values and their difference is normed, a learned bias joins every
+score by the key's distance.
 
 :class:`WindowAttention` holds what a layer fixes; :func:`proj_norm_write` normalises the whole q and k projections of new tokens
-and fills the pages, :func:`rope_write` rotates them instead; :func:`window_attention` runs query rows at given positions against the
+and fills the pages, :func:`rope_write` rotates them instead (``ops/gated_attention.py`` norms them per head);
+:func:`window_attention` runs query rows at given positions against the
 pages, :func:`window_attention_tiles` the many rows of a prompt.  CUDA tensors run the kernels, CPU tensors the plain math."""
 from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass
+from fractions import Fraction
 from typing import List, Optional, Tuple
 
 import torch
@@ -24,10 +27,10 @@ UNBOUNDED = 1 << 30                    # a window that never ends
 class WindowArgs(C.Structure):
     """``PtbWindowAttn`` of csrc/ptb200_types.h."""
     _fields_ = [(n, C.c_void_p) for n in ("q", "out", "k_pages", "v_pages", "page_table", "pos", "req", "sink", "gate")] + \
-        [("gate_ld", C.c_longlong), ("work", C.c_void_p), ("status", C.c_void_p), ("tiles", C.c_void_p), ("k_rot", C.c_void_p)] + \
+        [("gate_ld", C.c_longlong), ("work", C.c_void_p), ("status", C.c_void_p), ("tiles", C.c_void_p), ("rel", C.c_void_p), ("k_rot", C.c_void_p)] + \
         [(n, C.c_longlong) for n in ("k_ld", "v_row", "rot_ld")] + \
         [(n, C.c_int) for n in ("n", "H", "G", "D", "Dp", "Dv", "Dvp", "v_ld", "maps", "pos_stride", "req_stride", "pt_stride", "n_pages", "window", "keep", "chunked",
-                                "max_keys", "nsplit", "bf16", "n_tiles", "flat_rows", "rot_dim")] + \
+                                "max_keys", "nsplit", "bf16", "rel_n", "n_tiles", "flat_rows", "rot_dim")] + \
         [(n, C.c_float) for n in ("scale", "mix", "mix_gain", "mix_eps")]
 
 
@@ -66,6 +69,7 @@ class WindowAttention:
     mix: float = 0.0
     mix_gain: float = 1.0
     mix_eps: float = 0.0
+    rel: Optional[torch.Tensor] = None       # [heads, distances] fp32: added to a scaled score, the last one for all distances beyond
 
     @property
     def dim_stored(self) -> int:
@@ -142,6 +146,24 @@ def rope_write(p: torch.Tensor, cols: Tuple[int, int, int], a: WindowAttention, 
     return q
 
 
+def distance_bias(table: torch.Tensor, far: float) -> torch.Tensor:
+    """``table [rows, heads]`` by bucket of distances -> ``[heads, distances]`` fp32 by distance: one bucket per distance below half the rows,
+    above it buckets at equal steps of the logarithm up to ``far``, the last one for all beyond.  The buckets' borders are exact."""
+    rows, half = table.shape[0], table.shape[0] // 2
+    span, ratio = rows - half, Fraction(far) / max(half, 1)
+    first = list(range(half)) or [0]                            # first distance of every bucket
+    for m in range(span) if half and ratio > 1 else ():
+        # distance n lies m buckets above the first half where ln(n / half) / ln(far / half) * span >= m
+        n = max(half, int(half * float(ratio) ** (m / span)) - 1)
+        while Fraction(n, half) ** span < ratio ** m:
+            n += 1
+        first.append(n)
+    if len(first) < rows:
+        first = (first + [max(half, 1)] * rows)[:rows] if half else [0] * rows
+    bucket = torch.searchsorted(torch.tensor(first), torch.arange(first[-1] + 1), right=True) - 1
+    return table.float()[bucket.to(table.device)].t().contiguous()
+
+
 def pick_splits(rows: int, kv_heads: int, keys: int, sms: int = 148) -> int:
     """CTAs that share a row's keys: as many as bring the grid to about four per SM while a CTA keeps 32 keys, and at least as many
     as the kernel's limit of keys per CTA asks for.  The number of keys is rounded up to a power of two so that the choice (part of
@@ -158,7 +180,7 @@ def _args(q: torch.Tensor, a: WindowAttention, page_table: torch.Tensor, k_pages
                       n_pages=k_pages.shape[0], sink=N.ptr(a.sink), gate=N.ptr(gate), gate_ld=gate.stride(0) if gate is not None else 0, H=a.heads, G=a.kv_heads,
                       D=a.dim, Dp=a.dim_stored, Dv=a.vdim, Dvp=a.vdim_stored, v_ld=a.vdim_stored, maps=a.maps, window=a.window, keep=a.keep,
                       chunked=int(a.chunked), scale=float(a.scale), mix=float(a.mix), mix_gain=float(a.mix_gain), mix_eps=float(a.mix_eps),
-                      bf16=int(q.dtype == torch.bfloat16), status=_status(q.device).data_ptr())
+                      bf16=int(q.dtype == torch.bfloat16), status=_status(q.device).data_ptr(), rel=N.ptr(a.rel), rel_n=a.rel.shape[1] if a.rel is not None else 0)
 
 
 def run_rows(args: WindowArgs, q: torch.Tensor, out: torch.Tensor, pos: torch.Tensor, req: torch.Tensor, nsplit: int, gate=None,
@@ -194,6 +216,7 @@ def window_attention(q: torch.Tensor, a: WindowAttention, pos: torch.Tensor, req
 
 
 QUERY_TILE = 128                       # queries per tile of csrc/window_attn_sm100.cu
+TILE_DISTANCES = 8192                  # entries of a head's distance bias that its tiles hold (MAX_REL there)
 TILES_FROM = 16                        # rows of a prompt pass from which the tile kernel is the better choice
 
 
@@ -213,7 +236,8 @@ class PromptTiles:
 
 
 def tiles_supported(q: torch.Tensor, a: WindowAttention) -> bool:
-    return q.is_cuda and q.dtype == torch.bfloat16 and a.dim_stored <= 128 and a.vdim_stored <= 128
+    return q.is_cuda and q.dtype == torch.bfloat16 and a.dim_stored <= 128 and a.vdim_stored <= 128 and \
+        (a.rel is None or (a.maps == 1 and a.rel.shape[1] <= TILE_DISTANCES))
 
 
 def window_attention_tiles(q: torch.Tensor, a: WindowAttention, tiles: PromptTiles, page_table: torch.Tensor, k_pages: torch.Tensor,
@@ -245,7 +269,10 @@ def window_attention_reference(q, a: WindowAttention, pos, req, page_table, k_pa
         o = []
         for m in range(a.maps):
             km = k[:, :, m].transpose(0, 1).repeat_interleave(R, 0)                                        # [H, keys, D]
-            s = (torch.einsum("nhd,hjd->hnj", qs[rows, :, m], km) * a.scale).masked_fill(~see, float("-inf"))
+            s = torch.einsum("nhd,hjd->hnj", qs[rows, :, m], km) * a.scale
+            if a.rel is not None:
+                s = s + a.rel[:, (p[:, None] - j[None, :]).clamp(0, a.rel.shape[1] - 1)]
+            s = s.masked_fill(~see, float("-inf"))
             if a.sink is not None:
                 s = torch.cat([s, a.sink.float()[:, None, None].expand(H, len(rows), 1)], -1)
             o.append(torch.einsum("hnj,hjd->nhd", torch.softmax(s, -1)[..., :len(j)], v))

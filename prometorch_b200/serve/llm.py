@@ -1,5 +1,5 @@
 """Continuous-batching engine with a paged KV cache for the models registered in ``models/paged.py`` (Hugging Face Llama
-checkpoints, Kifusun, Gelutar, Budorax).
+checkpoints, Kifusun, Gelutar, Budorax, Tifepel).
 
 Same public surface as the reference's ``LLMEngine`` (torch/serve/llm.h:33-57 for the request types, :299-334 for the
 64-token page pool, :352-437 for ``load / set_weights / generate / submit_request / step / poll_responses``).  The
