@@ -115,8 +115,9 @@ class Output:
     rows: Optional[ExpertRows] = None
 
 
-def _value(b: Branch) -> torch.Tensor:
-    return b.y.float().sum(0) if b.y.dim() == 3 else b.y.float()
+def _value(b: Branch, W: int) -> torch.Tensor:
+    """The first ``W`` columns: the rows of a matrix may have been rounded up."""
+    return (b.y.float().sum(0) if b.y.dim() == 3 else b.y.float())[:, :W]
 
 
 def _norm(u: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
@@ -159,8 +160,8 @@ def step(x: torch.Tensor, before: Optional[Output], nxt: Optional[Connection], e
     else:
         if before is not None:
             link = before.link
-            y = sum(v for v in (_value(before.y) if before.y else None, before.rows.combine() if before.rows else None) if v is not None)
-            y = y * torch.sigmoid(_value(before.gate) + link.gate_bias)
+            y = sum(v for v in (_value(before.y, x.shape[2]) if before.y else None, before.rows.combine() if before.rows else None) if v is not None)
+            y = y * torch.sigmoid(_value(before.gate, x.shape[2]) + link.gate_bias)
             x.copy_(torch.einsum("nsw,st->ntw", x, link.mix) + link.way_out[:, None] * y[:, None, :])
         h = hc = None
         if nxt is not None:
