@@ -320,6 +320,9 @@ def served_native_figure(path, prompt_ids, n_new):
             p.kill()
 
 
+BESIDE_LLAMA = ("kifusun", "gelutar", "budorax", "tifepel")
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -327,8 +330,8 @@ def main():
     ap.add_argument("--warmup", type=int, default=16)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--prompt-len", type=int, default=128)
-    ap.add_argument("--model", default="qwen3-4b", choices=["qwen3-4b", "tiny", "kifusun", "gelutar", "budorax"],
-                    help="kifusun, gelutar, budorax: that model beside Llama of equal size in the batching engine (benchmarks/*_bench.py), 1 GPU")
+    ap.add_argument("--model", default="qwen3-4b", choices=["qwen3-4b", "tiny", *BESIDE_LLAMA],
+                    help=", ".join(BESIDE_LLAMA) + ": that model beside Llama of equal size in the batching engine (benchmarks/*_bench.py), 1 GPU")
     ap.add_argument("--max-seq", type=int, default=4096)
     ap.add_argument("--repeats", type=int, default=5, help="timed regions of --steps steps each (median is reported)")
     ap.add_argument("--train-steps", type=int, default=5, help="timed steps of the Llama-1.1B FSDP half (0 = skip)")
@@ -338,18 +341,10 @@ def main():
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
-    if args.model == "kifusun":
+    if args.model in BESIDE_LLAMA:
+        import importlib
         sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
-        import kifusun_bench
-        return kifusun_bench.main([])
-    if args.model == "gelutar":
-        sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
-        import gelutar_bench
-        return gelutar_bench.main([])
-    if args.model == "budorax":
-        sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
-        import budorax_bench
-        return budorax_bench.main([])
+        return importlib.import_module(args.model + "_bench").main([])
     args.warmup = max(args.warmup, 3)
 
     import torch

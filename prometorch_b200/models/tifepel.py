@@ -26,7 +26,7 @@ from ..ops import recurrence as R
 from ..ops import residual as S
 from ..ops import streams as H
 from ..ops import window_attention as A
-from ..ops.gated_attention import head_norm_write
+from ..ops.gated_attention import distance_bias, head_norm_write
 from .paged import PagedModel, PromptBatch, RowPack, register_model
 
 
@@ -303,7 +303,8 @@ class PagedTifepel(PagedModel):
             else:
                 d["pack"] = RowPack({n: mix[n].shape[0] for n in "qkv"})
                 d["w_in"] = d["pack"].pack({n: mix[n] for n in "qkv"})
-                d["attn"] = A.WindowAttention(m.heads, m.kv_heads, m.dim, m.vdim, A.UNBOUNDED, 0, m.scale, rel=A.distance_bias(mix["rel"], m.bias_max))
+                d["attn"] = A.WindowAttention(m.heads, m.kv_heads, m.dim, m.vdim, A.UNBOUNDED, 0, m.scale, 
+                                              rel=distance_bias(mix["rel"], m.bias_max, c.max_position_embeddings))
                 d["gain"] = gain(m.temp_coef, m.temp_every)
             if x:
                 parts = lambda n: [L[f"mlp.e{i}.{n}"] for i in range(x.experts)]

@@ -179,7 +179,7 @@ def run_shared(h: torch.Tensor, e: SharedExpert) -> Branch:
     F = e.down.shape[1]
     if h.is_cuda and h.dtype == torch.bfloat16 and n > GATED_FROM and W % 8 == 0 and h.stride(0) % 8 == 0:
         act = torch.empty(n, F, dtype=h.dtype, device=h.device)
-        offsets = torch.tensor([0, n], dtype=torch.int32).to(h.device)
+        offsets = torch.arange(0, n + 1, n, dtype=torch.int32, device=h.device)          # [0, n]
         N.check(N.lib().ptb_expert_gemm(h.data_ptr(), h.stride(0), e.gate_up.data_ptr(), 1, act.data_ptr(), offsets.data_ptr(), n, 1, F, W, 0, 0,
                                         _status(h.device).data_ptr(), _st(h)), "expert_gemm")
     else:

@@ -11,7 +11,6 @@ from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass
-from fractions import Fraction
 from typing import List, Optional, Tuple
 
 import torch
@@ -69,7 +68,7 @@ class WindowAttention:
     mix: float = 0.0
     mix_gain: float = 1.0
     mix_eps: float = 0.0
-    rel: Optional[torch.Tensor] = None       # [heads, distances] fp32: added to a scaled score, the last one for all distances beyond
+    rel: Optional[torch.Tensor] = None       # [heads, distances] fp32: added to a scaled score, the last one for all beyond (ops/gated_attention.py makes it)
 
     @property
     def dim_stored(self) -> int:
@@ -144,24 +143,6 @@ def rope_write(p: torch.Tensor, cols: Tuple[int, int, int], a: WindowAttention, 
     k_pages[pages, :, at % PAGE] = turn(cols[1], Gm).reshape(n, G, a.maps * Dp).to(k_pages.dtype)
     v_pages[pages, :, at % PAGE] = torch.nn.functional.pad(x[:, cols[2]:cols[2] + G * Dv].reshape(n, G, Dv), (0, Dvp - Dv)).to(v_pages.dtype)
     return q
-
-
-def distance_bias(table: torch.Tensor, far: float) -> torch.Tensor:
-    """``table [rows, heads]`` by bucket of distances -> ``[heads, distances]`` fp32 by distance: one bucket per distance below half the rows,
-    above it buckets at equal steps of the logarithm up to ``far``, the last one for all beyond.  The buckets' borders are exact."""
-    rows, half = table.shape[0], table.shape[0] // 2
-    span, ratio = rows - half, Fraction(far) / max(half, 1)
-    first = list(range(half)) or [0]                            # first distance of every bucket
-    for m in range(span) if half and ratio > 1 else ():
-        # distance n lies m buckets above the first half where ln(n / half) / ln(far / half) * span >= m
-        n = max(half, int(half * float(ratio) ** (m / span)) - 1)
-        while Fraction(n, half) ** span < ratio ** m:
-            n += 1
-        first.append(n)
-    if len(first) < rows:
-        first = (first + [max(half, 1)] * rows)[:rows] if half else [0] * rows
-    bucket = torch.searchsorted(torch.tensor(first), torch.arange(first[-1] + 1), right=True) - 1
-    return table.float()[bucket.to(table.device)].t().contiguous()
 
 
 def pick_splits(rows: int, kv_heads: int, keys: int, sms: int = 148) -> int:

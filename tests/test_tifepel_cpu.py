@@ -120,24 +120,19 @@ def test_step_between_sublayers(streams):
 
 
 # ------------------------------------------------------------------------------------------ attention
-@pytest.mark.parametrize("n_rows,far", [(16, 120), (16, 128), (32, 1000), (10, 37), (7, 50), (2, 9), (4, 2), (5, 2.5), (1, 10), (64, 64.5)])
+@pytest.mark.parametrize("n_rows,far", [(16, 120), (16, 128), (32, 1000), (10, 37), (7, 50), (2, 9), (5, 2.5), (64, 64.5)])
 def test_bias_by_distance(n_rows, far):
     table = torch.arange(2 * n_rows).view(n_rows, 2)
-    got = A.distance_bias(table, far)
-    if n_rows == 1:
-        assert got.tolist() == [[0.0], [1.0]]
-        return
-    half = n_rows // 2
+    got = GA.distance_bias(table, far, 6000)
     for n in list(range(min(300, 3 * int(far)))) + [int(far) - 1, int(far), int(far) + 1, 5000]:
-        want = oracle.bucket(n, n_rows, far) if far > half else min(n, half - 1) if n < half else n_rows - 1
-        assert got[1, min(n, got.shape[1] - 1)] == 2 * want + 1, n
-    assert got.shape[1] <= max(far, half) + 2 and int(got[0, -1]) == 2 * (n_rows - 1)
+        assert got[1, min(n, got.shape[1] - 1)] == 2 * oracle.bucket(n, n_rows, far) + 1, n
+    assert got.shape[1] <= far + 2 and int(got[0, -1]) == 2 * (n_rows - 1)
 
 
 def attention_case(Hh, G, D, Dv, n, rel_rows=8, far=30, scale=0.4, seed=1, every=10, coef=0.5):
     g = torch.Generator().manual_seed(seed)
     rel = torch.randn(rel_rows, Hh, generator=g) * 2
-    a = A.WindowAttention(Hh, G, D, Dv, A.UNBOUNDED, 0, scale, rel=A.distance_bias(rel, far))
+    a = A.WindowAttention(Hh, G, D, Dv, A.UNBOUNDED, 0, scale, rel=GA.distance_bias(rel, far, 1024))
     kc, vc = Hh * D + 3, Hh * D + 3 + G * D
     p = torch.randn(n, vc + G * Dv + 2, generator=g) * 1.5
     gain = torch.tensor([oracle.temperature(i, coef, every) for i in range(256)])
@@ -170,7 +165,7 @@ def test_a_bucket_that_stands_out():
     q = GA.head_norm_write(p, a, None, None, 1e-6, *rows(n), table, kp, vp, cols=cols, gain=gain)
     v = p[:, cols[1]:cols[1] + D].double()
     for b in range(8):
-        a.rel = A.distance_bias(torch.where(torch.arange(8)[:, None] == b, 60.0, 0.0), 40)
+        a.rel = GA.distance_bias(torch.where(torch.arange(8)[:, None] == b, 60.0, 0.0), 40, 1024)
         out = A.window_attention(q, a, *rows(n), table, kp, vp, 1, n)
         for i in range(n):
             there = [j for j in range(i + 1) if oracle.bucket(i - j, 8, 40) == b] or list(range(i + 1))

@@ -145,10 +145,10 @@ def test_convolution_with_bias_or_sum(C, taps, add, dtype):
 
 # ------------------------------------------------------------------------------------------ attention
 def biased(Hh, G, D, Dv, lens, starts, far=100, rel_rows=16, scale=None, seed=0):
-    from prometorch_b200.ops import window_attention as A
+    from prometorch_b200.ops import gated_attention as GA, window_attention as A
     g, pages, table, pos, req, offs = layout(lens, starts, seed)
     rnd = lambda *s: torch.randn(*s, generator=g)
-    a = A.WindowAttention(Hh, G, D, Dv, A.UNBOUNDED, 0, scale or D ** -0.5, rel=A.distance_bias(rnd(rel_rows, Hh) * 2, far).cuda())
+    a = A.WindowAttention(Hh, G, D, Dv, A.UNBOUNDED, 0, scale or D ** -0.5, rel=GA.distance_bias(rnd(rel_rows, Hh) * 2, far, 30000).cuda())
     n, Dp = sum(lens), a.dim_stored
     k, v, q = torch.zeros(pages, G, 64, Dp), torch.zeros(pages, G, 64, a.vdim_stored), torch.zeros(n, Hh, Dp)
     k[..., :D], v[..., :Dv], q[..., :D] = rnd(pages, G, 64, D) * 1.5, rnd(pages, G, 64, Dv), rnd(n, Hh, D) * 1.5
@@ -181,14 +181,14 @@ def test_biased_attention_kernels(shape):
 @pytest.mark.parametrize("far,rel_rows", [(40, 8), (64, 16), (65, 6), (200, 16)])
 def test_a_bucket_that_stands_out(far, rel_rows):
     """One bucket's bias far above the others: rows return the mean of the values at its distances, in both kernels, across pages and tiles."""
-    from prometorch_b200.ops import window_attention as A
+    from prometorch_b200.ops import gated_attention as GA, window_attention as A
     n = 430
     a, q, k, v, pos, req, table, offs = biased(2, 1, 64, 64, [n], [0], scale=1e-5)
     tiles = A.PromptTiles.of(offs, [0], [0], "cuda")
     at = torch.arange(n)
     val = v[table[0, at.cuda() // 64].long(), 0, at.cuda() % 64].double().cpu()
     for b in range(rel_rows):
-        a.rel = A.distance_bias(torch.where(torch.arange(rel_rows)[:, None] == b, 60.0, 0.0).expand(rel_rows, 2), far).cuda()
+        a.rel = GA.distance_bias(torch.where(torch.arange(rel_rows)[:, None] == b, 60.0, 0.0).expand(rel_rows, 2), far, 1024).cuda()
         where = torch.tensor([oracle.bucket(d, rel_rows, far) == b for d in range(n)])
         for out in (A.window_attention(q, a, pos, req, table, k, v, 4, n), A.window_attention_tiles(q, a, tiles, table, k, v)):
             for i in (0, 1, 62, 63, 64, 65, 127, 128, 129, 200, 300, 429):
