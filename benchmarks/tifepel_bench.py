@@ -115,19 +115,20 @@ def kernel_rows(z, prompt=4096, ctx=4096):
     # ---- router, experts' products and the shared expert
     wr = lambda *s: torch.randn(*s, device="cuda", dtype=torch.bfloat16).mul_(s[-1] ** -0.5)
     O = EXPERTS + IDENTITY
-    ex = [X.Experts(wr(EXPERTS, 2 * ff, W), wr(EXPERTS, W, ff), wr(-(-O // 8) * 8, W), f32(O) * 0.01, TOP, 1.0, True) for _ in range(2)]
-    eb = [X.Experts(e.gate_up, e.down, wr(EXPERTS, W), f32(EXPERTS) * 0.1, TOP + 1, 1.0) for e in ex]
-    sh = [X.SharedExpert(wr(2 * ff, W), wr(W, ff)) for _ in range(8)]
+    ex = [X.Experts(wr(EXPERTS + 1, 2 * ff, W), wr(EXPERTS + 1, W, ff), wr(-(-O // 8) * 8, W), f32(O) * 0.01, TOP, 1.0, True, 1) for _ in range(2)]
+    eb = [X.Experts(e.gate_up[:EXPERTS], e.down[:EXPERTS], wr(EXPERTS, W), f32(EXPERTS) * 0.1, TOP + 1, 1.0) for e in ex]
+    sh = [X.SharedExpert(wr(2 * z["ff"], W), wr(W, z["ff"])) for _ in range(3)]
     for n in (4096, 32, 1):
         h = rand(n, W)
         add(f"router (softmax) and order, {n} rows", per_launch_us([lambda i=i: X.route(h, ex[i]) for i in range(2)], 6), 2 * n * W + 2 * O * W)
         add(f"router (sigmoid) and order, {n} rows (budorax)", per_launch_us([lambda i=i: X.route(h, eb[i]) for i in range(2)], 6), 2 * n * W + 2 * EXPERTS * W)
-        for name, es in (("with identities", ex), ("(budorax)", eb)):
+        for name, es in (("with identities and the shared one", ex), ("(budorax)", eb)):
             rt = [X.route(h, e) for e in es]
             live, held = int((rt[0].offsets[1:] > rt[0].offsets[:-1]).sum()), int(rt[0].offsets[-1])
             add(f"experts' products, {n} rows {name}", per_launch_us([lambda i=i: X.products(h, es[i], rt[i]) for i in range(2)], 6),
                 2 * (4 * held * W + live * 3 * ff * W + 2 * held * ff), 6.0 * held * ff * W)
-        add(f"shared expert, {n} rows", per_launch_us([lambda e=e: X.run_shared(h, e) for e in sh], 8), 2 * (2 * n * W + 3 * ff * W + 2 * n * ff), 6.0 * n * ff * W)
+        add(f"shared expert by itself, {PARTS} times the others' width, {n} rows", per_launch_us([lambda e=e: X.run_shared(h, e) for e in sh], 6),
+            2 * (2 * n * W + 3 * z["ff"] * W + 2 * n * z["ff"]), 6.0 * n * z["ff"] * W)
         wg, wd = [rand(2 * z["ff"], W) for _ in range(2)], [rand(W, z["ff"]) for _ in range(2)]
         add(f"feed-forward, {n} rows (llama)", per_launch_us([lambda i=i: gemm.linear(gemm.linear_swiglu(h, wg[i]), wd[i]) for i in range(2)], 4),
             2 * (2 * n * W + 3 * z["ff"] * W + 2 * n * z["ff"]), 6.0 * n * z["ff"] * W)
@@ -175,10 +176,10 @@ def kernel_rows(z, prompt=4096, ctx=4096):
         add(f"streams: gate + sum + layer norm{'' if big else ' + input convolution'}, {n} rows",
             per_launch_us([lambda i=i: H._launch(xs[i], H.Output(link, S.Branch(g[i]), S.Branch(y[i])), link.way_in, link.norm, 1e-5, torch.bfloat16, None, None if big else link.conv, canon,
                                                  pos, req) for i in range(sets)]), step_bytes + 4 * n * W)
-        rows_ = X.ExpertRows(rand(n * TOP, W), torch.randperm(n * TOP, device="cuda").int().view(n, TOP), torch.rand(n, TOP, device="cuda"), rand(n, W))
-        add(f"streams: experts' sum + shared + gate + sum + layer norm{'' if big else ' + input convolution'}, {n} rows",
-            per_launch_us([lambda i=i: H._launch(xs[i], H.Output(link, S.Branch(g[i]), S.Branch(y[i]), rows_), link.way_in, link.norm, 1e-5, torch.bfloat16, None,
-                                                 None if big else link.conv, canon, pos, req) for i in range(sets)]), step_bytes + n * W * (4 + 2 * TOP))
+        rows_ = X.ExpertRows(rand(n * PARTS, W), torch.randperm(n * PARTS, device="cuda").int().view(n, PARTS), torch.rand(n, PARTS, device="cuda"), rand(n, W))
+        add(f"streams: experts' sum + gate + sum + layer norm{'' if big else ' + input convolution'}, {n} rows",
+            per_launch_us([lambda i=i: H._launch(xs[i], H.Output(link, S.Branch(g[i]), None, rows_), link.way_in, link.norm, 1e-5, torch.bfloat16, None,
+                                                 None if big else link.conv, canon, pos, req) for i in range(sets)]), step_bytes + n * W * (2 + 2 * PARTS))
         x1 = [f32(n, W) for _ in range(sets)]
         add(f"tanh norm + fp32 residual + tanh norm, {n} rows (budorax)", per_launch_us([lambda i=i: T.residual(x1[i], S.Branch(y[i]), norm, norm, torch.bfloat16) for i in range(sets)]),
             n * W * 12)

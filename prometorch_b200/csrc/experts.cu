@@ -6,7 +6,8 @@
 //   route_small_kernel  both for few tokens in one CTA;
 //   route_rows_kernel   the router's product as well, for few tokens;
 //   expert_simt_kernel  a grouped product over the sorted rows with FMAs in fp32 (fp32 models, sizes the tensor-core kernel cannot address).
-// The router may have more outputs than there are experts: those behind them are identities, without rows; their place is -1.
+// The router may have more outputs than there are experts: those behind them are identities, without rows; their place is -1.  `always` more
+// experts follow the routed ones in the order of rows; every token uses them, with the weight 1.
 // Where a row lies inside its expert depends on the order of atomics; what is computed for it does not.
 #include "common.cuh"
 #include <algorithm>
@@ -22,17 +23,31 @@ struct Route {
     long long stride, ld;
     const float* correction;           // [O]
     int n, E, top;
-    int O, softmax;                    // router outputs: the experts and the identities behind them
+    int O, softmax, always;            // router outputs: the experts and the identities behind them
     float scale;                       // weights: scores over their sum times scale; softmax: the scores times scale
-    int* index;                        // [n][top] out: place in the order by expert
-    float* weight;                     // [n][top] out
-    int* token;                        // [n top] out
-    int* offsets;                      // [E + 1] out
-    int* expert;                       // [n][top] between the kernels
-    int* rank;                         // [n][top]
+    int* index;                        // [n][K] out: place in the order by expert, K = top + always
+    float* weight;                     // [n][K] out
+    int* token;                        // [n K] out
+    int* offsets;                      // [E + always + 1] out
+    int* expert;                       // [n][K] between the kernels, the first `top` of a row
+    int* rank;                         // [n][K] likewise
     int* counts;                       // [E], zero at the start
     int* status;
+    __host__ __device__ int K() const { return top + always; }
 };
+
+// Pair p of a token goes to its place; off: first place of every expert.
+__device__ __forceinline__ void put(const Route& R, long long p, const int* off) {
+    const int K = R.K(), i = (int)(p / K), k = (int)(p % K);
+    int at;
+    if (k >= R.top) at = off[R.E + k - R.top] + i;
+    else {
+        const int e = __ldcg(R.expert + p);
+        at = e < R.E ? off[e] + R.rank[p] : -1;
+    }
+    R.index[p] = at;
+    if (at >= 0) R.token[at] = i;
+}
 
 // The logit of token i and expert e.
 struct Logits {
@@ -92,12 +107,13 @@ __device__ __forceinline__ void choose(const Route& R, int i, float* c_s, Z logi
             chosen(k, at);
         }
         __syncwarp();
-        if ((k & 31) == 31 && k + 1 < R.top) R.weight[(size_t)i * R.top + k - 31 + lane] = mine;      // unscaled: the sum is not known yet
+        if ((k & 31) == 31 && k + 1 < R.top) R.weight[(size_t)i * R.K() + k - 31 + lane] = mine;      // unscaled: the sum is not known yet
     }
     const float f = R.softmax ? R.scale : R.scale / (sum + 1e-20f);
     const int k0 = (R.top - 1) & ~31;                  // the last ones are still in registers
-    for (int k = lane; k < k0; k += 32) R.weight[(size_t)i * R.top + k] *= f;
-    if (k0 + lane < R.top) R.weight[(size_t)i * R.top + k0 + lane] = mine * f;
+    for (int k = lane; k < k0; k += 32) R.weight[(size_t)i * R.K() + k] *= f;
+    if (k0 + lane < R.top) R.weight[(size_t)i * R.K() + k0 + lane] = mine * f;
+    for (int k = R.top + lane; k < R.K(); k += 32) R.weight[(size_t)i * R.K() + k] = 1.f;
 }
 
 __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const __grid_constant__ Route R) {
@@ -113,25 +129,26 @@ __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const __grid_const
     const int i = blockIdx.x * RT_WARPS + warp;
     if (i < R.n)
         choose(R, i, c_s, Logits{R, i}, [&](int k, int e) {
-            R.expert[(size_t)i * R.top + k] = e;
-            if (e < R.E) R.rank[(size_t)i * R.top + k] = atomicAdd(&count[e], 1);
+            R.expert[(size_t)i * R.K() + k] = e;
+            if (e < R.E) R.rank[(size_t)i * R.K() + k] = atomicAdd(&count[e], 1);
         });
     __syncthreads();
     for (int e = threadIdx.x; e < R.E; e += blockDim.x) base[e] = count[e] ? atomicAdd(&R.counts[e], count[e]) : 0;
     __syncthreads();
     if (i < R.n)
         for (int k = threadIdx.x & 31; k < R.top; k += 32) {
-            const size_t p = (size_t)i * R.top + k;
+            const size_t p = (size_t)i * R.K() + k;
             if (R.expert[p] < R.E) R.rank[p] += base[R.expert[p]];
         }
 }
 
-// Exclusive sums of count[0 .. E) to off[0 .. E], by the first warp.
-__device__ __forceinline__ void prefix(const int* count, int* off, int E) {
+// Exclusive sums of the experts' rows to off[0 .. E + always], by the first warp; count: of the routed ones.
+__device__ __forceinline__ void prefix(const Route& R, const int* count, int* off) {
     if (threadIdx.x < 32) {
+        const int E = R.E + R.always;
         int run = 0;
         for (int e0 = 0; e0 < E; e0 += 32) {
-            const int e = e0 + threadIdx.x, v = e < E ? count[e] : 0;
+            const int e = e0 + threadIdx.x, v = e < R.E ? count[e] : e < E ? R.n : 0;
             int s = v;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -149,16 +166,12 @@ __global__ void __launch_bounds__(256) place_kernel(const __grid_constant__ Rout
     extern __shared__ int off[];
     pdl_wait();
     pdl_launch_dependents();
-    prefix(R.counts, off, R.E);
+    prefix(R, R.counts, off);
     __syncthreads();
     if (blockIdx.x == 0)
-        for (int e = threadIdx.x; e <= R.E; e += blockDim.x) R.offsets[e] = off[e];
-    const long long total = (long long)R.n * R.top;
-    for (long long p = (long long)blockIdx.x * blockDim.x + threadIdx.x; p < total; p += (long long)gridDim.x * blockDim.x) {
-        const int e = R.expert[p], at = e < R.E ? off[e] + R.rank[p] : -1;
-        R.index[p] = at;
-        if (at >= 0) R.token[at] = (int)(p / R.top);
-    }
+        for (int e = threadIdx.x; e <= R.E + R.always; e += blockDim.x) R.offsets[e] = off[e];
+    const long long total = (long long)R.n * R.K();
+    for (long long p = (long long)blockIdx.x * blockDim.x + threadIdx.x; p < total; p += (long long)gridDim.x * blockDim.x) put(R, p, off);
 }
 
 __global__ void __launch_bounds__(RS_WARPS * 32) route_small_kernel(const __grid_constant__ Route R) {
@@ -173,18 +186,14 @@ __global__ void __launch_bounds__(RS_WARPS * 32) route_small_kernel(const __grid
     __syncthreads();
     for (int i = warp; i < R.n; i += RS_WARPS)
         choose(R, i, c_s, Logits{R, i}, [&](int k, int e) {
-            R.expert[(size_t)i * R.top + k] = e;
-            if (e < R.E) R.rank[(size_t)i * R.top + k] = atomicAdd(&count[e], 1);
+            R.expert[(size_t)i * R.K() + k] = e;
+            if (e < R.E) R.rank[(size_t)i * R.K() + k] = atomicAdd(&count[e], 1);
         });
     __syncthreads();
-    prefix(count, off, R.E);
+    prefix(R, count, off);
     __syncthreads();
-    for (int e = threadIdx.x; e <= R.E; e += blockDim.x) R.offsets[e] = off[e];
-    for (int p = threadIdx.x; p < R.n * R.top; p += blockDim.x) {
-        const int e = R.expert[p], at = e < R.E ? off[e] + R.rank[p] : -1;
-        R.index[p] = at;
-        if (at >= 0) R.token[at] = p / R.top;
-    }
+    for (int e = threadIdx.x; e <= R.E + R.always; e += blockDim.x) R.offsets[e] = off[e];
+    for (int p = threadIdx.x; p < R.n * R.K(); p += blockDim.x) put(R, p, off);
 }
 
 constexpr int RR_THREADS = 128, RR_WARPS = RR_THREADS / 32;
@@ -195,7 +204,7 @@ constexpr int RR_THREADS = 128, RR_WARPS = RR_THREADS / 32;
 template <typename T>
 __global__ void __launch_bounds__(RR_THREADS) route_rows_kernel(const __grid_constant__ Route R, const T* __restrict__ h, long long ldh, const T* __restrict__ w, int W,
                                                                 float* z, unsigned* done) {
-    extern __shared__ float c_s[];                     // [2 O], later counts [E] and offsets [E + 1]
+    extern __shared__ float c_s[];                     // [2 O], later counts [E] and offsets [E + always + 1]
     __shared__ int last;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, i = blockIdx.y;
     constexpr int V = 16 / sizeof(T);                  // elements of a 16-byte load
@@ -232,25 +241,22 @@ __global__ void __launch_bounds__(RR_THREADS) route_rows_kernel(const __grid_con
         return last != 0;
     };
     if (!finished(done + i, gridDim.x)) return;
-    if (warp == 0) choose(R, i, c_s, [&](int e) { return __ldcg(z + (size_t)i * R.O + e); }, [&](int k, int e) { R.expert[(size_t)i * R.top + k] = e; });
+    if (warp == 0) choose(R, i, c_s, [&](int e) { return __ldcg(z + (size_t)i * R.O + e); }, [&](int k, int e) { R.expert[(size_t)i * R.K() + k] = e; });
     if (!finished(done + R.n, gridDim.y)) return;
     int *count = reinterpret_cast<int*>(c_s), *off = count + R.E;
     for (int e = threadIdx.x; e < R.E; e += RR_THREADS) count[e] = 0;
     __syncthreads();
-    const int pairs = R.n * R.top;
+    const int K = R.K(), pairs = R.n * K;
     for (int p = threadIdx.x; p < pairs; p += RR_THREADS) {
+        if (p % K >= R.top) continue;
         const int e = __ldcg(R.expert + p);
         if (e < R.E) R.rank[p] = atomicAdd(&count[e], 1);
     }
     __syncthreads();
-    prefix(count, off, R.E);
+    prefix(R, count, off);
     __syncthreads();
-    for (int e = threadIdx.x; e <= R.E; e += RR_THREADS) R.offsets[e] = off[e];
-    for (int p = threadIdx.x; p < pairs; p += RR_THREADS) {
-        const int e = __ldcg(R.expert + p), at = e < R.E ? off[e] + R.rank[p] : -1;
-        R.index[p] = at;
-        if (at >= 0) R.token[at] = p / R.top;
-    }
+    for (int e = threadIdx.x; e <= R.E + R.always; e += RR_THREADS) R.offsets[e] = off[e];
+    for (int p = threadIdx.x; p < pairs; p += RR_THREADS) put(R, p, off);
 }
 
 // ---------------------------------------------------------------------------------------------- grouped product, any size
@@ -326,20 +332,23 @@ __global__ void __launch_bounds__(256) expert_simt_kernel(const T* __restrict__ 
 
 using namespace ptb;
 
-// Routing of n tokens over O >= E router outputs: z [splits][n] fp32 logits (rows of pitch ld, splits `stride` apart), correction [O].  index
-// [n, top]: the place of a token's i-th expert in the order by expert, -1 for an output behind the experts; weight [n, top]: its sigmoid score over
-// the sum of the chosen ones, times scale (softmax: its score times scale); token [n top]: the token of every place; offsets [E + 1].  work:
-// 2 n top + E ints.
-PTB_API int ptb_expert_route(const float* z, int splits, long long stride, long long ld, const float* correction, int n, int E, int O, int softmax, int top, float scale,
+// Routing of n tokens over O >= E router outputs: z [splits][n] fp32 logits (rows of pitch ld, splits `stride` apart), correction [O].  `always`
+// experts behind the E routed ones serve every token; K = top + always.  index [n, K]: the place of a token's i-th expert in the order by expert, -1
+// for an output behind the routed experts; weight [n, K]: its sigmoid score over the sum of the chosen ones, times scale (softmax: its score times
+// scale), 1 for the last `always`; token [n K]: the token of every place; offsets [E + always + 1].  work: 2 n K + E ints.
+PTB_API int ptb_expert_route(const float* z, int splits, long long stride, long long ld, const float* correction, int n, int E, int O, int always, int softmax, int top, float scale,
                              int* index, float* weight, int* token, int* offsets, int* work, int* status, cudaStream_t st) {
     using namespace ptb::moe;
     if (n <= 0) return 0;
-    if (E < 1 || O < E || top < 1 || top > O || O > 1024) { ptb_set_error("experts: %d of %d outputs (at most 1024), %d experts", top, O, E); return -1; }
-    const size_t pairs = (size_t)n * top;
-    Route r{z, splits, stride, ld, correction, n, E, top, O, softmax, scale, index, weight, token, offsets, work, work + pairs, work + 2 * pairs, status};
+    if (E < 1 || O < E || top < 1 || top > O || O > 1024 || always < 0 || E + always > 1024) {
+        ptb_set_error("experts: %d of %d outputs (at most 1024), %d and %d experts", top, O, E, always);
+        return -1;
+    }
+    const size_t pairs = (size_t)n * (top + always);
+    Route r{z, splits, stride, ld, correction, n, E, top, O, softmax, always, scale, index, weight, token, offsets, work, work + pairs, work + 2 * pairs, status};
     const bool pdl = ptb_pdl_enabled();
     if (n <= SMALL_TOKENS && O <= 256) {
-        const size_t smem = ((size_t)RS_WARPS * 2 * O + 2 * E + 1) * 4;
+        const size_t smem = ((size_t)RS_WARPS * 2 * O + 2 * E + always + 1) * 4;
         if (smem > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(route_small_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
         PTB_CUDA_OK(ptb_launch(route_small_kernel, dim3(1), dim3(RS_WARPS * 32), smem, st, pdl, r));
     } else {
@@ -347,29 +356,29 @@ PTB_API int ptb_expert_route(const float* z, int splits, long long stride, long 
         const size_t smem = ((size_t)RT_WARPS * 2 * O + 2 * E) * 4;
         if (smem > 48 * 1024) PTB_CUDA_OK(cudaFuncSetAttribute(route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024));
         PTB_CUDA_OK(ptb_launch(route_kernel, dim3((n + RT_WARPS - 1) / RT_WARPS), dim3(RT_WARPS * 32), smem, st, false, r));
-        PTB_CUDA_OK(ptb_launch(place_kernel, dim3((unsigned)std::min<size_t>(1024, (pairs + 255) / 256)), dim3(256), (size_t)(E + 1) * 4, st, pdl, r));
+        PTB_CUDA_OK(ptb_launch(place_kernel, dim3((unsigned)std::min<size_t>(1024, (pairs + 255) / 256)), dim3(256), (size_t)(E + always + 1) * 4, st, pdl, r));
     }
     PTB_CUDA_OK(cudaGetLastError());
     return 0;
 }
 
-// The same from the rows themselves, for few tokens: h [n, W] (pitch ldh) and the router w [O, W], both bf16 or fp32.  work: 2 n top ints and n O floats;
+// The same from the rows themselves, for few tokens: h [n, W] (pitch ldh) and the router w [O, W], both bf16 or fp32.  work: 2 n K ints and n O floats;
 // done: n + 1 unsigned that are zero between calls, used by one stream at a time.
-PTB_API int ptb_expert_route_rows(const void* h, long long ldh, const void* w, int W, const float* correction, int n, int E, int O, int softmax, int top,
+PTB_API int ptb_expert_route_rows(const void* h, long long ldh, const void* w, int W, const float* correction, int n, int E, int O, int always, int softmax, int top,
                                   float scale, int* index, float* weight, int* token, int* offsets, int* work, unsigned* done, int bf16, cudaStream_t st) {
     using namespace ptb::moe;
     if (n <= 0) return 0;
-    const size_t pairs = (size_t)n * top;
-    if (E < 1 || O < E || top < 1 || top > O || O > 1024 || n > 65535 || W < 1) {
-        ptb_set_error("experts: %d of %d outputs (at most 1024), %d experts, %d columns", top, O, E, W);
+    const size_t pairs = (size_t)n * (top + always);
+    if (E < 1 || O < E || top < 1 || top > O || O > 1024 || always < 0 || E + always > 1024 || n > 65535 || W < 1) {
+        ptb_set_error("experts: %d of %d outputs (at most 1024), %d and %d experts, %d columns", top, O, E, always, W);
         return -1;
     }
-    const Route r{nullptr, 0, 0, 0, correction, n, E, top, O, softmax, scale, index, weight, token, offsets, work, work + pairs, nullptr, nullptr};
+    const Route r{nullptr, 0, 0, 0, correction, n, E, top, O, softmax, always, scale, index, weight, token, offsets, work, work + pairs, nullptr, nullptr};
     const bool pdl = ptb_pdl_enabled();
     auto go = [&](auto k, auto t) {
         using T = decltype(t);
         const int groups = std::max(1, std::min((O + RR_WARPS - 1) / RR_WARPS, 148 * 8 / n));
-        return ptb_launch(k, dim3(groups, n), dim3(RR_THREADS), (2 * (size_t)O + 1) * 4, st, pdl, r, (const T*)h, ldh, (const T*)w, W,
+        return ptb_launch(k, dim3(groups, n), dim3(RR_THREADS), (2 * (size_t)O + always + 1) * 4, st, pdl, r, (const T*)h, ldh, (const T*)w, W,
                           reinterpret_cast<float*>(work + 2 * pairs), done);
     };
     PTB_CUDA_OK(bf16 ? go(route_rows_kernel<__nv_bfloat16>, __nv_bfloat16()) : go(route_rows_kernel<float>, 0.f));

@@ -46,7 +46,7 @@ __device__ __forceinline__ void st(T* p, const Vals<V>& r) {
 template <typename T> __device__ __forceinline__ float rounded(float v) { return (float)(T)v; }
 
 // ---------------------------------------------------------------------------------------------- into the streams
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(256) pair_embed_kernel(const __grid_constant__ PtbPairEmbed P) {
     pdl_wait();
     pdl_launch_dependents();
@@ -70,9 +70,12 @@ __global__ void __launch_bounds__(256) pair_embed_kernel(const __grid_constant__
     }
     const T *a = (const T*)P.table + (size_t)id * P.W, *b = (const T*)P.pairs + (size_t)row * P.W, *c = (const T*)P.at + (size_t)pos * P.W;
     float* x = P.x + i * P.streams * P.W;
-    for (int e = threadIdx.x; e < P.W; e += blockDim.x) {
-        const float v = (float)a[e] + (float)b[e] + (float)c[e];
-        for (int s = 0; s < P.streams; ++s) x[(size_t)s * P.W + e] = v;
+    for (int e = threadIdx.x * V; e < P.W; e += blockDim.x * V) {
+        Vals<V> v = ld<V>(a + e);
+        const Vals<V> p = ld<V>(b + e), q = ld<V>(c + e);
+#pragma unroll
+        for (int k = 0; k < V; ++k) v.v[k] += p.v[k] + q.v[k];
+        for (int s = 0; s < P.streams; ++s) st<V>(x + (size_t)s * P.W + e, v);
     }
 }
 
@@ -277,7 +280,10 @@ PTB_API int ptb_pair_embed(const PtbPairEmbed* args, cudaStream_t s) {
         return -1;
     }
     const bool pdl = ptb_pdl_enabled();
-    PTB_CUDA_OK(ptb_launch(p.bf16 ? streams::pair_embed_kernel<__nv_bfloat16> : streams::pair_embed_kernel<float>, dim3(p.n), dim3(256), 0, s, pdl, p));
+    const bool vec = p.W % 4 == 0 && (((uintptr_t)p.table | (uintptr_t)p.pairs | (uintptr_t)p.at | (uintptr_t)p.x) & 15) == 0;
+    auto kern = p.bf16 ? (vec ? streams::pair_embed_kernel<__nv_bfloat16, 4> : streams::pair_embed_kernel<__nv_bfloat16, 1>)
+                       : (vec ? streams::pair_embed_kernel<float, 4> : streams::pair_embed_kernel<float, 1>);
+    PTB_CUDA_OK(ptb_launch(kern, dim3(p.n), dim3(256), 0, s, pdl, p));
     if (p.seqs && p.n_seqs > 0) PTB_CUDA_OK(ptb_launch(streams::pair_tail_kernel, dim3((p.n_seqs + 255) / 256), dim3(256), 0, s, pdl, p));
     PTB_CUDA_OK(cudaGetLastError());
     return 0;

@@ -308,9 +308,12 @@ class PagedTifepel(PagedModel):
                 d["gain"] = gain(m.temp_coef, m.temp_every)
             if x:
                 parts = lambda n: [L[f"mlp.e{i}.{n}"] for i in range(x.experts)]
-                d["experts"] = X.Experts.of(parts("gate"), parts("up"), parts("down"), L["mlp.router"], L["mlp.correction"], x.top, 1.0, softmax=True)
-                if x.shared:
-                    d["shared"] = X.SharedExpert.of(*(L["mlp.shared." + n] for n in ("gate", "up", "down")))
+                shared = tuple(L["mlp.shared." + n] for n in ("gate", "up", "down")) if x.shared else None
+                join = x.shared <= X.SHARED_PARTS * x.ff
+                d["experts"] = X.Experts.of(parts("gate"), parts("up"), parts("down"), L["mlp.router"], L["mlp.correction"], x.top, 1.0, softmax=True,
+                                            shared=shared if join else None)
+                if shared and not join:
+                    d["shared"] = X.SharedExpert.of(*shared)
                 for k in [k for k in L if k.startswith("mlp.e")]:
                     L[k] = L[k][:0]                        # the packed copy is what runs
             self.prep.append(d)

@@ -252,6 +252,8 @@ def test_experts(E, identity, top, ff, shared):
         t.update({"shared." + k: v.double() for k, v in zip(("gate", "up", "down"), three)})
         m["shared"] = {"ff": shared}
         got = got + X.run_shared(h, X.SharedExpert.of(*three)).y
+        joined = X.run(h, X.Experts.of(gate, up, down, router, corr, top, 1.0, softmax=True, shared=tuple(three)))       # as more experts of the same products
+        assert close(joined.combine(), oracle.moe(h.double(), t, "", m)) and joined.index.shape[1] == top + -(-shared // ff)
     assert close(got, oracle.moe(h.double(), t, "", m))
     held = out.index[out.index >= 0]
     assert sorted(held.tolist()) == list(range(held.numel())) and (identity > 0) == bool((out.index < 0).any())

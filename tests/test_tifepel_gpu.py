@@ -258,40 +258,44 @@ def test_gate_ahead_of_a_grouped_norm(K, groups, dtype):
 
 
 # ------------------------------------------------------------------------------------------ experts
-def expert_case(n, W, ff, E, identity, top, dtype, seed=0, spread=0.3):
+def expert_case(n, W, ff, E, identity, top, dtype, seed=0, spread=0.3, shared=0):
     from prometorch_b200.ops import experts as X
     g = torch.Generator().manual_seed(seed)
     r = lambda *s, by=1.0: (torch.randn(*s, generator=g) * by).to(dtype)
     gate, up, down = ([r(*s, by=s[1] ** -0.5) for _ in range(E)] for s in ((ff, W), (ff, W), (W, ff)))
+    three = [r(*s, by=s[1] ** -0.5) for s in ((shared, W), (shared, W), (W, shared))] if shared else None
     O = E + identity
     h, router, corr = r(n, W), r(O, W, by=2 * W ** -0.5), torch.randn(O, generator=g) * spread
-    make = lambda dev, dt: X.Experts.of(*([t.to(dev, dt) for t in m] for m in (gate, up, down)), router.to(dev, dt), corr.to(dev), top, 1.0, softmax=True)
+    make = lambda dev, dt: X.Experts.of(*([t.to(dev, dt) for t in m] for m in (gate, up, down)), router.to(dev, dt), corr.to(dev), top, 1.0, softmax=True,
+                                        shared=tuple(t.to(dev, dt) for t in three) if three else None)
     return h, make("cpu", torch.float32), make("cuda", dtype)
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("n,E,identity,top", [(1, 4, 2, 2), (7, 8, 0, 3), (64, 64, 16, 8), (65, 64, 16, 8), (500, 5, 2, 7), (300, 200, 100, 40), (33, 1, 1, 1), (20, 250, 6, 4),
-                                              (64, 3, 60, 5), (200, 300, 1, 2)])
-def test_softmax_routing_with_identities(n, E, identity, top, dtype):
+@pytest.mark.parametrize("n,E,identity,top,shared", [(1, 4, 2, 2, 8), (7, 8, 0, 3, 0), (64, 64, 16, 8, 20), (65, 64, 16, 8, 16), (500, 5, 2, 7, 0), (300, 200, 100, 40, 9), (33, 1, 1, 1, 8),
+                                                     (20, 250, 6, 4, 1), (64, 3, 60, 5, 0), (200, 300, 1, 2, 70)])
+def test_softmax_routing_with_identities(n, E, identity, top, shared, dtype):
     """Against the plain choice from the same logits, except where the last score chosen and the next are all but equal."""
     from prometorch_b200.ops import experts as X, paged as P
-    h, c, g = expert_case(n, 64, 8, E, identity, top, dtype)
-    O = E + identity
+    h, c, g = expert_case(n, 64, 8, E, identity, top, dtype, shared=shared)
+    O, parts, K = E + identity, -(-shared // 8), top + -(-shared // 8)
     r = X.route(h.cuda(), g)
     z = h.double() @ c.router[:O].double().t()
     s = torch.softmax(z, -1)
     order = torch.sort(s + c.correction, descending=True)
     clear = order.values[:, top - 1] - order.values[:, top] > 1e-4 if top < O else torch.ones(n, dtype=torch.bool)
     off, token, index, weight = r.offsets.cpu(), r.token.cpu(), r.index.cpu(), r.weight.cpu()
+    assert g.always == parts and off.shape[0] == E + parts + 1 and index.shape[1] == K
     held = (index >= 0).flatten()
-    assert int(off[0]) == 0 and int(off[E]) == int(held.sum()) and bool((off[1:] >= off[:-1]).all())
+    assert int(off[0]) == 0 and int(off[-1]) == int(held.sum()) and bool((off[1:] >= off[:-1]).all())
     assert sorted(index.flatten()[held].tolist()) == list(range(int(held.sum())))
-    assert torch.equal(token[index.flatten()[held].long()], torch.arange(n).repeat_interleave(top).int()[held])
-    expert = torch.where(index < 0, E, torch.searchsorted(off[1:].contiguous(), index, right=True))
+    assert torch.equal(token[index.flatten()[held].long()], torch.arange(n).repeat_interleave(K).int()[held])
+    expert = torch.where(index < 0, -1, torch.searchsorted(off[1:].contiguous(), index, right=True))
+    assert torch.equal(expert[:, top:], torch.arange(E, E + parts).expand(n, parts)) and bool((weight[:, top:] == 1).all())
     for i in clear.nonzero()[:, 0].tolist():
-        want = sorted(min(o, E) for o in order.indices[i, :top].tolist())
-        assert sorted(expert[i].tolist()) == want
-        assert torch.allclose(weight[i].sort().values.double(), s[i, order.indices[i, :top]].sort().values, rtol=1e-4, atol=1e-9)
+        want = sorted(o if o < E else -1 for o in order.indices[i, :top].tolist())
+        assert sorted(expert[i, :top].tolist()) == want
+        assert torch.allclose(weight[i, :top].sort().values.double(), s[i, order.indices[i, :top]].sort().values, rtol=1e-4, atol=1e-9)
     P.check_status("cuda")
 
 
@@ -299,16 +303,20 @@ def test_softmax_routing_with_identities(n, E, identity, top, dtype):
 @pytest.mark.parametrize("n,W,ff,E,identity,top,shared", [(1, 64, 128, 4, 2, 2, 64), (5, 192, 96, 8, 3, 4, 100), (40, 128, 200, 3, 1, 4, 0), (300, 128, 256, 6, 6, 2, 256),
                                                           (1500, 256, 136, 4, 1, 1, 520), (70, 50, 20, 7, 2, 3, 12), (200, 64, 33, 64, 16, 8, 33), (16, 520, 1032, 2, 0, 1, 2048)])
 def test_expert_and_shared_products(n, W, ff, E, identity, top, shared, dtype):
+    """Experts, and a shared expert both among them and by itself."""
     from prometorch_b200.ops import experts as X, paged as P
-    h, c, g = expert_case(n, W, ff, E, identity, top, dtype, spread=0.2)
-    r = X.route(h.cuda(), g)
-    cpu = X.Routing(*(t.cpu() for t in (r.index, r.weight, r.token, r.offsets)))
-    live = int(cpu.offsets[-1])
-    want = X.products(h.float(), c, X.Routing(cpu.index, cpu.weight, cpu.token.clamp(0, n - 1), cpu.offsets))[:live]
     tol = 2e-6 if dtype == torch.float32 else 1e-2
-    for simt in (False, True):
-        got = X.products(h.cuda(), g, r, simt=simt)[:live]
-        assert torch.isfinite(got).all() and (live == 0 or rel(got, want) < tol), simt
+    for wide in {0, shared}:
+        h, c, g = expert_case(n, W, ff, E, identity, top, dtype, spread=0.2, shared=wide)
+        r = X.route(h.cuda(), g)
+        cpu = X.Routing(*(t.cpu() for t in (r.index, r.weight, r.token, r.offsets)))
+        live = int(cpu.offsets[-1])
+        want = X.products(h.float(), c, X.Routing(cpu.index, cpu.weight, cpu.token.clamp(0, n - 1), cpu.offsets))[:live]
+        for simt in (False, True):
+            got = X.products(h.cuda(), g, r, simt=simt)[:live]
+            assert torch.isfinite(got).all() and (live == 0 or rel(got, want) < tol), simt
+        total = X.ExpertRows(X.products(h.cuda(), g, r), r.index, r.weight, h.cuda()).combine()
+        assert rel(total, X.ExpertRows(X.products(h.float(), c, X.Routing(cpu.index, cpu.weight, cpu.token.clamp(0, n - 1), cpu.offsets)), cpu.index, cpu.weight, h).combine()) < tol
     if shared:
         three = [(torch.randn(*s) * s[1] ** -0.5).to(dtype) for s in ((shared, W), (shared, W), (W, shared))]
         got = X.run_shared(h.cuda(), X.SharedExpert.of(*(t.cuda() for t in three))).y
