@@ -13,7 +13,9 @@
 namespace ptb {
 namespace streams {
 
-constexpr int MAX_STREAMS = 16, MAX_THREADS = 1024;
+constexpr int MAX_STREAMS = 16;
+// Most threads of a row's CTA: a thread holds its columns of all streams in registers.
+__host__ __device__ constexpr int max_threads(int S) { return S == 0 ? 256 : S > 2 ? 512 : 1024; }
 
 template <int V> struct Vals { float v[V]; };
 template <int V, typename T>
@@ -116,7 +118,7 @@ __device__ __forceinline__ Vals<V> dense_load(const PtbDense& D, size_t row, int
 
 // One CTA per row.  T: the compute type; V elements per access; S streams (0: any number up to MAX_STREAMS).
 template <typename T, int V, int S>
-__global__ void __launch_bounds__(MAX_THREADS) stream_step_kernel(const __grid_constant__ PtbStreamStep P) {
+__global__ void __launch_bounds__(max_threads(S)) stream_step_kernel(const __grid_constant__ PtbStreamStep P) {
     extern __shared__ __align__(16) float u_s[];       // [W] what the next sublayer reads
     __shared__ float mix_s[MAX_STREAMS * MAX_STREAMS], out_s[MAX_STREAMS], in_s[MAX_STREAMS], red[2][32];
     const int streams = S ? S : P.streams, W = P.W;
@@ -247,7 +249,7 @@ __global__ void __launch_bounds__(MAX_THREADS) stream_step_kernel(const __grid_c
 
 template <typename T, int V>
 static cudaError_t step_launch(const PtbStreamStep& p, cudaStream_t s) {
-    const int lanes = (p.W + V - 1) / V, most = p.m <= 256 ? MAX_THREADS : 256;
+    const int lanes = (p.W + V - 1) / V, most = p.m <= 256 ? max_threads(p.streams > 4 ? 0 : p.streams) : 256;
     const int threads = std::min(most, (lanes + 31) / 32 * 32);
     const size_t smem = p.norm ? (size_t)p.W * 4 : 0;
     auto go = [&](auto k) {

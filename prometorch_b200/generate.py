@@ -1,5 +1,5 @@
 """Command-line text generation from a GGUF file (or an Ollama model name), or from a directory with ``config.json`` and
-safetensors (the models of the batching engine: Hugging Face Llama, Kifusun, Gelutar, Budorax).
+safetensors (the models of the batching engine: Hugging Face Llama, Kifusun, Gelutar, Budorax, Tifepel).
 
     python -m prometorch_b200.generate MODEL [PROMPT] [--device cuda|cpu] [--greedy] [--max-tokens N] [--temp T]
         [--top-k K] [--top-p P] [--chat | --raw] [--info] [--tensors] [--profile] [--nprocs N]
